@@ -68,6 +68,7 @@ SIGNATURES = {
     "axb200_decode_step_host": (_i, [_vp] * 12 + [_vp, _vp, _f, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i64, _i,
                                           _vp, _sz, _vp]),
     "axb200_kv_arena_create": (_i, [_i, _i, _i, _i, _i, _i, _i, _i, _i, C.POINTER(_vp)]),
+    "axb200_kv_arena_create_rows": (_i, [_i, _vp, _i, _i, _i, _i, _i, _i, C.POINTER(_vp)]),
     "axb200_kv_arena_destroy": (_i, [_vp]),
     "axb200_kv_arena_alloc_seq": (_i, [_vp, _i64, C.POINTER(_i)]),
     "axb200_kv_arena_reserve": (_i, [_vp, _i, _i64]),
@@ -91,6 +92,22 @@ SIGNATURES = {
     "axb200_embedding": (_i, [_vp, _i, _vp, _vp, _i64, _i64, _i, _i, _vp]),
     "axb200_argmax_last_dim": (_i, [_vp, _vp, _i64, _i, _i, _vp]),
     "axb200_linear_nobias": (_i, [_vp, _vp, _vp, _i64, _i64, _i64, _i, _vp]),
+    # x, w, out | rows, out, in, x_ld, w_ld, out_ld, batch, x_stride, w_stride, out_stride | w_in_major, dtypes
+    "axb200_linear_strided": (_i, [_vp] * 3 + [_i64] * 10 + [_i] * 3 + [_vp]),
+    "axb200_embed_layer_norm": (_i, [_vp, _vp, _vp, _f, _vp, _i64, _i64, _i, _i, _vp]),
+    "axb200_residual_layer_norm": (_i, [_vp] * 6 + [_i] + [_vp] * 4 + [_f, _i64, _i, _i, _vp]),
+    "axb200_latent_prepare": (_i, [_vp, _i64, _i, _i, _vp, _i64, _i, _vp, _vp, _vp, _i64, _i, _vp, _f] + [_vp] * 5 +
+                              [_i, _i, _i64] + [_i] * 5 + [_vp]),
+    "axb200_latent_attend_workspace_bytes": (_sz, [_i, _i, _i, _i, _i64, _i]),
+    "axb200_latent_attend": (_i, [_vp, _vp, _i64, _i] + [_vp] * 5 + [_i] * 4 + [_f] + [_i] * 4 + [_i64, _i, _vp, _sz, _vp]),
+    "axb200_latent_gather": (_i, [_vp, _vp, _vp, _i64, _i, _i, _i, _i, _i, _vp]),
+    "axb200_latent_prefill_supported": (_i, [_i] * 5),
+    "axb200_latent_prefill": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _i, _i64, _i, _i, _i, _i, _f, _i, _vp]),
+    "axb200_moe_route": (_i, [_vp] * 6 + [_i64, _i, _i, _i, _i, _f, _vp]),
+    "axb200_moe_tile_rows": (_i, [_i64, _i, _i, _i, _i]),
+    "axb200_moe_sort": (_i, [_vp] * 9 + [_i64, _i, _i, _i, _i, _i, _vp]),
+    "axb200_moe_gate_up": (_i, [_vp] * 5 + [_i64, _i, _i, _i, _i, _f, _f, _f, _i, _vp]),
+    "axb200_moe_down": (_i, [_vp] * 5 + [_i64, _i, _i, _i, _i, _i, _vp]),
     "axb200_randn": (_i, [_vp, _i64, _i, _f, _f, C.c_uint64, _vp]),
     "axb200_cast": (_i, [_vp, _i, _vp, _i, _i64, _vp]),
     "axb200_concat": (_i, [_vp, _vp, _vp, _i64, _sz, _sz, _vp]),
@@ -101,12 +118,25 @@ STATUS_NAMES = ["OK", "INVALID_ARGUMENT", "OUT_OF_MEMORY", "UNSUPPORTED_TYPE", "
 
 # axono::core::DataType values (include/axono/core/types.h:18-27 of the reference)
 INT8, INT16, INT32, INT64, FLOAT16, FLOAT32, FLOAT64, BOOLEAN = range(8)
+BFLOAT16 = 8  # extension, for the language-model operators
 
 _lib = None
 
 
+_path = None
+
+
 def library_path() -> str:
-    return _build.LIB
+    return _path or _build.LIB
+
+
+def use_serving_library() -> str:
+    """For processes that serve a model: builds what they need if it is missing or stale (the full library when
+    that is up to date) and makes it the one `lib()` loads.  Without effect once a library is loaded."""
+    global _path
+    if _lib is None:
+        _path = _build.build_serving()
+    return library_path()
 
 
 def lib() -> C.CDLL:
@@ -120,6 +150,8 @@ def lib() -> C.CDLL:
                 "axono_b200 has no fallback path.")
         handle = C.CDLL(path)
         for name, (res, args) in SIGNATURES.items():
+            if path == _build.SERVING_LIB and not hasattr(handle, name):
+                continue  # the subset library has no such operator
             fn = getattr(handle, name)
             fn.restype = res
             fn.argtypes = args

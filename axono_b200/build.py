@@ -1,15 +1,22 @@
 """Builds the C-ABI library (axono_b200/lib/libaxono_b200.so) for sm_100a with nvcc, and the native
 Python module `libaxono` (host runtime + operator adapters + pybind11 binding) that links against it.
 
-    python -m axono_b200.build [--force] [--verbose]
+    python -m axono_b200.build [--force] [--verbose] [--serving]
 
 nvcc cross-compiles without a GPU; the library is kept in-tree so it travels with the
-source checkout.  Rebuilds only when a source or header is newer than the library.
+source checkout.  Sources compile to objects side by side and only where a source or header is newer.
+
+`build_serving()` links the subset of the same objects that the language-model serving path calls into
+libaxono_b200_lm.so: a fresh checkout that only serves a model compiles that much and no more.
 """
 from __future__ import annotations
 
+import concurrent.futures
+import contextlib
+import fcntl
 import glob
 import os
+import shutil
 import subprocess
 import sys
 
@@ -17,12 +24,16 @@ PKG = os.path.dirname(os.path.abspath(__file__))
 ROOT = os.path.dirname(PKG)
 CSRC = os.path.join(PKG, "csrc")
 LIB_DIR = os.path.join(PKG, "lib")
+OBJ_DIR = os.path.join(LIB_DIR, "obj")
 LIB = os.path.join(LIB_DIR, "libaxono_b200.so")
+SERVING_LIB = os.path.join(LIB_DIR, "libaxono_b200_lm.so")
+SERVING_SOURCES = ("core.cu", "fused.cu", "kv_arena.cu", "latent_attn.cu", "latent_prefill.cu", "linear_lt.cpp", "moe.cu",
+                   "moe_umma.cu", "residual_norm.cu")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
     "-O3", "-std=c++17", "-lineinfo",
-    "-Xcompiler", "-fPIC", "-shared",
+    "-Xcompiler", "-fPIC",
 ]
 
 
@@ -30,26 +41,65 @@ def sources():
     return sorted(glob.glob(os.path.join(CSRC, "*.cu")) + glob.glob(os.path.join(CSRC, "*.cpp")))
 
 
-def _stale() -> bool:
-    if not os.path.exists(LIB):
+def serving_sources():
+    return [os.path.join(CSRC, name) for name in SERVING_SOURCES]
+
+
+def _headers():
+    return (glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h")) +
+            glob.glob(os.path.join(ROOT, "include", "*.h")))
+
+
+def _newer(deps, target) -> bool:
+    if not os.path.exists(target):
         return True
-    t = os.path.getmtime(LIB)
-    deps = sources() + glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
-    deps += glob.glob(os.path.join(ROOT, "include", "*.h"))
+    t = os.path.getmtime(target)
     return any(os.path.getmtime(d) > t for d in deps)
 
 
+@contextlib.contextmanager
+def _build_lock():
+    os.makedirs(OBJ_DIR, exist_ok=True)
+    with open(os.path.join(OBJ_DIR, ".lock"), "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        yield
+
+
+def _link(lib: str, srcs, force: bool, verbose: bool) -> str:
+    if not force and not _newer(list(srcs) + _headers(), lib):
+        return lib
+    with _build_lock():
+        nvcc = os.environ.get("NVCC") or shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
+        headers = _headers()
+
+        def compile_one(src):
+            obj = os.path.join(OBJ_DIR, os.path.basename(src) + ".o")
+            if force or _newer([src] + headers, obj):
+                cmd = [nvcc, *NVCC_FLAGS, "-I", os.path.join(ROOT, "include"), "-I", CSRC]
+                if verbose:
+                    cmd += ["-Xptxas", "-v"]
+                part = f"{obj}.{os.getpid()}"
+                subprocess.check_call([*cmd, "-c", src, "-o", part])
+                os.replace(part, obj)
+            return obj
+
+        with concurrent.futures.ThreadPoolExecutor(max(1, min(len(srcs), os.cpu_count() or 1))) as pool:
+            objs = list(pool.map(compile_one, srcs))
+        part = f"{lib}.{os.getpid()}"
+        subprocess.check_call([nvcc, *NVCC_FLAGS, "-shared", "-o", part, *objs, "-ldl"])
+        os.replace(part, lib)
+    return lib
+
+
 def build(force: bool = False, verbose: bool = False) -> str:
-    if not force and not _stale():
+    return _link(LIB, sources(), force, verbose)
+
+
+def build_serving(force: bool = False, verbose: bool = False) -> str:
+    """The library a serving process loads: the full one when it is there and up to date, else the subset."""
+    if not force and not _newer(sources() + _headers(), LIB):
         return LIB
-    os.makedirs(LIB_DIR, exist_ok=True)
-    nvcc = os.environ.get("NVCC", "nvcc")
-    cmd = [nvcc, *NVCC_FLAGS, "-I", os.path.join(ROOT, "include"), "-I", CSRC]
-    if verbose:
-        cmd += ["-Xptxas", "-v"]
-    cmd += ["-o", LIB, *sources(), "-ldl"]
-    subprocess.check_call(cmd)
-    return LIB
+    return _link(SERVING_LIB, serving_sources(), force, verbose)
 
 
 HOST = os.path.join(CSRC, "host")
@@ -86,5 +136,8 @@ def build_native(force: bool = False) -> str:
 
 
 if __name__ == "__main__":
+    if "--serving" in sys.argv:
+        print(build_serving(force="--force" in sys.argv, verbose="--verbose" in sys.argv))
+        sys.exit(0)
     print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv))
     print(build_native(force="--force" in sys.argv))

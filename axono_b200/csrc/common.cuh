@@ -4,6 +4,7 @@
 #pragma once
 
 #include <cuda.h>
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -19,6 +20,10 @@ static __device__ unsigned int g_error_word = 0;
 
 using ErrorReader = unsigned int (*)();
 void register_error_reader(ErrorReader fn);  // defined once, beside axb200_last_error()
+// Called by axb200_last_error() after a wait ran out: restores device-side counters that the CTAs which gave
+// up left half-counted.
+using TimeoutHook = void (*)();
+void register_timeout_hook(TimeoutHook fn);
 
 static unsigned int read_clear_error_word() {
   unsigned int word = 0, zero = 0;
@@ -53,10 +58,37 @@ int decode_step_try_fused(const void *q, const void *k_new, const void *v_new, v
 
 inline size_t dtype_size(int dtype) {
   switch (dtype) {
-    case AXB200_FLOAT16: return 2;
+    case AXB200_FLOAT16:
+    case AXB200_BFLOAT16: return 2;
     case AXB200_FLOAT32: return 4;
     default: return 0;
   }
+}
+
+// One element of a stored type as a float, and back (round to nearest even).
+__device__ __forceinline__ float ldf(const float *p) { return *p; }
+__device__ __forceinline__ float ldf(const __half *p) { return __half2float(*p); }
+__device__ __forceinline__ float ldf(const __nv_bfloat16 *p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void stf(float *p, float v) { *p = v; }
+__device__ __forceinline__ void stf(__half *p, float v) { *p = __float2half_rn(v); }
+__device__ __forceinline__ void stf(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
+  return v;
+}
+
+// Sum over the CTA; every thread gets the total.
+__device__ __forceinline__ float block_sum(float v, float *scratch /* >= 32 floats */) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+  v = warp_sum(v);
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  float t = lane < nwarps ? scratch[lane] : 0.f;
+  t = warp_sum(t);
+  __syncthreads();
+  return t;
 }
 
 inline int launch_status() {
@@ -142,6 +174,27 @@ __device__ __forceinline__ bool mbar_wait_bounded(uint64_t *bar, uint32_t parity
 __device__ __forceinline__ void grid_dependency_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void grid_dependency_launch() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
+// Launches `kernel` as a programmatic dependent of the kernel before it in the stream (see above); the kernel
+// must call grid_dependency_wait() before it touches anything an earlier kernel wrote.
+template <typename... KArgs, typename... Args>
+inline int launch_dependent(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args &&...args) {
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  if (cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...) != cudaSuccess) {
+    cudaGetLastError();
+    return AXB200_DEVICE_ERROR;
+  }
+  return AXB200_OK;
+}
+
 // ---- rotary position embedding: the arithmetic every kernel that rotates shares ------------------
 // Pair (a, b) = (x[i], x[i + half]) turned by the angle whose cosine and sine are (c, s).  The
 // roundings are spelled out (one product rounded, then one fused multiply-add) so that the append
@@ -200,6 +253,20 @@ __device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4],
       "{%0,%1,%2,%3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// D(16x8,f32) += A(16x16,bf16,row) * B(16x8,bf16,col)
+__device__ __forceinline__ void mma_16816_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
+      "{%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+__device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
+  __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<uint32_t *>(&h);
 }
 
 __device__ __forceinline__ uint32_t pack_half2(float lo, float hi) {

@@ -31,37 +31,6 @@ struct Vec<__half> {
   }
 };
 
-template <typename T>
-__device__ __forceinline__ float ldf(const T *p);
-template <>
-__device__ __forceinline__ float ldf<float>(const float *p) { return *p; }
-template <>
-__device__ __forceinline__ float ldf<__half>(const __half *p) { return __half2float(*p); }
-template <typename T>
-__device__ __forceinline__ void stf(T *p, float v);
-template <>
-__device__ __forceinline__ void stf<float>(float *p, float v) { *p = v; }
-template <>
-__device__ __forceinline__ void stf<__half>(__half *p, float v) { *p = __float2half_rn(v); }
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
-  return v;
-}
-
-// Sum over the CTA; every thread gets the total.
-__device__ __forceinline__ float block_sum(float v, float *scratch /* >= 32 floats */) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
-  v = warp_sum(v);
-  if (lane == 0) scratch[warp] = v;
-  __syncthreads();
-  float t = lane < nwarps ? scratch[lane] : 0.f;
-  t = warp_sum(t);
-  __syncthreads();
-  return t;
-}
-
 // ---- add_rms_norm: y = x + res; out = y * rsqrt(mean(y^2) + eps) * w -----------------------------
 // One CTA per row.  Vector path: each thread keeps up to kMaxVec 16-byte vectors of y in
 // registers between the two phases, so x and res are read once and y/out written once.

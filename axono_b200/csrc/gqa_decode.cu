@@ -28,16 +28,6 @@
 namespace axb {
 
 namespace {
-constexpr int kMaxErrorReaders = 16;
-ErrorReader g_error_readers[kMaxErrorReaders];
-int g_num_error_readers = 0;
-}  // namespace
-
-void register_error_reader(ErrorReader fn) {
-  if (g_num_error_readers < kMaxErrorReaders) g_error_readers[g_num_error_readers++] = fn;
-}
-
-namespace {
 
 constexpr int kHeadDim = 128;
 constexpr int kConsumerWarps = 4;
@@ -128,6 +118,14 @@ __global__ void zero_arrival_kernel() {
        i += gridDim.x * blockDim.x)
     g_arrival[i] = g_step_readers[i] = 0u;
 }
+
+namespace {
+// after a wait that ran out: a CTA that gave up never counted itself in
+struct ArrivalReset {
+  ArrivalReset() { register_timeout_hook([] { zero_arrival_kernel<<<64, 256>>>(); }); }
+};
+static ArrivalReset g_arrival_reset;
+}  // namespace
 
 __device__ __forceinline__ int seq_len_raw(const DecodeParams &p, int b) {
   if (p.seq_lens) return p.seq_lens[b];
@@ -1760,7 +1758,6 @@ bool make_map(CUtensorMap *map, const void *base, int dtype, bool paged, int d, 
 
 // ---- host settings -------------------------------------------------------------------------------
 std::mutex g_settings_mu;
-unsigned long long g_wait_limit_ns = kWaitNanos;
 bool g_fused_merge = true;
 bool g_merge_pairs = true;
 bool g_step_fused = true;  // axb200_decode_step_paged may use the one-launch form
@@ -1985,7 +1982,7 @@ int decode_impl(bool paged, const void *q, void *out, const void *k, const void 
   p.row_offset = row_offset;
   {
     std::lock_guard<std::mutex> lock(g_settings_mu);
-    p.wait_ns = g_wait_limit_ns;
+    p.wait_ns = wait_limit_ns();
   }
   const bool need_ws = pl.max_chunks > 1;
   if (need_ws) {
@@ -2199,7 +2196,7 @@ int axb200_qkv_decode_step_paged(const void *qkv, int64_t ld, const void *q_norm
                                  int rank, int hq_total, void *stream) {
   using namespace axb;
   const size_t es = dtype_size(dtype);
-  if (es == 0) return AXB200_UNSUPPORTED_TYPE;
+  if (es == 0 || dtype == AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
   if (!qkv || !k_pages || !v_pages || !block_table || !seq_lens || !workspace) return AXB200_INVALID_PTR;
   if (batch <= 0 || hq <= 0 || hkv <= 0 || d <= 0 || max_seq_len <= 0 || ld < (int64_t)(hq + 2 * hkv) * d)
     return AXB200_INVALID_ARGUMENT;
@@ -2275,7 +2272,7 @@ int axb200_set_step_fused(int on) {
 
 size_t axb200_decode_step_workspace_bytes(int batch, int hq, int hkv, int d, int64_t max_seq_len, int dtype) {
   const size_t es = axb::dtype_size(dtype);
-  if (es == 0 || batch <= 0 || hq <= 0 || hkv <= 0 || d <= 0 || max_seq_len <= 0) return 0;
+  if (es == 0 || dtype == AXB200_BFLOAT16 || batch <= 0 || hq <= 0 || hkv <= 0 || d <= 0 || max_seq_len <= 0) return 0;
   const size_t attn = (axb200_gqa_workspace_bytes(batch, hq, hkv, d, max_seq_len, dtype) + 255) & ~size_t(255);
   return attn + (((size_t)batch * hq * d * es + 255) & ~size_t(255));  // + the rotated q of the two-launch form
 }
@@ -2300,7 +2297,7 @@ int axb200_decode_step_paged(const void *q, const void *k_new, const void *v_new
                              int max_blocks, int num_pages, int64_t max_seq_len, int dtype, void *workspace,
                              size_t workspace_bytes, void *stream) {
   const size_t es = axb::dtype_size(dtype);
-  if (es == 0) return AXB200_UNSUPPORTED_TYPE;
+  if (es == 0 || dtype == AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
   if (!q || !k_new || !v_new || !out || !k_pages || !v_pages || !block_table || !seq_lens || !workspace)
     return AXB200_INVALID_PTR;
   if (batch <= 0 || hq <= 0 || hkv <= 0 || d <= 0 || max_seq_len <= 0) return AXB200_INVALID_ARGUMENT;
@@ -2327,13 +2324,6 @@ int axb200_decode_step_paged(const void *q, const void *k_new, const void *v_new
   if (rc != AXB200_OK) return rc;
   return axb200_gqa_decode_paged(q_attn, out, k_pages, v_pages, block_table, seq_lens, batch, hq, hkv, d, page_tokens,
                                  max_blocks, num_pages, max_seq_len, dtype, workspace, attn_bytes, stream);
-}
-
-int axb200_set_wait_limit_ns(uint64_t ns) {
-  if (ns == 0) return AXB200_INVALID_ARGUMENT;
-  std::lock_guard<std::mutex> lock(axb::g_settings_mu);
-  axb::g_wait_limit_ns = ns;
-  return AXB200_OK;
 }
 
 int axb200_set_dependent_launch(int on) {
@@ -2503,20 +2493,6 @@ int axb200_p2p_close(void *dev_ptr) {
 
 int axb200_p2p_free(void *dev_ptr) {
   return cudaFree(dev_ptr) == cudaSuccess ? AXB200_OK : AXB200_DEVICE_ERROR;
-}
-
-const char *axb200_version(void) { return "axono_b200 0.2 (sm_100a)"; }
-
-unsigned int axb200_last_error(void) {
-  if (cudaDeviceSynchronize() != cudaSuccess) return 0x80000000u;
-  unsigned int word = 0;
-  for (int i = 0; i < axb::g_num_error_readers; ++i) word |= axb::g_error_readers[i]();
-  if (word & AXB200_ERR_WAIT_TIMEOUT) {
-    // a CTA that gave up never counted itself in: put the fused merge's counters back to zero
-    axb::zero_arrival_kernel<<<64, 256>>>();
-    cudaDeviceSynchronize();
-  }
-  return word;
 }
 
 int axb200_profile_enable(int on) {

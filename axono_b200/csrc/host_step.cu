@@ -35,7 +35,7 @@ extern "C" int axb200_decode_step_host(
     int page_tokens, int max_blocks, int num_pages, int64_t max_seq_len, int dtype, void *workspace,
     size_t workspace_bytes, void *stream) {
   const size_t es = axb::dtype_size(dtype);
-  if (es == 0) return AXB200_UNSUPPORTED_TYPE;
+  if (es == 0 || dtype == AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
   if (!q_host || !k_new_host || !v_new_host || !out_host || !q_dev || !k_new_dev || !v_new_dev ||
       !out_dev)
     return AXB200_INVALID_PTR;

@@ -28,10 +28,11 @@ struct axb200_kv_arena {
   std::vector<int32_t> blocks_of;            // pages held per sequence slot
   std::vector<uint8_t> live;                 // slot in use
   int dirty_lo, dirty_hi;                    // rows whose device copy is stale: [lo, hi)
-  std::vector<void *> k_pools, v_pools;      // per layer
+  std::vector<void *> k_pools, v_pools;      // per layer (no v_pools in an arena of rows)
   int32_t *table_dev = nullptr;
   int32_t *seq_lens_dev = nullptr;
-  size_t pool_bytes = 0;
+  std::vector<size_t> pool_bytes;            // per layer, of each of its pools
+  bool has_v = true;
 };
 
 namespace {
@@ -58,17 +59,14 @@ int reserve_locked(axb200_kv_arena *a, int seq, int64_t tokens) {
   return AXB200_OK;
 }
 
-}  // namespace
-
-extern "C" {
-
-int axb200_kv_arena_create(int n_layers, int num_pages, int hkv, int page_tokens, int d, int dtype,
-                           int max_seqs, int max_blocks, int device_memory,
-                           axb200_kv_arena **out) {
-  if (!out) return AXB200_INVALID_PTR;
+// row_elems[l]: elements of one token's row in layer l's pool (K pool, and V pool when has_v)
+int create_arena(int n_layers, const int32_t *row_elems, bool has_v, int num_pages, int hkv, int page_tokens, int d,
+                 int dtype, int max_seqs, int max_blocks, int device_memory, axb200_kv_arena **out) {
   if (n_layers <= 0 || num_pages <= 0 || hkv <= 0 || page_tokens <= 0 || page_tokens % 64 != 0 ||
       d <= 0 || max_seqs <= 0 || max_blocks <= 0 || axb::dtype_size(dtype) == 0)
     return AXB200_INVALID_ARGUMENT;
+  for (int l = 0; l < n_layers; ++l)
+    if (row_elems[l] <= 0) return AXB200_INVALID_ARGUMENT;
   axb200_kv_arena *a = new (std::nothrow) axb200_kv_arena();
   if (!a) return AXB200_OUT_OF_MEMORY;
   a->n_layers = n_layers;
@@ -87,15 +85,18 @@ int axb200_kv_arena_create(int n_layers, int num_pages, int hkv, int page_tokens
   a->live.assign(max_seqs, 0);
   a->dirty_lo = 0;
   a->dirty_hi = max_seqs;
-  a->pool_bytes = (size_t)num_pages * hkv * page_tokens * d * axb::dtype_size(dtype);
+  a->has_v = has_v;
+  for (int l = 0; l < n_layers; ++l)
+    a->pool_bytes.push_back((size_t)num_pages * page_tokens * row_elems[l] * axb::dtype_size(dtype));
   if (a->device) {
     bool ok = true;
     for (int l = 0; l < n_layers && ok; ++l) {
       void *k = nullptr, *v = nullptr;
-      ok = cudaMalloc(&k, a->pool_bytes) == cudaSuccess && cudaMalloc(&v, a->pool_bytes) == cudaSuccess;
+      const size_t bytes = a->pool_bytes[l];
+      ok = cudaMalloc(&k, bytes) == cudaSuccess && (!has_v || cudaMalloc(&v, bytes) == cudaSuccess);
       if (k) a->k_pools.push_back(k);
       if (v) a->v_pools.push_back(v);
-      if (ok) ok = cudaMemset(k, 0, a->pool_bytes) == cudaSuccess && cudaMemset(v, 0, a->pool_bytes) == cudaSuccess;
+      if (ok) ok = cudaMemset(k, 0, bytes) == cudaSuccess && (!has_v || cudaMemset(v, 0, bytes) == cudaSuccess);
     }
     ok = ok && cudaMalloc(&a->table_dev, a->table.size() * sizeof(int32_t)) == cudaSuccess &&
          cudaMalloc(&a->seq_lens_dev, max_seqs * sizeof(int32_t)) == cudaSuccess &&
@@ -112,6 +113,27 @@ int axb200_kv_arena_create(int n_layers, int num_pages, int hkv, int page_tokens
   }
   *out = a;
   return AXB200_OK;
+}
+
+}  // namespace
+
+extern "C" {
+
+int axb200_kv_arena_create(int n_layers, int num_pages, int hkv, int page_tokens, int d, int dtype,
+                           int max_seqs, int max_blocks, int device_memory,
+                           axb200_kv_arena **out) {
+  if (!out) return AXB200_INVALID_PTR;
+  if (n_layers <= 0 || hkv <= 0 || d <= 0) return AXB200_INVALID_ARGUMENT;
+  const std::vector<int32_t> rows(n_layers, hkv * d);
+  return create_arena(n_layers, rows.data(), true, num_pages, hkv, page_tokens, d, dtype, max_seqs, max_blocks,
+                      device_memory, out);
+}
+
+int axb200_kv_arena_create_rows(int n_layers, const int32_t *row_elems, int num_pages, int page_tokens, int dtype,
+                                int max_seqs, int max_blocks, int device_memory, axb200_kv_arena **out) {
+  if (!out || !row_elems) return AXB200_INVALID_PTR;
+  return create_arena(n_layers, row_elems, false, num_pages, 1, page_tokens, n_layers > 0 ? row_elems[0] : 0, dtype, max_seqs,
+                      max_blocks, device_memory, out);
 }
 
 int axb200_kv_arena_shuffle_free(axb200_kv_arena *a, uint64_t seed) {
@@ -215,7 +237,10 @@ int axb200_kv_arena_stats(axb200_kv_arena *a, int64_t *pages_total, int64_t *pag
   if (pages_total) *pages_total = a->num_pages;
   if (pages_free) *pages_free = (int64_t)a->free_pages.size();
   if (seqs_live) *seqs_live = live;
-  if (device_bytes) *device_bytes = a->device ? (int64_t)(2 * a->pool_bytes * a->n_layers) : 0;
+  if (device_bytes) {
+    *device_bytes = 0;
+    for (size_t bytes : a->pool_bytes) *device_bytes += a->device ? (int64_t)(bytes * (a->has_v ? 2 : 1)) : 0;
+  }
   return AXB200_OK;
 }
 
@@ -247,7 +272,7 @@ void *axb200_kv_arena_k_pages(axb200_kv_arena *a, int layer) {
   return (a && a->device && layer >= 0 && layer < a->n_layers) ? a->k_pools[layer] : nullptr;
 }
 void *axb200_kv_arena_v_pages(axb200_kv_arena *a, int layer) {
-  return (a && a->device && layer >= 0 && layer < a->n_layers) ? a->v_pools[layer] : nullptr;
+  return (a && a->device && a->has_v && layer >= 0 && layer < a->n_layers) ? a->v_pools[layer] : nullptr;
 }
 int32_t *axb200_kv_arena_block_table(axb200_kv_arena *a) { return a ? a->table_dev : nullptr; }
 int32_t *axb200_kv_arena_seq_lens(axb200_kv_arena *a) { return a ? a->seq_lens_dev : nullptr; }

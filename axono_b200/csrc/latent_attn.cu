@@ -1,0 +1,317 @@
+// Attention over a cache of latents: every token caches one row [c (kv_rank) | rotated key part (rot_dim)] that
+// all heads share, and a head's key and value are linear maps of c.  Folding the key map into the query
+// (q_lat = q . W_uk) and the value map behind the sum turns it into attention of H queries per token over ONE
+// key row of kv_rank + rot_dim elements whose first kv_rank elements are also the value:
+//     score = (q_lat . c + q_rot . k_rot) * scale,   out_lat = sum softmax(score) c.
+// This file holds the kernels of that form: the step's norms, rotation and append in one launch; the
+// tensor-core split kernel (bf16) with its merge; an evaluation for every other size and for fp32; and the
+// gather that the expanded form (latent_prefill.cu) reads from.
+//
+// Rows are independent: row r belongs to sequence row_seq[r] (its block-table row) and sees the cached tokens
+// 0 .. row_pos[r], so one launch serves decode batches, portions of prompts and mixtures of both.
+#include <math.h>
+
+#include "tcgen05.cuh"
+
+namespace axb {
+namespace {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// ---- norms, rotation, append -----------------------------------------------------------------------
+template <typename T>
+struct PrepareParams {
+  T *q;  // (rows, q_ld): heads of [dim plain | rot_dim rotated], rotated in place; null: none
+  int64_t q_ld;
+  int heads, dim;
+  const T *dq;  // (rows, dq_ld): query latent to norm into cq (rows, q_rank); null: none
+  int64_t dq_ld;
+  int q_rank;
+  const T *dq_w;
+  T *cq;
+  const T *dkv;  // (rows, dkv_ld): [kv_rank | rot_dim] to norm, rotate and append; null: none
+  int64_t dkv_ld;
+  int kv_rank;
+  const T *dkv_w;
+  T *pages;  // (num_pages, page_tokens, kv_rank + rot_dim)
+  const int32_t *block_table, *row_seq, *row_pos;
+  const double *inv_freq;  // (rot_pairs)
+  int rot_dim, rot_pairs, max_blocks, page_tokens, num_pages, max_seqs;
+  float eps;
+};
+
+constexpr int kPrepThreads = 256, kMaxRotPairs = 256;
+
+// One CTA per row.  The angle position * frequency is formed and reduced to one turn in double, so that far
+// positions lose nothing; its sine and cosine are evaluated in fp32, once per pair for all heads.
+template <typename T>
+__global__ void __launch_bounds__(kPrepThreads) latent_prepare_kernel(const PrepareParams<T> p) {
+  __shared__ float scratch[32], cs[kMaxRotPairs], sn[kMaxRotPairs];
+  const int64_t r = blockIdx.x;
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const int pos = p.row_pos[r];
+  for (int i = threadIdx.x; i < p.rot_pairs; i += kPrepThreads) {
+    const double turns = (double)pos * p.inv_freq[i] * 0.15915494309189533577;  // 1 / (2 pi)
+    const float a = (float)((turns - rint(turns)) * 6.28318530717958647692);
+    sincosf(a, &sn[i], &cs[i]);
+  }
+  __syncthreads();
+  if (p.q) {
+    const int per = p.rot_pairs, n = p.heads * per;
+    for (int i = threadIdx.x; i < n; i += kPrepThreads) {
+      const int h = i / per, j = i % per;
+      T *e = p.q + r * p.q_ld + (int64_t)h * (p.dim + p.rot_dim) + p.dim + 2 * j;
+      const float u = ldf(e), v = ldf(e + 1);
+      stf(e, u * cs[j] - v * sn[j]);
+      stf(e + 1, v * cs[j] + u * sn[j]);
+    }
+  }
+  if (p.dq) {
+    const T *src = p.dq + r * p.dq_ld;
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < p.q_rank; i += kPrepThreads) {
+      const float v = ldf(src + i);
+      sq = fmaf(v, v, sq);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)p.q_rank + p.eps);
+    for (int i = threadIdx.x; i < p.q_rank; i += kPrepThreads)
+      stf(p.cq + r * p.q_rank + i, ldf(src + i) * inv * ldf(p.dq_w + i));
+  }
+  if (p.dkv) {
+    const T *src = p.dkv + r * p.dkv_ld;
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < p.kv_rank; i += kPrepThreads) {
+      const float v = ldf(src + i);
+      sq = fmaf(v, v, sq);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)p.kv_rank + p.eps);
+    const int seq = p.row_seq[r], blk = pos / p.page_tokens;
+    if (seq < 0 || seq >= p.max_seqs || pos < 0 || blk >= p.max_blocks) {
+      if (threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_CAPACITY);
+      return;
+    }
+    const int page = p.block_table[(size_t)seq * p.max_blocks + blk];
+    if (page < 0 || page >= p.num_pages) {
+      if (threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
+      return;
+    }
+    T *dst = p.pages + ((size_t)page * p.page_tokens + pos % p.page_tokens) * (p.kv_rank + p.rot_dim);
+    for (int i = threadIdx.x; i < p.kv_rank; i += kPrepThreads) stf(dst + i, ldf(src + i) * inv * ldf(p.dkv_w + i));
+    src += p.kv_rank;
+    dst += p.kv_rank;
+    for (int j = threadIdx.x; j < p.rot_pairs; j += kPrepThreads) {
+      const float u = ldf(src + 2 * j), v = ldf(src + 2 * j + 1);
+      stf(dst + 2 * j, u * cs[j] - v * sn[j]);
+      stf(dst + 2 * j + 1, v * cs[j] + u * sn[j]);
+    }
+    for (int i = 2 * p.rot_pairs + threadIdx.x; i < p.rot_dim; i += kPrepThreads) stf(dst + i, ldf(src + i));
+  }
+}
+
+// ---- attention in latent form -------------------------------------------------------------------------
+struct AttendParams {
+  const void *q_lat;  // (rows, heads, kv_rank)
+  const void *q;      // (rows, q_ld): the rotated part of head h starts at h * (dim + rot_dim) + dim
+  int64_t q_ld;
+  void *out;  // (rows, heads, kv_rank)
+  const void *pages;
+  const int32_t *block_table, *row_seq, *row_pos;
+  int rows, heads, dim, kv_rank, rot_dim, page_tokens, max_blocks, num_pages, max_seqs, max_len;
+  float scale;
+  float *part_o, *part_ml;
+  int splits, split_tokens;
+  unsigned long long wait_ns;
+};
+
+// Keys row r may read: 0 .. row_pos[r], never beyond the block table's reach or the host's bound.
+__device__ __forceinline__ int visible_keys(const AttendParams &p, int r) {
+  const int seq = p.row_seq[r];
+  if (seq < 0 || seq >= p.max_seqs) return 0;
+  const int cover = min(p.max_blocks * p.page_tokens, p.max_len);
+  return max(0, min(p.row_pos[r] + 1, cover));
+}
+
+// Any size, fp32 or bf16: one CTA per (row, head); 64 keys at a time, one warp per key for the scores, one
+// thread per latent element for the sum.  fp32 arithmetic throughout.
+constexpr int kGenThreads = 256, kGenTile = 64;
+
+template <typename T>
+__global__ void __launch_bounds__(kGenThreads) latent_attend_generic_kernel(const AttendParams p) {
+  extern __shared__ float sm[];
+  __shared__ float scratch[32], score[kGenTile];
+  __shared__ const T *key[kGenTile];
+  const int row_elems = p.kv_rank + p.rot_dim;
+  float *q = sm, *acc = sm + row_elems;
+  const int r = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const T *ql = static_cast<const T *>(p.q_lat) + ((size_t)r * p.heads + h) * p.kv_rank;
+  const T *qr = static_cast<const T *>(p.q) + (size_t)r * p.q_ld + (size_t)h * (p.dim + p.rot_dim) + p.dim;
+  for (int i = threadIdx.x; i < row_elems; i += kGenThreads) q[i] = i < p.kv_rank ? ldf(ql + i) : ldf(qr + i - p.kv_rank);
+  for (int i = threadIdx.x; i < p.kv_rank; i += kGenThreads) acc[i] = 0.f;
+  const int keys = visible_keys(p, r);
+  const int32_t *table = p.block_table + (size_t)max(0, min(p.row_seq[r], p.max_seqs - 1)) * p.max_blocks;
+  const T *pages = static_cast<const T *>(p.pages);
+  float m = -INFINITY, l = 0.f;
+  for (int k0 = 0; k0 < keys; k0 += kGenTile) {
+    const int n = min(kGenTile, keys - k0);
+    __syncthreads();
+    if (threadIdx.x < n) {
+      const int t = k0 + threadIdx.x;
+      int page = table[t / p.page_tokens];
+      if (page < 0 || page >= p.num_pages) {
+        atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
+        page = 0;
+      }
+      key[threadIdx.x] = pages + ((size_t)page * p.page_tokens + t % p.page_tokens) * row_elems;
+    }
+    __syncthreads();
+    for (int j = warp; j < n; j += kGenThreads / 32) {
+      float s = 0.f;
+      for (int i = lane; i < row_elems; i += 32) s = fmaf(q[i], ldf(key[j] + i), s);
+      s = warp_sum(s);
+      if (lane == 0) score[j] = s * p.scale;
+    }
+    __syncthreads();
+    float mt = m;
+    for (int j = 0; j < n; ++j) mt = fmaxf(mt, score[j]);
+    const float corr = expf(m - mt);  // 0 at the first tile
+    m = mt;
+    __syncthreads();
+    if (threadIdx.x < n) score[threadIdx.x] = expf(score[threadIdx.x] - m);
+    __syncthreads();
+    l = l * corr + block_sum(threadIdx.x < n ? score[threadIdx.x] : 0.f, scratch);
+    for (int i = threadIdx.x; i < p.kv_rank; i += kGenThreads) {
+      float a = acc[i] * corr;
+      for (int j = 0; j < n; ++j) a = fmaf(score[j], ldf(key[j] + i), a);
+      acc[i] = a;
+    }
+  }
+  const float inv = l > 0.f ? 1.0f / l : 0.f;
+  T *out = static_cast<T *>(p.out) + ((size_t)r * p.heads + h) * p.kv_rank;
+  for (int i = threadIdx.x; i < p.kv_rank; i += kGenThreads) stf(out + i, acc[i] * inv);
+}
+
+// ---- gather: cached rows 0 .. n-1 of one sequence, contiguous -----------------------------------------
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint8_t *pages, const int32_t *table, uint8_t *out, int n, int row_bytes, int page_tokens,
+                     int max_blocks, int num_pages, int unit) {
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const int per = row_bytes / unit;
+  const int64_t total = (int64_t)n * per;
+  for (int64_t i = blockIdx.x * 256ll + threadIdx.x; i < total; i += gridDim.x * 256ll) {
+    const int t = (int)(i / per), c = (int)(i % per), blk = t / page_tokens;
+    const int page = blk < max_blocks ? table[blk] : -1;
+    if (page < 0 || page >= num_pages) {
+      atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
+      continue;
+    }
+    const uint8_t *src = pages + ((size_t)page * page_tokens + t % page_tokens) * row_bytes + (size_t)c * unit;
+    uint8_t *dst = out + (size_t)t * row_bytes + (size_t)c * unit;
+    if (unit == 16)
+      *reinterpret_cast<uint4 *>(dst) = *reinterpret_cast<const uint4 *>(src);
+    else
+      *reinterpret_cast<uint16_t *>(dst) = *reinterpret_cast<const uint16_t *>(src);
+  }
+}
+
+}  // namespace
+}  // namespace axb
+
+extern "C" {
+
+int axb200_latent_prepare(void *q, int64_t q_ld, int heads, int dim, const void *dq, int64_t dq_ld, int q_rank,
+                          const void *dq_w, void *cq, const void *dkv, int64_t dkv_ld, int kv_rank, const void *dkv_w,
+                          float eps, void *pages, const int32_t *block_table, const int32_t *row_seq,
+                          const int32_t *row_pos, const double *inv_freq, int rot_dim, int rot_pairs, int64_t rows,
+                          int page_tokens, int max_blocks, int num_pages, int max_seqs, int dtype, void *stream) {
+  if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
+  if (!row_pos || (rot_pairs > 0 && !inv_freq) || (dq && (!dq_w || !cq)) ||
+      (dkv && (!dkv_w || !pages || !block_table || !row_seq)))
+    return AXB200_INVALID_PTR;
+  if (rows < 0 || rows > 0x7fffffff || rot_pairs < 0 || rot_pairs > axb::kMaxRotPairs || 2 * rot_pairs > rot_dim ||
+      (q && (heads <= 0 || dim < 0)) || (dq && q_rank <= 0) ||
+      (dkv && (kv_rank <= 0 || page_tokens <= 0 || max_blocks <= 0 || num_pages <= 0 || max_seqs <= 0)))
+    return AXB200_INVALID_ARGUMENT;
+  if ((q && q_ld < (int64_t)heads * (dim + rot_dim)) || (dq && dq_ld < q_rank) || (dkv && dkv_ld < kv_rank + rot_dim))
+    return AXB200_SHAPE_MISMATCH;
+  if (rows == 0) return AXB200_OK;
+  auto go = [&](auto tag) {
+    using T = decltype(tag);
+    axb::PrepareParams<T> p{static_cast<T *>(q), q_ld, heads, dim, static_cast<const T *>(dq), dq_ld, q_rank,
+                            static_cast<const T *>(dq_w), static_cast<T *>(cq), static_cast<const T *>(dkv), dkv_ld, kv_rank,
+                            static_cast<const T *>(dkv_w), static_cast<T *>(pages), block_table, row_seq, row_pos, inv_freq,
+                            rot_dim, rot_pairs, max_blocks, page_tokens, num_pages, max_seqs, eps};
+    return axb::launch_dependent(axb::latent_prepare_kernel<T>, dim3((unsigned)rows), dim3(axb::kPrepThreads), 0,
+                                 static_cast<cudaStream_t>(stream), p);
+  };
+  return dtype == AXB200_FLOAT32 ? go(float{}) : go(__nv_bfloat16{});
+}
+
+size_t axb200_latent_attend_workspace_bytes(int rows, int heads, int kv_rank, int rot_dim, int64_t max_len, int dtype) {
+  return 0;
+}
+
+int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim, void *out, const void *pages,
+                         const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, int rows, int heads,
+                         int kv_rank, int rot_dim, float scale, int page_tokens, int max_blocks, int num_pages,
+                         int max_seqs, int64_t max_len, int dtype, void *workspace, size_t workspace_bytes, void *stream) {
+  if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
+  if (!q_lat || !q || !out || !pages || !block_table || !row_seq || !row_pos) return AXB200_INVALID_PTR;
+  if (rows < 0 || heads <= 0 || heads > 65535 || kv_rank <= 0 || rot_dim < 0 || dim < 0 || page_tokens <= 0 || max_blocks <= 0 ||
+      num_pages <= 0 || max_seqs <= 0 || max_len <= 0 || max_len > 0x7fffffff - 4096)
+    return AXB200_INVALID_ARGUMENT;
+  if (q_ld < (int64_t)heads * (dim + rot_dim)) return AXB200_SHAPE_MISMATCH;
+  if (rows == 0) return AXB200_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  axb::AttendParams p{};
+  p.q_lat = q_lat;
+  p.q = q;
+  p.q_ld = q_ld;
+  p.out = out;
+  p.pages = pages;
+  p.block_table = block_table;
+  p.row_seq = row_seq;
+  p.row_pos = row_pos;
+  p.rows = rows;
+  p.heads = heads;
+  p.dim = dim;
+  p.kv_rank = kv_rank;
+  p.rot_dim = rot_dim;
+  p.page_tokens = page_tokens;
+  p.max_blocks = max_blocks;
+  p.num_pages = num_pages;
+  p.max_seqs = max_seqs;
+  p.max_len = (int)max_len;
+  p.scale = scale;
+  p.wait_ns = axb::wait_limit_ns();
+  const size_t smem = (size_t)(2 * kv_rank + rot_dim) * sizeof(float);
+  if (smem > 200 * 1024) return AXB200_INVALID_ARGUMENT;
+  auto *kernel = dtype == AXB200_FLOAT32 ? axb::latent_attend_generic_kernel<float>
+                                         : axb::latent_attend_generic_kernel<__nv_bfloat16>;
+  if (smem > 40 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    return AXB200_DEVICE_ERROR;
+  return axb::launch_dependent(kernel, dim3(rows, heads), dim3(axb::kGenThreads), smem, st, p);
+}
+
+int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out, int64_t n, int row_elems, int page_tokens,
+                         int max_blocks, int num_pages, int dtype, void *stream) {
+  const size_t es = axb::dtype_size(dtype);
+  if (es == 0) return AXB200_UNSUPPORTED_TYPE;
+  if (!pages || !block_row || !out) return AXB200_INVALID_PTR;
+  if (n < 0 || n > (int64_t)max_blocks * page_tokens || row_elems <= 0 || page_tokens <= 0 || max_blocks <= 0 || num_pages <= 0)
+    return AXB200_INVALID_ARGUMENT;
+  if (n == 0) return AXB200_OK;
+  const int row_bytes = (int)(row_elems * es);
+  const bool vec = row_bytes % 16 == 0 && ((reinterpret_cast<uintptr_t>(pages) | reinterpret_cast<uintptr_t>(out)) & 15u) == 0;
+  const int unit = vec ? 16 : 2;
+  const int64_t items = n * (row_bytes / unit);
+  const int grid = (int)(items / 256 + 1 < 148 * 8 ? items / 256 + 1 : 148 * 8);
+  return axb::launch_dependent(axb::latent_gather_kernel, dim3(grid), dim3(256), 0, static_cast<cudaStream_t>(stream),
+                               static_cast<const uint8_t *>(pages), block_row, static_cast<uint8_t *>(out), (int)n, row_bytes,
+                               page_tokens, max_blocks, num_pages, unit);
+}
+
+}  // extern "C"

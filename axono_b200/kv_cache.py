@@ -239,6 +239,40 @@ class KVArena:
         self._h = h
         self._cache = None
 
+    @classmethod
+    def of_rows(cls, row_elems, num_pages, max_seqs, max_seq_len, dtype=torch.bfloat16, page_tokens=64, device_memory=True):
+        """An arena whose layer l caches one row of row_elems[l] elements per token, with no value pool (latent
+        caches); `row_pages(l)` and `table()` are its device memory."""
+        a = cls.__new__(cls)
+        a.n_layers, a.num_pages, a.n_kv_heads, a.head_dim = len(row_elems), num_pages, 1, row_elems[0]
+        a.row_elems = list(row_elems)
+        a.max_seqs, a.page_tokens, a.dtype = max_seqs, page_tokens, dtype
+        a.max_blocks = (max_seq_len + page_tokens - 1) // page_tokens
+        a.device_memory = device_memory
+        code = {torch.bfloat16: _capi.BFLOAT16, torch.float16: _capi.FLOAT16, torch.float32: _capi.FLOAT32}[dtype]
+        h = C.c_void_p()
+        _capi.check(_capi.lib().axb200_kv_arena_create_rows(len(row_elems), (C.c_int32 * len(row_elems))(*row_elems), num_pages,
+                                                            page_tokens, code, max_seqs, a.max_blocks, int(device_memory),
+                                                            C.byref(h)), "kv_arena_create_rows")
+        a._h, a._cache = h, None
+        return a
+
+    def row_pages(self, layer: int):
+        """Layer `layer`'s pool (num_pages, page_tokens, row_elems[layer]) of an arena of rows."""
+        view = {torch.bfloat16: "<i2", torch.float16: "<f2", torch.float32: "<f4"}[self.dtype]
+        ptr = _capi.lib().axb200_kv_arena_k_pages(self._h, layer)
+        t = torch.as_tensor(_DeviceView(ptr, (self.num_pages, self.page_tokens, self.row_elems[layer]), view),
+                            device=torch.device("cuda", torch.cuda.current_device()))
+        return t.view(torch.bfloat16) if self.dtype == torch.bfloat16 else t
+
+    def table(self):
+        """The device block table (max_seqs, max_blocks), refreshed by `sync()`."""
+        return torch.as_tensor(_DeviceView(_capi.lib().axb200_kv_arena_block_table(self._h), (self.max_seqs, self.max_blocks),
+                                           "<i4"), device=torch.device("cuda", torch.cuda.current_device()))
+
+    def shuffle_free(self, seed: int) -> None:
+        _capi.check(_capi.lib().axb200_kv_arena_shuffle_free(self._h, seed), "kv_arena_shuffle_free")
+
     def _stream(self):
         return torch.cuda.current_stream().cuda_stream if self.device_memory else None
 

@@ -510,7 +510,7 @@ def concat(a, b, axis: int):
 def embedding(ids, table):
     """table[ids]: ids int32/int64 of any shape, table (vocab, hidden) -> ids.shape + (hidden,)."""
     op = "embedding"
-    dt = _dt(table, op)
+    dt = _capi.BFLOAT16 if table.is_cuda and table.dtype == torch.bfloat16 else _dt(table, op)
     if table.dim() != 2 or ids.dim() < 1:
         _capi.check(1, op)
     code = {torch.int64: _capi.INT64, torch.int32: _capi.INT32}.get(ids.dtype)
@@ -556,3 +556,202 @@ def scaled_dot_product_attention(q, k, v, is_causal: bool = False):
     _call(lib.axb200_sdpa(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), sq, hq, hkv, d, skv,
                           int(bool(is_causal)), dt, ws.data_ptr(), ws.numel(), _stream(q)), op)
     return out
+
+
+# ---- operators of the language models (fp32 or bf16; residual, scores, norms and routers in fp32) -----------
+_LM_DTYPES = {torch.bfloat16: _capi.BFLOAT16, torch.float32: _capi.FLOAT32}
+
+
+def _lm_dt(t: torch.Tensor, op: str) -> int:
+    if not t.is_cuda:
+        raise RuntimeError(f"{op}: expected a CUDA tensor (this package has no CPU path)")
+    code = _LM_DTYPES.get(t.dtype)
+    if code is None:
+        _capi.check(3, op)  # UNSUPPORTED_TYPE
+    return code
+
+
+def linear(x, weight, out_dtype=None):
+    """x (rows, in), rows may be strided, . weight (out, in)^T -> (rows, out) of out_dtype (x's type or fp32)."""
+    op = "linear"
+    dt = _lm_dt(x, op)
+    if x.dim() != 2 or weight.dim() != 2 or x.shape[1] != weight.shape[1] or weight.dtype != x.dtype or x.stride(1) != 1:
+        _capi.check(4, op)
+    rows, k = x.shape
+    n = weight.shape[0]
+    out = torch.empty((rows, n), dtype=out_dtype or x.dtype, device=x.device)
+    if rows:
+        _call(_capi.lib().axb200_linear_strided(x.data_ptr(), weight.data_ptr(), out.data_ptr(), rows, n, k, x.stride(0),
+                                                weight.stride(0), n, 1, 0, 0, 0, 0, dt, _LM_DTYPES[out.dtype], _stream(x)), op)
+    return out
+
+
+def linear_heads(x, x_ld, x_stride, weight, out, rows, in_major):
+    """One product per head: out[:, h] (rows, heads, n) = x_h . weight[h]^T, where x_h (rows, k) starts
+    h * x_stride elements into x with row stride x_ld; weight (heads, n, k), or (heads, k, n) with in_major."""
+    op = "linear_heads"
+    dt = _lm_dt(x, op)
+    heads, n = out.shape[1], out.shape[2]
+    k = weight.shape[1] if in_major else weight.shape[2]
+    if weight.shape[0] != heads or weight.shape[2 if in_major else 1] != n or out.dtype != x.dtype:
+        _capi.check(4, op)
+    if rows:
+        _call(_capi.lib().axb200_linear_strided(
+            x.data_ptr(), weight.data_ptr(), out.data_ptr(), rows, n, k, x_ld, weight.shape[2], heads * n, heads, x_stride,
+            n * k, n, int(in_major), dt, dt, _stream(x)), op)
+    return out
+
+
+def embed_layer_norm(ids, table, weight, eps):
+    """layer_norm(table[ids]) * weight as the fp32 residual stream (n, width)."""
+    op = "embed_layer_norm"
+    dt = _lm_dt(table, op)
+    if ids.dtype != torch.int64 or weight.dtype != table.dtype:
+        _capi.check(3, op)
+    x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    _call(_capi.lib().axb200_embed_layer_norm(ids.data_ptr(), table.data_ptr(), weight.data_ptr(), float(eps), x.data_ptr(),
+                                              ids.numel(), table.shape[0], table.shape[1], dt, _stream(table)), op)
+    return x
+
+
+def residual_layer_norm(x, w1, w2, eps, a=None, b=None, experts=None):
+    """x (rows, width) fp32 += a + b + sum of the routed experts' rows, in place; returns (h1, h2), the layer norm of
+    the new x times w1 and w2 (None where the weight is None).  experts = (rows, slot, weight) of `MoE`."""
+    op = "residual_layer_norm"
+    dt = _lm_dt(w1 if w1 is not None else w2, op)
+    dtype = (w1 if w1 is not None else w2).dtype
+    for t in (a, b, w2, experts[0] if experts is not None else None):
+        if t is not None and (t.dtype != dtype or not t.is_contiguous()):
+            _capi.check(3, op)
+    h1 = torch.empty(x.shape, dtype=dtype, device=x.device) if w1 is not None else None
+    h2 = torch.empty(x.shape, dtype=dtype, device=x.device) if w2 is not None else None
+    er, slot, weight = experts if experts is not None else (None, None, None)
+    _call(_capi.lib().axb200_residual_layer_norm(
+        x.data_ptr(), _ptr(a), _ptr(b), _ptr(er), _ptr(slot), _ptr(weight), slot.shape[1] if slot is not None else 0, _ptr(w1),
+        _ptr(h1), _ptr(w2), _ptr(h2), float(eps), x.shape[0], x.shape[1], dt, _stream(x)), op)
+    return h1, h2
+
+
+def latent_prepare(rows, inv_freq, rot_dim, q=None, heads=0, dim=0, dq=None, dq_weight=None, dkv=None, dkv_weight=None,
+                   pages=None, eps=1e-5):
+    """The step's norms, rotation and append of latent attention in one launch; each of q (rows, >= heads *
+    (dim + rot_dim)), dq (rows, q_rank) and dkv (rows, kv_rank + rot_dim) is optional and may be a column slice of
+    a wider matrix.  q is rotated in place; returns the normed query latent (or None)."""
+    op = "latent_prepare"
+    ref = next(t for t in (q, dq, dkv) if t is not None)
+    dt = _lm_dt(ref, op)
+    for t in (q, dq, dkv):
+        if t is not None and (t.dim() != 2 or t.stride(1) != 1 or t.dtype != ref.dtype):
+            _capi.check(4, op)
+    n = ref.shape[0]
+    cq = torch.empty((n, dq.shape[1]), dtype=ref.dtype, device=ref.device) if dq is not None else None
+    ld = lambda t: t.stride(0) if t is not None else 0  # noqa: E731
+    geo = (pages.shape[1], rows.block_table.shape[1], pages.shape[0]) if pages is not None else (1, 1, 1)
+    _call(_capi.lib().axb200_latent_prepare(
+        _ptr(q), ld(q), heads, dim, _ptr(dq), ld(dq), dq.shape[1] if dq is not None else 0, _ptr(dq_weight), _ptr(cq),
+        _ptr(dkv), ld(dkv), dkv.shape[1] - rot_dim if dkv is not None else 0, _ptr(dkv_weight), float(eps), _ptr(pages),
+        rows.block_table.data_ptr(), rows.seq.data_ptr(), rows.pos.data_ptr(), inv_freq.data_ptr(), rot_dim,
+        inv_freq.numel(), n, *geo, rows.block_table.shape[0], dt, _stream(ref)), op)
+    return cq
+
+
+def latent_attend(q_lat, q, dim, rot_dim, scale, pages, rows, n):
+    """Latent attention of the first n rows: q_lat (n, heads, kv_rank), the rotated query parts inside q (strided
+    rows of heads x (dim + rot_dim)) -> (n, heads, kv_rank)."""
+    op = "latent_attend"
+    dt = _lm_dt(q_lat, op)
+    heads, rank = q_lat.shape[1], q_lat.shape[2]
+    out = torch.empty_like(q_lat)
+    lib = _capi.lib()
+    ws = workspace(q.device, lib.axb200_latent_attend_workspace_bytes(n, heads, rank, rot_dim, rows.max_len, dt))
+    _call(lib.axb200_latent_attend(
+        q_lat.data_ptr(), q.data_ptr(), q.stride(0), dim, out.data_ptr(), pages.data_ptr(), rows.block_table.data_ptr(),
+        rows.seq.data_ptr(), rows.pos.data_ptr(), n, heads, rank, rot_dim, float(scale), pages.shape[1],
+        rows.block_table.shape[1], pages.shape[0], rows.block_table.shape[0], int(rows.max_len), dt, ws.data_ptr(), ws.numel(),
+        _stream(q)), op)
+    return out
+
+
+def latent_gather(pages, block_row, n):
+    """The first n cached rows of the sequence whose block-table row is block_row, contiguous."""
+    op = "latent_gather"
+    out = torch.empty((n, pages.shape[2]), dtype=pages.dtype, device=pages.device)
+    _call(_capi.lib().axb200_latent_gather(pages.data_ptr(), block_row.data_ptr(), out.data_ptr(), n, pages.shape[2],
+                                           pages.shape[1], block_row.numel(), pages.shape[0], _lm_dt(pages, op), _stream(pages)), op)
+    return out
+
+
+def latent_prefill_supported(heads, dim, rot_dim, vdim, dtype) -> bool:
+    return bool(_capi.lib().axb200_latent_prefill_supported(heads, dim, rot_dim, vdim, _LM_DTYPES[dtype]))
+
+
+def latent_prefill(q, start, k, v, rot, heads, dim, rot_dim, vdim, scale):
+    """Expanded form of one sequence's portion: q (n, >= heads * (dim + rot_dim)) at positions start.., k (start + n,
+    heads * dim), v (start + n, heads * vdim), rot (start + n, rot_dim), strided rows -> (n, heads * vdim)."""
+    op = "latent_prefill"
+    dt = _lm_dt(q, op)
+    n = q.shape[0]
+    if k.shape[0] != start + n or v.shape[0] != start + n or rot.shape[0] != start + n or not (k.is_contiguous() and v.is_contiguous()):
+        _capi.check(4, op)
+    out = torch.empty((n, heads * vdim), dtype=q.dtype, device=q.device)
+    _call(_capi.lib().axb200_latent_prefill(q.data_ptr(), q.stride(0), k.data_ptr(), v.data_ptr(), rot.data_ptr(), rot.stride(0),
+                                            out.data_ptr(), n, int(start), heads, dim, rot_dim, vdim, float(scale), dt,
+                                            _stream(q)), op)
+    return out
+
+
+def moe_route(logits, correction, groups, keep, top, scale):
+    """Grouped top-k routing over sigmoid scores: (ids, weights, place, counts) of axb200_moe_route."""
+    op = "moe_route"
+    n, experts = logits.shape
+    ids = torch.empty((n, top), dtype=torch.int32, device=logits.device)
+    place = torch.empty_like(ids)
+    weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
+    counts = torch.empty((experts,), dtype=torch.int32, device=logits.device)
+    if logits.dtype != torch.float32 or (correction is not None and correction.dtype != torch.float32):
+        _capi.check(3, op)
+    _call(_capi.lib().axb200_moe_route(logits.data_ptr(), _ptr(correction), ids.data_ptr(), weights.data_ptr(), place.data_ptr(),
+                                       counts.data_ptr(), n, experts, groups, keep, top, float(scale), _stream(logits)), op)
+    return ids, weights, place, counts
+
+
+def moe_tile_rows(rows, experts, width, ff, dtype) -> int:
+    return int(_capi.lib().axb200_moe_tile_rows(rows, experts, width, ff, _LM_DTYPES[dtype]))
+
+
+def moe_sort(x, ids, place, counts, tile_rows):
+    """Rows of x once per chosen expert, in expert order: (sorted, row_of, offsets, tiles, n_tiles)."""
+    op = "moe_sort"
+    n, top = ids.shape
+    experts = counts.numel()
+    srt = torch.empty((n * top, x.shape[1]), dtype=x.dtype, device=x.device)
+    row_of = torch.empty_like(ids)
+    ints = lambda *s: torch.empty(s, dtype=torch.int32, device=x.device)  # noqa: E731
+    offsets, tiles, n_tiles = ints(experts + 1), ints(n * top // tile_rows + min(experts, n * top), 4), ints(1)
+    _call(_capi.lib().axb200_moe_sort(x.data_ptr(), srt.data_ptr(), ids.data_ptr(), place.data_ptr(), counts.data_ptr(),
+                                      row_of.data_ptr(), offsets.data_ptr(), tiles.data_ptr(), n_tiles.data_ptr(), n, experts, top,
+                                      tile_rows, x.shape[1], _lm_dt(x, op), _stream(x)), op)
+    return srt, row_of, offsets, tiles, n_tiles
+
+
+def moe_gate_up(x, weight, limit, slope=1.702, offset=1.0, tiles=None, n_tiles=None, tile_rows=0):
+    """Gate, up and clamped-gate activation of every row's expert: weight (experts, 2, ff, width) -> (rows, ff)."""
+    op = "moe_gate_up"
+    experts, _, ff, width = weight.shape
+    act = torch.empty((x.shape[0], ff), dtype=x.dtype, device=x.device)
+    dt = _lm_dt(x, op)
+    tile_rows = tile_rows or moe_tile_rows(x.shape[0], 1, width, ff, x.dtype)
+    _call(_capi.lib().axb200_moe_gate_up(x.data_ptr(), weight.data_ptr(), act.data_ptr(), _ptr(tiles), _ptr(n_tiles), x.shape[0],
+                                         experts, width, ff, tile_rows, float(limit), float(slope), float(offset), dt, _stream(x)), op)
+    return act
+
+
+def moe_down(act, weight, tiles=None, n_tiles=None, tile_rows=0):
+    """Down product of every row's expert: weight (experts, width, ff) -> (rows, width)."""
+    op = "moe_down"
+    experts, width, ff = weight.shape
+    y = torch.empty((act.shape[0], width), dtype=act.dtype, device=act.device)
+    tile_rows = tile_rows or moe_tile_rows(act.shape[0], 1, width, ff, act.dtype)
+    _call(_capi.lib().axb200_moe_down(act.data_ptr(), weight.data_ptr(), y.data_ptr(), _ptr(tiles), _ptr(n_tiles), act.shape[0],
+                                      experts, width, ff, tile_rows, _lm_dt(act, op), _stream(act)), op)
+    return y

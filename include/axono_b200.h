@@ -45,7 +45,8 @@ enum {
   AXB200_FLOAT16 = 4,
   AXB200_FLOAT32 = 5,
   AXB200_FLOAT64 = 6,
-  AXB200_BOOLEAN = 7
+  AXB200_BOOLEAN = 7,
+  AXB200_BFLOAT16 = 8  /* extension: no value of the reference's enum; the language-model operators take it */
 };
 
 /* Bits of the device error word returned by axb200_last_error(). */
@@ -463,6 +464,94 @@ int axb200_randn(void *out, int64_t n, int dtype, float mean, float stddev, uint
 int axb200_linear_nobias(const void *x, const void *w, void *out, int64_t rows, int64_t out_features,
                          int64_t in_features, int dtype, void *stream);
 
+/* The general form of that call: `batch` products out[b] = x[b] . w[b]^T with row strides (x_ld, w_ld, out_ld)
+ * and batch strides in elements, w[b] stored (out_features, in_features) or, with w_in_major,
+ * (in_features, out_features); FLOAT16, BFLOAT16 or FLOAT32 operands (FLOAT32 in full fp32 arithmetic), result
+ * in the same type or FLOAT32.  Candidates are timed up to 512 rows; above that the heuristic's first choice
+ * is taken, since prompts come in every length.  No counterpart in the reference. */
+int axb200_linear_strided(const void *x, const void *w, void *out, int64_t rows, int64_t out_features,
+                          int64_t in_features, int64_t x_ld, int64_t w_ld, int64_t out_ld, int64_t batch,
+                          int64_t x_stride, int64_t w_stride, int64_t out_stride, int w_in_major, int dtype,
+                          int out_dtype, void *stream);
+
+/* ---- residual stream in fp32 with layer norms --------------------------------------------------------
+ * For decoders outside the reference's models: FLOAT32 or BFLOAT16 activations and weights (`dtype`), the
+ * residual x always fp32 (rows, width).  Layer norm: (x - mean) / sqrt(mean((x - mean)^2) + eps) * w, no bias.
+ *   embed_layer_norm: x = layer_norm(table[ids]) * weight; an id outside the table sets AXB200_ERR_BAD_INDEX
+ *     and counts as a zero row.
+ *   residual_layer_norm: x += a + b + sum_k weight[r, k] * expert_rows[slot[r, k]] (each addend optional), then
+ *     h1 = layer_norm(x) * w1 and h2 = layer_norm(x) * w2 (each optional).  One launch between two layers. */
+int axb200_embed_layer_norm(const int64_t *ids, const void *table, const void *weight, float eps, float *x,
+                            int64_t n, int64_t vocab, int width, int dtype, void *stream);
+int axb200_residual_layer_norm(float *x, const void *a, const void *b, const void *expert_rows,
+                               const int32_t *slot, const float *weight, int top, const void *w1, void *h1,
+                               const void *w2, void *h2, float eps, int64_t rows, int width, int dtype,
+                               void *stream);
+
+/* ---- latent attention ----------------------------------------------------------------------------------
+ * Attention whose cache holds one row [c (kv_rank) | rotated key part (rot_dim)] per token, shared by all heads:
+ * head h's key is [W_uk c | rotated part], its value W_uv c.  Row r of a launch belongs to sequence
+ * row_seq[r] (row of block_table) and stands at position row_pos[r]; pages (num_pages, page_tokens,
+ * kv_rank + rot_dim).  FLOAT32 or BFLOAT16; scores, weights and sums in fp32.
+ *
+ *   latent_prepare: per row, any of: rotate the last rot_dim elements of every head of q (rows, q_ld) in place
+ *     (heads of [dim | rot_dim]); cq = rms_norm(dq) * dq_w over q_rank; append [rms_norm(dkv[:kv_rank]) * dkv_w |
+ *     rotate(dkv[kv_rank:])] at the row's position.  Rotation turns the pairs (2i, 2i + 1), i < rot_pairs, by
+ *     position * inv_freq[i] (device, double); elements past 2 * rot_pairs pass unchanged.
+ *   latent_attend: out (rows, heads, kv_rank) = sum over j <= row_pos[r] of softmax((q_lat . c_j +
+ *     q_rot . rot_j) * scale) c_j, with q_lat (rows, heads, kv_rank) = q . W_uk and q_rot read from q.
+ *     max_len bounds row_pos + 1 and sizes the grid.
+ *   latent_gather: rows 0 .. n-1 of one sequence's pages, contiguous.
+ *   latent_prefill: the expanded form for n rows of ONE sequence at positions start .. start + n - 1: q (n, q_ld)
+ *     rotated, k (skv, heads * dim) and v (skv, heads * vdim) expanded from the latents of positions 0 .. skv - 1
+ *     (skv = start + n), rot = the rotated key parts, row stride rot_ld; out (n, heads, vdim).  BFLOAT16 on
+ *     tcgen05; latent_prefill_supported tells which sizes. */
+int axb200_latent_prepare(void *q, int64_t q_ld, int heads, int dim, const void *dq, int64_t dq_ld, int q_rank,
+                          const void *dq_w, void *cq, const void *dkv, int64_t dkv_ld, int kv_rank,
+                          const void *dkv_w, float eps, void *pages, const int32_t *block_table,
+                          const int32_t *row_seq, const int32_t *row_pos, const double *inv_freq, int rot_dim,
+                          int rot_pairs, int64_t rows, int page_tokens, int max_blocks, int num_pages, int max_seqs,
+                          int dtype, void *stream);
+size_t axb200_latent_attend_workspace_bytes(int rows, int heads, int kv_rank, int rot_dim, int64_t max_len, int dtype);
+int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim, void *out, const void *pages,
+                         const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, int rows,
+                         int heads, int kv_rank, int rot_dim, float scale, int page_tokens, int max_blocks,
+                         int num_pages, int max_seqs, int64_t max_len, int dtype, void *workspace,
+                         size_t workspace_bytes, void *stream);
+int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out, int64_t n, int row_elems,
+                         int page_tokens, int max_blocks, int num_pages, int dtype, void *stream);
+int axb200_latent_prefill_supported(int heads, int dim, int rot_dim, int vdim, int dtype);
+int axb200_latent_prefill(const void *q, int64_t q_ld, const void *k, const void *v, const void *rot, int64_t rot_ld,
+                          void *out, int n, int64_t start, int heads, int dim, int rot_dim, int vdim, float scale,
+                          int dtype, void *stream);
+
+/* ---- mixture of experts ---------------------------------------------------------------------------------
+ *   moe_route: per token, scores s = sigmoid(logits), choices s + correction; the experts form `groups` equal
+ *     groups of neighbours, a group is worth its two largest choices, only the best `keep` groups are open;
+ *     the `top` largest choices among their experts are taken.  ids, weights = s * scale, place (rows, top);
+ *     counts (experts).
+ *   moe_tile_rows: rows per tile the products want for this many routed rows.
+ *   moe_sort: copies each token's row once per chosen expert into `sorted` (rows * top, width), in expert order;
+ *     row_of (rows, top) = where; offsets (experts + 1); tiles (at most rows * top / tile_rows +
+ *     min(experts, rows * top) entries of int32 x 4), n_tiles (1).
+ *   moe_gate_up: act (rows, ff) = g * sigmoid(slope * g) * (u + offset), g = min(x . W_gate^T, limit),
+ *     u = clamp(x . W_up^T, -limit, limit); w (experts, 2, ff, width) = gate, up.
+ *   moe_down: y (rows, width) = act . W_down^T; w (experts, width, ff).
+ * In the products `rows` counts rows of x; tiles == NULL means one expert over all rows.  FLOAT32, or BFLOAT16
+ * with fp32 accumulation (tcgen05 when width and ff are multiples of 8).  No counterparts in the reference. */
+int axb200_moe_route(const float *logits, const float *correction, int32_t *ids, float *weights, int32_t *place,
+                     int32_t *counts, int64_t rows, int experts, int groups, int keep, int top, float scale,
+                     void *stream);
+int axb200_moe_tile_rows(int64_t rows, int experts, int width, int ff, int dtype);
+int axb200_moe_sort(const void *x, void *sorted, const int32_t *ids, const int32_t *place, const int32_t *counts,
+                    int32_t *row_of, int32_t *offsets, int32_t *tiles, int32_t *n_tiles, int64_t rows, int experts,
+                    int top, int tile_rows, int width, int dtype, void *stream);
+int axb200_moe_gate_up(const void *x, const void *w, void *act, const int32_t *tiles, const int32_t *n_tiles,
+                       int64_t rows, int experts, int width, int ff, int tile_rows, float limit, float slope,
+                       float offset, int dtype, void *stream);
+int axb200_moe_down(const void *act, const void *w, void *y, const int32_t *tiles, const int32_t *n_tiles,
+                    int64_t rows, int experts, int width, int ff, int tile_rows, int dtype, void *stream);
+
 /* axono::ops::cuda::Concat, src/ops/cuda/sequence.cu:474-521, on bytes: out (outer, a_bytes +
  * b_bytes) = a (outer, a_bytes) ++ b (outer, b_bytes).  Axis 0 is outer == 1. */
 int axb200_concat(const void *a, const void *b, void *out, int64_t outer,
@@ -481,6 +570,10 @@ int axb200_concat(const void *a, const void *b, void *out, int64_t outer,
 typedef struct axb200_kv_arena axb200_kv_arena;
 int axb200_kv_arena_create(int n_layers, int num_pages, int hkv, int page_tokens, int d, int dtype,
                            int max_seqs, int max_blocks, int device_memory, axb200_kv_arena **out);
+/* An arena whose layers hold one row of row_elems[l] elements per token and no V pool (latent caches): k_pages
+ * gives the pool (num_pages, page_tokens, row_elems[l]).  Everything else is the same. */
+int axb200_kv_arena_create_rows(int n_layers, const int32_t *row_elems, int num_pages, int page_tokens, int dtype,
+                                int max_seqs, int max_blocks, int device_memory, axb200_kv_arena **out);
 int axb200_kv_arena_destroy(axb200_kv_arena *arena);
 /* Takes the lowest free sequence slot and pages for reserve_tokens; OUT_OF_MEMORY when slots or
  * pages run out (nothing is taken then). */
