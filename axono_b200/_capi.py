@@ -106,8 +106,8 @@ SIGNATURES = {
     "axb200_moe_route": (_i, [_vp] * 6 + [_i64, _i, _i, _i, _i, _f, _vp]),
     "axb200_moe_tile_rows": (_i, [_i64, _i, _i, _i, _i]),
     "axb200_moe_sort": (_i, [_vp] * 9 + [_i64, _i, _i, _i, _i, _i, _vp]),
-    "axb200_moe_gate_up": (_i, [_vp] * 5 + [_i64, _i, _i, _i, _i, _f, _f, _f, _i, _vp]),
-    "axb200_moe_down": (_i, [_vp] * 5 + [_i64, _i, _i, _i, _i, _i, _vp]),
+    "axb200_moe_gate_up": (_i, [_vp] * 5 + [_i64, _i, _i, _f, _vp, _vp, _vp, _i64, _i, _f, _i, _i, _f, _f, _i, _vp]),
+    "axb200_moe_down": (_i, [_vp] * 5 + [_i64, _i, _i, _vp, _vp, _vp, _i64, _i, _i, _i, _i, _vp]),
     "axb200_randn": (_i, [_vp, _i64, _i, _f, _f, C.c_uint64, _vp]),
     "axb200_cast": (_i, [_vp, _i, _vp, _i, _i64, _vp]),
     "axb200_concat": (_i, [_vp, _vp, _vp, _i64, _sz, _sz, _vp]),

@@ -217,22 +217,39 @@ int launch_generic(const MoeProduct &p, bool gate_up, cudaStream_t st) {
                  : launch_dependent(moe_product_generic_kernel<T, false>, grid, dim3(kGenThreads), 0, st, p);
 }
 
-int product(const MoeProduct &q, bool gate_up, int dtype, void *stream) {
-  if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
-  if (!q.x || !q.w || !q.y || (q.tiles && !q.n_tiles)) return AXB200_INVALID_PTR;
-  if (q.rows < 0 || q.experts <= 0 || q.in <= 0 || q.out <= 0 || q.tile_rows <= 0 || (!q.tiles && q.experts != 1))
-    return AXB200_INVALID_ARGUMENT;
-  if (q.rows == 0) return AXB200_OK;
-  MoeProduct p = q;
+// The grid bound of a product, in tiles; < 0: invalid.
+int check_product(MoeProduct &p) {
+  if (!p.x || !p.w || !p.y || (p.tiles && !p.n_tiles)) return -AXB200_INVALID_PTR;
+  if (p.rows <= 0 || p.experts <= 0 || p.in <= 0 || p.out <= 0 || p.tile_rows <= 0 || (!p.tiles && p.experts != 1))
+    return -AXB200_INVALID_ARGUMENT;
   const int64_t bound = p.tiles ? (int64_t)p.rows / p.tile_rows + (p.experts < p.rows ? p.experts : p.rows)
                                 : ((int64_t)p.rows + p.tile_rows - 1) / p.tile_rows;
-  if (bound > 65535) return AXB200_INVALID_ARGUMENT;
+  if (bound > 65535) return -AXB200_INVALID_ARGUMENT;
   p.max_tiles = (int)bound;
   p.wait_ns = wait_limit_ns();
+  return AXB200_OK;
+}
+
+int products(MoeProduct routed, MoeProduct shared, bool gate_up, int dtype, void *stream) {
+  if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
+  if (routed.rows == 0 && shared.rows == 0) return AXB200_OK;
+  int rc = check_product(routed);
+  if (rc == AXB200_OK && shared.rows > 0) rc = check_product(shared);
+  if (rc != AXB200_OK) return -rc;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dtype == AXB200_BFLOAT16 && moe_umma_supported(p, gate_up)) return moe_umma(p, gate_up, st);
-  if (p.tile_rows > kGenRows) return AXB200_INVALID_ARGUMENT;
-  return dtype == AXB200_FLOAT32 ? launch_generic<float>(p, gate_up, st) : launch_generic<__nv_bfloat16>(p, gate_up, st);
+  const bool umma = dtype == AXB200_BFLOAT16 && moe_umma_supported(routed, gate_up);
+  if (umma && (shared.rows == 0 || moe_umma_supported(shared, gate_up))) return moe_umma(routed, shared, gate_up, st);
+  if (umma) {
+    rc = moe_umma(routed, MoeProduct{}, gate_up, st);
+  } else {
+    if (routed.tile_rows > kGenRows) return AXB200_INVALID_ARGUMENT;
+    rc = dtype == AXB200_FLOAT32 ? launch_generic<float>(routed, gate_up, st) : launch_generic<__nv_bfloat16>(routed, gate_up, st);
+  }
+  if (rc != AXB200_OK || shared.rows == 0) return rc;
+  shared.tile_rows = kGenRows;
+  rc = check_product(shared);
+  if (rc != AXB200_OK) return -rc;
+  return dtype == AXB200_FLOAT32 ? launch_generic<float>(shared, gate_up, st) : launch_generic<__nv_bfloat16>(shared, gate_up, st);
 }
 
 }  // namespace
@@ -284,23 +301,30 @@ int axb200_moe_sort(const void *x, void *sorted, const int32_t *ids, const int32
 }
 
 int axb200_moe_gate_up(const void *x, const void *w, void *act, const int32_t *tiles, const int32_t *n_tiles, int64_t rows,
-                       int experts, int width, int ff, int tile_rows, float limit, float slope, float offset, int dtype,
-                       void *stream) {
-  axb::MoeProduct p{};
+                       int experts, int ff, float limit, const void *shared_x, const void *shared_w, void *shared_act,
+                       int64_t shared_rows, int shared_ff, float shared_limit, int width, int tile_rows, float slope,
+                       float offset, int dtype, void *stream) {
+  if (rows < 0 || rows > 0x7fffffff || shared_rows < 0 || shared_rows > 0x7fffffff) return AXB200_INVALID_ARGUMENT;
+  axb::MoeProduct p{}, s{};
   p.x = x, p.w = w, p.y = act, p.tiles = reinterpret_cast<const int4 *>(tiles), p.n_tiles = n_tiles;
-  if (rows > 0x7fffffff) return AXB200_INVALID_ARGUMENT;
   p.rows = (int)rows, p.experts = experts, p.in = width, p.out = ff, p.tile_rows = tile_rows;
   p.act = {limit, slope, offset};
-  return axb::product(p, true, dtype, stream);
+  s.x = shared_x, s.w = shared_w, s.y = shared_act, s.rows = (int)shared_rows, s.experts = 1, s.in = width, s.out = shared_ff;
+  s.tile_rows = tile_rows;
+  s.act = {shared_limit, slope, offset};
+  return axb::products(p, s, true, dtype, stream);
 }
 
 int axb200_moe_down(const void *act, const void *w, void *y, const int32_t *tiles, const int32_t *n_tiles, int64_t rows,
-                    int experts, int width, int ff, int tile_rows, int dtype, void *stream) {
-  axb::MoeProduct p{};
+                    int experts, int ff, const void *shared_act, const void *shared_w, void *shared_y, int64_t shared_rows,
+                    int shared_ff, int width, int tile_rows, int dtype, void *stream) {
+  if (rows < 0 || rows > 0x7fffffff || shared_rows < 0 || shared_rows > 0x7fffffff) return AXB200_INVALID_ARGUMENT;
+  axb::MoeProduct p{}, s{};
   p.x = act, p.w = w, p.y = y, p.tiles = reinterpret_cast<const int4 *>(tiles), p.n_tiles = n_tiles;
-  if (rows > 0x7fffffff) return AXB200_INVALID_ARGUMENT;
   p.rows = (int)rows, p.experts = experts, p.in = ff, p.out = width, p.tile_rows = tile_rows;
-  return axb::product(p, false, dtype, stream);
+  s.x = shared_act, s.w = shared_w, s.y = shared_y, s.rows = (int)shared_rows, s.experts = 1, s.in = shared_ff, s.out = width;
+  s.tile_rows = tile_rows;
+  return axb::products(p, s, false, dtype, stream);
 }
 
 }  // extern "C"

@@ -49,6 +49,7 @@ __device__ __forceinline__ bool moe_tile(const MoeProduct &p, int t, int tile_ro
 bool moe_umma_takes(int width, int ff);
 int moe_umma_tile_rows(int64_t rows, int experts);
 bool moe_umma_supported(const MoeProduct &p, bool gate_up);
-int moe_umma(const MoeProduct &p, bool gate_up, cudaStream_t st);
+// Both in one launch; shared.rows == 0: no shared expert.
+int moe_umma(const MoeProduct &routed, const MoeProduct &shared, bool gate_up, cudaStream_t st);
 
 }  // namespace axb

@@ -126,10 +126,10 @@ class MixtureOfExperts:
         experts, _, ff, width = self.gate_up.shape
         tile = ops.moe_tile_rows(h.shape[0] * ids.shape[1], experts, width, ff, h.dtype)
         srt, row_of, _, tiles, n_tiles = ops.moe_sort(h, ids, place, counts, tile)
-        act = ops.moe_gate_up(srt, self.gate_up, self.limit, self.slope, self.offset, tiles, n_tiles, tile)
-        y = ops.moe_down(act, self.down, tiles, n_tiles, tile)
-        shared = None
-        if self.shared_gate_up is not None:
-            shared = ops.moe_down(ops.moe_gate_up(h, self.shared_gate_up, self.shared_limit, self.slope, self.offset),
-                                  self.shared_down)
+        has_shared = self.shared_gate_up is not None
+        act, shared_act = ops.moe_gate_up(srt, self.gate_up, self.limit, tiles, n_tiles, tile,
+                                          (h, self.shared_gate_up, self.shared_limit) if has_shared else None, self.slope,
+                                          self.offset)
+        y, shared = ops.moe_down(act, self.down, tiles, n_tiles, tile,
+                                 (shared_act, self.shared_down) if has_shared else None)
         return (y, row_of, weights), shared

@@ -734,24 +734,32 @@ def moe_sort(x, ids, place, counts, tile_rows):
     return srt, row_of, offsets, tiles, n_tiles
 
 
-def moe_gate_up(x, weight, limit, slope=1.702, offset=1.0, tiles=None, n_tiles=None, tile_rows=0):
-    """Gate, up and clamped-gate activation of every row's expert: weight (experts, 2, ff, width) -> (rows, ff)."""
+def moe_gate_up(x, weight, limit, tiles, n_tiles, tile_rows, shared=None, slope=1.702, offset=1.0):
+    """Gate, up and clamped-gate activation of every routed row's expert: weight (experts, 2, ff, width) -> (rows, ff).
+    shared = (x, weight (1, 2, ff, width), limit): one more expert over all rows of its x, in the same launch; returns
+    (routed, shared) activations."""
     op = "moe_gate_up"
     experts, _, ff, width = weight.shape
-    act = torch.empty((x.shape[0], ff), dtype=x.dtype, device=x.device)
-    dt = _lm_dt(x, op)
-    tile_rows = tile_rows or moe_tile_rows(x.shape[0], 1, width, ff, x.dtype)
-    _call(_capi.lib().axb200_moe_gate_up(x.data_ptr(), weight.data_ptr(), act.data_ptr(), _ptr(tiles), _ptr(n_tiles), x.shape[0],
-                                         experts, width, ff, tile_rows, float(limit), float(slope), float(offset), dt, _stream(x)), op)
-    return act
+    sx, sw, slimit = shared if shared is not None else (None, None, 0.0)
+    new = lambda n, f: torch.empty((n, f), dtype=x.dtype, device=x.device)  # noqa: E731
+    act, sact = new(x.shape[0], ff), new(sx.shape[0], sw.shape[2]) if sx is not None else None
+    _call(_capi.lib().axb200_moe_gate_up(
+        x.data_ptr(), weight.data_ptr(), act.data_ptr(), _ptr(tiles), _ptr(n_tiles), x.shape[0], experts, ff, float(limit),
+        _ptr(sx), _ptr(sw), _ptr(sact), sx.shape[0] if sx is not None else 0, sw.shape[2] if sw is not None else 0, float(slimit),
+        width, tile_rows, float(slope), float(offset), _lm_dt(x, op), _stream(x)), op)
+    return act, sact
 
 
-def moe_down(act, weight, tiles=None, n_tiles=None, tile_rows=0):
-    """Down product of every row's expert: weight (experts, width, ff) -> (rows, width)."""
+def moe_down(act, weight, tiles, n_tiles, tile_rows, shared=None):
+    """Down product of every routed row's expert: weight (experts, width, ff) -> (rows, width).  shared = (act, weight
+    (1, width, ff)) as in `moe_gate_up`; returns (routed, shared)."""
     op = "moe_down"
     experts, width, ff = weight.shape
-    y = torch.empty((act.shape[0], width), dtype=act.dtype, device=act.device)
-    tile_rows = tile_rows or moe_tile_rows(act.shape[0], 1, width, ff, act.dtype)
-    _call(_capi.lib().axb200_moe_down(act.data_ptr(), weight.data_ptr(), y.data_ptr(), _ptr(tiles), _ptr(n_tiles), act.shape[0],
-                                      experts, width, ff, tile_rows, _lm_dt(act, op), _stream(act)), op)
-    return y
+    sact, sw = shared if shared is not None else (None, None)
+    new = lambda n: torch.empty((n, width), dtype=act.dtype, device=act.device)  # noqa: E731
+    y, sy = new(act.shape[0]), new(sact.shape[0]) if sact is not None else None
+    _call(_capi.lib().axb200_moe_down(
+        act.data_ptr(), weight.data_ptr(), y.data_ptr(), _ptr(tiles), _ptr(n_tiles), act.shape[0], experts, ff, _ptr(sact),
+        _ptr(sw), _ptr(sy), sact.shape[0] if sact is not None else 0, sw.shape[2] if sw is not None else 0, width, tile_rows,
+        _lm_dt(act, op), _stream(act)), op)
+    return y, sy

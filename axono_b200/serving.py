@@ -150,17 +150,23 @@ class Request:
         return len(self.out) >= self.max_new
 
 
+def greedy(logits) -> List[int]:
+    return ops.argmax_last_dim(logits).tolist()
+
+
 class Engine:
-    def __init__(self, runner: ModelRunner, token_budget: int = 2048, use_graphs: bool = True):
-        """token_budget: the most tokens one step brings (decoded tokens first, then portions of prompts)."""
+    def __init__(self, runner: ModelRunner, token_budget: int = 2048, use_graphs: bool = True, sample=greedy):
+        """token_budget: the most tokens one step brings (decoded tokens first, then portions of prompts); sample:
+        logits (rows, vocab) -> list of ids (the graph form of decoding is greedy and only used with `greedy`)."""
         if token_budget < 1:
             raise ValueError("token_budget must be positive")
-        self.runner, self.token_budget, self.use_graphs = runner, token_budget, use_graphs
+        self.runner, self.token_budget, self.sample = runner, token_budget, sample
+        self.use_graphs = use_graphs and sample is greedy
         self.waiting = collections.deque()
         self.running: List[Request] = []
         self._graph: Optional[DecodeGraph] = None
         self._steady = 0  # decode-only steps since the batch last changed
-        self._held = 0    # pages' worth of tokens promised to running requests
+        self._held = 0  # pages promised to running requests
 
     def submit(self, tokens: Sequence[int], max_new: int) -> Request:
         need = len(tokens) + max_new
@@ -217,7 +223,7 @@ class Engine:
                 last = True
             reqs.append((req, n, last))
         logits = self.runner.step(entries)
-        nxt = iter(ops.argmax_last_dim(logits).tolist() if logits is not None else [])
+        nxt = iter(self.sample(logits) if logits is not None else [])
         for req, n, last in reqs:
             if req.prompt_left:
                 req.done += n

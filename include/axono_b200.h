@@ -537,8 +537,9 @@ int axb200_latent_prefill(const void *q, int64_t q_ld, const void *k, const void
  *   moe_gate_up: act (rows, ff) = g * sigmoid(slope * g) * (u + offset), g = min(x . W_gate^T, limit),
  *     u = clamp(x . W_up^T, -limit, limit); w (experts, 2, ff, width) = gate, up.
  *   moe_down: y (rows, width) = act . W_down^T; w (experts, width, ff).
- * In the products `rows` counts rows of x; tiles == NULL means one expert over all rows.  FLOAT32, or BFLOAT16
- * with fp32 accumulation (tcgen05 when width and ff are multiples of 8).  No counterparts in the reference. */
+ * In the products `rows` counts rows of x; tiles == NULL means one expert over all rows.  shared_*: one more
+ * expert of the same form over shared_rows rows of its own input, in the same launch (shared_rows == 0: none).
+ * FLOAT32, or BFLOAT16 with fp32 accumulation (tcgen05 when width and ff are multiples of 8).  No counterparts in the reference. */
 int axb200_moe_route(const float *logits, const float *correction, int32_t *ids, float *weights, int32_t *place,
                      int32_t *counts, int64_t rows, int experts, int groups, int keep, int top, float scale,
                      void *stream);
@@ -547,10 +548,12 @@ int axb200_moe_sort(const void *x, void *sorted, const int32_t *ids, const int32
                     int32_t *row_of, int32_t *offsets, int32_t *tiles, int32_t *n_tiles, int64_t rows, int experts,
                     int top, int tile_rows, int width, int dtype, void *stream);
 int axb200_moe_gate_up(const void *x, const void *w, void *act, const int32_t *tiles, const int32_t *n_tiles,
-                       int64_t rows, int experts, int width, int ff, int tile_rows, float limit, float slope,
-                       float offset, int dtype, void *stream);
+                       int64_t rows, int experts, int ff, float limit, const void *shared_x, const void *shared_w,
+                       void *shared_act, int64_t shared_rows, int shared_ff, float shared_limit, int width,
+                       int tile_rows, float slope, float offset, int dtype, void *stream);
 int axb200_moe_down(const void *act, const void *w, void *y, const int32_t *tiles, const int32_t *n_tiles,
-                    int64_t rows, int experts, int width, int ff, int tile_rows, int dtype, void *stream);
+                    int64_t rows, int experts, int ff, const void *shared_act, const void *shared_w, void *shared_y,
+                    int64_t shared_rows, int shared_ff, int width, int tile_rows, int dtype, void *stream);
 
 /* axono::ops::cuda::Concat, src/ops/cuda/sequence.cu:474-521, on bytes: out (outer, a_bytes +
  * b_bytes) = a (outer, a_bytes) ++ b (outer, b_bytes).  Axis 0 is outer == 1. */

@@ -1,0 +1,194 @@
+"""The Nuderax model on the GPU against the plain CPU evaluation (tests/plain_nuderax.py): whole prompts, token
+by token, portions, batches, pages and slots used again, and generation through the scheduler.
+
+fp32 comparisons are sharp.  In bf16 a rounded activation can turn a close choice of the router, which
+moves single positions by far more than rounding: there most positions have to be close and all bounded."""
+import numpy as np
+import pytest
+import torch
+
+import nuderax_cases as cases
+import plain_nuderax as plain
+
+pytestmark = pytest.mark.gpu
+
+F32_TOL = 2e-5
+
+
+@pytest.fixture(scope="module")
+def built():
+    """name -> (config, weights as stored, prompt, plain logits of the whole prompt)."""
+    made = {}
+
+    def get(name, n):
+        if (name, n) not in made:
+            cfg = getattr(cases, name)()
+            w = plain.random_weights(cfg, seed=len(name))
+            rng = np.random.default_rng(n)
+            tokens = rng.integers(0, cfg["vocab"], n).tolist()
+            ref = plain.forward(cfg, {k: v.double() for k, v in w.items()}, tokens).numpy()
+            made[(name, n)] = (cfg, w, tokens, ref)
+        return made[(name, n)]
+
+    return get
+
+
+def runner_of(cfg, w, dtype, max_tokens, **kw):
+    from axono_b200 import models
+    from axono_b200.serving import ModelRunner
+
+    return ModelRunner(models.create(cfg, w, dtype), max_tokens, **kw)
+
+
+def feed(runner, seq, tokens, portions):
+    """All logits of `tokens` brought in portions of the given sizes (the last size repeats)."""
+    out, at, sizes = [], 0, list(portions)
+    while at < len(tokens):
+        n = min(sizes.pop(0) if len(sizes) > 1 else sizes[0], len(tokens) - at)
+        out.append(runner.step([(seq, tokens[at:at + n], list(range(n)))]).cpu().numpy())
+        at += n
+    assert runner.error_word() == 0
+    return np.concatenate(out)
+
+
+def check(got, ref, dtype):
+    err = cases.position_errors(got, ref)
+    if dtype == torch.float32:
+        assert err.max() <= F32_TOL, f"worst {err.max():.2e} at {int(err.argmax())}"
+    else:
+        assert np.quantile(err, 0.8) <= 0.04 and err.max() <= 1.0, f"{np.quantile(err, 0.8):.3f} {err.max():.3f}"
+
+
+SCHEDULES = {"whole": [10000], "tokens": [1], "twos": [2], "mixed": [5, 2, 64, 1, 63, 3, 17, 65, 2, 1], "prompt_then_tokens": [120, 1]}
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("schedule", sorted(SCHEDULES))
+@pytest.mark.parametrize("name", ["odd", "tiles"])
+def test_schedules(built, name, schedule, dtype):
+    cfg, w, tokens, ref = built(name, 150)
+    r = runner_of(cfg, w, dtype, 192, shuffle_pages=3)
+    check(feed(r, r.open(), tokens, SCHEDULES[schedule]), ref, dtype)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("schedule", ["whole", "prompt_then_tokens", "long_portions"])
+def test_schedules_at_tensor_core_sizes(built, schedule, dtype):
+    cfg, w, tokens, ref = built("fast", 420)
+    sizes = {"whole": [10000], "prompt_then_tokens": [390, 1], "long_portions": [257, 3, 130, 30]}[schedule]
+    r = runner_of(cfg, w, dtype, 512, shuffle_pages=5)
+    check(feed(r, r.open(), tokens, sizes), ref, dtype)
+
+
+def test_residual_after_every_layer(built):
+    cfg, w, tokens, _ = built("odd", 150)
+    want, got = [], []
+    plain.forward(cfg, {k: v.double() for k, v in w.items()}, tokens[:40], want)
+    r = runner_of(cfg, w, torch.float32, 64)
+    r.step([(r.open(), tokens[:40], [])], trace=got)
+    assert len(got) == len(want) == len(cfg["layers"])
+    for a, b in zip(got, want):
+        assert (a.cpu().double() - b).abs().max() <= 2e-5 * b.abs().max()
+
+
+def test_first_tokens(built):
+    cfg, w, tokens, ref = built("odd", 150)
+    r = runner_of(cfg, w, torch.float32, 64)
+    for n in (1, 2, 3):
+        s = r.open()
+        got = r.step([(s, tokens[:n], list(range(n)))]).cpu().numpy()
+        check(got, ref[:n], torch.float32)
+        r.close(s)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_unequal_batch_equals_each_alone(built, dtype):
+    """Prompts, portions and decoded tokens of different requests in the same steps."""
+    cfg, w, tokens, _ = built("tiles", 150)
+    spans = [(0, 150), (3, 83), (10, 140), (1, 2)]
+    steps = [[150, 7, 0, 1], [0, 70, 100, 0], [0, 1, 1, 0], [0, 2, 29, 0]]
+    r = runner_of(cfg, w, dtype, 448, max_seqs=4, shuffle_pages=1)
+    seqs, at, got = [r.open() for _ in spans], [0] * 4, [[] for _ in spans]
+    for step in steps:
+        entries = []
+        for i, n in enumerate(step):
+            if n:
+                lo = spans[i][0] + at[i]
+                entries.append((seqs[i], tokens[lo:lo + n], list(range(n))))
+        logits = r.step(entries).cpu().numpy()
+        k = 0
+        for i, n in enumerate(step):
+            got[i].append(logits[k:k + n])
+            k, at[i] = k + n, at[i] + n
+    for i, (lo, hi) in enumerate(spans):
+        alone = runner_of(cfg, w, dtype, 192)
+        ref = feed(alone, alone.open(), tokens[lo:hi], [10000])
+        assert at[i] == hi - lo
+        check(np.concatenate(got[i]), ref, dtype)
+
+
+def test_pages_and_slots_used_again(built):
+    """Freed pages hold another request's rows; nothing of them may show."""
+    cfg, w, tokens, ref = built("tiles", 150)
+    r = runner_of(cfg, w, torch.float32, 192, max_seqs=2, shuffle_pages=7)
+    rng = np.random.default_rng(4)
+    for trial in range(3):
+        s = r.open()
+        feed(r, s, rng.integers(0, cfg["vocab"], 90 + 31 * trial).tolist(), [50, 1, 40])
+        r.close(s)
+        s = r.open()
+        check(feed(r, s, tokens, [70, 2, 1, 30]), ref, torch.float32)
+        r.close(s)
+    assert r.arena.stats()["pages_free"] == r.arena.num_pages
+
+
+def test_cache_overflow_is_an_error(built):
+    cfg, w, tokens, _ = built("odd", 150)
+    r = runner_of(cfg, w, torch.float32, 64)
+    s = r.open()
+    with pytest.raises(RuntimeError):
+        r.step([(s, (tokens * 2)[:200], [])])
+
+
+def test_greedy_generation(built):
+    """The scheduler's tokens (portions of prompts beside decoding, then graph replays) are the plain ones."""
+    from axono_b200.serving import generate
+
+    cfg, w, tokens, _ = built("odd", 150)
+    wd = {k: v.double() for k, v in w.items()}
+    prompts = [tokens[:5], tokens[20:90], tokens[7:8], tokens[60:75]]
+    want = [plain.greedy(cfg, wd, p, 12) for p in prompts]
+    for kw in (dict(token_budget=16), dict(token_budget=4096), dict(token_budget=4096, use_graphs=False)):
+        r = runner_of(cfg, w, torch.float32, 384, max_seqs=3, max_seq_len=128, shuffle_pages=2)
+        assert generate(r, prompts, 12, **kw) == want
+        assert r.error_word() == 0
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_long_decoding_by_graph(built, dtype):
+    """Hundreds of tokens decoded by one captured graph, over page borders, against the whole sequence at once."""
+    from axono_b200.serving import DecodeGraph
+
+    cfg, w, tokens, _ = built("tiles", 150)
+    r = runner_of(cfg, w, dtype, 1024, max_seqs=2, max_seq_len=512, shuffle_pages=9)
+    seqs = [r.open(), r.open()]
+    outs = [tokens[:30], tokens[:61]]
+    first = []
+    for s, t in zip(seqs, outs):
+        first.append(int(torch.argmax(r.step([(s, t, [len(t) - 1])]))))
+    g = DecodeGraph(r, seqs, first, [400, 400])
+    got = [[f] for f in first]
+    for _ in range(300):
+        for o, t in zip(got, g.step().tolist()):
+            o.append(t)
+    assert r.error_word() == 0
+    for s, prompt, out in zip(seqs, outs, got):
+        fresh = runner_of(cfg, w, dtype, 512)
+        logits = fresh.step([(fresh.open(), prompt + out[:-1], list(range(len(prompt) - 1, len(prompt) + len(out) - 1)))])
+        pick = torch.argmax(logits, -1).cpu().tolist()
+        # a tie within rounding may go either way: the decoded token must be (nearly) the largest logit
+        gap = [float(logits[i].max() - logits[i, t]) for i, t in enumerate(out)]
+        scale = float(logits.std())
+        limit = 1e-4 if dtype == torch.float32 else 0.5
+        assert max(gap) <= limit * scale, max(gap) / scale
+        assert np.mean([a == b for a, b in zip(pick, out)]) >= (0.99 if dtype == torch.float32 else 0.7)
