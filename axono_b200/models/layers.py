@@ -49,7 +49,7 @@ class LatentAttention:
         self.wuk = wuk.reshape(heads, dim, kv_rank).contiguous()
         self.wuv = wuv.reshape(heads, vdim, kv_rank).contiguous()
         self.wo = wo.contiguous()
-        self.expandable = ops.latent_prefill_supported(heads, dim, rot_dim, vdim, wo.dtype)
+        self.expandable = ops.latent_prefill_supported(heads, dim, rot_dim, vdim, wo.dtype) and kv_rank % 8 == 0 and scale > 0
         # a portion of n rows pays the expansion of every cached token once, (dim + vdim) * kv_rank products per
         # token and head, and saves the difference of the two forms' products per key, head and row
         saved = 2 * kv_rank - dim - vdim
