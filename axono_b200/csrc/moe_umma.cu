@@ -37,13 +37,6 @@ struct UmmaParams {
   int shared_tiles;    // grid rows of the shared expert, before the routed ones
 };
 
-__device__ __forceinline__ void tma_load_2d(void *dst, const CUtensorMap *map, uint64_t *bar, int c0, int c1) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
-      ::"r"(smem_u32(dst)), "l"(reinterpret_cast<uint64_t>(map)), "r"(smem_u32(bar)), "r"(c0), "r"(c1)
-      : "memory");
-}
-
 template <int kN, bool kGateUp>
 __global__ void __launch_bounds__(kThreads, Shape<kN>::kCtasPerSm)
 moe_umma_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
