@@ -94,6 +94,42 @@ class NuderaxConfig:
         return cls(int(config["vocab"]), int(config["width"]), float(config["norm"]["eps"]), layers)
 
 
+def tensor_shapes(cfg: NuderaxConfig):
+    """(name, shape) of every tensor a model of this configuration has."""
+    width = cfg.width
+    yield "embed", (cfg.vocab, width)
+    yield "embed.norm", (width,)
+    yield "final.norm", (width,)
+    for i, layer in enumerate(cfg.layers):
+        m, f, p = layer.mixer, layer.mlp, f"l{i}."
+        q = m.heads * (m.dim + m.rot_dim)
+        yield p + "norm1", (width,)
+        if m.low_rank_q:
+            yield p + "mix.dq", (m.q_rank, width)
+            yield p + "mix.dq.norm", (m.q_rank,)
+            yield p + "mix.uq", (q, m.q_rank)
+        else:
+            yield p + "mix.q", (q, width)
+        if m.kv_from is None:
+            yield p + "mix.dkv", (m.kv_rank + m.rot_dim, width)
+            yield p + "mix.dkv.norm", (m.kv_rank,)
+        yield p + "mix.uk", (m.heads * m.dim, m.kv_rank)
+        yield p + "mix.uv", (m.heads * m.vdim, m.kv_rank)
+        yield p + "mix.o", (width, m.heads * m.vdim)
+        if f is None:
+            continue
+        yield p + "norm2", (width,)
+        yield p + "mlp.router", (f.experts, width)
+        yield p + "mlp.correction", (f.experts,)
+        forms = [(f"e{j}", f.ff) for j in range(f.experts)]
+        if f.shared_ff is not None:
+            forms.append(("shared", f.shared_ff))
+        for name, ff in forms:
+            yield f"{p}mlp.{name}.gate", (ff, width)
+            yield f"{p}mlp.{name}.up", (ff, width)
+            yield f"{p}mlp.{name}.down", (width, ff)
+
+
 @register("Nuderax")
 class Nuderax:
     config_class = NuderaxConfig

@@ -33,7 +33,8 @@ batch of 64 sequences per step.
 Other workloads, each with its own JSON line: `c2_block` (the fused decode block, batch 8, KV 8192, one
 CUDA graph), `c5_tower` (the text-tower step by itself; `--runtime torch` runs it on the torch-tensor
 mirror), `prefill` (causal prefill attention; `--dtype f32` for the reference's own type), `ops` (the
-standalone operators at the multimodal prompt's shapes); `--impl reference-cuda` times the reference's
+standalone operators at the multimodal prompt's shapes), `nuderax` (decode and prefill of the Nuderax
+layers beside the text tower's at equal size); `--impl reference-cuda` times the reference's
 own CUDA kernels compiled for sm_100; `--runtime torch` runs the attention workload on the torch mirror.
 """
 from __future__ import annotations
@@ -1295,14 +1296,293 @@ def run_small_ops(args):
     }), flush=True)
 
 
+# ---- language models: the Nuderax layers beside the text tower's at equal size -------------------------
+LM_SIZES = {
+    # name: width, heads, q_rank of the low-rank layers, ff of an expert, ff of the shared expert, experts, top, groups, keep;
+    # tower: intermediate, KV heads.  Head sizes 128 + 64 rotated, 128 for values, latent 512 in all.
+    "2k": dict(width=2048, heads=16, q_rank=1536, ff=1408, shared_ff=2816, experts=64, top=6, groups=8, keep=3, inter=6144, hkv=8),
+    "4k": dict(width=4096, heads=32, q_rank=1536, ff=2048, shared_ff=2048, experts=64, top=8, groups=8, keep=4, inter=12288, hkv=8),
+    "5k": dict(width=5120, heads=128, q_rank=1536, ff=1536, shared_ff=3072, experts=160, top=6, groups=8, keep=3, inter=12288, hkv=8),
+}
+
+
+def lm_config(size, n_layers):
+    z = LM_SIZES[size]
+    mlp = {"kind": "moe", "expert": {"ff": z["ff"], "limit": 7.0}, "shared": {"ff": z["shared_ff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 1.5, "groups": {"count": z["groups"], "keep": z["keep"]}}}
+    layers = []
+    for i in range(n_layers):
+        m = {"heads": z["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+             "rot": {"base": 10000.0, "dims": 64}}
+        low_rank = i % 2 == 1
+        if low_rank:
+            m["q_rank"] = z["q_rank"]
+        layers.append({"type": "latent_attention_2" if low_rank else "latent_attention", "mixer": m, "mlp": mlp})
+    return {"architecture": "Nuderax", "vocab": 32768, "width": z["width"], "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def run_lm(args):
+    """`nuderax`: decode and prefill throughput of Nuderax layers with random bf16 weights, beside the text tower
+    (fp16, the framework's other decoder) with the same width, heads and context; and the kernels of both alone
+    against the measured peaks.  Decode: CUDA-graph replays of whole steps, batch --lm-batch at context --lm-len.
+    Prefill: one prompt of --prefill-len tokens through the runner (the tower has no prefill step: its prefill
+    attention kernel stands beside).  Kernels: event pairs around single calls, L2 flushed before each."""
+    import math
+
+    import torch
+
+    from axono_b200 import models, ops
+    from axono_b200.cuda_graph import CUDAGraph
+    from axono_b200.decode import TextTower, TextTowerConfig
+    from axono_b200.models.layers import Rows
+    from axono_b200.models.nuderax import tensor_shapes
+    from axono_b200.serving import DecodeGraph, ModelRunner
+
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    gen = torch.Generator(device=dev).manual_seed(3)
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            peaks = json.load(f)
+        gbs_peak, tf_peak, kind = float(peaks["hbm_gbs"]), float(peaks["bf16_tflops"]), "measured"
+    except Exception:
+        gbs_peak, tf_peak, kind = FALLBACK_HBM_GBS, 1590.0, "fallback"
+    B, L, S, n_layers = args.lm_batch, args.lm_len, args.prefill_len, args.lm_layers
+    warmup = max(3, args.warmup)
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)  # 256 MB, twice the L2
+    sampler = ClockSampler(0)
+    launches = 0
+
+    def timed(fn, n=20):
+        """Mean milliseconds of one call, L2 flushed before each."""
+        for _ in range(3):
+            fn()
+        pairs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(n)]
+        sampler.start()
+        for e0, e1 in pairs:
+            flush.zero_()
+            e0.record()
+            fn()
+            e1.record()
+        torch.cuda.synchronize()
+        sampler.pause()
+        return statistics.median(e0.elapsed_time(e1) for e0, e1 in pairs)
+
+    def replayed(graph, steps):
+        for _ in range(warmup):
+            graph()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        sampler.start()
+        e0.record()
+        for _ in range(steps):
+            graph()
+        e1.record()
+        torch.cuda.synchronize()
+        sampler.pause()
+        return e0.elapsed_time(e1) / steps
+
+    class RandomWeights(dict):
+        def __missing__(self, name):
+            shape = shapes[name]
+            if len(shape) == 1:
+                return (0.0 if name.endswith("correction") else 1.0) + 0.1 * torch.randn(shape, generator=gen, device=dev)
+            gain = 1.0 if name == "embed" else 1.0 / math.sqrt(shape[1])
+            return (gain * torch.randn(shape, generator=gen, device=dev)).to(torch.bfloat16)
+
+    results, total_steps = {}, args.steps + warmup + 8
+    for size in (args.lm_sizes.split(",") if args.lm_sizes else ["2k", "4k"]):
+        z = LM_SIZES[size]
+        cfg = lm_config(size, n_layers)
+        shapes = dict(tensor_shapes(models.config_of(cfg)))
+        model = models.create(cfg, RandomWeights(), torch.bfloat16)
+        res = {"decode": {}, "prefill": {}, "kernels": {}}
+
+        # ---- decode: whole steps as graph replays ----
+        runner = ModelRunner(model, B * (L + total_steps + 64), max_seqs=B, max_seq_len=L + total_steps + 64, shuffle_pages=1)
+        for pool in runner.pages:
+            pool.normal_(generator=gen)
+        seqs = [runner.open() for _ in range(B)]
+        for s in seqs:
+            runner.lengths[s] = L
+        g = DecodeGraph(runner, seqs, torch.randint(0, 32768, (B,)).tolist(), [L + total_steps] * B)
+        ms = replayed(g.step, args.steps)
+        launches += g.graph.num_nodes * args.steps
+        # what a step has to read: the latents once per layer, dense weights, the experts that were chosen
+        mlp0 = model.layers[0][3]
+        moe_bytes = sum(2.0 * (m.gate_up.numel() + m.down.numel()) for _, _, _, m in model.layers)
+        touched = 1.0 - (1.0 - z["top"] / z["experts"]) ** B
+        need = model.weight_bytes() - moe_bytes * (1 - touched) + n_layers * B * L * 576 * 2.0
+        res["decode"]["nuderax"] = {"ms_per_step": ms, "tokens_per_s": B / ms * 1e3, "bytes_per_step": need, "launches": g.graph.num_nodes,
+                                    "frac_of_hbm": need / (ms * 1e6) / gbs_peak}
+        g.graph.reset()
+
+        # ---- its kernels at decode sizes ----
+        K = res["kernels"]
+
+        def bandwidth(name, ms, nbytes, like=None):
+            K[name] = {"us": ms * 1e3, "gbs": nbytes / (ms * 1e6), "frac": nbytes / (ms * 1e6) / gbs_peak, "bound": "hbm", "like": like}
+
+        def tensor(name, ms, flops, like=None):
+            K[name] = {"us": ms * 1e3, "tflops": flops / (ms * 1e9), "frac": flops / (ms * 1e9) / tf_peak, "bound": "tensor", "like": like}
+
+        bf = lambda *sh: torch.randn(sh, generator=gen, device=dev).to(torch.bfloat16)  # noqa: E731
+        rows = Rows(torch.tensor(seqs, dtype=torch.int32, device=dev), torch.full((B,), L - 1, dtype=torch.int32, device=dev),
+                    runner.block_table, L, B)
+        H, per, width = z["heads"], 192, z["width"]
+        mixer = model.layers[0][2]
+        ql, q = bf(B, H, 512), bf(B, H * per)
+        bandwidth("decode latent_attend (+ merge)", timed(lambda: ops.latent_attend(ql, q, 128, 64, 0.07, runner.pages[0], rows, B)),
+                  B * L * 1152.0 + 2 * ql.numel() * 2, "gqa decode")
+        K["decode latent_attend (+ merge)"]["tflops"] = 2.0 * B * L * H * 1088 / (K["decode latent_attend (+ merge)"]["us"] * 1e6)
+
+        def moe_kernels(n, tag):
+            h = bf(n, width)
+            logits = torch.randn((n, z["experts"]), generator=gen, device=dev)
+            corr = torch.zeros(z["experts"], device=dev)
+            route = lambda: ops.moe_route(logits, corr, z["groups"], z["keep"], z["top"], 1.5)  # noqa: E731
+            ids, wts, place, counts = route()
+            tile = ops.moe_tile_rows(n * z["top"], z["experts"], width, z["ff"], torch.bfloat16)
+            srt, row_of, _, tiles, n_tiles = ops.moe_sort(h, ids, place, counts, tile)
+            gu = lambda: ops.moe_gate_up(srt, mlp0.gate_up, 7.0, tiles, n_tiles, tile, (h, mlp0.shared_gate_up, 7.0))  # noqa: E731
+            act, sact = gu()
+            down = lambda: ops.moe_down(act, mlp0.down, tiles, n_tiles, tile, (sact, mlp0.shared_down))  # noqa: E731
+            y, sy = down()
+            used = int((counts > 0).sum())
+            products = n * (z["top"] * z["ff"] + z["shared_ff"]) * width
+            w1 = 2.0 * (used * z["ff"] + z["shared_ff"]) * width * 2
+            t_gu, t_down = timed(gu), timed(down)
+            if n <= 256:
+                bandwidth(f"{tag} experts gate/up", t_gu, w1, "decode GEMM")
+                bandwidth(f"{tag} experts down", t_down, w1 / 2, "decode GEMM")
+            else:
+                tensor(f"{tag} experts gate/up", t_gu, 4.0 * products, "prefill GEMM")
+                tensor(f"{tag} experts down", t_down, 2.0 * products, "prefill GEMM")
+            x = torch.randn((n, width), generator=gen, device=dev)
+            a = bf(n, width)
+            nw = bf(width)
+            bandwidth(f"{tag} residual + experts + 2 norms", timed(lambda: ops.residual_layer_norm(x, nw, nw, 1e-5, a=a, b=sy,
+                                                                                                   experts=(y, row_of, wts))),
+                      n * width * (8.0 + 4 + 2 * z["top"] + 4), "add_rms_norm")
+            bandwidth(f"{tag} route", timed(route), n * z["experts"] * 4.0 + n * z["top"] * 12.0, None)
+            bandwidth(f"{tag} sort", timed(lambda: ops.moe_sort(h, ids, place, counts, tile)), n * width * 2.0 * (1 + z["top"]), "add_rms_norm")
+
+        def prepare_kernel(n, tag):
+            prows = Rows(torch.zeros(n, dtype=torch.int32, device=dev), torch.arange(n, dtype=torch.int32, device=dev) % L,
+                         runner.block_table, L, n)
+            proj = bf(n, H * per + 576)
+            bandwidth(f"{tag} norm + rotate + append", timed(lambda: ops.latent_prepare(
+                prows, mixer.inv_freq, 64, q=proj[:, :H * per], heads=H, dim=128, dkv=proj[:, H * per:], dkv_weight=mixer.dkv_norm,
+                pages=runner.pages[0])), n * (H * 64 * 4.0 + 576 * 4), "rope + append")
+
+        moe_kernels(B, "decode")
+        prepare_kernel(B, "decode")
+
+        # ---- prefill: whole prompts through the runner ----
+        for s in seqs:
+            runner.close(s)
+        prompt = torch.randint(0, 32768, (S,)).tolist()
+
+        def prefill(portion):
+            s = runner.open()
+            for at in range(0, S, portion):
+                runner.step([(s, prompt[at:at + portion], [len(prompt[at:at + portion]) - 1] if at + portion >= S else [])])
+            runner.close(s)
+
+        for portion in (S, min(2048, S)):
+            for _ in range(2):
+                prefill(portion)
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            reps = 5
+            sampler.start()
+            e0.record()
+            for _ in range(reps):
+                prefill(portion)
+            e1.record()
+            torch.cuda.synchronize()
+            sampler.pause()
+            pms = e0.elapsed_time(e1) / reps
+            dense = sum(t.numel() for _, _, m, _ in model.layers for t in (m.w_in, m.wo, m.wuq, m.wuk, m.wuv) if t is not None)
+            dense += n_layers * ((z["top"] * z["ff"] + z["shared_ff"]) * 3 + z["experts"]) * width
+            flops = 2.0 * S * dense + n_layers * H * (S * (S + 1) / 2) * 2 * (192 + 128)
+            res["prefill"][f"portion {portion}"] = {"tokens": S, "ms": pms, "tokens_per_s": S / pms * 1e3, "tflops": flops / (pms * 1e9),
+                                                    "frac_of_tensor": flops / (pms * 1e9) / tf_peak}
+        moe_kernels(S, "prefill")
+        prepare_kernel(min(S, L), "prefill")
+        qp, kp, vp, cp = bf(S, H * per), bf(S, H * 128), bf(S, H * 128), bf(S, 576)
+        tensor("prefill attention (expanded)", timed(lambda: ops.latent_prefill(qp, 0, kp, vp, cp[:, 512:], H, 128, 64, 128, 0.07)),
+               H * (S * (S + 1) / 2) * 2.0 * (192 + 128), "prefill attention (tower)")
+        del qp, kp, vp, cp, runner, model, mixer, mlp0, ql, q
+        torch.cuda.empty_cache()
+
+        # ---- the text tower at the same width, heads and context ----
+        tcfg = TextTowerConfig(hidden=width, intermediate=z["inter"], n_q_heads=H, n_kv_heads=z["hkv"], vocab=32768, n_layers=n_layers)
+        tower = TextTower(tcfg, B, L + total_steps + 64, device=dev, seed=5)
+        for li in range(n_layers):
+            tower.cache.k_pages[li].normal_(generator=gen)
+            tower.cache.v_pages[li].normal_(generator=gen)
+        tower.set_state(np.arange(B) % 32768, [L] * B)
+        ops.workspace(dev, ops.gqa_workspace_bytes(B, H, z["hkv"], 128, tower.cache.max_seq_len))
+        tg = CUDAGraph().capture(tower.decode_step)
+        tower.cache.note_replayed()
+        tms = replayed(tg.replay_async, args.steps)
+        launches += tg.num_nodes * args.steps
+        tneed = tower.kv_bytes_per_step([L] * B) + tower.weight_bytes()
+        res["decode"]["tower"] = {"ms_per_step": tms, "tokens_per_s": B / tms * 1e3, "bytes_per_step": tneed, "launches": tg.num_nodes,
+                                  "frac_of_hbm": tneed / (tms * 1e6) / gbs_peak}
+        tg.reset()
+        f16 = lambda *sh: torch.randn(sh, generator=gen, device=dev).half()  # noqa: E731
+        tq = f16(B, H, 128)
+        tower.cache.seq_lens.fill_(L)
+        tower.cache._host_len_bound = L
+        bandwidth("tower gqa decode", timed(lambda: tower.cache.attend(0, tq)), B * L * z["hkv"] * 512.0 + 2 * tq.numel() * 2)
+        lw = tower.layers[0]
+        xb, xs = f16(B, width), f16(S, width)
+        bandwidth("tower decode GEMM (gate|up)", timed(lambda: ops.linear_nobias(xb, lw["gate_up"])), lw["gate_up"].numel() * 2.0)
+        tensor("tower prefill GEMM (gate|up)", timed(lambda: ops.linear_nobias(xs, lw["gate_up"])), 2.0 * S * lw["gate_up"].numel())
+        bandwidth("tower add_rms_norm (decode)", timed(lambda: ops.add_rms_norm(xb, xb, lw["input_ln"], 1e-6)), B * width * 8.0)
+        bandwidth("tower add_rms_norm (prefill)", timed(lambda: ops.add_rms_norm(xs, xs, lw["input_ln"], 1e-6)), S * width * 8.0)
+        qkv = f16(B, (H + 2 * z["hkv"]) * 128)
+        bandwidth("tower norm + rope + append (decode)", timed(lambda: tower.cache.append_qkv(
+            1, qkv, H, lw["q_norm"], lw["k_norm"], 1e-6, pos=tower.pos3[0], theta=1e6)), qkv.numel() * 4.0)
+        tk, tv = f16(S, z["hkv"], 128), f16(S, z["hkv"], 128)
+        tqp = f16(S, H, 128)
+        bandwidth("tower rope + append (prefill)", timed(lambda: ops.kv_prefill_write(
+            tqp, tk, tv, tower.cache.k_pages[0], tower.cache.v_pages[0], tower.cache.block_table[0], theta=1e6)) if S <= L else 1e9,
+            (tqp.numel() + 2 * tk.numel()) * 4.0)
+        tensor("tower prefill attention", timed(lambda: ops.scaled_dot_product_attention(tqp, tk, tv, True)),
+               4.0 * H * 128 * (S * (S + 1) / 2))
+        del tower, tq, tqp, tk, tv, lw, tg
+        torch.cuda.empty_cache()
+        results[size] = res
+    err = ops.last_error()
+    if err:
+        raise SystemExit(f"device error word {err:#x}")
+    first = next(iter(results.values()))["decode"]["nuderax"]
+    round_ = lambda v: {k: round_(x) for k, x in v.items()} if isinstance(v, dict) else float(f"{v:.4g}") if isinstance(v, float) else v  # noqa: E731
+    print(json.dumps({
+        "metric": "nuderax_decode_tokens_per_s", "value": first["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+        "warmup": warmup, "ms_per_step": first["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "nuderax", "sizes": list(results), "layers": n_layers, "batch": B, "kv_len": L, "prefill_len": S,
+                   "l2": "steps read more than L2; single kernels after an L2 flush", "peaks": f"of {kind}"},
+        "results": round_(results), "gpu_launches": launches, "clocks": sampler.summary(),
+    }), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=200)
     ap.add_argument("--warmup", type=int, default=10)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "reference-cuda"])
-    ap.add_argument("--workload", default="c3_ragged", choices=sorted(WORKLOADS) + ["c2_block", "c5_tower", "prefill", "ops"])
+    ap.add_argument("--workload", default="c3_ragged", choices=sorted(WORKLOADS) + ["c2_block", "c5_tower", "prefill", "ops", "nuderax"])
     ap.add_argument("--prefill-len", type=int, default=8192)
+    ap.add_argument("--lm-sizes", default="", help="nuderax: comma-separated sizes out of " + ", ".join(LM_SIZES) + " (default 2k,4k)")
+    ap.add_argument("--lm-batch", type=int, default=32, help="nuderax: sequences that decode together")
+    ap.add_argument("--lm-len", type=int, default=16384, help="nuderax: context length of decoding")
+    ap.add_argument("--lm-layers", type=int, default=4, help="nuderax: layers (even ones with direct, odd ones with low-rank queries)")
     ap.add_argument("--ops-once", action="store_true",
                     help="ops: launch every operator once inside the profiler range and exit (for ncu)")
     ap.add_argument("--runtime", default="native", choices=["native", "torch"],
@@ -1335,9 +1615,12 @@ def main():
         if rank0:
             run_reference_cuda(args)
     elif args.impl == "reference":
-        if args.workload in ("c2_block", "c5_tower", "prefill", "ops"):
+        if args.workload in ("c2_block", "c5_tower", "prefill", "ops", "nuderax"):
             args.workload = "c2_b8_l8k" if args.workload == "c2_block" else "c3_ragged"
         run_reference_arm(args)
+    elif args.workload == "nuderax":
+        if rank0:
+            run_lm(args)
     elif args.workload == "prefill":
         if rank0:
             run_prefill(args)
