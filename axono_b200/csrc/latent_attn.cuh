@@ -1,0 +1,33 @@
+// What the kernels of latent attention in its cached (latent) form share; see latent_attn.cu.
+#pragma once
+
+#include "tcgen05.cuh"
+
+namespace axb {
+
+struct AttendParams {
+  const void *q_lat;  // (rows, heads, kv_rank)
+  const void *q;      // (rows, q_ld): the rotated part of head h starts at h * (dim + rot_dim) + dim
+  int64_t q_ld;
+  void *out;  // (rows, heads, kv_rank)
+  const void *pages;
+  const int32_t *block_table, *row_seq, *row_pos;
+  int rows, heads, dim, kv_rank, rot_dim, page_tokens, max_blocks, num_pages, max_seqs, max_len;
+  float scale;
+  unsigned long long wait_ns;
+};
+
+// Keys row r may read: 0 .. row_pos[r], never beyond the block table's reach or the host's bound.
+__device__ __forceinline__ int visible_keys(const AttendParams &p, int r) {
+  const int seq = p.row_seq[r];
+  if (seq < 0 || seq >= p.max_seqs) return 0;
+  const int cover = min(p.max_blocks * p.page_tokens, p.max_len);
+  return max(0, min(p.row_pos[r] + 1, cover));
+}
+
+// tcgen05 form for bf16 (latent_umma.cu)
+size_t latent_umma_workspace_bytes(int heads, int kv_rank, int rot_dim);
+bool latent_umma_supported(const AttendParams &p);
+int latent_umma(const AttendParams &p, void *workspace, cudaStream_t st);
+
+}  // namespace axb

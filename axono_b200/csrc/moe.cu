@@ -27,7 +27,7 @@ struct RouteParams {
   float *weights;           // (rows, top)
   int32_t *place;           // (rows, top): place in the expert's list
   int32_t *counts;          // (experts), zero on entry
-  int rows, experts, groups, keep, top;
+  int rows, experts, groups, keep, top, rows_per_warp;
   float scale;
 };
 
@@ -46,63 +46,74 @@ __device__ __forceinline__ void warp_argmax(float &v, int &i) {
 // Weights are the scores without the correction, times scale.
 __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const RouteParams p) {
   extern __shared__ float sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x * kRouteWarps + warp;
-  float *score = sm + (size_t)warp * (2 * p.experts + p.groups), *choice = score + p.experts, *group = choice + p.experts;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row0 = blockIdx.x * kRouteWarps * p.rows_per_warp;
+  int *count = reinterpret_cast<int *>(sm);  // rows of this CTA per expert; then the CTA's first place there
+  float *score = sm + p.experts + (size_t)warp * (2 * p.experts + p.groups), *choice = score + p.experts, *group = choice + p.experts;
+  for (int e = threadIdx.x; e < p.experts; e += kRouteWarps * 32) count[e] = 0;
   grid_dependency_wait();
   grid_dependency_launch();
-  if (row >= p.rows) return;
-  for (int e = lane; e < p.experts; e += 32) {
-    const float s = 1.0f / (1.0f + expf(-p.logits[(size_t)row * p.experts + e]));
-    score[e] = s;
-    choice[e] = s + (p.correction ? p.correction[e] : 0.f);
-  }
-  __syncwarp();
-  if (p.keep < p.groups) {
-    const int size = p.experts / p.groups;
-    for (int g = lane; g < p.groups; g += 32) {
-      float a = -INFINITY, b = -INFINITY;  // the two largest
-      for (int e = g * size; e < (g + 1) * size; ++e) {
-        const float c = choice[e];
-        if (c > a)
-          b = a, a = c;
-        else if (c > b)
-          b = c;
-      }
-      group[g] = size > 1 ? a + b : a;
+  __syncthreads();
+  const int row_end = min(p.rows, row0 + kRouteWarps * p.rows_per_warp);
+#pragma unroll 1
+  for (int row = row0 + warp; row < row_end; row += kRouteWarps) {
+    for (int e = lane; e < p.experts; e += 32) {
+      const float s = 1.0f / (1.0f + expf(-p.logits[(size_t)row * p.experts + e]));
+      score[e] = s;
+      choice[e] = s + (p.correction ? p.correction[e] : 0.f);
     }
     __syncwarp();
-    // close all but the `keep` best groups: an open group is marked by a NaN-free flag in its score
-    for (int k = 0; k < p.keep; ++k) {
+    if (p.keep < p.groups) {
+      const int size = p.experts / p.groups;
+      for (int g = lane; g < p.groups; g += 32) {
+        float a = -INFINITY, b = -INFINITY;  // the two largest
+        for (int e = g * size; e < (g + 1) * size; ++e) {
+          const float c = choice[e];
+          if (c > a)
+            b = a, a = c;
+          else if (c > b)
+            b = c;
+        }
+        group[g] = size > 1 ? a + b : a;
+      }
+      __syncwarp();
+      // close all but the `keep` best groups: an open group is marked by a NaN-free flag in its score
+      for (int k = 0; k < p.keep; ++k) {
+        float best = -INFINITY;
+        int at = INT_MAX;
+        for (int g = lane; g < p.groups; g += 32)
+          if (group[g] > best || (group[g] == best && g < at)) best = group[g], at = g;
+        warp_argmax(best, at);
+        __syncwarp();
+        if (lane == 0 && at != INT_MAX) group[at] = -INFINITY;
+        __syncwarp();
+      }
+      for (int e = lane; e < p.experts; e += 32)
+        if (group[e / size] != -INFINITY) choice[e] = -INFINITY;
+      __syncwarp();
+    }
+    for (int k = 0; k < p.top; ++k) {
       float best = -INFINITY;
       int at = INT_MAX;
-      for (int g = lane; g < p.groups; g += 32)
-        if (group[g] > best || (group[g] == best && g < at)) best = group[g], at = g;
+      for (int e = lane; e < p.experts; e += 32)
+        if (choice[e] > best) best = choice[e], at = e;
       warp_argmax(best, at);
+      if (at == INT_MAX) at = 0;  // only with NaN logits: stay in bounds
       __syncwarp();
-      if (lane == 0 && at != INT_MAX) group[at] = -INFINITY;
+      if (lane == 0) {
+        choice[at] = -INFINITY;
+        const int64_t o = (int64_t)row * p.top + k;
+        p.ids[o] = at;
+        p.weights[o] = score[at] * p.scale;
+        p.place[o] = atomicAdd(&count[at], 1);
+      }
       __syncwarp();
     }
-    for (int e = lane; e < p.experts; e += 32)
-      if (group[e / size] != -INFINITY) choice[e] = -INFINITY;
-    __syncwarp();
   }
-  for (int k = 0; k < p.top; ++k) {
-    float best = -INFINITY;
-    int at = INT_MAX;
-    for (int e = lane; e < p.experts; e += 32)
-      if (choice[e] > best) best = choice[e], at = e;
-    warp_argmax(best, at);
-    if (at == INT_MAX) at = 0;  // only with NaN logits: stay in bounds
-    __syncwarp();
-    if (lane == 0) {
-      choice[at] = -INFINITY;
-      const int64_t o = (int64_t)row * p.top + k;
-      p.ids[o] = at;
-      p.weights[o] = score[at] * p.scale;
-      p.place[o] = atomicAdd(&p.counts[at], 1);
-    }
-    __syncwarp();
-  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < p.experts; e += kRouteWarps * 32) count[e] = count[e] ? atomicAdd(&p.counts[e], count[e]) : 0;
+  __syncthreads();
+  for (int64_t o = (int64_t)row0 * p.top + threadIdx.x; o < (int64_t)row_end * p.top; o += kRouteWarps * 32)
+    p.place[o] += count[p.ids[o]];
 }
 
 // offsets[e] = start of expert e's rows in the sorted order; tiles of up to tile_rows rows in expert order.
@@ -266,13 +277,16 @@ int axb200_moe_route(const float *logits, const float *correction, int32_t *ids,
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (cudaMemsetAsync(counts, 0, (size_t)experts * sizeof(int32_t), st) != cudaSuccess) return AXB200_DEVICE_ERROR;
   if (rows == 0) return AXB200_OK;
-  axb::RouteParams p{logits, correction, ids, weights, place, counts, (int)rows, experts, groups, keep, top, scale};
-  const size_t smem = (size_t)axb::kRouteWarps * (2 * experts + groups) * sizeof(float);
+  // enough rows per CTA that its experts' places come in one round of global atomics, and enough CTAs
+  const int per_warp = rows >= 148 * 2 * axb::kRouteWarps * 4 ? 4 : rows >= 148 * axb::kRouteWarps * 2 ? 2 : 1;
+  axb::RouteParams p{logits, correction, ids, weights, place, counts, (int)rows, experts, groups, keep, top, per_warp, scale};
+  const size_t smem = ((size_t)experts + axb::kRouteWarps * (2 * experts + groups)) * sizeof(float);
   if (smem > 48 * 1024 && cudaFuncSetAttribute(axb::moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                (int)smem) != cudaSuccess)
     return AXB200_DEVICE_ERROR;
-  return axb::launch_dependent(axb::moe_route_kernel, dim3((unsigned)((rows + axb::kRouteWarps - 1) / axb::kRouteWarps)),
-                               dim3(axb::kRouteWarps * 32), smem, st, p);
+  const int per_cta = axb::kRouteWarps * per_warp;
+  return axb::launch_dependent(axb::moe_route_kernel, dim3((unsigned)((rows + per_cta - 1) / per_cta)), dim3(axb::kRouteWarps * 32),
+                               smem, st, p);
 }
 
 int axb200_moe_tile_rows(int64_t rows, int experts, int width, int ff, int dtype) {

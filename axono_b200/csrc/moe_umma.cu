@@ -8,8 +8,8 @@
 // exchange.  The shared expert's tiles ride in the same launch (first in the grid: with few rows its CTAs alone
 // could not fill the GPU), through tensor maps of their own.
 //
-// Warps 0-3 read the accumulators and store; one lane of warp 4 issues the MMAs, one lane of warp 5 the TMA
-// loads, 64 elements of K per stage with 128-byte swizzle.  Sizes that are no multiple of the tile are
+// Warps 0-7 read the accumulators and store (every other 16 columns each four); warp 8 issues the MMAs, one lane of
+// warp 9 the TMA loads, 64 elements of K per stage with 128-byte swizzle.  Sizes that are no multiple of the tile are
 // zero-filled by TMA on the way in and masked on the way out.  Every wait is bounded.
 #include <mutex>
 
@@ -18,7 +18,7 @@
 namespace axb {
 namespace {
 
-constexpr int kThreads = 192, kMmaWarp = 4, kLoadWarp = 5;
+constexpr int kThreads = 320, kMmaWarp = 8, kLoadWarp = 9;
 constexpr int kMTile = 128, kKTile = 64, kATile = kMTile * kKTile * 2;
 
 template <int kN>
@@ -99,47 +99,53 @@ moe_umma_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
           }
     }
   } else if (warp == kMmaWarp) {
-    if (lane == 0) {
+    const uint32_t lead = lane == 0;  // the warp walks, one lane issues
+    {
       // fp32 accumulate, bf16 operands, both K-major, M = 128, N = kN
       constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(kN >> 3) << 17) | ((kMTile >> 4) << 24);
       const uint64_t base = smem_desc(smem_u32(smem), 16, 1024);
       bool ok = true;
       for (int k = 0; k < steps && ok; ++k) {
         const int s = k % S::kStages;
-        ok = mbar_wait_bounded(&full[s], (k / S::kStages) & 1, abort_flag, p.wait_ns);
+        ok = mbar_wait_warp(&full[s], (k / S::kStages) & 1, abort_flag, p.wait_ns);
         if (!ok) break;
         tc_fence_after();
         const uint64_t a0 = base + (uint64_t)(s * (S::kStageBytes >> 4)), a1 = a0 + (kATile >> 4), b = a0 + (2 * kATile >> 4);
 #pragma unroll
-        for (int ks = 0; ks < kKTile / 16; ++ks) umma_f16(tmem, a0 + ks * 2, b + ks * 2, idesc, k > 0 || ks > 0);
+        for (int ks = 0; ks < kKTile / 16; ++ks) umma_f16_lead(tmem, a0 + ks * 2, b + ks * 2, idesc, k > 0 || ks > 0, lead);
 #pragma unroll
-        for (int ks = 0; ks < kKTile / 16; ++ks) umma_f16(tmem + kN, a1 + ks * 2, b + ks * 2, idesc, k > 0 || ks > 0);
-        umma_commit(&empty[s]);
+        for (int ks = 0; ks < kKTile / 16; ++ks) umma_f16_lead(tmem + kN, a1 + ks * 2, b + ks * 2, idesc, k > 0 || ks > 0, lead);
+        umma_commit_lead(&empty[s], lead);
       }
-      if (ok) umma_commit(done);
+      if (ok) umma_commit_lead(done, lead);
     }
   } else if (__all_sync(0xffffffffu, mbar_wait_bounded(done, 0, abort_flag, p.wait_ns))) {
     tc_fence_after();
-    const uint32_t base = tmem + ((uint32_t)(warp * 32) << 16);
-    const int f0 = m0 + warp * 32 + lane;
-    __nv_bfloat16 *y = static_cast<__nv_bfloat16 *>(p.y) + (size_t)tile.y * p.out;
+    // warps w and w + 4 share a quarter of the lanes (features) and take every other 16 columns (rows)
+    const uint32_t base = tmem + ((uint32_t)((warp & 3) * 32) << 16);
+    const int f0 = m0 + (warp & 3) * 32 + lane;
+    const bool in0 = f0 < p.out, in1 = f0 + kMTile < p.out;
+    __nv_bfloat16 *y = static_cast<__nv_bfloat16 *>(p.y) + (size_t)tile.y * p.out + f0;
 #pragma unroll 1
-    for (int c = 0; c < kN && c < tile.z; c += 16) {
+    for (int c = (warp >> 2) * 16; c < kN && c < tile.z; c += 32) {
       uint32_t a[16], b[16];
       tmem_ld16_async(base + c, a);
       tmem_ld16_async(base + kN + c, b);
       tmem_wait_ld();
+      __nv_bfloat16 *row = y + (size_t)c * p.out;
+      if (kGateUp) {
+        __nv_bfloat16 v[16];
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const int n = c + i;
-        if (n >= tile.z) break;
-        __nv_bfloat16 *row = y + (size_t)n * p.out;
-        const float va = __uint_as_float(a[i]), vb = __uint_as_float(b[i]);
-        if (kGateUp) {
-          if (f0 < p.out) row[f0] = __float2bfloat16_rn(clamped_gate<false>(va, vb, p.act));
-        } else {
-          if (f0 < p.out) row[f0] = __float2bfloat16_rn(va);
-          if (f0 + kMTile < p.out) row[f0 + kMTile] = __float2bfloat16_rn(vb);
+        for (int i = 0; i < 16; ++i)
+          v[i] = __float2bfloat16_rn(clamped_gate<false>(__uint_as_float(a[i]), __uint_as_float(b[i]), p.act));
+#pragma unroll
+        for (int i = 0; i < 16; ++i)
+          if (in0 && c + i < tile.z) row[(size_t)i * p.out] = v[i];
+      } else {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          if (in0 && c + i < tile.z) row[(size_t)i * p.out] = __float2bfloat16_rn(__uint_as_float(a[i]));
+          if (in1 && c + i < tile.z) row[(size_t)i * p.out + kMTile] = __float2bfloat16_rn(__uint_as_float(b[i]));
         }
       }
     }

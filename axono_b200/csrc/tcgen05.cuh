@@ -54,6 +54,39 @@ __device__ __forceinline__ void umma_commit(uint64_t *bar) {
                : "memory");
 }
 
+// The same three for a warp that walks its loop as a whole, with `lead` set in one lane: the instruction is
+// predicated, not branched around, so descriptors and counters stay warp-uniform for the compiler (inside a branch
+// for one lane it rebuilds every operand per instruction, and the issue of small products, not the tensor core, sets
+// their pace).
+__device__ __forceinline__ void umma_f16_lead(uint32_t tmem_d, uint64_t da, uint64_t db, uint32_t idesc, bool accumulate,
+                                              uint32_t lead) {
+  asm volatile(
+      "{\n.reg .pred p, q;\nsetp.ne.b32 p, %4, 0;\nsetp.ne.b32 q, %5, 0;\n"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}\n"
+      ::"r"(tmem_d), "l"(da), "l"(db), "r"(idesc), "r"((uint32_t)accumulate), "r"(lead)
+      : "memory");
+}
+__device__ __forceinline__ void umma_f16_ts_lead(uint32_t tmem_d, uint32_t tmem_a, uint64_t db, uint32_t idesc, bool accumulate,
+                                                 uint32_t lead) {
+  asm volatile(
+      "{\n.reg .pred p, q;\nsetp.ne.b32 p, %4, 0;\nsetp.ne.b32 q, %5, 0;\n"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n"
+      ::"r"(tmem_d), "r"(tmem_a), "l"(db), "r"(idesc), "r"((uint32_t)accumulate), "r"(lead)
+      : "memory");
+}
+__device__ __forceinline__ void umma_commit_lead(uint64_t *bar, uint32_t lead) {
+  asm volatile(
+      "{\n.reg .pred q;\nsetp.ne.b32 q, %1, 0;\n"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n}\n"
+      ::"r"(smem_u32(bar)), "r"(lead)
+      : "memory");
+}
+
+// A bounded wait of the whole warp.
+__device__ __forceinline__ bool mbar_wait_warp(uint64_t *bar, uint32_t parity, volatile int *abort_flag, unsigned long long limit_ns) {
+  return __all_sync(0xffffffffu, mbar_wait_bounded(bar, parity, abort_flag, limit_ns));
+}
+
 __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
   asm volatile(
       "tcgen05.ld.sync.aligned.32x32b.x32.b32 "

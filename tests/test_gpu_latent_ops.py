@@ -93,17 +93,19 @@ class Pages:
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_prepare_norms_rotates_and_appends(dtype):
+@pytest.mark.parametrize("heads,dim,rot,pairs,rank,q_rank", [(3, 20, 12, 4, 44, 36), (16, 128, 64, 32, 512, 1536), (5, 24, 16, 8, 136, 88),
+                                                             (7, 8, 64, 20, 264, 2048)])
+def test_prepare_norms_rotates_and_appends(heads, dim, rot, pairs, rank, q_rank, dtype):
     from axono_b200 import ops
 
-    heads, dim, rot, pairs, rank, q_rank, base, eps = 3, 20, 12, 4, 44, 36, 700.0, 1e-3
+    base, eps = 700.0, 1e-3
     pos = [0, 1, 63, 64, 65, 5000]
     n = len(pos)
     pages = Pages([6000], rank + rot, dtype)
     rows = pages.rows([0] * n, pos, 6000)
     inv = torch.tensor([base ** (-i / pairs) for i in range(pairs)], dtype=torch.float64).cuda()
     per = dim + rot
-    wide = rnd((n, heads * per + q_rank + rank + rot + 5), dtype, 1)  # one matrix, columns side by side
+    wide = rnd((n, heads * per + q_rank + rank + rot + 8), dtype, 1)  # one matrix, columns side by side
     wd = wide.cuda()
     dq_w, dkv_w = rnd((q_rank,), dtype, 2), rnd((rank,), dtype, 3)
     pool = pages.pool.cuda()
@@ -270,6 +272,20 @@ def test_route(experts, groups, keep, top):
         assert counts.tolist() == torch.bincount(ids.flatten().long(), minlength=experts).tolist()
         for e in range(experts):
             assert sorted(place[ids == e].tolist()) == list(range(int(counts[e])))
+
+
+def test_route_many_rows():
+    from axono_b200 import ops
+
+    n, experts = 9601, 64
+    logits = torch.randn(n, experts, generator=torch.Generator().manual_seed(1)) * 2
+    corr = torch.randn(experts, generator=torch.Generator().manual_seed(2)) - 2
+    ids, _, place, counts = (t.cpu() for t in ops.moe_route(logits.cuda(), corr.cuda(), 8, 3, 6, 1.0))
+    for t in range(0, n, 37):
+        assert ids[t].tolist() == plain.route_token(logits[t].double(), corr.double(), 6, 8, 3, 1.0)[0]
+    assert counts.tolist() == torch.bincount(ids.flatten().long(), minlength=experts).tolist()
+    for e in range(experts):
+        assert sorted(place[ids == e].tolist()) == list(range(int(counts[e])))
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
