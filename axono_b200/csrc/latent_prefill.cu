@@ -59,7 +59,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   }
   // heaviest blocks first: the last query block has the most key tiles
   const int h = blockIdx.y, q0 = (gridDim.x - 1 - blockIdx.x) * 2 * kRows;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = uniform_warp(), lane = threadIdx.x & 31;
   int nkv_g[2];
 #pragma unroll
   for (int g = 0; g < 2; ++g) {

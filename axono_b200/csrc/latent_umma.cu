@@ -158,7 +158,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
     if (threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_WAIT_TIMEOUT);
     return;
   }
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = uniform_warp(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     for (int i = 0; i < 4 * kMaxSlots + 2; ++i) mbar_init(&full_p[i], 1);  // rings and bar_s
     mbar_init(bar_p, 4);
@@ -201,7 +201,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
     // ================= loader (one lane) =================
     if (lane == 0) {
       tma_prefetch_descriptor(&tmPages);
-      int np = 0, ns = 0;  // chunk pairs and singles issued
+      RingPos rp, rs;      // chunk pairs and singles
+      int np = 0, ns = 0;  // how many were issued
       bool ok = true;
       for (int r = r_first, g = lo; g < hi && ok; ++r) {
         const int keys = visible_keys(p, r);
@@ -224,16 +225,16 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
           auto load_chunk = [&](uint8_t *dst, uint64_t *bar, int c) {
             for (int i = 0; i < halves; ++i) tma_load_2d(dst + i * (kChunk / 2), &tmPages, bar, c * 64, at[i]);
           };
-          for (int i = 0; i < u.singles && ok; ++i, ++ns) {
-            const int s = ns % u.single_slots;
-            if (ns >= u.single_slots) ok = mbar_wait_bounded(&empty_s[s], (ns / u.single_slots - 1) & 1, abort_flag, p.wait_ns);
+          for (int i = 0; i < u.singles && ok; ++i, ++ns, rs.next(u.single_slots)) {
+            const int s = rs.slot;
+            if (ns >= u.single_slots) ok = mbar_wait_bounded(&empty_s[s], rs.parity ^ 1, abort_flag, p.wait_ns);
             if (!ok) break;
             mbar_arrive_expect_tx(&full_s[s], halves * (kChunk / 2));
             load_chunk(smem + off_single + s * kChunk, &full_s[s], 2 * u.pairs + i);
           }
-          for (int i = 0; i < u.pairs && ok; ++i, ++np) {
-            const int s = np % u.pair_slots, n = min(2, u.chunks - 2 * i);
-            if (np >= u.pair_slots) ok = mbar_wait_bounded(&empty_p[s], (np / u.pair_slots - 1) & 1, abort_flag, p.wait_ns);
+          for (int i = 0; i < u.pairs && ok; ++i, ++np, rp.next(u.pair_slots)) {
+            const int s = rp.slot, n = min(2, u.chunks - 2 * i);
+            if (np >= u.pair_slots) ok = mbar_wait_bounded(&empty_p[s], rp.parity ^ 1, abort_flag, p.wait_ns);
             if (!ok) break;
             mbar_arrive_expect_tx(&full_p[s], n * halves * (kChunk / 2));
             for (int c = 0; c < n; ++c) load_chunk(smem + s * 2 * kChunk + c * kChunk, &full_p[s], 2 * i + c);
@@ -259,7 +260,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
     const uint64_t da = smem_desc(smem_u32(smem), 16, 1024);           // a chunk as [keys][elements]
     const uint64_t dv = smem_desc(smem_u32(smem), kChunk, 1024);       // a pair as latent elements x keys
     const uint64_t dq = smem_desc(smem_u32(smem + S::off_q(u)), 16, 1024), dp = smem_desc(smem_u32(smem + S::off_p(u)), 16, 1024);
-    int np = 0, ns = 0, tile = 0, seg = 0, pv = 0;
+    RingPos rp, rs, pv;  // pairs and singles of the scores, pairs of the sum
+    int tile = 0, seg = 0;
     bool ok = true;
     for (int r = r_first, g = lo; g < hi && ok; ++r) {
       if (start[r + 1] <= g) continue;
@@ -275,17 +277,17 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
           for (int ks = 0; ks < 4; ++ks) umma_f16_lead(ts, a + ks * 2, b + ks * 2, idesc_s, !first || ks > 0, lead);
           first = false;
         };
-        for (int i = 0; i < u.singles && ok; ++i, ++ns) {
-          const int s = ns % u.single_slots;
-          ok = mbar_wait_warp(&full_s[s], (ns / u.single_slots) & 1, abort_flag, p.wait_ns);
+        for (int i = 0; i < u.singles && ok; ++i, rs.next(u.single_slots)) {
+          const int s = rs.slot;
+          ok = mbar_wait_warp(&full_s[s], rs.parity, abort_flag, p.wait_ns);
           if (!ok) break;
           tc_fence_after();
           score_chunk(off_single + s * kChunk, 2 * u.pairs + i);
           umma_commit_lead(&empty_s[s], lead);
         }
-        for (int i = 0; i < u.pairs && ok; ++i, ++np) {
-          const int s = np % u.pair_slots;
-          ok = mbar_wait_warp(&full_p[s], (np / u.pair_slots) & 1, abort_flag, p.wait_ns);
+        for (int i = 0; i < u.pairs && ok; ++i, rp.next(u.pair_slots)) {
+          const int s = rp.slot;
+          ok = mbar_wait_warp(&full_p[s], rp.parity, abort_flag, p.wait_ns);
           if (!ok) break;
           tc_fence_after();
           for (int c = 0; c < 2 && 2 * i + c < u.chunks; ++c) score_chunk(s * 2 * kChunk + c * kChunk, 2 * i + c);
@@ -295,8 +297,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         ok = mbar_wait_warp(bar_p, tile & 1, abort_flag, p.wait_ns);
         if (!ok) break;
         tc_fence_after();
-        for (int i = 0; i < u.pairs; ++i, ++pv) {
-          const int s = pv % u.pair_slots;
+        for (int i = 0; i < u.pairs; ++i, pv.next(u.pair_slots)) {
+          const int s = pv.slot;
           const uint64_t a = dv + (uint64_t)(s * (2 * kChunk >> 4));
 #pragma unroll
           for (int ks = 0; ks < kKeys / 16; ++ks)  // 16 keys: 2 KB of the chunk, 32 bytes of P

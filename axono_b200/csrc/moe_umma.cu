@@ -51,7 +51,7 @@ moe_umma_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
     if (threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_WAIT_TIMEOUT);
     return;
   }
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = uniform_warp(), lane = threadIdx.x & 31;
   const bool shared = (int)blockIdx.y < up.shared_tiles;
   const MoeProduct &p = up.p[shared ? 1 : 0];
   constexpr int kMStep = kGateUp ? kMTile : 2 * kMTile;

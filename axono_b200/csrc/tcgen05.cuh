@@ -82,6 +82,22 @@ __device__ __forceinline__ void umma_commit_lead(uint64_t *bar, uint32_t lead) {
       : "memory");
 }
 
+// The warp's number as a value the compiler knows to be the same in all lanes: code behind a branch on it stays
+// warp-uniform.
+__device__ __forceinline__ int uniform_warp() { return __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0); }
+
+// Position in a ring of stages: slot, and the parity its barriers have there.
+struct RingPos {
+  int slot = 0;
+  uint32_t parity = 0;
+  __device__ __forceinline__ void next(int slots) {
+    if (++slot == slots) {
+      slot = 0;
+      parity ^= 1;
+    }
+  }
+};
+
 // A bounded wait of the whole warp.
 __device__ __forceinline__ bool mbar_wait_warp(uint64_t *bar, uint32_t parity, volatile int *abort_flag, unsigned long long limit_ns) {
   return __all_sync(0xffffffffu, mbar_wait_bounded(bar, parity, abort_flag, limit_ns));
