@@ -110,7 +110,7 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prepare_kernel(const Prep
 // bf16 with sizes and addresses that allow 16-byte accesses and at most 32 rotated pairs: one CTA per row, its warps
 // take turns at the row's jobs - the cached row, the query latent, then 32 chunks of 8 query elements at a time.
 // Lane i holds the sine and cosine of pair i; the sums of the norms stay inside a warp.
-constexpr int kPrepVecWarps = 4, kPrepVecChunks = 8;  // a warp norms up to 8 x 256 elements out of registers
+constexpr int kPrepVecWarps = 4;
 
 struct Bf16x8 {
   uint4 raw;
@@ -124,7 +124,7 @@ struct Bf16x8 {
   }
 };
 
-__global__ void __launch_bounds__(kPrepVecWarps * 32) latent_prepare_vec_kernel(const PrepareParams<__nv_bfloat16> p) {
+__global__ void __launch_bounds__(kPrepVecWarps * 32, 10) latent_prepare_vec_kernel(const PrepareParams<__nv_bfloat16> p) {
   const int64_t r = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   grid_dependency_wait();
@@ -146,34 +146,28 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32) latent_prepare_vec_kernel(
     }
   };
   auto norm = [&](const __nv_bfloat16 *src, const __nv_bfloat16 *weight, __nv_bfloat16 *dst, int n) {
-    Bf16x8 x[kPrepVecChunks];
+    // the source is read twice, the second time from L1: holding it would cost the registers that keep enough
+    // rows in flight
+    Bf16x8 x, ww;
     float v[8], w[8], sq = 0.f;
-#pragma unroll
-    for (int k = 0; k < kPrepVecChunks; ++k) {
-      const int e = (k * 32 + lane) * 8;
-      if (e >= n) break;
-      x[k].raw = *reinterpret_cast<const uint4 *>(src + e);
-    }
-#pragma unroll
-    for (int k = 0; k < kPrepVecChunks; ++k) {
-      if ((k * 32 + lane) * 8 >= n) break;
-      x[k].get(v);
+#pragma unroll 2
+    for (int e = lane * 8; e < n; e += 256) {
+      x.raw = *reinterpret_cast<const uint4 *>(src + e);
+      x.get(v);
 #pragma unroll
       for (int i = 0; i < 8; ++i) sq = fmaf(v[i], v[i], sq);
     }
     const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)n + p.eps);
-#pragma unroll
-    for (int k = 0; k < kPrepVecChunks; ++k) {
-      const int e = (k * 32 + lane) * 8;
-      if (e >= n) break;
-      Bf16x8 ww;
+#pragma unroll 2
+    for (int e = lane * 8; e < n; e += 256) {
+      x.raw = *reinterpret_cast<const uint4 *>(src + e);
       ww.raw = *reinterpret_cast<const uint4 *>(weight + e);
-      x[k].get(v);
+      x.get(v);
       ww.get(w);
 #pragma unroll
       for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * w[i];
-      x[k].set(v);
-      *reinterpret_cast<uint4 *>(dst + e) = x[k].raw;
+      x.set(v);
+      *reinterpret_cast<uint4 *>(dst + e) = x.raw;
     }
   };
   const int rot_chunks = p.rot_dim / 8;
@@ -228,11 +222,10 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32) latent_prepare_vec_kernel(
 
 bool prepare_vec_takes(const PrepareParams<__nv_bfloat16> &p) {
   const auto al = [](const void *q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
-  const int limit = kPrepVecChunks * 256;
   return p.rot_pairs <= 32 && p.rot_dim > 0 && p.rot_dim % 8 == 0 && p.rot_pairs * 2 == p.rot_dim &&
          (!p.q || (al(p.q) && p.dim % 8 == 0 && p.q_ld % 8 == 0)) &&
-         (!p.dq || (al(p.dq) && al(p.dq_w) && al(p.cq) && p.q_rank % 8 == 0 && p.dq_ld % 8 == 0 && p.q_rank <= limit)) &&
-         (!p.dkv || (al(p.dkv) && al(p.dkv_w) && al(p.pages) && p.kv_rank % 8 == 0 && p.dkv_ld % 8 == 0 && p.kv_rank <= limit));
+         (!p.dq || (al(p.dq) && al(p.dq_w) && al(p.cq) && p.q_rank % 8 == 0 && p.dq_ld % 8 == 0)) &&
+         (!p.dkv || (al(p.dkv) && al(p.dkv_w) && al(p.pages) && p.kv_rank % 8 == 0 && p.dkv_ld % 8 == 0));
 }
 
 // ---- attention in latent form -------------------------------------------------------------------------

@@ -319,10 +319,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
     const int tid = threadIdx.x, elems = p.kv_rank + p.rot_dim;
     int tile = 0, seg = 0, np = 0;
     bool ok = true;
-    for (int r = r_first, g = lo; g < hi && ok; ++r) {
-      if (start[r + 1] <= g) continue;
-      const int k_first = g - start[r], g_end = min(hi, start[r + 1]), keys = visible_keys(p, r);
-      // ---- the item's queries, heads x elements, 16-byte pieces into the swizzled boxes ----
+    // an item's queries, heads x elements, in 16-byte pieces into the swizzled boxes
+    auto put_queries = [&](int r) {
       for (int i = tid; i < kN * u.chunks * 8; i += kSoftmax) {
         const int h = i / (u.chunks * 8), e = (i - h * (u.chunks * 8)) * 8;
         uint4 v = make_uint4(0, 0, 0, 0);
@@ -336,6 +334,11 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_q);
+    };
+    for (int r = r_first, g = lo; g < hi && ok; ++r) {
+      if (start[r + 1] <= g) continue;
+      const int k_first = g - start[r], g_end = min(hi, start[r + 1]), keys = visible_keys(p, r);
+      if (seg == 0) put_queries(r);
       ++seg;
       float l[kN];
 #pragma unroll
@@ -420,6 +423,13 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         if (lane == 0) mbar_arrive(bar_p);
       }
       if (!ok) break;
+      // The scores of the item's last tile are done (bar_s), so its queries may be replaced: the next item's first
+      // scores are then computed while this item's result is stored.
+      if (g < hi) {
+        int r_next = r + 1;
+        while (start[r_next + 1] <= g) ++r_next;
+        put_queries(r_next);
+      }
       // ---- the item, or this range's part of it ----
       const float sum = reduce_heads<kN>(l, lane, [](float a, float b) { return a + b; });
       if (kN == 32 || (lane & 1) == 0) red[warp][lane * kN / 32] = sum;
