@@ -119,35 +119,39 @@ moe_umma_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
       }
       if (ok) umma_commit_lead(done, lead);
     }
-  } else if (__all_sync(0xffffffffu, mbar_wait_bounded(done, 0, abort_flag, p.wait_ns))) {
+  } else {
+    mbar_wait_bounded(done, 0, abort_flag, p.wait_ns);
+    named_bar_sync(1, 256);  // a wait that ran out raised the flag before this: all eight warps see the same
     tc_fence_after();
-    // warps w and w + 4 share a quarter of the lanes (features) and take every other 16 columns (rows)
+    const int rows = *abort_flag ? 0 : tile.z;
+    // warps w and w + 4 share a quarter of the lanes (features) and take every other 16 columns (rows); the results
+    // cross shared memory - every stage has been consumed - so that whole rows of features leave in 16-byte pieces
     const uint32_t base = tmem + ((uint32_t)((warp & 3) * 32) << 16);
-    const int f0 = m0 + (warp & 3) * 32 + lane;
-    const bool in0 = f0 < p.out, in1 = f0 + kMTile < p.out;
-    __nv_bfloat16 *y = static_cast<__nv_bfloat16 *>(p.y) + (size_t)tile.y * p.out + f0;
+    constexpr int kPitch = kMStep * 2, kPieces = kPitch / 16;
+    uint8_t *mine = smem + ((warp & 3) * 32 + lane) * 2;
 #pragma unroll 1
-    for (int c = (warp >> 2) * 16; c < kN && c < tile.z; c += 32) {
+    for (int c = (warp >> 2) * 16; c < kN && c < rows; c += 32) {
       uint32_t a[16], b[16];
       tmem_ld16_async(base + c, a);
       tmem_ld16_async(base + kN + c, b);
       tmem_wait_ld();
-      __nv_bfloat16 *row = y + (size_t)c * p.out;
-      if (kGateUp) {
-        __nv_bfloat16 v[16];
 #pragma unroll
-        for (int i = 0; i < 16; ++i)
-          v[i] = __float2bfloat16_rn(clamped_gate<false>(__uint_as_float(a[i]), __uint_as_float(b[i]), p.act));
-#pragma unroll
-        for (int i = 0; i < 16; ++i)
-          if (in0 && c + i < tile.z) row[(size_t)i * p.out] = v[i];
-      } else {
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          if (in0 && c + i < tile.z) row[(size_t)i * p.out] = __float2bfloat16_rn(__uint_as_float(a[i]));
-          if (in1 && c + i < tile.z) row[(size_t)i * p.out + kMTile] = __float2bfloat16_rn(__uint_as_float(b[i]));
+      for (int i = 0; i < 16; ++i) {
+        __nv_bfloat16 *row = reinterpret_cast<__nv_bfloat16 *>(mine + (c + i) * kPitch);
+        const float va = __uint_as_float(a[i]), vb = __uint_as_float(b[i]);
+        if (kGateUp) {
+          row[0] = __float2bfloat16_rn(clamped_gate<false>(va, vb, p.act));
+        } else {
+          row[0] = __float2bfloat16_rn(va);
+          row[kMTile] = __float2bfloat16_rn(vb);
         }
       }
+    }
+    named_bar_sync(1, 256);
+    __nv_bfloat16 *y = static_cast<__nv_bfloat16 *>(p.y) + (size_t)tile.y * p.out + m0;
+    for (int i = threadIdx.x; i < rows * kPieces; i += 256) {
+      const int n = i / kPieces, f = i % kPieces * 8;
+      if (m0 + f < p.out) *reinterpret_cast<uint4 *>(y + (size_t)n * p.out + f) = *reinterpret_cast<const uint4 *>(smem + n * kPitch + f * 2);
     }
   }
   tc_fence_before();
