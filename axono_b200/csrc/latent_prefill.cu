@@ -139,8 +139,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       }
     }
   } else if (warp == kMmaWarp) {
-    const uint32_t lead = lane == 0;  // the warp walks, one lane issues
-    {
+    if (lane == 0) {
       // fp32 accumulate, bf16 operands, M = 128.  Q.K^T: N = 128, B K-major; P.V: N = kVB * 64, B MN-major
       constexpr uint32_t kBf16 = (1u << 4) | (1u << 7) | (1u << 10) | ((kRows >> 4) << 24);
       constexpr uint32_t idesc_qk = kBf16 | ((kKeys >> 3) << 17), idesc_pv = kBf16 | (1u << 16) | ((kVB * 64 >> 3) << 17);
@@ -152,16 +151,16 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 #pragma unroll
         for (int ks = 0; ks < L::kBlocks * 4; ++ks) {
           const uint32_t off = ((ks >> 2) * kBox + (ks & 3) * 32) >> 4;
-          umma_f16_lead(tmem + g * 128, dqg + off, dks + off, idesc_qk, ks > 0, lead);
+          umma_f16(tmem + g * 128, dqg + off, dks + off, idesc_qk, ks > 0);
         }
-        umma_commit_lead(&bar_s[g], lead);
+        umma_commit(&bar_s[g]);
       };
-      bool ok = mbar_wait_warp(bar_q, 0, abort_flag, p.wait_ns) && mbar_wait_warp(&full_k[0], 0, abort_flag, p.wait_ns);
+      bool ok = mbar_wait_bounded(bar_q, 0, abort_flag, p.wait_ns) && mbar_wait_bounded(&full_k[0], 0, abort_flag, p.wait_ns);
       if (ok) {
         tc_fence_after();
         if (nkv_g[0] > 0) issue_s(0, 0);
         if (nkv_g[1] > 0) issue_s(1, 0);
-        umma_commit_lead(&empty_k[0], lead);
+        umma_commit(&empty_k[0]);
       }
       for (int j = 0; j < nkv && ok; ++j) {
         const int last_g = nkv_g[1] > j ? 1 : 0;
@@ -169,31 +168,31 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 #pragma unroll
         for (int g = 0; g < 2; ++g) {
           if (j >= nkv_g[g]) continue;
-          ok = mbar_wait_warp(&bar_p[g], j & 1, abort_flag, p.wait_ns);
+          ok = mbar_wait_bounded(&bar_p[g], j & 1, abort_flag, p.wait_ns);
           if (!ok) break;
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
-            ok = ok && mbar_wait_warp(&full_v[half], j & 1, abort_flag, p.wait_ns);
+            ok = ok && mbar_wait_bounded(&full_v[half], j & 1, abort_flag, p.wait_ns);
             if (!ok) break;
             tc_fence_after();
             const uint64_t dvh = dv + (uint64_t)(half * (L::kVHalf >> 4));
 #pragma unroll
             for (int ks = 0; ks < 4; ++ks)  // 16 keys: 8 columns of P, 2 KB of V
-              umma_f16_ts_lead(tmem_o(g), tmem_p(g) + half * 32 + ks * 8, dvh + (uint64_t)(ks * (2048 >> 4)), idesc_pv,
-                          j > 0 || half > 0 || ks > 0, lead);
-            if (g == last_g) umma_commit_lead(&empty_v[half], lead);
+              umma_f16_ts(tmem_o(g), tmem_p(g) + half * 32 + ks * 8, dvh + (uint64_t)(ks * (2048 >> 4)), idesc_pv,
+                          j > 0 || half > 0 || ks > 0);
+            if (g == last_g) umma_commit(&empty_v[half]);
           }
           if (!ok) break;
-          if (j == nkv_g[g] - 1) umma_commit_lead(&bar_fin[g], lead);
+          if (j == nkv_g[g] - 1) umma_commit(&bar_fin[g]);
           if (j + 1 < nkv_g[g]) {
-            if (!have_k) ok = mbar_wait_warp(&full_k[(j + 1) & 1], ((j + 1) >> 1) & 1, abort_flag, p.wait_ns);
+            if (!have_k) ok = mbar_wait_bounded(&full_k[(j + 1) & 1], ((j + 1) >> 1) & 1, abort_flag, p.wait_ns);
             if (!ok) break;
             have_k = true;
             tc_fence_after();
             issue_s(g, j + 1);
           }
         }
-        if (ok && j + 1 < nkv) umma_commit_lead(&empty_k[(j + 1) & 1], lead);
+        if (ok && j + 1 < nkv) umma_commit(&empty_k[(j + 1) & 1]);
       }
     }
   } else {
