@@ -213,11 +213,17 @@ int launch_n(int n, const UmmaParams &up, const CUtensorMap (&maps)[4], dim3 gri
 
 bool moe_umma_takes(int width, int ff) { return width % 8 == 0 && ff % 8 == 0; }
 
-// Rows per tile: about twice what an expert gets on average, so that few experts need a second tile (which
-// reads the weights again) and little of the MMA is spent on empty columns.
+// Rows per tile.  Few rows per expert: the time is the reading of the weights, and a tile that holds nearly every
+// expert's rows reads them once at the least cost per column.  Many: the columns that the tiles of an expert with a
+// typical number of rows (average plus two standard deviations) cover, those of 128 weighted with what they lose to
+// operand traffic against 256.
 int moe_umma_tile_rows(int64_t rows, int experts) {
   const int64_t avg = rows / experts;
-  return avg <= 10 ? 16 : avg <= 22 ? 32 : avg <= 48 ? 64 : avg <= 110 ? 128 : 256;
+  if (avg <= 36) return avg <= 7 ? 16 : avg <= 30 ? 32 : 64;
+  int64_t sd = 1;
+  while (sd * sd < avg) ++sd;
+  const int64_t typical = avg + 2 * sd;
+  return 10 * ((typical + 255) / 256) * 256 <= 12 * ((typical + 127) / 128) * 128 ? 256 : 128;
 }
 
 bool moe_umma_supported(const MoeProduct &p, bool gate_up) {

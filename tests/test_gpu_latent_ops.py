@@ -290,7 +290,7 @@ def test_route_many_rows():
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("width,ff,experts,top,n", [(76, 44, 6, 3, 50), (200, 72, 12, 3, 9), (256, 96, 8, 3, 1), (384, 192, 16, 4, 300),
-                                                    (512, 384, 4, 2, 1500), (256, 128, 3, 3, 33), (128, 256, 32, 1, 40)])
+                                                    (512, 384, 4, 2, 1500), (256, 128, 8, 2, 60), (256, 128, 3, 3, 33), (128, 256, 32, 1, 40)])
 def test_experts(dtype, width, ff, experts, top, n):
     """Routed and shared expert products, with gates and ups on both sides of the clamps; some experts get no row."""
     from axono_b200 import ops
@@ -298,7 +298,7 @@ def test_experts(dtype, width, ff, experts, top, n):
 
     x = rnd((n, width), dtype, 1)
     gu, down = rnd((experts, 2, ff, width), dtype, 2, 1.5 / math.sqrt(width)), rnd((experts, width, ff), dtype, 3, 1 / math.sqrt(ff))
-    sff = ff + 8
+    sff = ff + (4 if n == 9 else 8)  # 4: a shared expert whose size the tensor-core form does not take beside routed ones it does
     sgu, sdown = rnd((1, 2, sff, width), dtype, 4, 1.5 / math.sqrt(width)), rnd((1, width, sff), dtype, 5, 1 / math.sqrt(sff))
     corr = torch.linspace(0, 1, experts)
     corr[0] = -9.0  # never chosen while others are left
