@@ -124,12 +124,30 @@ struct Bf16x8 {
   }
 };
 
-__global__ void __launch_bounds__(kPrepVecWarps * 32, 10) latent_prepare_vec_kernel(const PrepareParams<__nv_bfloat16> p) {
+__global__ void __launch_bounds__(kPrepVecWarps * 32, 9) latent_prepare_vec_kernel(const PrepareParams<__nv_bfloat16> p) {
   const int64_t r = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   grid_dependency_wait();
   grid_dependency_launch();
   const int pos = p.row_pos[r];
+  // what a warp needs first is on its way while the angles are evaluated
+  const int rot_chunks = p.rot_dim / 8, q_chunks = p.q ? p.heads * rot_chunks : 0;
+  auto q_chunk = [&](int i) {  // address of chunk i of the rotated query parts
+    const int h = i / rot_chunks;
+    return p.q + r * p.q_ld + (int64_t)h * (p.dim + p.rot_dim) + p.dim + (i - h * rot_chunks) * 8;
+  };
+  const int first_q = warp < 2 ? warp + kPrepVecWarps : warp;  // the first of this warp's jobs from 2 on
+  Bf16x8 ahead;
+  ahead.raw = make_uint4(0, 0, 0, 0);
+  if ((first_q - 2) * 32 + lane < q_chunks) ahead.raw = *reinterpret_cast<const uint4 *>(q_chunk((first_q - 2) * 32 + lane));
+  Bf16x8 ahead_norm[2];  // warp 0: of the row to cache, warp 1: of the query latent
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int e = (k * 32 + lane) * 8;
+    ahead_norm[k].raw = make_uint4(0, 0, 0, 0);
+    if (warp == 0 && p.dkv && e < p.kv_rank) ahead_norm[k].raw = *reinterpret_cast<const uint4 *>(p.dkv + r * p.dkv_ld + e);
+    if (warp == 1 && p.dq && e < p.q_rank) ahead_norm[k].raw = *reinterpret_cast<const uint4 *>(p.dq + r * p.dq_ld + e);
+  }
   float c = 1.f, s = 0.f;
   if (lane < p.rot_pairs) {
     const double turns = (double)pos * p.inv_freq[lane] * 0.15915494309189533577;  // 1 / (2 pi)
@@ -146,21 +164,25 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 10) latent_prepare_vec_ker
     }
   };
   auto norm = [&](const __nv_bfloat16 *src, const __nv_bfloat16 *weight, __nv_bfloat16 *dst, int n) {
-    // the source is read twice, the second time from L1: holding it would cost the registers that keep enough
-    // rows in flight
-    Bf16x8 x, ww;
-    float v[8], w[8], sq = 0.f;
-#pragma unroll 2
-    for (int e = lane * 8; e < n; e += 256) {
-      x.raw = *reinterpret_cast<const uint4 *>(src + e);
+    // the first 512 elements are in registers, the rest is read twice, the second time from L1: holding more would
+    // cost the registers that keep enough rows in flight
+    float v[8], sq = 0.f;
+    auto square = [&](const Bf16x8 &x) {
       x.get(v);
 #pragma unroll
       for (int i = 0; i < 8; ++i) sq = fmaf(v[i], v[i], sq);
+    };
+#pragma unroll
+    for (int k = 0; k < 2; ++k) square(ahead_norm[k]);  // zeros past the end
+    Bf16x8 x;
+    for (int e = 512 + lane * 8; e < n; e += 256) {
+      x.raw = *reinterpret_cast<const uint4 *>(src + e);
+      square(x);
     }
     const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)n + p.eps);
-#pragma unroll 2
-    for (int e = lane * 8; e < n; e += 256) {
-      x.raw = *reinterpret_cast<const uint4 *>(src + e);
+    auto scale_store = [&](Bf16x8 x, int e) {
+      Bf16x8 ww;
+      float w[8];
       ww.raw = *reinterpret_cast<const uint4 *>(weight + e);
       x.get(v);
       ww.get(w);
@@ -168,9 +190,15 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 10) latent_prepare_vec_ker
       for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * w[i];
       x.set(v);
       *reinterpret_cast<uint4 *>(dst + e) = x.raw;
+    };
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      if ((k * 32 + lane) * 8 < n) scale_store(ahead_norm[k], (k * 32 + lane) * 8);
+    for (int e = 512 + lane * 8; e < n; e += 256) {
+      x.raw = *reinterpret_cast<const uint4 *>(src + e);
+      scale_store(x, e);
     }
   };
-  const int rot_chunks = p.rot_dim / 8;
   for (int job = warp;; job += kPrepVecWarps) {
     if (job == 0) {
       if (!p.dkv) continue;
@@ -201,20 +229,16 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 10) latent_prepare_vec_ker
     } else if (job == 1) {
       if (p.dq) norm(p.dq + r * p.dq_ld, p.dq_w, p.cq + r * p.q_rank, p.q_rank);
     } else {
-      const int total = p.q ? p.heads * rot_chunks : 0, i = (job - 2) * 32 + lane;
-      if ((job - 2) * 32 >= total) break;
-      Bf16x8 x;
-      float v[8] = {};
-      const int h = i / rot_chunks, j = i - h * rot_chunks;
-      __nv_bfloat16 *e = p.q + r * p.q_ld + (int64_t)h * (p.dim + p.rot_dim) + p.dim + j * 8;
-      if (i < total) {
-        x.raw = *reinterpret_cast<const uint4 *>(e);
-        x.get(v);
-      }
-      rotate(v, j);
-      if (i < total) {
+      const int i = (job - 2) * 32 + lane;
+      if ((job - 2) * 32 >= q_chunks) break;
+      Bf16x8 x = ahead;
+      if (job != first_q && i < q_chunks) x.raw = *reinterpret_cast<const uint4 *>(q_chunk(i));
+      float v[8];
+      x.get(v);
+      rotate(v, i % rot_chunks);
+      if (i < q_chunks) {
         x.set(v);
-        *reinterpret_cast<uint4 *>(e) = x.raw;
+        *reinterpret_cast<uint4 *>(q_chunk(i)) = x.raw;
       }
     }
   }
