@@ -69,6 +69,7 @@ SIGNATURES = {
                                           _vp, _sz, _vp]),
     "axb200_kv_arena_create": (_i, [_i, _i, _i, _i, _i, _i, _i, _i, _i, C.POINTER(_vp)]),
     "axb200_kv_arena_create_rows": (_i, [_i, _vp, _i, _i, _i, _i, _i, _i, C.POINTER(_vp)]),
+    "axb200_kv_arena_add_state": (_i, [_vp, _i64, C.POINTER(_vp)]),
     "axb200_kv_arena_destroy": (_i, [_vp]),
     "axb200_kv_arena_alloc_seq": (_i, [_vp, _i64, C.POINTER(_i)]),
     "axb200_kv_arena_reserve": (_i, [_vp, _i, _i64]),
@@ -96,13 +97,25 @@ SIGNATURES = {
     "axb200_linear_strided": (_i, [_vp] * 3 + [_i64] * 10 + [_i] * 3 + [_vp]),
     "axb200_embed_layer_norm": (_i, [_vp, _vp, _vp, _f, _vp, _i64, _i64, _i, _i, _vp]),
     "axb200_residual_layer_norm": (_i, [_vp] * 6 + [_i] + [_vp] * 4 + [_f, _i64, _i, _i, _vp]),
+    "axb200_embed_residual": (_i, [_vp] * 4 + [_i64, _i64, _i, _i, _vp]),
+    "axb200_residual_post_norm": (_i, [_vp, _vp, _vp, _f, _f, _vp, _vp, _i64, _i, _i, _vp]),
     "axb200_latent_prepare": (_i, [_vp, _i64, _i, _i, _vp, _i64, _i, _vp, _vp, _vp, _i64, _i, _vp, _f] + [_vp] * 5 +
                               [_i, _i, _i64] + [_i] * 5 + [_vp]),
     "axb200_latent_attend_workspace_bytes": (_sz, [_i, _i, _i, _i, _i64, _i]),
-    "axb200_latent_attend": (_i, [_vp, _vp, _i64, _i] + [_vp] * 5 + [_i] * 4 + [_f] + [_i] * 4 + [_i64, _i, _vp, _sz, _vp]),
-    "axb200_latent_gather": (_i, [_vp, _vp, _vp, _i64, _i, _i, _i, _i, _i, _vp]),
+    # q_lat, q, q_ld, dim | out, pages, block_table, row_seq, row_pos, sink | rows, heads, kv_heads, kv_rank, rot_dim,
+    # row_elems, key_scale, window | scale | page_tokens, max_blocks, num_pages, max_seqs | max_len, dtype, workspace
+    "axb200_latent_attend": (_i, [_vp, _vp, _i64, _i] + [_vp] * 6 + [_i] * 8 + [_f] + [_i] * 4 + [_i64, _i, _vp, _sz, _vp]),
+    "axb200_latent_gather": (_i, [_vp, _vp, _vp, _i64, _i64, _i, _i, _i, _i, _i, _vp]),
     "axb200_latent_prefill_supported": (_i, [_i] * 5),
-    "axb200_latent_prefill": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _i, _i64, _i, _i, _i, _i, _f, _i, _vp]),
+    "axb200_latent_prefill": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _i, _i64] + [_i] * 6 + [_f, _i, _vp]),
+    "axb200_shared_kv_prepare": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _f] + [_vp] * 4 + [_i64] + [_i] * 10 + [_vp]),
+    "axb200_shared_kv_gather": (_i, [_vp] * 4 + [_i64] * 2 + [_i] * 8 + [_vp]),
+    # proj, ld, row_seq, row_pos[, row_back, first], rows, conv, a_log, dt_bias, norm, ring, state | operands | heads,
+    # kv_heads, dim, vdim, taps, max_seqs, eps, dtype, stream
+    "axb200_delta_step": (_i, [_vp, _i64, _vp, _vp, _i] + [_vp] * 6 + [_vp] + [_i] * 6 + [_f, _i, _vp]),
+    "axb200_delta_prepare": (_i, [_vp, _i64, _vp, _vp, _vp, _i, _i] + [_vp] * 6 + [_vp] * 4 + [_i] * 6 + [_f, _i, _vp]),
+    "axb200_delta_scan": (_i, [_vp, _i, _i] + [_vp] * 6 + [_i] * 6 + [_vp]),
+    "axb200_delta_finish": (_i, [_vp, _i64, _vp, _vp, _vp, _i, _i] + [_vp] * 6 + [_vp] * 2 + [_i] * 6 + [_f, _i, _vp]),
     "axb200_moe_route": (_i, [_vp] * 6 + [_i64, _i, _i, _i, _i, _f, _vp]),
     "axb200_moe_tile_rows": (_i, [_i64, _i, _i, _i, _i]),
     "axb200_moe_sort": (_i, [_vp] * 9 + [_i64, _i, _i, _i, _i, _i, _vp]),

@@ -31,6 +31,18 @@ struct Vec<__half> {
   }
 };
 
+template <>
+struct Vec<__nv_bfloat16> {
+  static constexpr int kN = 8;
+  uint4 raw;
+  __device__ __forceinline__ float get(int i) const {
+    return __bfloat162float(reinterpret_cast<const __nv_bfloat16 *>(&raw)[i]);
+  }
+  __device__ __forceinline__ void set(int i, float v) {
+    reinterpret_cast<__nv_bfloat16 *>(&raw)[i] = __float2bfloat16_rn(v);
+  }
+};
+
 // ---- add_rms_norm: y = x + res; out = y * rsqrt(mean(y^2) + eps) * w -----------------------------
 // One CTA per row.  Vector path: each thread keeps up to kMaxVec 16-byte vectors of y in
 // registers between the two phases, so x and res are read once and y/out written once.
@@ -424,21 +436,20 @@ int axb200_silu_mul(const void *gate, const void *up, void *out, int64_t n, int 
 
 int axb200_silu_mul_rows(const void *gate_up, int64_t ld, int n, int64_t rows, void *out, int dtype,
                          void *stream) {
-  if (dtype != AXB200_FLOAT32 && dtype != AXB200_FLOAT16) return AXB200_UNSUPPORTED_TYPE;
+  if (axb::dtype_size(dtype) == 0) return AXB200_UNSUPPORTED_TYPE;
   if (!gate_up || !out) return AXB200_INVALID_PTR;
   if (n <= 0 || rows < 0 || ld < 2 * (int64_t)n) return AXB200_INVALID_ARGUMENT;
   if (rows == 0) return AXB200_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dtype == AXB200_FLOAT32) {
-    const bool vec = n % 4 == 0 && ld % 4 == 0 && axb::al16(gate_up) && axb::al16(out);
-    axb::silu_mul_rows_kernel<float><<<axb::blocks_for(rows * n / (vec ? 4 : 1), 256), 256, 0, st>>>(
-        static_cast<const float *>(gate_up), ld, n, rows, static_cast<float *>(out), vec);
-  } else {
-    const bool vec = n % 8 == 0 && ld % 8 == 0 && axb::al16(gate_up) && axb::al16(out);
-    axb::silu_mul_rows_kernel<__half><<<axb::blocks_for(rows * n / (vec ? 8 : 1), 256), 256, 0, st>>>(
-        static_cast<const __half *>(gate_up), ld, n, rows, static_cast<__half *>(out), vec);
-  }
-  return axb::launch_status();
+  auto go = [&](auto tag) {
+    using T = decltype(tag);
+    constexpr int kN = axb::Vec<T>::kN;
+    const bool vec = n % kN == 0 && ld % kN == 0 && axb::al16(gate_up) && axb::al16(out);
+    axb::silu_mul_rows_kernel<T><<<axb::blocks_for(rows * n / (vec ? kN : 1), 256), 256, 0, st>>>(
+        static_cast<const T *>(gate_up), ld, n, rows, static_cast<T *>(out), vec);
+    return axb::launch_status();
+  };
+  return dtype == AXB200_FLOAT32 ? go(float{}) : dtype == AXB200_FLOAT16 ? go(__half{}) : go(__nv_bfloat16{});
 }
 
 int axb200_embedding(const void *ids, int ids_dtype, const void *table, void *out, int64_t n,

@@ -8,6 +8,8 @@
 //     kernels mask by sequence length, so stale bytes in a recycled page cannot be read);
 //   * sequences own pages through a block table (max_seqs, max_blocks) shared by all layers; a
 //     sequence slot is the batch row the kernels see;
+//   * state that does not grow with a sequence (recurrent mixers) has a pool of fixed size per slot
+//     (add_state); it is not cleared between sequences, the kernels start a sequence's first token from zero;
 //   * alloc / reserve / free are host-side and O(pages touched); the device copies of the block
 //     table are refreshed by axb200_kv_arena_sync (one H2D copy of the dirty rows' span).
 // With device_memory == 0 only the bookkeeping exists (no CUDA call is made): that mode is what the
@@ -33,6 +35,8 @@ struct axb200_kv_arena {
   int32_t *seq_lens_dev = nullptr;
   std::vector<size_t> pool_bytes;            // per layer, of each of its pools
   bool has_v = true;
+  std::vector<void *> states;                // pools of per-slot state
+  std::vector<size_t> state_bytes;           // per slot
 };
 
 namespace {
@@ -62,7 +66,7 @@ int reserve_locked(axb200_kv_arena *a, int seq, int64_t tokens) {
 // row_elems[l]: elements of one token's row in layer l's pool (K pool, and V pool when has_v)
 int create_arena(int n_layers, const int32_t *row_elems, bool has_v, int num_pages, int hkv, int page_tokens, int d,
                  int dtype, int max_seqs, int max_blocks, int device_memory, axb200_kv_arena **out) {
-  if (n_layers <= 0 || num_pages <= 0 || hkv <= 0 || page_tokens <= 0 || page_tokens % 64 != 0 ||
+  if (n_layers < 0 || (n_layers == 0 && has_v) || num_pages <= 0 || hkv <= 0 || page_tokens <= 0 || page_tokens % 64 != 0 ||
       d <= 0 || max_seqs <= 0 || max_blocks <= 0 || axb::dtype_size(dtype) == 0)
     return AXB200_INVALID_ARGUMENT;
   for (int l = 0; l < n_layers; ++l)
@@ -131,9 +135,29 @@ int axb200_kv_arena_create(int n_layers, int num_pages, int hkv, int page_tokens
 
 int axb200_kv_arena_create_rows(int n_layers, const int32_t *row_elems, int num_pages, int page_tokens, int dtype,
                                 int max_seqs, int max_blocks, int device_memory, axb200_kv_arena **out) {
-  if (!out || !row_elems) return AXB200_INVALID_PTR;
-  return create_arena(n_layers, row_elems, false, num_pages, 1, page_tokens, n_layers > 0 ? row_elems[0] : 0, dtype, max_seqs,
+  if (!out || (!row_elems && n_layers > 0)) return AXB200_INVALID_PTR;
+  return create_arena(n_layers, row_elems, false, num_pages, 1, page_tokens, n_layers > 0 ? row_elems[0] : 1, dtype, max_seqs,
                       max_blocks, device_memory, out);
+}
+
+int axb200_kv_arena_add_state(axb200_kv_arena *a, int64_t bytes_per_seq, void **pool) {
+  if (!a || !pool) return AXB200_INVALID_PTR;
+  if (bytes_per_seq <= 0) return AXB200_INVALID_ARGUMENT;
+  std::lock_guard<std::mutex> lock(a->mu);
+  *pool = nullptr;
+  if (a->device) {
+    const size_t bytes = (size_t)bytes_per_seq * a->max_seqs;
+    void *p = nullptr;
+    if (cudaMalloc(&p, bytes) != cudaSuccess || cudaMemset(p, 0, bytes) != cudaSuccess) {
+      cudaGetLastError();
+      if (p) cudaFree(p);
+      return AXB200_OUT_OF_MEMORY;
+    }
+    *pool = p;
+    a->states.push_back(p);
+  }
+  a->state_bytes.push_back((size_t)bytes_per_seq);
+  return AXB200_OK;
 }
 
 int axb200_kv_arena_shuffle_free(axb200_kv_arena *a, uint64_t seed) {
@@ -156,6 +180,7 @@ int axb200_kv_arena_destroy(axb200_kv_arena *a) {
     cudaDeviceSynchronize();
     for (void *p : a->k_pools) cudaFree(p);
     for (void *p : a->v_pools) cudaFree(p);
+    for (void *p : a->states) cudaFree(p);
     cudaFree(a->table_dev);
     cudaFree(a->seq_lens_dev);
   }
@@ -240,6 +265,7 @@ int axb200_kv_arena_stats(axb200_kv_arena *a, int64_t *pages_total, int64_t *pag
   if (device_bytes) {
     *device_bytes = 0;
     for (size_t bytes : a->pool_bytes) *device_bytes += a->device ? (int64_t)(bytes * (a->has_v ? 2 : 1)) : 0;
+    for (size_t bytes : a->state_bytes) *device_bytes += a->device ? (int64_t)(bytes * a->max_seqs) : 0;
   }
   return AXB200_OK;
 }

@@ -8,7 +8,11 @@
 // (latent_prefill.cu) reads from.
 //
 // Rows are independent: row r belongs to sequence row_seq[r] (its block-table row) and sees the cached tokens
-// 0 .. row_pos[r], so one launch serves decode batches, portions of prompts and mixtures of both.
+// 0 .. row_pos[r], or the last `window` of them, so one launch serves decode batches, portions of prompts and
+// mixtures of both.  A per-head sink may join the denominator.
+//
+// The same kernels attend plain cached keys that are also the values: kv_heads parts per row, each read by its group of
+// query heads, and a factor per row that turns its keys - not its values - into normed ones (shared_kv.cu).
 #include <math.h>
 
 #include "latent_attn.cuh"
@@ -246,7 +250,7 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 9) latent_prepare_vec_kern
 
 bool prepare_vec_takes(const PrepareParams<__nv_bfloat16> &p) {
   const auto al = [](const void *q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
-  return p.rot_pairs <= 32 && p.rot_dim > 0 && p.rot_dim % 8 == 0 && p.rot_pairs * 2 == p.rot_dim &&
+  return p.rot_pairs <= 32 && p.rot_dim % 8 == 0 && p.rot_pairs * 2 == p.rot_dim &&
          (!p.q || (al(p.q) && p.dim % 8 == 0 && p.q_ld % 8 == 0)) &&
          (!p.dq || (al(p.dq) && al(p.dq_w) && al(p.cq) && p.q_rank % 8 == 0 && p.dq_ld % 8 == 0)) &&
          (!p.dkv || (al(p.dkv) && al(p.dkv_w) && al(p.pages) && p.kv_rank % 8 == 0 && p.dkv_ld % 8 == 0));
@@ -260,22 +264,23 @@ constexpr int kGenThreads = 256, kGenTile = 64;
 template <typename T>
 __global__ void __launch_bounds__(kGenThreads) latent_attend_generic_kernel(const AttendParams p) {
   extern __shared__ float sm[];
-  __shared__ float scratch[32], score[kGenTile];
+  __shared__ float scratch[32], score[kGenTile], factor[kGenTile];
   __shared__ const T *key[kGenTile];
-  const int row_elems = p.kv_rank + p.rot_dim;
-  float *q = sm, *acc = sm + row_elems;
+  const int part_elems = p.kv_rank + p.rot_dim;
+  float *q = sm, *acc = sm + part_elems;
   const int r = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int part = h / (p.heads / p.kv_heads) * p.kv_rank;
   grid_dependency_wait();
   grid_dependency_launch();
   const T *ql = static_cast<const T *>(p.q_lat) + ((size_t)r * p.heads + h) * p.kv_rank;
   const T *qr = static_cast<const T *>(p.q) + (size_t)r * p.q_ld + (size_t)h * (p.dim + p.rot_dim) + p.dim;
-  for (int i = threadIdx.x; i < row_elems; i += kGenThreads) q[i] = i < p.kv_rank ? ldf(ql + i) : ldf(qr + i - p.kv_rank);
+  for (int i = threadIdx.x; i < part_elems; i += kGenThreads) q[i] = i < p.kv_rank ? ldf(ql + i) : ldf(qr + i - p.kv_rank);
   for (int i = threadIdx.x; i < p.kv_rank; i += kGenThreads) acc[i] = 0.f;
   const int keys = visible_keys(p, r);
   const int32_t *table = p.block_table + (size_t)max(0, min(p.row_seq[r], p.max_seqs - 1)) * p.max_blocks;
   const T *pages = static_cast<const T *>(p.pages);
-  float m = -INFINITY, l = 0.f;
-  for (int k0 = 0; k0 < keys; k0 += kGenTile) {
+  float m = p.sink ? p.sink[h] : -INFINITY, l = p.sink ? 1.f : 0.f;
+  for (int k0 = first_key(p, r); k0 < keys; k0 += kGenTile) {
     const int n = min(kGenTile, keys - k0);
     __syncthreads();
     if (threadIdx.x < n) {
@@ -285,19 +290,21 @@ __global__ void __launch_bounds__(kGenThreads) latent_attend_generic_kernel(cons
         atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
         page = 0;
       }
-      key[threadIdx.x] = pages + ((size_t)page * p.page_tokens + t % p.page_tokens) * row_elems;
+      const T *row = pages + ((size_t)page * p.page_tokens + t % p.page_tokens) * p.row_elems;
+      key[threadIdx.x] = row + part;
+      factor[threadIdx.x] = p.key_scale >= 0 ? p.scale * *reinterpret_cast<const float *>(row + p.key_scale) : p.scale;
     }
     __syncthreads();
     for (int j = warp; j < n; j += kGenThreads / 32) {
       float s = 0.f;
-      for (int i = lane; i < row_elems; i += 32) s = fmaf(q[i], ldf(key[j] + i), s);
+      for (int i = lane; i < part_elems; i += 32) s = fmaf(q[i], ldf(key[j] + i), s);
       s = warp_sum(s);
-      if (lane == 0) score[j] = s * p.scale;
+      if (lane == 0) score[j] = s * factor[j];
     }
     __syncthreads();
     float mt = m;
     for (int j = 0; j < n; ++j) mt = fmaxf(mt, score[j]);
-    const float corr = expf(m - mt);  // 0 at the first tile
+    const float corr = expf(m - mt);  // 0 at the first tile without a sink
     m = mt;
     __syncthreads();
     if (threadIdx.x < n) score[threadIdx.x] = expf(score[threadIdx.x] - m);
@@ -314,23 +321,23 @@ __global__ void __launch_bounds__(kGenThreads) latent_attend_generic_kernel(cons
   for (int i = threadIdx.x; i < p.kv_rank; i += kGenThreads) stf(out + i, acc[i] * inv);
 }
 
-// ---- gather: cached rows 0 .. n-1 of one sequence, contiguous -----------------------------------------
+// ---- gather: cached rows first .. first + n - 1 of one sequence, contiguous -----------------------------------------
 __global__ void __launch_bounds__(256)
-latent_gather_kernel(const uint8_t *pages, const int32_t *table, uint8_t *out, int n, int row_bytes, int page_tokens,
+latent_gather_kernel(const uint8_t *pages, const int32_t *table, uint8_t *out, int first, int n, int row_bytes, int page_tokens,
                      int max_blocks, int num_pages, int unit) {
   grid_dependency_wait();
   grid_dependency_launch();
   const int per = row_bytes / unit;
   const int64_t total = (int64_t)n * per;
   for (int64_t i = blockIdx.x * 256ll + threadIdx.x; i < total; i += gridDim.x * 256ll) {
-    const int t = (int)(i / per), c = (int)(i % per), blk = t / page_tokens;
+    const int t = first + (int)(i / per), c = (int)(i % per), blk = t / page_tokens;
     const int page = blk < max_blocks ? table[blk] : -1;
     if (page < 0 || page >= num_pages) {
       atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
       continue;
     }
     const uint8_t *src = pages + ((size_t)page * page_tokens + t % page_tokens) * row_bytes + (size_t)c * unit;
-    uint8_t *dst = out + (size_t)t * row_bytes + (size_t)c * unit;
+    uint8_t *dst = out + (size_t)(t - first) * row_bytes + (size_t)c * unit;
     if (unit == 16)
       *reinterpret_cast<uint4 *>(dst) = *reinterpret_cast<const uint4 *>(src);
     else
@@ -382,18 +389,33 @@ size_t axb200_latent_attend_workspace_bytes(int rows, int heads, int kv_rank, in
 }
 
 int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim, void *out, const void *pages,
-                         const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, int rows, int heads,
-                         int kv_rank, int rot_dim, float scale, int page_tokens, int max_blocks, int num_pages,
-                         int max_seqs, int64_t max_len, int dtype, void *workspace, size_t workspace_bytes, void *stream) {
+                         const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, const float *sink,
+                         int rows, int heads, int kv_heads, int kv_rank, int rot_dim, int row_elems, int key_scale, int window,
+                         float scale, int page_tokens, int max_blocks, int num_pages, int max_seqs, int64_t max_len, int dtype,
+                         void *workspace, size_t workspace_bytes, void *stream) {
   if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
-  if (!q_lat || !q || !out || !pages || !block_table || !row_seq || !row_pos) return AXB200_INVALID_PTR;
+  if (!q_lat || (!q && rot_dim > 0) || !out || !pages || !block_table || !row_seq || !row_pos) return AXB200_INVALID_PTR;
+  if (kv_heads <= 0 || heads % kv_heads != 0 || (kv_heads > 1 && rot_dim > 0) || window < 0 ||
+      row_elems < kv_heads * kv_rank + rot_dim)
+    return AXB200_INVALID_ARGUMENT;
+  // the factor is an aligned float inside the row, behind its parts
+  if (key_scale >= 0) {
+    const int es = (int)axb::dtype_size(dtype), per = 4 / es;
+    if (key_scale < kv_heads * kv_rank + rot_dim || key_scale + per > row_elems || key_scale % per || row_elems % per)
+      return AXB200_INVALID_ARGUMENT;
+  }
   if (rows < 0 || heads <= 0 || heads > 65535 || kv_rank <= 0 || rot_dim < 0 || dim < 0 || page_tokens <= 0 || max_blocks <= 0 ||
       num_pages <= 0 || max_seqs <= 0 || max_len <= 0 || max_len > 0x7fffffff - 4096)
     return AXB200_INVALID_ARGUMENT;
-  if (q_ld < (int64_t)heads * (dim + rot_dim)) return AXB200_SHAPE_MISMATCH;
+  if (rot_dim > 0 && q_ld < (int64_t)heads * (dim + rot_dim)) return AXB200_SHAPE_MISMATCH;
   if (rows == 0) return AXB200_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   axb::AttendParams p{};
+  p.kv_heads = kv_heads;
+  p.row_elems = row_elems;
+  p.key_scale = key_scale < 0 ? -1 : key_scale;
+  p.window = window;
+  p.sink = sink;
   p.q_lat = q_lat;
   p.q = q;
   p.q_ld = q_ld;
@@ -415,7 +437,7 @@ int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim
   p.scale = scale;
   p.wait_ns = axb::wait_limit_ns();
   if (dtype == AXB200_BFLOAT16 && axb::latent_umma_supported(p)) {
-    if (!workspace || workspace_bytes < axb200_latent_attend_workspace_bytes(rows, heads, kv_rank, rot_dim, max_len, dtype))
+    if (!workspace || workspace_bytes < axb200_latent_attend_workspace_bytes(rows, heads / kv_heads, kv_rank, rot_dim, max_len, dtype))
       return AXB200_OUT_OF_MEMORY;
     if ((reinterpret_cast<uintptr_t>(workspace) & 15u) == 0) return axb::latent_umma(p, workspace, st);
   }
@@ -428,12 +450,12 @@ int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim
   return axb::launch_dependent(kernel, dim3(rows, heads), dim3(axb::kGenThreads), smem, st, p);
 }
 
-int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out, int64_t n, int row_elems, int page_tokens,
+int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out, int64_t first, int64_t n, int row_elems, int page_tokens,
                          int max_blocks, int num_pages, int dtype, void *stream) {
   const size_t es = axb::dtype_size(dtype);
   if (es == 0) return AXB200_UNSUPPORTED_TYPE;
   if (!pages || !block_row || !out) return AXB200_INVALID_PTR;
-  if (n < 0 || n > (int64_t)max_blocks * page_tokens || row_elems <= 0 || page_tokens <= 0 || max_blocks <= 0 || num_pages <= 0)
+  if (n < 0 || first < 0 || first + n > (int64_t)max_blocks * page_tokens || row_elems <= 0 || page_tokens <= 0 || max_blocks <= 0 || num_pages <= 0)
     return AXB200_INVALID_ARGUMENT;
   if (n == 0) return AXB200_OK;
   const int row_bytes = (int)(row_elems * es);
@@ -442,7 +464,7 @@ int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out,
   const int64_t items = n * (row_bytes / unit);
   const int grid = (int)(items / 256 + 1 < 148 * 8 ? items / 256 + 1 : 148 * 8);
   return axb::launch_dependent(axb::latent_gather_kernel, dim3(grid), dim3(256), 0, static_cast<cudaStream_t>(stream),
-                               static_cast<const uint8_t *>(pages), block_row, static_cast<uint8_t *>(out), (int)n, row_bytes,
+                               static_cast<const uint8_t *>(pages), block_row, static_cast<uint8_t *>(out), (int)first, (int)n, row_bytes,
                                page_tokens, max_blocks, num_pages, unit);
 }
 

@@ -1,4 +1,5 @@
-// What the kernels of latent attention in its cached (latent) form share; see latent_attn.cu.
+// What the kernels of attention over cached rows (latent attention in its cached form, keys that are also the values)
+// share; see latent_attn.cu.
 #pragma once
 
 #include "tcgen05.cuh"
@@ -15,6 +16,11 @@ struct AttendParams {
   int rows, heads, dim, kv_rank, rot_dim, page_tokens, max_blocks, num_pages, max_seqs, max_len;
   float scale;
   unsigned long long wait_ns;
+  int kv_heads;       // a cached row holds kv_heads parts of kv_rank elements, each for heads / kv_heads query heads
+  int row_elems;      // elements from one cached row to the next
+  int key_scale;      // element of the row at which the fp32 factor of its keys stands, or -1: none
+  int window;         // keys a row sees, itself included; 0: all
+  const float *sink;  // (heads): logit that takes part in the softmax's denominator only, or null
 };
 
 // Keys row r may read: 0 .. row_pos[r], never beyond the block table's reach or the host's bound.
@@ -25,8 +31,13 @@ __device__ __forceinline__ int visible_keys(const AttendParams &p, int r) {
   return max(0, min(p.row_pos[r] + 1, cover));
 }
 
+// The first key row r sees.
+__device__ __forceinline__ int first_key(const AttendParams &p, int r) {
+  return p.window > 0 ? max(0, p.row_pos[r] + 1 - p.window) : 0;
+}
+
 // tcgen05 form for bf16 (latent_umma.cu)
-size_t latent_umma_workspace_bytes(int heads, int kv_rank, int rot_dim);
+size_t latent_umma_workspace_bytes(int part_heads, int kv_rank, int rot_dim);
 bool latent_umma_supported(const AttendParams &p);
 int latent_umma(const AttendParams &p, void *workspace, cudaStream_t st);
 

@@ -4,7 +4,11 @@
 // their own - the shared part is read from the cached rows and never copied per head - and meet in shared
 // memory as neighbouring 64-wide blocks of the K dimension; likewise the two parts of a query.  Blocks that are
 // not full (dim 32, rot 16, ...) are zero-filled by TMA, so any sizes that are multiples of 8 up to
-// dim 128, rot 64, vdim 128 run.
+// dim 128, rot 64, vdim 128 run.  Without a rotated part the key is its own elements alone; kv_heads below heads shares
+// a key and value head among a group of query heads, which makes this the prompt form of grouped attention too.
+//
+// A row may see only the last `window` keys (a CTA starts at the tile that holds its first row's first key), and a
+// per-head sink may join the denominator.
 //
 // Structure as the 256-row form of prefill_attn.cu: one CTA per (256 query rows, head) works on two query tiles
 // against key tiles of 128; S_g and O_g in tensor memory; warps 0-7 own one query row per thread and do the
@@ -14,6 +18,7 @@
 #include <math.h>
 
 #include <mutex>
+#include <type_traits>
 
 #include "tcgen05.cuh"
 
@@ -26,27 +31,29 @@ constexpr float kLog2e = 1.4426950408889634f, kLazy = 8.0f;
 
 struct Params {
   __nv_bfloat16 *out;
-  int n, start, skv, heads, vdim;
+  int n, start, skv, heads, group, vdim;  // group: query heads per key and value head
+  int window;                             // 0: all
+  const float *sink;                      // (heads), or null
   float scale_log2;
   unsigned long long wait_ns;
 };
 
-// kQB / kVB: 64-wide blocks of the heads' own key part and of the values (one more block holds the rotated part)
-template <int kQB, int kVB>
+// kQB / kVB: 64-wide blocks of the heads' own key part and of the values; kRot: one more block for the rotated part
+template <int kQB, int kVB, int kRot>
 struct Layout {
-  static constexpr int kBlocks = kQB + 1;
+  static constexpr int kBlocks = kQB + kRot;
   static constexpr int kTile = kBlocks * kBox;        // a query tile or a key tile
   static constexpr int kVHalf = 64 * kVB * 64 * 2;    // 64 keys: kVB boxes of [64 keys][64]
   static constexpr int kOffK = 2 * kTile, kOffV = kOffK + 2 * kTile, kOffBar = kOffV + 2 * kVHalf;
   static constexpr int kSmem = kOffBar + 256;
 };
 
-template <int kQB, int kVB>
+template <int kQB, int kVB, int kRot>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmQr,
                       const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmKr,
                       const __grid_constant__ CUtensorMap tmV, const Params p) {
-  using L = Layout<kQB, kVB>;
+  using L = Layout<kQB, kVB, kRot>;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint64_t *bars = reinterpret_cast<uint64_t *>(smem + L::kOffBar);
   uint64_t *bar_q = bars, *full_k = bars + 1, *empty_k = bars + 3, *full_v = bars + 5, *empty_v = bars + 7;
@@ -60,11 +67,13 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   // heaviest blocks first: the last query block has the most key tiles
   const int h = blockIdx.y, q0 = (gridDim.x - 1 - blockIdx.x) * 2 * kRows;
   const int warp = uniform_warp(), lane = threadIdx.x & 31;
+  const int hk = h / p.group;
+  const int tile0 = p.window > 0 ? max(0, p.start + q0 + 1 - p.window) / kKeys : 0;  // the first key tile
   int nkv_g[2];
 #pragma unroll
   for (int g = 0; g < 2; ++g) {
     const int first = q0 + g * kRows, last = min(first + kRows, p.n) - 1;
-    nkv_g[g] = first < p.n ? (min(p.start + last + 1, p.skv) + kKeys - 1) / kKeys : 0;
+    nkv_g[g] = first < p.n ? (min(p.start + last + 1, p.skv) + kKeys - 1) / kKeys - tile0 : 0;
   }
   const int nkv = max(nkv_g[0], nkv_g[1]);
 
@@ -94,14 +103,14 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   if (warp == kLoadWarp) {
     if (lane == 0) {
       tma_prefetch_descriptor(&tmK);
-      tma_prefetch_descriptor(&tmKr);
+      if (kRot) tma_prefetch_descriptor(&tmKr);
       tma_prefetch_descriptor(&tmV);
       mbar_arrive_expect_tx(bar_q, 2 * L::kTile);
 #pragma unroll
       for (int g = 0; g < 2; ++g) {  // rows past n are zero-filled
         uint8_t *dst = smem + g * L::kTile;
         for (int b = 0; b < kQB; ++b) tma_load_3d(dst + b * kBox, &tmQ, bar_q, b * 64, h, q0 + g * kRows);
-        tma_load_3d(dst + kQB * kBox, &tmQr, bar_q, 0, h, q0 + g * kRows);
+        if (kRot) tma_load_3d(dst + kQB * kBox, &tmQr, bar_q, 0, h, q0 + g * kRows);
       }
       bool ok = true;
       auto load_k = [&](int t) {
@@ -110,8 +119,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         if (!ok) return;
         uint8_t *dst = smem + L::kOffK + s * L::kTile;
         mbar_arrive_expect_tx(&full_k[s], L::kTile);
-        for (int b = 0; b < kQB; ++b) tma_load_3d(dst + b * kBox, &tmK, &full_k[s], b * 64, h, t * kKeys);
-        tma_load_3d(dst + kQB * kBox, &tmKr, &full_k[s], 0, 0, t * kKeys);
+        for (int b = 0; b < kQB; ++b) tma_load_3d(dst + b * kBox, &tmK, &full_k[s], b * 64, hk, (tile0 + t) * kKeys);
+        if (kRot) tma_load_3d(dst + kQB * kBox, &tmKr, &full_k[s], 0, 0, (tile0 + t) * kKeys);
       };
       load_k(0);
       int j = 0;
@@ -123,7 +132,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
           if (!ok) break;
           uint8_t *dst = smem + L::kOffV + half * L::kVHalf;
           mbar_arrive_expect_tx(&full_v[half], L::kVHalf);
-          for (int b = 0; b < kVB; ++b) tma_load_3d(dst + b * (64 * 64 * 2), &tmV, &full_v[half], b * 64, h, j * kKeys + half * 64);
+          for (int b = 0; b < kVB; ++b) tma_load_3d(dst + b * (64 * 64 * 2), &tmV, &full_v[half], b * 64, hk, (tile0 + j) * kKeys + half * 64);
         }
         if (!ok) break;
       }
@@ -200,7 +209,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     const int g = warp >> 2, row = threadIdx.x & (kRows - 1);
     const int my_nkv = g ? nkv_g[1] : nkv_g[0];
     const int t_row = q0 + g * kRows + row;
-    const int kv_end = min(p.start + t_row + 1, p.skv);
+    const int kv_end = min(p.start + t_row + 1, p.skv), kv_begin = p.window > 0 ? max(0, p.start + t_row + 1 - p.window) : 0;
     const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t ts = tmem + g * 128 + lane_base, to = tmem_o(g) + lane_base, tp = tmem_p(g) + lane_base;
     float m_run = -INFINITY, l_run = 0.f;
@@ -213,7 +222,14 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld32_async(ts + c * 32, sr[c]);
       tmem_wait_ld();
-      const int n0 = j * kKeys;
+      const int n0 = (tile0 + j) * kKeys;
+      if (n0 < kv_begin) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (n0 + c * 32 + i < kv_begin) sr[c][i] = 0xff800000u;  // -inf
+      }
       if (n0 + kKeys > kv_end) {
 #pragma unroll
         for (int c = 0; c < 4; ++c)
@@ -270,7 +286,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     if (ok && my_nkv > 0) ok = __all_sync(0xffffffffu, mbar_wait_bounded(&bar_fin[g], 0, abort_flag, p.wait_ns));
     tc_fence_after();
     if (ok && my_nkv > 0) {
-      const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      if (p.sink) {
+        const float s = p.sink[h] * kLog2e, top = fmaxf(m_run, s), w = fast_exp2(m_run - top);
+        inv = w / fmaf(l_run, w, fast_exp2(s - top));
+      }
       __nv_bfloat16 *dst = p.out + ((size_t)t_row * p.heads + h) * p.vdim;
 #pragma unroll
       for (int c = 0; c < kVB * 2; ++c) {
@@ -309,9 +329,10 @@ bool map_of(CUtensorMap *map, const void *base, int elems, int heads, int64_t ro
                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int kQB, int kVB>
+template <int kQB, int kVB, int kRot>
 int launch(const CUtensorMap (&m)[5], const Params &p, cudaStream_t st) {
-  auto *kernel = latent_prefill_kernel<kQB, kVB>;
+  using L = Layout<kQB, kVB, kRot>;
+  auto *kernel = latent_prefill_kernel<kQB, kVB, kRot>;
   static std::mutex mu;
   static bool opted[64] = {false};
   int dev = 0;
@@ -319,13 +340,13 @@ int launch(const CUtensorMap (&m)[5], const Params &p, cudaStream_t st) {
   {
     std::lock_guard<std::mutex> lock(mu);
     if (!opted[dev]) {
-      if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Layout<kQB, kVB>::kSmem) != cudaSuccess)
+      if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kSmem) != cudaSuccess)
         return AXB200_DEVICE_ERROR;
       opted[dev] = true;
     }
   }
   const dim3 grid((p.n + 2 * kRows - 1) / (2 * kRows), p.heads);
-  return launch_dependent(kernel, grid, dim3(kThreads), Layout<kQB, kVB>::kSmem, st, m[0], m[1], m[2], m[3], m[4], p);
+  return launch_dependent(kernel, grid, dim3(kThreads), L::kSmem, st, m[0], m[1], m[2], m[3], m[4], p);
 }
 
 bool al16(const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
@@ -336,33 +357,41 @@ bool al16(const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 extern "C" {
 
 int axb200_latent_prefill_supported(int heads, int dim, int rot_dim, int vdim, int dtype) {
-  return dtype == AXB200_BFLOAT16 && heads > 0 && heads <= 65535 && dim >= 8 && dim <= 128 && dim % 8 == 0 && rot_dim >= 8 &&
+  return dtype == AXB200_BFLOAT16 && heads > 0 && heads <= 65535 && dim >= 8 && dim <= 128 && dim % 8 == 0 && rot_dim >= 0 &&
          rot_dim <= 64 && rot_dim % 8 == 0 && vdim >= 8 && vdim <= 128 && vdim % 8 == 0;
 }
 
-int axb200_latent_prefill(const void *q, int64_t q_ld, const void *k, const void *v, const void *rot, int64_t rot_ld, void *out,
-                          int n, int64_t start, int heads, int dim, int rot_dim, int vdim, float scale, int dtype, void *stream) {
+int axb200_latent_prefill(const void *q, int64_t q_ld, const void *k, const void *v, const void *rot, int64_t rot_ld,
+                          const float *sink, void *out, int n, int64_t start, int heads, int kv_heads, int dim, int rot_dim,
+                          int vdim, int window, float scale, int dtype, void *stream) {
   if (!axb200_latent_prefill_supported(heads, dim, rot_dim, vdim, dtype)) return AXB200_UNSUPPORTED_TYPE;
-  if (!q || !k || !v || !rot || !out) return AXB200_INVALID_PTR;
-  if (n < 0 || start < 0 || start + n > 0x7fffffff - 4096 || !(scale > 0.f)) return AXB200_INVALID_ARGUMENT;
+  if (!q || !k || !v || (rot_dim > 0 && !rot) || !out) return AXB200_INVALID_PTR;
+  if (n < 0 || start < 0 || start + n > 0x7fffffff - 4096 || !(scale > 0.f) || kv_heads <= 0 || heads % kv_heads != 0 || window < 0)
+    return AXB200_INVALID_ARGUMENT;
   if (q_ld < (int64_t)heads * (dim + rot_dim) || rot_ld < rot_dim) return AXB200_SHAPE_MISMATCH;
   if (q_ld % 8 || rot_ld % 8 || !axb::al16(q) || !axb::al16(k) || !axb::al16(v) || !axb::al16(rot) || !axb::al16(out))
     return AXB200_UNSUPPORTED_TYPE;
   if (n == 0) return AXB200_OK;
   const int per = dim + rot_dim;
   const int64_t skv = start + n;
-  CUtensorMap m[5];
+  CUtensorMap m[5] = {};
   const __nv_bfloat16 *qb = static_cast<const __nv_bfloat16 *>(q);
   if (!axb::map_of(&m[0], qb, dim, heads, n, per, q_ld, axb::kRows) ||
-      !axb::map_of(&m[1], qb + dim, rot_dim, heads, n, per, q_ld, axb::kRows) ||
-      !axb::map_of(&m[2], k, dim, heads, skv, dim, (int64_t)heads * dim, axb::kKeys) ||
-      !axb::map_of(&m[3], rot, rot_dim, 1, skv, rot_ld, rot_ld, axb::kKeys) ||
-      !axb::map_of(&m[4], v, vdim, heads, skv, vdim, (int64_t)heads * vdim, 64))
+      !axb::map_of(&m[2], k, dim, kv_heads, skv, dim, (int64_t)kv_heads * dim, axb::kKeys) ||
+      !axb::map_of(&m[4], v, vdim, kv_heads, skv, vdim, (int64_t)kv_heads * vdim, 64))
     return AXB200_INTERNAL_ERROR;
-  axb::Params p{static_cast<__nv_bfloat16 *>(out), n, (int)start, (int)skv, heads, vdim, scale * axb::kLog2e, axb::wait_limit_ns()};
+  if (rot_dim > 0 && (!axb::map_of(&m[1], qb + dim, rot_dim, heads, n, per, q_ld, axb::kRows) ||
+                      !axb::map_of(&m[3], rot, rot_dim, 1, skv, rot_ld, rot_ld, axb::kKeys)))
+    return AXB200_INTERNAL_ERROR;
+  axb::Params p{static_cast<__nv_bfloat16 *>(out), n, (int)start, (int)skv, heads, heads / kv_heads, vdim, window, sink,
+                scale * axb::kLog2e, axb::wait_limit_ns()};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dim > 64) return vdim > 64 ? axb::launch<2, 2>(m, p, st) : axb::launch<2, 1>(m, p, st);
-  return vdim > 64 ? axb::launch<1, 2>(m, p, st) : axb::launch<1, 1>(m, p, st);
+  auto go = [&](auto rot_tag) {
+    constexpr int kRot = decltype(rot_tag)::value;
+    if (dim > 64) return vdim > 64 ? axb::launch<2, 2, kRot>(m, p, st) : axb::launch<2, 1, kRot>(m, p, st);
+    return vdim > 64 ? axb::launch<1, 2, kRot>(m, p, st) : axb::launch<1, 1, kRot>(m, p, st);
+  };
+  return rot_dim > 0 ? go(std::integral_constant<int, 1>{}) : go(std::integral_constant<int, 0>{});
 }
 
 }  // extern "C"

@@ -39,7 +39,8 @@ constexpr float kLog2e = 1.4426950408889634f, kLazy = 8.0f;
 
 struct UmmaAttend {
   AttendParams a;
-  int head_tiles, groups;
+  int part_tiles;          // tiles of heads that read one part of the rows
+  int head_tiles, groups;  // kv_heads * part_tiles
   int pairs, singles;            // per tile
   int pair_slots, single_slots;  // in the rings
   int chunks;                    // per row: ceil(elements / 64)
@@ -47,7 +48,11 @@ struct UmmaAttend {
   float2 *part_ml;               // (2 * CTAs, N): reference (log2 domain), sum
 };
 
-__device__ __forceinline__ int tiles_of(const AttendParams &p, int r) { return (visible_keys(p, r) + kKeys - 1) / kKeys; }
+// Tiles start at the multiple of 64 keys (half a tile lies in one page) at or before the row's first key.
+__device__ __forceinline__ int first_tile_key(const AttendParams &p, int r) { return first_key(p, r) & ~63; }
+__device__ __forceinline__ int tiles_of(const AttendParams &p, int r) {
+  return max(0, visible_keys(p, r) - first_tile_key(p, r) + kKeys - 1) / kKeys;
+}
 __device__ __forceinline__ int tiles_per_group(int total, int groups) { return max(kMinTiles, (total + groups - 1) / groups); }
 
 // start[r] = key tiles of the rows before r, r = 0 .. rows; all threads of the CTA.
@@ -75,6 +80,20 @@ __device__ __forceinline__ void scan_tiles(const AttendParams &p, int *start) {
     base = all;
     __syncthreads();
   }
+}
+
+// The factor of key t's row of row r's sequence (the loader reports a bad page).
+__device__ __forceinline__ float key_factor(const AttendParams &p, int r, int t) {
+  const int page = p.block_table[(size_t)p.row_seq[r] * p.max_blocks + t / p.page_tokens];
+  if (page < 0 || page >= p.num_pages) return 0.f;
+  const __nv_bfloat16 *row = static_cast<const __nv_bfloat16 *>(p.pages) + ((size_t)page * p.page_tokens + t % p.page_tokens) * p.row_elems;
+  return *reinterpret_cast<const float *>(row + p.key_scale);
+}
+
+// What un-normalised results with sum l at reference ref (log2 domain) are multiplied by when a sink joins the sum.
+__device__ __forceinline__ float inverse_with_sink(float ref, float l, float sink) {
+  const float s = sink * kLog2e, top = fmaxf(ref, s), w = fast_exp2(ref - top);
+  return w / fmaf(l, w, fast_exp2(s - top));
 }
 
 // Whether any of the 128 softmax threads says so.
@@ -174,7 +193,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
   const int total = start[p.rows], per = tiles_per_group(total, u.groups);
   const int lo = (int)(blockIdx.x / u.head_tiles) * per, hi = min(total, lo + per);
   if (lo >= hi) return;
-  const int h0 = (int)(blockIdx.x % u.head_tiles) * kN;
+  const int head_tile = (int)(blockIdx.x % u.head_tiles), part = head_tile / u.part_tiles, part_heads = p.heads / p.kv_heads;
+  const int h0 = part * part_heads + (head_tile - part * u.part_tiles) * kN, h_end = (part + 1) * part_heads;
   // the row that holds tile lo: the last r with start[r] <= lo
   int r_first = 0;
   for (int a = 0, b = p.rows - 1; a < b;) {
@@ -205,10 +225,10 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       int np = 0, ns = 0;  // how many were issued
       bool ok = true;
       for (int r = r_first, g = lo; g < hi && ok; ++r) {
-        const int keys = visible_keys(p, r);
+        const int keys = visible_keys(p, r), key0 = first_tile_key(p, r);
         const int32_t *table = p.block_table + (size_t)p.row_seq[r] * p.max_blocks;
         for (; g < hi && g < start[r + 1] && ok; ++g) {
-          const int t0 = (g - start[r]) * kKeys;
+          const int t0 = key0 + (g - start[r]) * kKeys;
           // two halves of 64 keys, each within one page; a half past the end is not loaded
           const int halves = keys - t0 > 64 ? 2 : 1;
           int at[2];
@@ -223,7 +243,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
             at[i] = page * p.page_tokens + t % p.page_tokens;
           }
           auto load_chunk = [&](uint8_t *dst, uint64_t *bar, int c) {
-            for (int i = 0; i < halves; ++i) tma_load_2d(dst + i * (kChunk / 2), &tmPages, bar, c * 64, at[i]);
+            for (int i = 0; i < halves; ++i) tma_load_3d(dst + i * (kChunk / 2), &tmPages, bar, c * 64, part, at[i]);
           };
           for (int i = 0; i < u.singles && ok; ++i, ++ns, rs.next(u.single_slots)) {
             const int s = rs.slot;
@@ -324,7 +344,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       for (int i = tid; i < kN * u.chunks * 8; i += kSoftmax) {
         const int h = i / (u.chunks * 8), e = (i - h * (u.chunks * 8)) * 8;
         uint4 v = make_uint4(0, 0, 0, 0);
-        if (h0 + h < p.heads && e < elems)
+        if (h0 + h < h_end && e < elems)
           v = e < p.kv_rank ? *reinterpret_cast<const uint4 *>(static_cast<const __nv_bfloat16 *>(p.q_lat) +
                                                                ((size_t)r * p.heads + h0 + h) * p.kv_rank + e)
                             : *reinterpret_cast<const uint4 *>(static_cast<const __nv_bfloat16 *>(p.q) + (size_t)r * p.q_ld +
@@ -338,15 +358,18 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
     for (int r = r_first, g = lo; g < hi && ok; ++r) {
       if (start[r + 1] <= g) continue;
       const int k_first = g - start[r], g_end = min(hi, start[r + 1]), keys = visible_keys(p, r);
+      const int key0 = first_tile_key(p, r), hidden = first_key(p, r) - key0;  // keys of the first tile before the window
       if (seg == 0) put_queries(r);
       ++seg;
       float l[kN];
 #pragma unroll
       for (int h = 0; h < kN; ++h) l[h] = 0.f;
       for (const int g_first = g; g < g_end; ++g, ++tile, np += u.pairs) {
+        const int t0 = key0 + (g - start[r]) * kKeys, valid = min(kKeys, keys - t0);
+        const bool seen = tid < valid && (g > start[r] || tid >= hidden);
+        const float factor = p.key_scale < 0 ? scale_log2 : seen ? scale_log2 * key_factor(p, r, t0 + tid) : 0.f;
         ok = mbar_wait_warp(&bar_s[tile & 1], (tile >> 1) & 1, abort_flag, p.wait_ns);
         tc_fence_after();
-        const int valid = min(kKeys, keys - (g - start[r]) * kKeys);
         float s[kN], rf[kN];
         load_refs<kN>(ref, rf);
         if (ok) {
@@ -358,7 +381,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         float most = -INFINITY;  // how far a score exceeds its head's reference
 #pragma unroll
         for (int h = 0; h < kN; ++h) {
-          s[h] = tid < valid ? s[h] * scale_log2 : -INFINITY;
+          s[h] = seen ? s[h] * factor : -INFINITY;
           most = fmaxf(most, s[h] - rf[h]);
         }
         const bool over = g == g_first || most > kLazy;
@@ -450,9 +473,10 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
 #pragma unroll
         for (int h = 0; h < kN; ++h) {
           if (whole) {
-            if (h0 + h < p.heads) {
+            if (h0 + h < h_end) {
               const float lt = red[0][h] + red[1][h] + red[2][h] + red[3][h];
-              static_cast<__nv_bfloat16 *>(p.out)[((size_t)r * p.heads + h0 + h) * p.kv_rank + e] = __float2bfloat16_rn(o[h] / lt);
+              const float inv = p.sink ? inverse_with_sink(ref[h], lt, p.sink[h0 + h]) : 1.0f / lt;
+              static_cast<__nv_bfloat16 *>(p.out)[((size_t)r * p.heads + h0 + h) * p.kv_rank + e] = __float2bfloat16_rn(o[h] * inv);
             }
           } else {
             u.part_o[((size_t)slot * kN + h) * p.kv_rank + e] = o[h];
@@ -503,7 +527,8 @@ __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const UmmaA
   const int first = before / per, last = (before + n - 1) / per, count = last - first + 1;
   if (count == 1) return;
   // records: the range that holds the item's first tile filed it under 1, the later ones under 0
-  auto slot = [&](int c) { return (((first + c) * u.head_tiles + h / kN) * 2 + (c == 0 ? 1 : 0)) * kN + h % kN; };
+  const int part_heads = p.heads / p.kv_heads, in_part = h % part_heads, head_tile = h / part_heads * u.part_tiles + in_part / kN;
+  auto slot = [&](int c) { return (((first + c) * u.head_tiles + head_tile) * 2 + (c == 0 ? 1 : 0)) * kN + in_part % kN; };
   float top = -INFINITY, sum = 0.f;
   for (int c = 0; c < count; ++c) top = fmaxf(top, u.part_ml[slot(c)].x);
   for (int c = 0; c < count; ++c) {
@@ -513,7 +538,7 @@ __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const UmmaA
     if (threadIdx.x == 0) weight[c] = w;
   }
   __syncthreads();
-  const float inv = sum > 0.f ? 1.0f / sum : 0.f;
+  const float inv = p.sink ? inverse_with_sink(top, sum, p.sink[h]) : sum > 0.f ? 1.0f / sum : 0.f;
   for (int e = threadIdx.x * 4; e < p.kv_rank; e += kMergeThreads * 4) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
@@ -576,11 +601,12 @@ int run(const AttendParams &p, void *workspace, cudaStream_t st) {
       opted[dev] = true;
     }
   }
-  const int elems = p.kv_rank + p.rot_dim;
+  // a part's elements, the parts of a row, the rows: a box ends with its part and is zero-filled beyond
   CUtensorMap map;
-  const cuuint64_t dims[2] = {(cuuint64_t)elems, (cuuint64_t)p.num_pages * p.page_tokens}, strides[1] = {(cuuint64_t)elems * 2};
-  const cuuint32_t box[2] = {64, 64}, es[2] = {1, 1};
-  if (tensor_map_encoder()(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(p.pages), dims, strides, box, es,
+  const cuuint64_t dims[3] = {(cuuint64_t)(p.kv_rank + p.rot_dim), (cuuint64_t)p.kv_heads, (cuuint64_t)p.num_pages * p.page_tokens};
+  const cuuint64_t strides[2] = {(cuuint64_t)(p.kv_heads > 1 ? p.kv_rank : p.row_elems) * 2, (cuuint64_t)p.row_elems * 2};
+  const cuuint32_t box[3] = {64, 1, 64}, es[3] = {1, 1, 1};
+  if (tensor_map_encoder()(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void *>(p.pages), dims, strides, box, es,
                            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
     return AXB200_INTERNAL_ERROR;
@@ -592,12 +618,13 @@ int run(const AttendParams &p, void *workspace, cudaStream_t st) {
     AttendParams &a = u.a;
     a.rows = p.rows - r0 < kMaxRows ? p.rows - r0 : kMaxRows;
     a.q_lat = static_cast<const __nv_bfloat16 *>(p.q_lat) + (size_t)r0 * p.heads * p.kv_rank;
-    a.q = static_cast<const __nv_bfloat16 *>(p.q) + (size_t)r0 * p.q_ld;
+    if (p.q) a.q = static_cast<const __nv_bfloat16 *>(p.q) + (size_t)r0 * p.q_ld;
     a.out = static_cast<__nv_bfloat16 *>(p.out) + (size_t)r0 * p.heads * p.kv_rank;
     a.row_seq = p.row_seq + r0;
     a.row_pos = p.row_pos + r0;
     if (!layout<kN>(u)) return AXB200_INTERNAL_ERROR;
-    u.head_tiles = (p.heads + kN - 1) / kN;
+    u.part_tiles = (p.heads / p.kv_heads + kN - 1) / kN;
+    u.head_tiles = p.kv_heads * u.part_tiles;
     u.groups = sms / u.head_tiles > 0 ? sms / u.head_tiles : 1;
     const int ctas = u.groups * u.head_tiles;
     u.part_ml = static_cast<float2 *>(workspace);
@@ -614,24 +641,24 @@ int heads_per_tile(int heads) { return heads <= 16 ? 16 : 32; }
 
 }  // namespace
 
-size_t latent_umma_workspace_bytes(int heads, int kv_rank, int rot_dim) {
-  return (size_t)2 * kMaxCtas * heads_per_tile(heads) * (sizeof(float2) + (size_t)kv_rank * sizeof(float));
+size_t latent_umma_workspace_bytes(int part_heads, int kv_rank, int rot_dim) {
+  return (size_t)2 * kMaxCtas * heads_per_tile(part_heads) * (sizeof(float2) + (size_t)kv_rank * sizeof(float));
 }
 
 bool latent_umma_supported(const AttendParams &p) {
   const uintptr_t bits = reinterpret_cast<uintptr_t>(p.q_lat) | reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.out) |
                          reinterpret_cast<uintptr_t>(p.pages);
-  const int n = heads_per_tile(p.heads), sms = sm_count();
+  const int n = heads_per_tile(p.heads / p.kv_heads), sms = sm_count();
   UmmaAttend u{};
   u.a = p;
-  return p.kv_rank % 8 == 0 && p.rot_dim % 8 == 0 && p.dim % 8 == 0 && p.q_ld % 8 == 0 && (bits & 15u) == 0 &&
-         p.page_tokens % 64 == 0 && (p.heads + n - 1) / n <= kMaxCtas && sms > 0 && sms <= kMaxCtas && tensor_map_encoder() &&
+  return p.kv_rank % 8 == 0 && p.rot_dim % 8 == 0 && p.row_elems % 8 == 0 && (p.rot_dim == 0 || (p.dim % 8 == 0 && p.q_ld % 8 == 0)) &&
+         (bits & 15u) == 0 && p.page_tokens % 64 == 0 && p.kv_heads * ((p.heads / p.kv_heads + n - 1) / n) <= kMaxCtas && sms > 0 && sms <= kMaxCtas && tensor_map_encoder() &&
          (int64_t)p.num_pages * p.page_tokens < 0x7fffffff && (p.max_len / kKeys + 1) * (int64_t)kMaxRows < 0x7fffffff &&
          (n == 16 ? layout<16>(u) : layout<32>(u));
 }
 
 int latent_umma(const AttendParams &p, void *workspace, cudaStream_t st) {
-  return heads_per_tile(p.heads) == 16 ? run<16>(p, workspace, st) : run<32>(p, workspace, st);
+  return heads_per_tile(p.heads / p.kv_heads) == 16 ? run<16>(p, workspace, st) : run<32>(p, workspace, st);
 }
 
 }  // namespace axb

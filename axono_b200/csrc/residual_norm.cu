@@ -2,45 +2,17 @@
 // kept in fp32: one launch between two layers adds everything the finished layer contributes - the mixer's
 // output, the weighted rows of the chosen experts, the shared expert's output - and writes the one or two
 // layer norms that the next layer (or the output projection) reads.  Both norms share the row's mean and
-// variance, so the second costs one multiply per element.  The other kernel is the start of the stream:
-// embedding gather + layer norm.  The operators of fused.cu are their RMS, fp16 / fp32-storage siblings.
-#include "common.cuh"
+// variance, so the second costs one multiply per element.  Another kernel is the start of the stream: embedding
+// gather + layer norm.  The operators of fused.cu are their RMS, fp16 / fp32-storage siblings.
+//
+// The other kind of stream norms what a sublayer puts out, not what it reads: x += rms_norm(y) * (offset + w), and the
+// next sublayer reads x itself (rounded to the activations' type), or after the last one the model's final norm of it.
+#include "vec.cuh"
 
 namespace axb {
 namespace {
 
 constexpr int kThreads = 256;
-
-// 8 consecutive elements (16 or 32 bytes), or one.
-template <int kVec, typename T>
-__device__ __forceinline__ void load_vec(const T *p, float (&v)[kVec]) {
-  if constexpr (kVec == 8 && sizeof(T) == 2) {
-    const uint4 raw = *reinterpret_cast<const uint4 *>(p);
-    const T *e = reinterpret_cast<const T *>(&raw);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = ldf(e + i);
-  } else if constexpr (kVec == 8) {
-    const float4 a = reinterpret_cast<const float4 *>(p)[0], b = reinterpret_cast<const float4 *>(p)[1];
-    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
-  } else {
-    v[0] = ldf(p);
-  }
-}
-template <int kVec, typename T>
-__device__ __forceinline__ void store_vec(T *p, const float (&v)[kVec]) {
-  if constexpr (kVec == 8 && sizeof(T) == 2) {
-    uint4 raw;
-    T *e = reinterpret_cast<T *>(&raw);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) stf(e + i, v[i]);
-    *reinterpret_cast<uint4 *>(p) = raw;
-  } else if constexpr (kVec == 8) {
-    reinterpret_cast<float4 *>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
-    reinterpret_cast<float4 *>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
-  } else {
-    stf(p, v[0]);
-  }
-}
 
 struct RowStats {
   float mean, inv;
@@ -169,6 +141,81 @@ embed_layer_norm_kernel(const int64_t *ids, const T *table, const T *w, float ep
   }
 }
 
+template <typename T>
+struct PostNormParams {
+  float *x;      // (rows, width), updated in place
+  const T *y;    // (rows, width): the sublayer's output
+  const T *w;    // its norm
+  const T *w2;   // norm of the new x in h, or null: h is x itself
+  T *h;          // or null
+  float offset;  // added to the stored weights (1 when they are stored around zero)
+  float eps;
+  int width;
+};
+
+template <typename T, int kVec>
+__global__ void __launch_bounds__(kThreads) residual_post_norm_kernel(const PostNormParams<T> p) {
+  extern __shared__ float row[];
+  __shared__ float scratch[32];
+  const size_t off = (size_t)blockIdx.x * p.width;
+  grid_dependency_wait();
+  grid_dependency_launch();
+  float sq = 0.f;
+  for (int c = threadIdx.x * kVec; c < p.width; c += kThreads * kVec) {
+    float v[kVec];
+    load_vec<kVec>(p.y + off + c, v);
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) {
+      row[c + i] = v[i];
+      sq = fmaf(v[i], v[i], sq);
+    }
+  }
+  const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)p.width + p.eps);
+  sq = 0.f;
+  for (int c = threadIdx.x * kVec; c < p.width; c += kThreads * kVec) {  // a thread reads back what it wrote
+    float v[kVec], w[kVec];
+    load_vec<kVec>(p.x + off + c, v);
+    load_vec<kVec>(p.w + c, w);
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) {
+      v[i] += row[c + i] * inv * (p.offset + w[i]);
+      row[c + i] = v[i];
+      sq = fmaf(v[i], v[i], sq);
+    }
+    store_vec<kVec>(p.x + off + c, v);
+    if (p.h && !p.w2) store_vec<kVec>(p.h + off + c, v);
+  }
+  if (!p.h || !p.w2) return;
+  const float inv2 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)p.width + p.eps);
+  for (int c = threadIdx.x * kVec; c < p.width; c += kThreads * kVec) {
+    float v[kVec], w[kVec];
+    load_vec<kVec>(p.w2 + c, w);
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) v[i] = row[c + i] * inv2 * (p.offset + w[i]);
+    store_vec<kVec>(p.h + off + c, v);
+  }
+}
+
+template <typename T, int kVec>
+__global__ void __launch_bounds__(kThreads)
+embed_residual_kernel(const int64_t *ids, const T *table, float *x, T *h, long long vocab, int width) {
+  const size_t off = (size_t)blockIdx.x * width;
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const long long id = ids[blockIdx.x];
+  const bool ok = id >= 0 && id < vocab;
+  if (!ok && threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_BAD_INDEX);
+  const T *src = table + (size_t)(ok ? id : 0) * width;
+  for (int c = threadIdx.x * kVec; c < width; c += kThreads * kVec) {
+    float v[kVec];
+    load_vec<kVec>(src + c, v);
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) v[i] = ok ? v[i] : 0.f;
+    store_vec<kVec>(x + off + c, v);
+    if (h) store_vec<kVec>(h + off + c, v);
+  }
+}
+
 bool al16(const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
 constexpr int kMaxWidth = 49152;  // the row is staged in shared memory as fp32
@@ -206,10 +253,56 @@ int residual_typed(float *x, const void *a, const void *b, const void *expert_ro
   return launch_residual(p, rows, st);
 }
 
+template <typename T>
+int launch_post_norm(const PostNormParams<T> &p, int64_t rows, cudaStream_t st) {
+  const bool vec = p.width % 8 == 0 && al16(p.x) && al16(p.y) && al16(p.w) && al16(p.w2) && al16(p.h);
+  auto *kernel = vec ? residual_post_norm_kernel<T, 8> : residual_post_norm_kernel<T, 1>;
+  const size_t smem = (size_t)p.width * sizeof(float);
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    return AXB200_DEVICE_ERROR;
+  return launch_dependent(kernel, dim3((unsigned)rows), dim3(kThreads), smem, st, p);
+}
+
+template <typename T>
+int launch_embed_residual(const int64_t *ids, const void *table, float *x, void *h, int64_t n, int64_t vocab, int width,
+                          cudaStream_t st) {
+  const bool vec = width % 8 == 0 && al16(table) && al16(x) && al16(h);
+  auto *kernel = vec ? embed_residual_kernel<T, 8> : embed_residual_kernel<T, 1>;
+  return launch_dependent(kernel, dim3((unsigned)n), dim3(kThreads), 0, st, ids, static_cast<const T *>(table), x,
+                          static_cast<T *>(h), (long long)vocab, width);
+}
+
 }  // namespace
 }  // namespace axb
 
 extern "C" {
+
+int axb200_embed_residual(const int64_t *ids, const void *table, float *x, void *h, int64_t n, int64_t vocab, int width,
+                          int dtype, void *stream) {
+  if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
+  if (!ids || !table || !x) return AXB200_INVALID_PTR;
+  if (n < 0 || n > 0x7fffffff || vocab <= 0 || width <= 0) return AXB200_INVALID_ARGUMENT;
+  if (n == 0) return AXB200_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return dtype == AXB200_FLOAT32 ? axb::launch_embed_residual<float>(ids, table, x, h, n, vocab, width, st)
+                                 : axb::launch_embed_residual<__nv_bfloat16>(ids, table, x, h, n, vocab, width, st);
+}
+
+int axb200_residual_post_norm(float *x, const void *y, const void *w, float offset, float eps, const void *w2, void *h,
+                              int64_t rows, int width, int dtype, void *stream) {
+  if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
+  if (!x || !y || !w || (w2 && !h)) return AXB200_INVALID_PTR;
+  if (rows < 0 || rows > 0x7fffffff || width <= 0 || width > axb::kMaxWidth) return AXB200_INVALID_ARGUMENT;
+  if (rows == 0) return AXB200_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  auto go = [&](auto tag) {
+    using T = decltype(tag);
+    axb::PostNormParams<T> p{x, static_cast<const T *>(y), static_cast<const T *>(w), static_cast<const T *>(w2),
+                             static_cast<T *>(h), offset, eps, width};
+    return axb::launch_post_norm(p, rows, st);
+  };
+  return dtype == AXB200_FLOAT32 ? go(float{}) : go(__nv_bfloat16{});
+}
 
 int axb200_embed_layer_norm(const int64_t *ids, const void *table, const void *weight, float eps, float *x, int64_t n,
                             int64_t vocab, int width, int dtype, void *stream) {

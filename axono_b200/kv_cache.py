@@ -244,7 +244,7 @@ class KVArena:
         """An arena whose layer l caches one row of row_elems[l] elements per token, with no value pool (latent
         caches); `row_pages(l)` and `table()` are its device memory."""
         a = cls.__new__(cls)
-        a.n_layers, a.num_pages, a.n_kv_heads, a.head_dim = len(row_elems), num_pages, 1, row_elems[0]
+        a.n_layers, a.num_pages, a.n_kv_heads, a.head_dim = len(row_elems), num_pages, 1, row_elems[0] if row_elems else 0
         a.row_elems = list(row_elems)
         a.max_seqs, a.page_tokens, a.dtype = max_seqs, page_tokens, dtype
         a.max_blocks = (max_seq_len + page_tokens - 1) // page_tokens
@@ -264,6 +264,22 @@ class KVArena:
         t = torch.as_tensor(_DeviceView(ptr, (self.num_pages, self.page_tokens, self.row_elems[layer]), view),
                             device=torch.device("cuda", torch.cuda.current_device()))
         return t.view(torch.bfloat16) if self.dtype == torch.bfloat16 else t
+
+    def add_state(self, shape, dtype):
+        """A pool of state that does not grow with a sequence: (max_seqs, *shape), one entry per slot.  Nothing clears an
+        entry between sequences: a layer starts a sequence's first token from zero by itself."""
+        count = 1
+        for n in shape:
+            count *= n
+        size = torch.empty((), dtype=dtype).element_size()
+        ptr = C.c_void_p()
+        _capi.check(_capi.lib().axb200_kv_arena_add_state(self._h, count * size, C.byref(ptr)), "kv_arena_add_state")
+        if not self.device_memory:
+            return None
+        view = {torch.bfloat16: "<i2", torch.float16: "<f2", torch.float32: "<f4"}[dtype]
+        t = torch.as_tensor(_DeviceView(ptr.value, (self.max_seqs, *shape), view),
+                            device=torch.device("cuda", torch.cuda.current_device()))
+        return t.view(torch.bfloat16) if dtype == torch.bfloat16 else t
 
     def table(self):
         """The device block table (max_seqs, max_blocks), refreshed by `sync()`."""

@@ -5,7 +5,8 @@
     models.create(config_dict, weights, dtype=...)                  # the same from memory
 
 A registered class takes (config, weights, dtype, device) and offers what `axono_b200.serving` drives:
-`cache_rows` (elements one token caches in each cache layer), `vocab` and `forward(tokens, rows, want)`.
+`cache_rows` (elements one token caches in each cache layer), `state_shapes` (what one sequence keeps in each state
+layer, as (shape, dtype) pairs), `vocab`, `takes_segment(n)` and `forward(tokens, rows, cache, want)`.
 `TextTower`, the decode step of the reference's own model, is listed by name for `config_of`; it makes its
 random weights itself and is stepped directly (axono_b200.decode, axono_b200.native_tower).
 """
@@ -26,7 +27,7 @@ def register(architecture: str):
 
 
 def architectures():
-    from . import nuderax  # noqa: F401 - registers itself
+    from . import nuderax, rigozen  # noqa: F401 - they register themselves
 
     return sorted(_REGISTRY)
 

@@ -15,7 +15,7 @@ import torch
 
 from .. import ops
 from . import register
-from .layers import GroupedSigmoidRouter, LatentAttention, MixtureOfExperts, Rows
+from .layers import Cache, GroupedSigmoidRouter, LatentAttention, MixtureOfExperts, Rows
 
 _MIXERS = {"latent_attention": False, "latent_attention_2": True}  # name -> queries through a latent
 
@@ -133,6 +133,7 @@ def tensor_shapes(cfg: NuderaxConfig):
 @register("Nuderax")
 class Nuderax:
     config_class = NuderaxConfig
+    state_shapes = ()  # no recurrent layers
 
     def __init__(self, cfg: NuderaxConfig, weights, dtype=torch.bfloat16, device="cuda"):
         self.cfg, self.dtype, self.device, self.vocab = cfg, dtype, torch.device(device), cfg.vocab
@@ -191,8 +192,8 @@ class Nuderax:
         """Whether a portion of n tokens of one sequence should go through attention's expanded form."""
         return all(mixer.takes_segment(n) for _, _, mixer, _ in self.layers)
 
-    def forward(self, tokens, rows: Rows, pages, want, trace=None):
-        """tokens int64 (rows) on the device; pages[c]: pool of cache layer c; want: int64 row indices whose logits
+    def forward(self, tokens, rows: Rows, cache: Cache, want, trace=None):
+        """tokens int64 (rows) on the device; cache.pages[c]: pool of cache layer c; want: int64 row indices whose logits
         are computed, or None for all.  Returns fp32 logits (wanted, vocab), or None when nothing is wanted.
         trace: list that receives a copy of the residual after every layer."""
         eps = self.cfg.eps
@@ -202,7 +203,7 @@ class Nuderax:
             h1, h2 = ops.residual_layer_norm(x, norm1, norm2, eps, **pending)
             if trace is not None and i:
                 trace.append(x.clone())
-            pending = {"a": mixer.forward(h1, rows, pages[mixer.cache_layer])}
+            pending = {"a": mixer.forward(h1, rows, cache)}
             if mlp is not None:
                 pending["experts"], pending["b"] = mlp.forward(h2)
         h, _ = ops.residual_layer_norm(x, self.final_norm, None, eps, **pending)

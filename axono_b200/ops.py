@@ -313,7 +313,7 @@ def silu_mul_rows(gate_up, n: int):
     """silu(gate) * up for gate = gate_up[:, :n], up = gate_up[:, n:2n] (one fused gate|up projection
     output, rows may be strided) -> (rows, n)."""
     op = "silu_mul_rows"
-    dt = _dt(gate_up, op)
+    dt = _capi.BFLOAT16 if gate_up.is_cuda and gate_up.dtype == torch.bfloat16 else _dt(gate_up, op)
     if gate_up.dim() != 2 or gate_up.stride(1) != 1 or gate_up.shape[1] != 2 * n:
         _capi.check(4, op)
     out = torch.empty((gate_up.shape[0], n), dtype=gate_up.dtype, device=gate_up.device)
@@ -632,6 +632,34 @@ def residual_layer_norm(x, w1, w2, eps, a=None, b=None, experts=None):
     return h1, h2
 
 
+def embed_residual(ids, table):
+    """(x, h): table[ids] as the fp32 residual stream (n, width) and in the table's type (x itself when that is fp32)."""
+    op = "embed_residual"
+    dt = _lm_dt(table, op)
+    if ids.dtype != torch.int64:
+        _capi.check(3, op)
+    x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    h = x if table.dtype == torch.float32 else torch.empty(x.shape, dtype=table.dtype, device=table.device)
+    _call(_capi.lib().axb200_embed_residual(ids.data_ptr(), table.data_ptr(), x.data_ptr(), None if h is x else h.data_ptr(),
+                                            ids.numel(), table.shape[0], table.shape[1], dt, _stream(table)), op)
+    return x, h
+
+
+def residual_post_norm(x, y, weight, eps, offset=0.0, final=None):
+    """x (rows, width) fp32 += rms_norm(y) * (offset + weight), in place; returns x in y's type (x itself when that is
+    fp32), or with `final` its rms norm times (offset + final)."""
+    op = "residual_post_norm"
+    dt = _lm_dt(y, op)
+    if x.dtype != torch.float32 or x.shape != y.shape or not y.is_contiguous() or weight.dtype != y.dtype or \
+            (final is not None and final.dtype != y.dtype):
+        _capi.check(4, op)
+    h = x if final is None and y.dtype == torch.float32 else torch.empty(x.shape, dtype=y.dtype, device=y.device)
+    _call(_capi.lib().axb200_residual_post_norm(x.data_ptr(), y.data_ptr(), weight.data_ptr(), float(offset), float(eps),
+                                                _ptr(final), None if h is x else h.data_ptr(), x.shape[0], x.shape[1], dt,
+                                                _stream(y)), op)
+    return h
+
+
 def latent_prepare(rows, inv_freq, rot_dim, q=None, heads=0, dim=0, dq=None, dq_weight=None, dkv=None, dkv_weight=None,
                    pages=None, eps=1e-5):
     """The step's norms, rotation and append of latent attention in one launch; each of q (rows, >= heads *
@@ -655,28 +683,33 @@ def latent_prepare(rows, inv_freq, rot_dim, q=None, heads=0, dim=0, dq=None, dq_
     return cq
 
 
-def latent_attend(q_lat, q, dim, rot_dim, scale, pages, rows, n):
+def latent_attend(q_lat, q, dim, rot_dim, scale, pages, rows, n, window=0, sink=None, kv_heads=1, key_scale=-1):
     """Latent attention of the first n rows: q_lat (n, heads, kv_rank), the rotated query parts inside q (strided
-    rows of heads x (dim + rot_dim)) -> (n, heads, kv_rank)."""
+    rows of heads x (dim + rot_dim); None without them) -> (n, heads, kv_rank).  window: keys a row sees (0: all); sink
+    (heads) fp32: logit in the denominator; kv_heads parts per cached row; key_scale: where its scores' factor stands."""
     op = "latent_attend"
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != q_lat.shape[1]):
+        _capi.check(4, op)
+    if not q_lat.is_contiguous() or q_lat.dtype != pages.dtype:
+        _capi.check(4, op)
     dt = _lm_dt(q_lat, op)
     heads, rank = q_lat.shape[1], q_lat.shape[2]
     out = torch.empty_like(q_lat)
     lib = _capi.lib()
-    ws = workspace(q.device, lib.axb200_latent_attend_workspace_bytes(n, heads, rank, rot_dim, rows.max_len, dt))
+    ws = workspace(q_lat.device, lib.axb200_latent_attend_workspace_bytes(n, heads // kv_heads, rank, rot_dim, rows.max_len, dt))
     _call(lib.axb200_latent_attend(
-        q_lat.data_ptr(), q.data_ptr(), q.stride(0), dim, out.data_ptr(), pages.data_ptr(), rows.block_table.data_ptr(),
-        rows.seq.data_ptr(), rows.pos.data_ptr(), n, heads, rank, rot_dim, float(scale), pages.shape[1],
-        rows.block_table.shape[1], pages.shape[0], rows.block_table.shape[0], int(rows.max_len), dt, ws.data_ptr(), ws.numel(),
-        _stream(q)), op)
+        q_lat.data_ptr(), _ptr(q), q.stride(0) if q is not None else 0, dim, out.data_ptr(), pages.data_ptr(),
+        rows.block_table.data_ptr(), rows.seq.data_ptr(), rows.pos.data_ptr(), _ptr(sink), n, heads, kv_heads, rank, rot_dim,
+        pages.shape[2], int(key_scale), int(window), float(scale), pages.shape[1], rows.block_table.shape[1], pages.shape[0],
+        rows.block_table.shape[0], int(rows.max_len), dt, ws.data_ptr(), ws.numel(), _stream(q_lat)), op)
     return out
 
 
-def latent_gather(pages, block_row, n):
-    """The first n cached rows of the sequence whose block-table row is block_row, contiguous."""
+def latent_gather(pages, block_row, n, first=0):
+    """The n cached rows from position `first` on of the sequence whose block-table row is block_row, contiguous."""
     op = "latent_gather"
     out = torch.empty((n, pages.shape[2]), dtype=pages.dtype, device=pages.device)
-    _call(_capi.lib().axb200_latent_gather(pages.data_ptr(), block_row.data_ptr(), out.data_ptr(), n, pages.shape[2],
+    _call(_capi.lib().axb200_latent_gather(pages.data_ptr(), block_row.data_ptr(), out.data_ptr(), int(first), n, pages.shape[2],
                                            pages.shape[1], block_row.numel(), pages.shape[0], _lm_dt(pages, op), _stream(pages)), op)
     return out
 
@@ -685,19 +718,110 @@ def latent_prefill_supported(heads, dim, rot_dim, vdim, dtype) -> bool:
     return bool(_capi.lib().axb200_latent_prefill_supported(heads, dim, rot_dim, vdim, _LM_DTYPES[dtype]))
 
 
-def latent_prefill(q, start, k, v, rot, heads, dim, rot_dim, vdim, scale):
+def latent_prefill(q, start, k, v, rot, heads, dim, rot_dim, vdim, scale, window=0, sink=None, kv_heads=None):
     """Expanded form of one sequence's portion: q (n, >= heads * (dim + rot_dim)) at positions start.., k (start + n,
-    heads * dim), v (start + n, heads * vdim), rot (start + n, rot_dim), strided rows -> (n, heads * vdim)."""
+    kv_heads * dim), v (start + n, kv_heads * vdim), rot (start + n, rot_dim) with strided rows (None without a rotated
+    part) -> (n, heads * vdim).  kv_heads defaults to heads; window and sink as in `latent_attend`."""
     op = "latent_prefill"
     dt = _lm_dt(q, op)
     n = q.shape[0]
-    if k.shape[0] != start + n or v.shape[0] != start + n or rot.shape[0] != start + n or not (k.is_contiguous() and v.is_contiguous()):
+    kv_heads = kv_heads or heads
+    if k.shape != (start + n, kv_heads * dim) or v.shape != (start + n, kv_heads * vdim) or not (k.is_contiguous() and v.is_contiguous()) \
+            or (rot is None) != (rot_dim == 0) or (rot is not None and rot.shape[0] != start + n):
+        _capi.check(4, op)
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != heads):
         _capi.check(4, op)
     out = torch.empty((n, heads * vdim), dtype=q.dtype, device=q.device)
-    _call(_capi.lib().axb200_latent_prefill(q.data_ptr(), q.stride(0), k.data_ptr(), v.data_ptr(), rot.data_ptr(), rot.stride(0),
-                                            out.data_ptr(), n, int(start), heads, dim, rot_dim, vdim, float(scale), dt,
-                                            _stream(q)), op)
+    _call(_capi.lib().axb200_latent_prefill(q.data_ptr(), q.stride(0), k.data_ptr(), v.data_ptr(), _ptr(rot),
+                                            rot.stride(0) if rot is not None else 0, _ptr(sink), out.data_ptr(), n, int(start),
+                                            heads, kv_heads, dim, rot_dim, vdim, int(window), float(scale), dt, _stream(q)), op)
     return out
+
+
+def shared_kv_row(kv_heads, dim, dtype):
+    """(elements of a cached row of raw keys, element at which its factor stands)."""
+    per = 16 // torch.empty((), dtype=dtype).element_size()
+    at = -(-kv_heads * dim // per) * per
+    return at + per, at
+
+
+def shared_kv_prepare(q, q_weight, k, k_weight, pages, rows, heads, kv_heads, dim, key_scale, eps):
+    """Norms q (rows, heads * dim) over the whole row with both weights folded in -> (rows, heads, dim), and appends the
+    raw k (rows, kv_heads * dim) with its factor; both may be column slices of a wider matrix."""
+    op = "shared_kv_prepare"
+    dt = _lm_dt(q, op)
+    n = q.shape[0]
+    if k.dtype != q.dtype or k.shape[0] != n or q.stride(1) != 1 or k.stride(1) != 1 or q.shape[1] != heads * dim or \
+            k.shape[1] != kv_heads * dim or pages.dtype != q.dtype or q_weight.dtype != q.dtype or k_weight.dtype != q.dtype:
+        _capi.check(4, op)
+    out = torch.empty((n, heads, dim), dtype=q.dtype, device=q.device)
+    _call(_capi.lib().axb200_shared_kv_prepare(
+        q.data_ptr(), q.stride(0), q_weight.data_ptr(), out.data_ptr(), k.data_ptr(), k.stride(0), k_weight.data_ptr(), float(eps),
+        pages.data_ptr(), rows.block_table.data_ptr(), rows.seq.data_ptr(), rows.pos.data_ptr(), n, heads, kv_heads, dim,
+        pages.shape[2], key_scale, pages.shape[1], rows.block_table.shape[1], pages.shape[0], rows.block_table.shape[0], dt,
+        _stream(q)), op)
+    return out
+
+
+def shared_kv_gather(pages, block_row, first, n, kv_heads, dim, key_scale):
+    """Cached rows first .. first + n - 1 of a sequence -> normed keys (without their weight), values; (n, kv_heads * dim)."""
+    op = "shared_kv_gather"
+    keys = torch.empty((n, kv_heads * dim), dtype=pages.dtype, device=pages.device)
+    values = torch.empty_like(keys)
+    _call(_capi.lib().axb200_shared_kv_gather(
+        pages.data_ptr(), block_row.data_ptr(), keys.data_ptr(), values.data_ptr(), int(first), n, kv_heads, dim, pages.shape[2],
+        key_scale, pages.shape[1], block_row.numel(), pages.shape[0], _lm_dt(pages, op), _stream(pages)), op)
+    return keys, values
+
+
+def _delta_args(m, proj, state, ring):
+    """(weights, sizes) shared by the operators of the gated delta rule; m holds conv (taps, channels), a_log, dt_bias, norm
+    and the sizes."""
+    if state.dtype != torch.float32 or ring.dtype != proj.dtype or proj.stride(1) != 1 or m.norm.dtype != proj.dtype:
+        _capi.check(3, "delta")
+    if tuple(state.shape[1:]) != (m.heads, m.dim, m.vdim) or tuple(ring.shape) != (state.shape[0],) + tuple(m.conv.shape):
+        _capi.check(4, "delta")
+    return ((m.conv.data_ptr(), m.a_log.data_ptr(), m.dt_bias.data_ptr(), m.norm.data_ptr(), ring.data_ptr(), state.data_ptr()),
+            (m.heads, m.kv_heads, m.dim, m.vdim, m.conv.shape[0], state.shape[0], float(m.eps)))
+
+
+def delta_step(m, proj, rows, n, state, ring, out):
+    """The gated delta rule for the first n rows, tokens of different sequences, into out[:n]."""
+    op = "delta_step"
+    weights, sizes = _delta_args(m, proj, state, ring)
+    _call(_capi.lib().axb200_delta_step(proj.data_ptr(), proj.stride(0), rows.seq.data_ptr(), rows.pos.data_ptr(), n, *weights,
+                                        out.data_ptr(), *sizes, _lm_dt(proj, op), _stream(proj)), op)
+
+
+def delta_prepare(m, proj, rows, first, state, ring):
+    """Rows first.. of a step: (qk fp32, v, log_g, beta) of axb200_delta_prepare."""
+    op = "delta_prepare"
+    weights, sizes = _delta_args(m, proj, state, ring)
+    n = proj.shape[0] - first
+    f32 = lambda cols: torch.empty((n, cols), dtype=torch.float32, device=proj.device)  # noqa: E731
+    qk, log_g, beta = f32(2 * m.kv_heads * m.dim), f32(m.heads), f32(m.heads)
+    v = torch.empty((n, m.heads * m.vdim), dtype=proj.dtype, device=proj.device)
+    _call(_capi.lib().axb200_delta_prepare(
+        proj.data_ptr(), proj.stride(0), rows.seq.data_ptr(), rows.pos.data_ptr(), rows.back.data_ptr(), first, proj.shape[0],
+        *weights, qk.data_ptr(), v.data_ptr(), log_g.data_ptr(), beta.data_ptr(), *sizes, _lm_dt(proj, op), _stream(proj)), op)
+    return qk, v, log_g, beta
+
+
+def delta_scan(m, portions, first, qk, v, log_g, beta, state, out):
+    """The recurrence of the portions (int32 (count, 4)), token by token, into out (rows - first, heads * vdim)."""
+    op = "delta_scan"
+    _call(_capi.lib().axb200_delta_scan(
+        portions.data_ptr(), portions.shape[0], first, qk.data_ptr(), v.data_ptr(), log_g.data_ptr(), beta.data_ptr(),
+        state.data_ptr(), out.data_ptr(), m.heads, m.kv_heads, m.dim, m.vdim, state.shape[0], _lm_dt(v, op), _stream(v)), op)
+
+
+def delta_finish(m, proj, rows, first, state, ring, o, out):
+    """Norm and gate of the recurrence's output o (rows - first, heads * vdim) into out (may be o), and the ring."""
+    op = "delta_finish"
+    weights, sizes = _delta_args(m, proj, state, ring)
+    _call(_capi.lib().axb200_delta_finish(
+        proj.data_ptr(), proj.stride(0), rows.seq.data_ptr(), rows.pos.data_ptr(), rows.back.data_ptr(), first, proj.shape[0],
+        *weights, o.data_ptr(), out.data_ptr(), *sizes, _lm_dt(proj, op), _stream(proj)), op)
 
 
 def moe_route(logits, correction, groups, keep, top, scale):

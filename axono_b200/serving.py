@@ -1,7 +1,7 @@
 """Serving of registered models: the step over cached sequences, and the scheduler above it.
 
-`ModelRunner` owns a model's cache (pages of a `KVArena`, one sequence slot per live request) and runs steps: a
-step brings each of some sequences its next tokens - a whole prompt, a portion of one, a decoded token - and
+`ModelRunner` owns a model's cache (pages of a `KVArena`, one sequence slot per live request, and that slot's state
+of recurrent layers) and runs steps: a step brings each of some sequences its next tokens - a whole prompt, a portion of one, a decoded token - and
 returns the logits asked for.  `Engine` schedules requests over it: every step decodes all running requests
 and fills the rest of its token budget with portions of waiting prompts; sampling is greedy (`argmax_last_dim`).
 While only decoding is left and the batch does not change, the engine replays the step as a CUDA graph.
@@ -17,7 +17,7 @@ import torch
 from . import ops
 from .cuda_graph import CUDAGraph
 from .kv_cache import KVArena
-from .models.layers import Rows
+from .models.layers import Cache, Rows
 
 
 class ModelRunner:
@@ -31,6 +31,8 @@ class ModelRunner:
         if shuffle_pages is not None:
             self.arena.shuffle_free(shuffle_pages)
         self.pages = [self.arena.row_pages(c) for c in range(len(model.cache_rows))]
+        self.states = [tuple(self.arena.add_state(shape, dtype) for shape, dtype in layer) for layer in model.state_shapes]
+        self.cache = Cache(self.pages, self.states)
         self.block_table = self.arena.table()
         self.lengths = {}
 
@@ -43,6 +45,16 @@ class ModelRunner:
     def close(self, seq: int) -> None:
         del self.lengths[seq]
         self.arena.free_seq(seq)
+
+    def copy_state(self, seqs):
+        """The recurrent state of some sequences, for `put_state`."""
+        at = torch.tensor(list(seqs), dtype=torch.int64, device=self.model.device)
+        return [(t, at, t.index_select(0, at)) for layer in self.states for t in layer]
+
+    @staticmethod
+    def put_state(saved) -> None:
+        for t, at, entries in saved:
+            t.index_copy_(0, at, entries)
 
     def capacity(self) -> int:
         return self.arena.max_blocks * self.page_tokens
@@ -60,29 +72,35 @@ class ModelRunner:
                 raise ValueError("an entry needs tokens, and wanted places among them")
             self.arena.reserve(seq, self.lengths[seq] + len(tokens))
         self.arena.sync()
-        # rows that attend through the cache first, then the long portions
-        long = [self.model.takes_segment(len(tokens)) for _, tokens, _ in entries]
-        order = sorted(range(len(entries)), key=lambda i: long[i])
-        ids, seqs, pos, first, segments, latent, max_len = [], [], [], {}, [], 0, 1
+        # single tokens first, then portions by length: those that attend through the cache, then the long ones
+        order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]))
+        ids, seqs, pos, back, first, segments, portions, latent, max_len = [], [], [], [], {}, [], [], 0, 1
         for i in order:
             seq, tokens, _ = entries[i]
             start, n = self.lengths[seq], len(tokens)
             first[i] = len(ids)
-            if long[i]:
+            if n > 1:
+                portions.append((seq, len(ids), n, start))
+            if self.model.takes_segment(n):
                 segments.append((seq, len(ids), n, start))
+            elif segments:
+                raise RuntimeError("a model that takes a portion as a segment must take every longer one")
             else:
                 latent += n
                 max_len = max(max_len, start + n)
             ids.extend(tokens)
             seqs.extend([seq] * n)
             pos.extend(range(start, start + n))
+            back.extend(range(n))
         want = [first[i] + w for i, (_, _, places) in enumerate(entries) for w in places]
         dev = self.model.device
-        # one copy for the step's integers: token ids and wanted rows (int64), sequences and positions
-        packed = torch.tensor([ids + want, seqs + [0] * len(want), pos + [0] * len(want)], dtype=torch.int64).to(dev)
-        n = len(ids)
-        rows = Rows(packed[1, :n].to(torch.int32), packed[2, :n].to(torch.int32), self.block_table, max_len, latent, segments)
-        logits = self.model.forward(packed[0, :n], rows, self.pages, packed[0, n:], trace=trace)
+        # two copies for the step's integers: token ids and wanted rows; portions, sequences, positions, rows before
+        wide = torch.tensor(ids + want, dtype=torch.int64).to(dev)
+        n, at = len(ids), 4 * len(portions)
+        ints = torch.tensor([v for p in portions for v in p] + seqs + pos + back, dtype=torch.int32).to(dev)
+        rows = Rows(ints[at:at + n], ints[at + n:at + 2 * n], self.block_table, max_len, latent, segments, n - sum(p[2] for p in portions),
+                    ints[at + 2 * n:], portions, ints[:at].view(-1, 4))
+        logits = self.model.forward(wide[:n], rows, self.cache, wide[n:], trace=trace)
         for seq, tokens, _ in entries:
             self.lengths[seq] += len(tokens)
         return logits
@@ -102,19 +120,21 @@ class DecodeGraph:
         self.tokens = torch.tensor(list(tokens), dtype=torch.int64, device=dev)
         self.rows = Rows(torch.tensor(self.seqs, dtype=torch.int32, device=dev),
                          torch.tensor([runner.lengths[s] for s in self.seqs], dtype=torch.int32, device=dev), runner.block_table,
-                         max(self.limits), len(self.seqs))
+                         max(self.limits), len(self.seqs), singles=len(self.seqs))
         if self.room() <= 0:
             raise ValueError("DecodeGraph: no room for a token")
         for s, limit in zip(self.seqs, self.limits):  # the pages the replays will write
             runner.arena.reserve(s, limit)
         runner.arena.sync()
         saved = (self.tokens.clone(), self.rows.pos.clone())
+        state = runner.copy_state(self.seqs)
         self.graph = CUDAGraph().capture(self._body)  # runs the step once before it records it
+        runner.put_state(state)
         self.tokens.copy_(saved[0])
         self.rows.pos.copy_(saved[1])
 
     def _body(self):
-        logits = self.runner.model.forward(self.tokens, self.rows, self.runner.pages, None)
+        logits = self.runner.model.forward(self.tokens, self.rows, self.runner.cache, None)
         nxt = ops.argmax_last_dim(logits)
         self.tokens.copy_(nxt)
         self.rows.pos.add_(1)

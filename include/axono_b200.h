@@ -488,11 +488,20 @@ int axb200_residual_layer_norm(float *x, const void *a, const void *b, const voi
                                const void *w2, void *h2, float eps, int64_t rows, int width, int dtype,
                                void *stream);
 
+/* The stream of layers that norm what a sublayer puts out:
+ *   embed_residual: x = table[ids] in fp32 and h (optional) the same in `dtype`; bad ids as above.
+ *   residual_post_norm: x += y / sqrt(mean(y^2) + eps) * (offset + w); then, where h is given, h = x in `dtype`, or with
+ *     w2 its norm x / sqrt(mean(x^2) + eps) * (offset + w2).  One launch per sublayer. */
+int axb200_embed_residual(const int64_t *ids, const void *table, float *x, void *h, int64_t n, int64_t vocab, int width,
+                          int dtype, void *stream);
+int axb200_residual_post_norm(float *x, const void *y, const void *w, float offset, float eps, const void *w2, void *h,
+                              int64_t rows, int width, int dtype, void *stream);
+
 /* ---- latent attention ----------------------------------------------------------------------------------
  * Attention whose cache holds one row [c (kv_rank) | rotated key part (rot_dim)] per token, shared by all heads:
  * head h's key is [W_uk c | rotated part], its value W_uv c.  Row r of a launch belongs to sequence
  * row_seq[r] (row of block_table) and stands at position row_pos[r]; pages (num_pages, page_tokens,
- * kv_rank + rot_dim).  FLOAT32 or BFLOAT16; scores, weights and sums in fp32.
+ * row_elems), row_elems = kv_rank + rot_dim.  FLOAT32 or BFLOAT16; scores, weights and sums in fp32.
  *
  *   latent_prepare: per row, any of: rotate the last rot_dim elements of every head of q (rows, q_ld) in place
  *     (heads of [dim | rot_dim]); cq = rms_norm(dq) * dq_w over q_rank; append [rms_norm(dkv[:kv_rank]) * dkv_w |
@@ -500,12 +509,17 @@ int axb200_residual_layer_norm(float *x, const void *a, const void *b, const voi
  *     position * inv_freq[i] (device, double); elements past 2 * rot_pairs pass unchanged.
  *   latent_attend: out (rows, heads, kv_rank) = sum over j <= row_pos[r] of softmax((q_lat . c_j +
  *     q_rot . rot_j) * scale) c_j, with q_lat (rows, heads, kv_rank) = q . W_uk and q_rot read from q.
- *     max_len bounds row_pos + 1 and sizes the grid.
- *   latent_gather: rows 0 .. n-1 of one sequence's pages, contiguous.
+ *     max_len bounds row_pos + 1 and sizes the grid.  window > 0: only the keys j > row_pos[r] - window take part.
+ *     sink (heads) or NULL: exp(sink_h) joins the denominator.  kv_heads > 1 (then rot_dim = 0): the row holds kv_heads
+ *     parts of kv_rank elements, query head h reads part h / (heads / kv_heads).  key_scale >= 0: the row's element at
+ *     which an fp32 factor of its scores stands (key_scale < 0: none).  workspace_bytes takes the heads per part.
+ *   latent_gather: rows first .. first + n - 1 of one sequence's pages, contiguous.
  *   latent_prefill: the expanded form for n rows of ONE sequence at positions start .. start + n - 1: q (n, q_ld)
  *     rotated, k (skv, heads * dim) and v (skv, heads * vdim) expanded from the latents of positions 0 .. skv - 1
- *     (skv = start + n), rot = the rotated key parts, row stride rot_ld; out (n, heads, vdim).  BFLOAT16 on
- *     tcgen05; latent_prefill_supported tells which sizes. */
+ *     (skv = start + n), rot = the rotated key parts, row stride rot_ld (NULL with rot_dim 0); out (n, heads, vdim).
+ *     kv_heads below heads: k and v have kv_heads heads, each for a group of query heads.  window, sink as above (a
+ *     caller that gathers only the keys a window needs counts positions from the first of them).  BFLOAT16 on tcgen05;
+ *     latent_prefill_supported tells which sizes. */
 int axb200_latent_prepare(void *q, int64_t q_ld, int heads, int dim, const void *dq, int64_t dq_ld, int q_rank,
                           const void *dq_w, void *cq, const void *dkv, int64_t dkv_ld, int kv_rank,
                           const void *dkv_w, float eps, void *pages, const int32_t *block_table,
@@ -514,16 +528,69 @@ int axb200_latent_prepare(void *q, int64_t q_ld, int heads, int dim, const void 
                           int dtype, void *stream);
 size_t axb200_latent_attend_workspace_bytes(int rows, int heads, int kv_rank, int rot_dim, int64_t max_len, int dtype);
 int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim, void *out, const void *pages,
-                         const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, int rows,
-                         int heads, int kv_rank, int rot_dim, float scale, int page_tokens, int max_blocks,
-                         int num_pages, int max_seqs, int64_t max_len, int dtype, void *workspace,
-                         size_t workspace_bytes, void *stream);
-int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out, int64_t n, int row_elems,
+                         const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, const float *sink,
+                         int rows, int heads, int kv_heads, int kv_rank, int rot_dim, int row_elems, int key_scale,
+                         int window, float scale, int page_tokens, int max_blocks, int num_pages, int max_seqs,
+                         int64_t max_len, int dtype, void *workspace, size_t workspace_bytes, void *stream);
+int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out, int64_t first, int64_t n, int row_elems,
                          int page_tokens, int max_blocks, int num_pages, int dtype, void *stream);
 int axb200_latent_prefill_supported(int heads, int dim, int rot_dim, int vdim, int dtype);
 int axb200_latent_prefill(const void *q, int64_t q_ld, const void *k, const void *v, const void *rot, int64_t rot_ld,
-                          void *out, int n, int64_t start, int heads, int dim, int rot_dim, int vdim, float scale,
-                          int dtype, void *stream);
+                          const float *sink, void *out, int n, int64_t start, int heads, int kv_heads, int dim,
+                          int rot_dim, int vdim, int window, float scale, int dtype, void *stream);
+
+/* ---- grouped attention whose values are the raw keys ------------------------------------------------------
+ * The cache row is [kv_heads parts of dim raw key elements | ... | fp32 factor at element key_scale], the factor
+ * 1 / rms of all raw elements of the row: factor * part * k_w is the normed key, the part itself the value.
+ *   shared_kv_prepare: per row q_out (rows, heads * dim) = rms_norm(q) * q_w * (k_w of the head's part), the norm over
+ *     all heads at once, and the append of the raw keys and their factor.  latent_attend with kv_rank = dim, kv_heads
+ *     and key_scale then is the attention.
+ *   shared_kv_gather: rows first .. first + n - 1 of one sequence as keys (part * factor) and values (part), both (n,
+ *     kv_heads * dim), for latent_prefill. */
+int axb200_shared_kv_prepare(const void *q, int64_t q_ld, const void *q_w, void *q_out, const void *k, int64_t k_ld,
+                             const void *k_w, float eps, void *pages, const int32_t *block_table,
+                             const int32_t *row_seq, const int32_t *row_pos, int64_t rows, int heads, int kv_heads,
+                             int dim, int row_elems, int key_scale, int page_tokens, int max_blocks, int num_pages,
+                             int max_seqs, int dtype, void *stream);
+int axb200_shared_kv_gather(const void *pages, const int32_t *block_row, void *keys, void *values, int64_t first,
+                            int64_t n, int kv_heads, int dim, int row_elems, int key_scale, int page_tokens,
+                            int max_blocks, int num_pages, int dtype, void *stream);
+
+/* ---- gated delta rule -------------------------------------------------------------------------------------
+ * A recurrent mixer.  proj (rows, ld) holds per row [q | k | v | gate | a | b]: kv_heads * dim twice, heads * vdim
+ * twice, heads twice.  q, k and v (the channels) pass a causal convolution over time - conv (taps, channels) fp32, the
+ * current token's tap last - and silu; q and k become unit vectors per head (x / sqrt(sum x^2 + 1e-6)), q times
+ * dim^-0.5.  Per head S (dim x vdim) <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q with g = exp(-exp(a_log)
+ * softplus(a + dt_bias)), beta = sigmoid(b); out = o / sqrt(mean(o^2) + eps) * norm * silu(gate).  Query head h uses
+ * q / k head h / (heads / kv_heads).
+ * Per sequence slot the caller keeps state (max_seqs, heads, dim, vdim) fp32 and ring (max_seqs, taps, channels) of
+ * `dtype`, the inputs of position p in slot p % taps.  A row at position 0 starts from nothing whatever they hold.
+ * FLOAT32 or BFLOAT16 activations; everything inside the recurrence in fp32.  dim <= 256.
+ *   delta_step: rows of different sequences, one token each, in one launch: out (rows, heads * vdim).
+ *   Rows first .. rows - 1 of a step that bring portions of sequences (row_back[r]: how many rows directly before r
+ *   are the same sequence's) go through
+ *   delta_prepare: qk (rows - first, 2 * kv_heads * dim) fp32 unit q and k, v (rows - first, heads * vdim), log_g and
+ *     beta (rows - first, heads) fp32;
+ *   delta_scan: the recurrence over portions (count x {sequence, first row, rows, start position}, int32), token by
+ *     token: out (rows - first, heads * vdim);
+ *   delta_finish: norm and gate of that output, and the ring's new entries. */
+int axb200_delta_step(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos, int rows,
+                      const float *conv, const float *a_log, const float *dt_bias, const void *norm, void *ring,
+                      float *state, void *out, int heads, int kv_heads, int dim, int vdim, int taps, int max_seqs,
+                      float eps, int dtype, void *stream);
+int axb200_delta_prepare(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos,
+                         const int32_t *row_back, int first, int rows, const float *conv, const float *a_log,
+                         const float *dt_bias, const void *norm, void *ring, float *state, float *qk, void *v,
+                         float *log_g, float *beta, int heads, int kv_heads, int dim, int vdim, int taps, int max_seqs,
+                         float eps, int dtype, void *stream);
+int axb200_delta_scan(const int32_t *portions, int count, int first, const float *qk, const void *v, const float *log_g,
+                      const float *beta, float *state, void *out, int heads, int kv_heads, int dim, int vdim,
+                      int max_seqs, int dtype, void *stream);
+int axb200_delta_finish(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos,
+                        const int32_t *row_back, int first, int rows, const float *conv, const float *a_log,
+                        const float *dt_bias, const void *norm, void *ring, float *state, const void *o, void *out,
+                        int heads, int kv_heads, int dim, int vdim, int taps, int max_seqs, float eps, int dtype,
+                        void *stream);
 
 /* ---- mixture of experts ---------------------------------------------------------------------------------
  *   moe_route: per token, scores s = sigmoid(logits), choices s + correction; the experts form `groups` equal
@@ -577,6 +644,10 @@ int axb200_kv_arena_create(int n_layers, int num_pages, int hkv, int page_tokens
  * gives the pool (num_pages, page_tokens, row_elems[l]).  Everything else is the same. */
 int axb200_kv_arena_create_rows(int n_layers, const int32_t *row_elems, int num_pages, int page_tokens, int dtype,
                                 int max_seqs, int max_blocks, int device_memory, axb200_kv_arena **out);
+/* Adds a pool of `bytes_per_seq` bytes per sequence slot (zero-filled), for state that does not grow
+ * with the sequence; *pool is its device address (max_seqs x bytes_per_seq), NULL without device memory.  An arena of
+ * rows may have no row layers (n_layers 0) when all its sequences keep is such state. */
+int axb200_kv_arena_add_state(axb200_kv_arena *arena, int64_t bytes_per_seq, void **pool);
 int axb200_kv_arena_destroy(axb200_kv_arena *arena);
 /* Takes the lowest free sequence slot and pages for reserve_tokens; OUT_OF_MEMORY when slots or
  * pages run out (nothing is taken then). */
