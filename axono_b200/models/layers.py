@@ -181,17 +181,19 @@ class GatedDelta:
         return ((self.heads, self.dim, self.vdim), torch.float32), (tuple(self.conv.shape), dtype)
 
     def forward(self, h, rows: Rows, cache: Cache) -> torch.Tensor:
-        state, ring = cache.states[self.state_layer]
-        proj = ops.linear(h, self.w_in)
-        n, m = h.shape[0], rows.singles
-        out = torch.empty((n, self.heads * self.vdim), dtype=h.dtype, device=h.device)
+        return ops.linear(self.recur(ops.linear(h, self.w_in), rows, *cache.states[self.state_layer]), self.wo)
+
+    def recur(self, proj, rows: Rows, state, ring) -> torch.Tensor:
+        """Everything between the two products: proj (rows, >= columns of w_in) -> (rows, heads * vdim)."""
+        n, m = proj.shape[0], rows.singles
+        out = torch.empty((n, self.heads * self.vdim), dtype=proj.dtype, device=proj.device)
         if m:
             ops.delta_step(self, proj, rows, m, state, ring, out)
         if m < n:
             qk, v, log_g, beta = ops.delta_prepare(self, proj, rows, m, state, ring)
             ops.delta_scan(self, rows.portion_table, m, qk, v, log_g, beta, state, out[m:])
             ops.delta_finish(self, proj, rows, m, state, ring, out[m:], out[m:])
-        return ops.linear(out, self.wo)
+        return out
 
 
 class GatedMLP:

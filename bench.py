@@ -34,7 +34,8 @@ Other workloads, each with its own JSON line: `c2_block` (the fused decode block
 CUDA graph), `c5_tower` (the text-tower step by itself; `--runtime torch` runs it on the torch-tensor
 mirror), `prefill` (causal prefill attention; `--dtype f32` for the reference's own type), `ops` (the
 standalone operators at the multimodal prompt's shapes), `nuderax` (decode and prefill of the Nuderax
-layers beside the text tower's at equal size); `--impl reference-cuda` times the reference's
+layers beside the text tower's at equal size), `rigozen` (the same for the Rigozen layers, beside Nuderax's);
+`--impl reference-cuda` times the reference's
 own CUDA kernels compiled for sm_100; `--runtime torch` runs the attention workload on the torch mirror.
 """
 from __future__ import annotations
@@ -1321,14 +1322,128 @@ def lm_config(size, n_layers):
     return {"architecture": "Nuderax", "vocab": 32768, "width": z["width"], "norm": {"eps": 1e-5}, "layers": layers}
 
 
+class LmLab:
+    """What the language-model workloads share: peaks, clocks, timing on the device, random weights."""
+
+    def __init__(self, args):
+        import torch
+
+        torch.cuda.set_device(0)
+        self.torch, self.dev = torch, torch.device("cuda", 0)
+        self.gen = torch.Generator(device=self.dev).manual_seed(3)
+        try:
+            with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+                peaks = json.load(f)
+            self.gbs_peak, self.tf_peak, self.kind = float(peaks["hbm_gbs"]), float(peaks["bf16_tflops"]), "measured"
+        except Exception:
+            self.gbs_peak, self.tf_peak, self.kind = FALLBACK_HBM_GBS, 1590.0, "fallback"
+        self.warmup = max(3, args.warmup)
+        self.flush = torch.empty(64 << 20, dtype=torch.float32, device=self.dev)  # 256 MB, twice the L2
+        self.sampler = ClockSampler(0)
+
+    def timed(self, fn, n=20):
+        """Median milliseconds of one call, L2 flushed before each."""
+        torch = self.torch
+        for _ in range(3):
+            fn()
+        pairs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(n)]
+        self.sampler.start()
+        for e0, e1 in pairs:
+            self.flush.zero_()
+            e0.record()
+            fn()
+            e1.record()
+        torch.cuda.synchronize()
+        self.sampler.pause()
+        return statistics.median(e0.elapsed_time(e1) for e0, e1 in pairs)
+
+    def replayed(self, step, steps, warmup=None):
+        """Mean milliseconds of consecutive calls."""
+        torch = self.torch
+        for _ in range(self.warmup if warmup is None else warmup):
+            step()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        self.sampler.start()
+        e0.record()
+        for _ in range(steps):
+            step()
+        e1.record()
+        torch.cuda.synchronize()
+        self.sampler.pause()
+        return e0.elapsed_time(e1) / steps
+
+    def weights(self, shapes, around_zero=("correction", "norm1", "norm2", "final.norm", "A_log", "dt_bias", "sink")):
+        """name -> random tensor; vectors named in around_zero have mean 0, the others 1."""
+        lab, torch = self, self.torch
+
+        class RandomWeights(dict):
+            def __missing__(self, name):
+                shape = shapes[name]
+                if len(shape) == 1:
+                    mean = 0.0 if name.endswith(around_zero) else 1.0
+                    return mean + 0.1 * torch.randn(shape, generator=lab.gen, device=lab.dev)
+                gain = 1.0 if name == "embed" else shape[1] ** -0.5
+                return (gain * torch.randn(shape, generator=lab.gen, device=lab.dev)).to(torch.bfloat16)
+
+        return RandomWeights()
+
+    def bandwidth(self, K, name, ms, nbytes, like=None):
+        K[name] = {"us": ms * 1e3, "gbs": nbytes / (ms * 1e6), "frac": nbytes / (ms * 1e6) / self.gbs_peak, "bound": "hbm", "like": like}
+
+    def tensor(self, K, name, ms, flops, like=None):
+        K[name] = {"us": ms * 1e3, "tflops": flops / (ms * 1e9), "frac": flops / (ms * 1e9) / self.tf_peak, "bound": "tensor", "like": like}
+
+    def decode(self, model, batch, length, steps):
+        """(ms per step, launches) of decoding a batch at a context length by graph replays."""
+        from axono_b200.serving import DecodeGraph, ModelRunner
+
+        total = length + steps + self.warmup + 8
+        runner = ModelRunner(model, batch * (total + 64), max_seqs=batch, max_seq_len=total + 64, shuffle_pages=1)
+        for pool in runner.pages:
+            pool.normal_(generator=self.gen)
+        for layer in runner.states:
+            for t in layer:
+                t.normal_(generator=self.gen)
+        seqs = [runner.open() for _ in range(batch)]
+        for s in seqs:
+            runner.lengths[s] = length
+        g = DecodeGraph(runner, seqs, self.torch.randint(0, model.vocab, (batch,)).tolist(), [total] * batch)
+        ms = self.replayed(g.step, steps)
+        nodes = g.graph.num_nodes
+        g.graph.reset()
+        runner.arena.close()
+        return ms, nodes
+
+    def prefill(self, model, tokens, portion):
+        """Milliseconds of bringing one prompt in portions."""
+        from axono_b200.serving import ModelRunner
+
+        runner = ModelRunner(model, tokens + 64, max_seqs=1)
+        prompt = self.torch.randint(0, model.vocab, (tokens,)).tolist()
+
+        def once():
+            s = runner.open()
+            for at in range(0, tokens, portion):
+                part = prompt[at:at + portion]
+                runner.step([(s, part, [len(part) - 1] if at + portion >= tokens else [])])
+            runner.close(s)
+
+        ms = self.replayed(once, 5, 2)
+        runner.arena.close()
+        return ms
+
+
+def rounded(v):
+    return {k: rounded(x) for k, x in v.items()} if isinstance(v, dict) else float(f"{v:.4g}") if isinstance(v, float) else v
+
+
 def run_lm(args):
     """`nuderax`: decode and prefill throughput of Nuderax layers with random bf16 weights, beside the text tower
     (fp16, the framework's other decoder) with the same width, heads and context; and the kernels of both alone
     against the measured peaks.  Decode: CUDA-graph replays of whole steps, batch --lm-batch at context --lm-len.
     Prefill: one prompt of --prefill-len tokens through the runner (the tower has no prefill step: its prefill
     attention kernel stands beside).  Kernels: event pairs around single calls, L2 flushed before each."""
-    import math
-
     import torch
 
     from axono_b200 import models, ops
@@ -1338,64 +1453,18 @@ def run_lm(args):
     from axono_b200.models.nuderax import tensor_shapes
     from axono_b200.serving import DecodeGraph, ModelRunner
 
-    torch.cuda.set_device(0)
-    dev = torch.device("cuda", 0)
-    gen = torch.Generator(device=dev).manual_seed(3)
-    try:
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
-            peaks = json.load(f)
-        gbs_peak, tf_peak, kind = float(peaks["hbm_gbs"]), float(peaks["bf16_tflops"]), "measured"
-    except Exception:
-        gbs_peak, tf_peak, kind = FALLBACK_HBM_GBS, 1590.0, "fallback"
+    lab = LmLab(args)
+    dev, gen, sampler, warmup, timed, replayed = lab.dev, lab.gen, lab.sampler, lab.warmup, lab.timed, lab.replayed
+    gbs_peak, tf_peak, kind = lab.gbs_peak, lab.tf_peak, lab.kind
     B, L, S, n_layers = args.lm_batch, args.lm_len, args.prefill_len, args.lm_layers
-    warmup = max(3, args.warmup)
-    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)  # 256 MB, twice the L2
-    sampler = ClockSampler(0)
     launches = 0
-
-    def timed(fn, n=20):
-        """Mean milliseconds of one call, L2 flushed before each."""
-        for _ in range(3):
-            fn()
-        pairs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(n)]
-        sampler.start()
-        for e0, e1 in pairs:
-            flush.zero_()
-            e0.record()
-            fn()
-            e1.record()
-        torch.cuda.synchronize()
-        sampler.pause()
-        return statistics.median(e0.elapsed_time(e1) for e0, e1 in pairs)
-
-    def replayed(graph, steps):
-        for _ in range(warmup):
-            graph()
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        torch.cuda.synchronize()
-        sampler.start()
-        e0.record()
-        for _ in range(steps):
-            graph()
-        e1.record()
-        torch.cuda.synchronize()
-        sampler.pause()
-        return e0.elapsed_time(e1) / steps
-
-    class RandomWeights(dict):
-        def __missing__(self, name):
-            shape = shapes[name]
-            if len(shape) == 1:
-                return (0.0 if name.endswith("correction") else 1.0) + 0.1 * torch.randn(shape, generator=gen, device=dev)
-            gain = 1.0 if name == "embed" else 1.0 / math.sqrt(shape[1])
-            return (gain * torch.randn(shape, generator=gen, device=dev)).to(torch.bfloat16)
 
     results, total_steps = {}, args.steps + warmup + 8
     for size in (args.lm_sizes.split(",") if args.lm_sizes else ["2k", "4k"]):
         z = LM_SIZES[size]
         cfg = lm_config(size, n_layers)
         shapes = dict(tensor_shapes(models.config_of(cfg)))
-        model = models.create(cfg, RandomWeights(), torch.bfloat16)
+        model = models.create(cfg, lab.weights(shapes), torch.bfloat16)
         res = {"decode": {}, "prefill": {}, "kernels": {}}
 
         # ---- decode: whole steps as graph replays ----
@@ -1420,11 +1489,8 @@ def run_lm(args):
         # ---- its kernels at decode sizes ----
         K = res["kernels"]
 
-        def bandwidth(name, ms, nbytes, like=None):
-            K[name] = {"us": ms * 1e3, "gbs": nbytes / (ms * 1e6), "frac": nbytes / (ms * 1e6) / gbs_peak, "bound": "hbm", "like": like}
-
-        def tensor(name, ms, flops, like=None):
-            K[name] = {"us": ms * 1e3, "tflops": flops / (ms * 1e9), "frac": flops / (ms * 1e9) / tf_peak, "bound": "tensor", "like": like}
+        bandwidth = lambda *a: lab.bandwidth(K, *a)  # noqa: E731
+        tensor = lambda *a: lab.tensor(K, *a)  # noqa: E731
 
         bf = lambda *sh: torch.randn(sh, generator=gen, device=dev).to(torch.bfloat16)  # noqa: E731
         rows = Rows(torch.tensor(seqs, dtype=torch.int32, device=dev), torch.full((B,), L - 1, dtype=torch.int32, device=dev),
@@ -1560,15 +1626,240 @@ def run_lm(args):
     if err:
         raise SystemExit(f"device error word {err:#x}")
     first = next(iter(results.values()))["decode"]["nuderax"]
-    round_ = lambda v: {k: round_(x) for k, x in v.items()} if isinstance(v, dict) else float(f"{v:.4g}") if isinstance(v, float) else v  # noqa: E731
     print(json.dumps({
         "metric": "nuderax_decode_tokens_per_s", "value": first["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
         "warmup": warmup, "ms_per_step": first["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic",
         "config": {"workload": "nuderax", "sizes": list(results), "layers": n_layers, "batch": B, "kv_len": L, "prefill_len": S,
                    "l2": "steps read more than L2; single kernels after an L2 flush", "peaks": f"of {kind}"},
-        "results": round_(results), "gpu_launches": launches, "clocks": sampler.summary(),
+        "results": rounded(results), "gpu_launches": launches, "clocks": sampler.summary(),
     }), flush=True)
+
+
+RIGOZEN_SIZES = {
+    # name: width, ff; delta heads and kv_heads (128 x 128 each); latent heads (dim and values 128, latent 512); attention
+    # heads and kv_heads (128); window of both.  The Nuderax and tower sizes of the same name have the same width and heads.
+    "2k": dict(width=2048, ff=6144, delta=(16, 8), latent=16, attn=(16, 8), window=4096),
+    "4k": dict(width=4096, ff=12288, delta=(32, 16), latent=32, attn=(32, 8), window=4096),
+    "5k": dict(width=5120, ff=12288, delta=(64, 16), latent=128, attn=(128, 8), window=4096),
+}
+
+
+def rigozen_config(size, n_layers):
+    """Layers in the order delta, delta, latent attention, attention."""
+    z = RIGOZEN_SIZES[size]
+    mask, scale = {"size": z["window"]}, 128 ** -0.5
+    kinds = [("delta", dict(heads=z["delta"][0], kv_heads=z["delta"][1], dim=128, vdim=128, conv=4))] * 2 + [
+        ("latent_attention", dict(heads=z["latent"], dim=128, vdim=128, kv_rank=512, scale=scale, mask=mask)),
+        ("attention", dict(heads=z["attn"][0], kv_heads=z["attn"][1], dim=128, vdim=128, scale=scale, mask=mask))]
+    layers = [dict(type=kinds[i % 4][0], mixer=kinds[i % 4][1], mlp=dict(kind="dense", ff=z["ff"])) for i in range(n_layers)]
+    return {"architecture": "Rigozen", "vocab": 32768, "width": z["width"], "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def run_rigozen(args):
+    """`rigozen`: decode and prefill throughput of Rigozen layers with random bf16 weights, beside Nuderax layers with the
+    same width and heads (and the text tower's kernels); and each kernel alone against the measured peaks."""
+    import torch
+
+    from axono_b200 import models, ops
+    from axono_b200.models.layers import Rows
+    from axono_b200.serving import ModelRunner
+
+    lab = LmLab(args)
+    dev, gen, timed = lab.dev, lab.gen, lab.timed
+    B, L, S, n_layers = args.lm_batch, args.lm_len, args.prefill_len, args.lm_layers
+    launches, results = 0, {}
+    bf = lambda *sh: torch.randn(sh, generator=gen, device=dev).to(torch.bfloat16)  # noqa: E731
+    ints = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)  # noqa: E731
+    for size in (args.lm_sizes.split(",") if args.lm_sizes else ["2k", "4k"]):
+        z = RIGOZEN_SIZES[size]
+        width, ff, W = z["width"], z["ff"], z["window"]
+        res = {"decode": {}, "prefill": {}, "kernels": {}}
+        for name, cfg in (("rigozen", rigozen_config(size, n_layers)), ("nuderax", lm_config(size, n_layers))):
+            parsed = models.config_of(cfg)
+            module = sys.modules[type(parsed).__module__]
+            model = models.create(cfg, lab.weights(dict(module.tensor_shapes(parsed))), torch.bfloat16)
+            ms, nodes = lab.decode(model, B, L, args.steps)
+            launches += nodes * args.steps
+            res["decode"][name] = {"ms_per_step": ms, "tokens_per_s": B / ms * 1e3, "launches": nodes}
+            if name == "rigozen":
+                cached = sum(B * min(L, m.window) * r * 2.0 for m, r in zip([m for _, m, _, _ in model.layers if hasattr(m, "window")],
+                                                                            model.cache_rows))
+                state = sum(2 * B * 4.0 * shape[0][0][0] * shape[0][0][1] * shape[0][0][2] for shape in model.state_shapes)
+                need = model.weight_bytes() + cached + state
+                res["decode"][name].update(bytes_per_step=need, frac_of_hbm=need / (ms * 1e6) / lab.gbs_peak)
+            for portion in (S, min(2048, S)):
+                ms = lab.prefill(model, S, portion)
+                entry = {"ms": ms, "tokens_per_s": S / ms * 1e3}
+                if name == "rigozen":
+                    dense = sum(t.numel() for _, m, _, f in model.layers for obj in (m, f) for k, t in vars(obj).items()
+                                if isinstance(t, torch.Tensor) and t.dim() >= 2 and k != "conv")
+                    pairs = sum(min(t + 1, W) for t in range(S))
+                    rule = sum(S * 2.0 * 4 * z["delta"][0] * 128 * 128 for _ in model.state_shapes)  # the rule token by token
+                    att = sum(pairs * 4.0 * 128 * m.heads for _, m, _, _ in model.layers if hasattr(m, "window"))
+                    flops = 2.0 * S * dense + rule + att
+                    entry.update(tflops=flops / (ms * 1e9), frac_of_tensor=flops / (ms * 1e9) / lab.tf_peak)
+                res["prefill"][f"{name}, portions of {portion}"] = entry
+            if name == "rigozen":
+                res["kernels"].update(rigozen_kernels(lab, model, z, B, S))
+            del model
+            torch.cuda.empty_cache()
+        K = res["kernels"]
+
+        # ---- the like kernels of the other decoders ----
+        runner_rows = Rows(ints(list(range(B))), ints([W - 1] * B), torch.randperm(B * (W // 64), device=dev).to(torch.int32).view(B, -1), W, B)
+        H = z["latent"]
+        pool, ql, q = bf(B * (W // 64), 64, 576), bf(B, H, 512), bf(B, H * 192)
+        lab.bandwidth(K, "nuderax latent_attend (decode)", timed(lambda: ops.latent_attend(ql, q, 128, 64, 0.07, pool, runner_rows, B)),
+                      B * W * 1152.0 + 4.0 * ql.numel())
+        inv = torch.ones(32, dtype=torch.float64, device=dev)
+        proj, dw = bf(B, H * 192 + 576), bf(512)
+        lab.bandwidth(K, "nuderax norm + rotate + append (decode)", timed(lambda: ops.latent_prepare(
+            runner_rows, inv, 64, q=proj[:, :H * 192], heads=H, dim=128, dkv=proj[:, H * 192:], dkv_weight=dw, pages=pool)),
+            B * (H * 64 * 4.0 + 576 * 4))
+        x, w, a = torch.randn((S, width), generator=gen, device=dev), bf(width), bf(S, width)
+        lab.bandwidth(K, "nuderax residual + norm (prefill)", timed(lambda: ops.residual_layer_norm(x, w, None, 1e-5, a=a)), S * width * 12.0)
+        xd, ad = x[:B].contiguous(), a[:B].contiguous()
+        lab.bandwidth(K, "nuderax residual + norm (decode)", timed(lambda: ops.residual_layer_norm(xd, w, None, 1e-5, a=ad)), B * width * 12.0)
+        n = min(S, W)
+        prows = Rows(ints([0] * n), ints(list(range(n))), runner_rows.block_table[:1], W, n)
+        pproj = bf(n, H * 192 + 576)
+        lab.bandwidth(K, "nuderax norm + rotate + append (prefill)", timed(lambda: ops.latent_prepare(
+            prows, inv, 64, q=pproj[:, :H * 192], heads=H, dim=128, dkv=pproj[:, H * 192:], dkv_weight=dw, pages=pool)),
+            n * (H * 64 * 4.0 + 576 * 4))
+        del pproj
+        qp, kp, vp, cp = bf(S, H * 192), bf(S, H * 128), bf(S, H * 128), bf(S, 576)
+        lab.tensor(K, "nuderax prefill attention", timed(lambda: ops.latent_prefill(qp, 0, kp, vp, cp[:, 512:], H, 128, 64, 128, 0.07)),
+                   H * (S * (S + 1) / 2) * 2.0 * (192 + 128))
+        del qp, kp, vp, cp, pool
+        f16 = lambda *sh: torch.randn(sh, generator=gen, device=dev).half()  # noqa: E731
+        from axono_b200.kv_cache import PagedKVCache
+
+        heads, kv = z["attn"]
+        cache = PagedKVCache(1, B, kv, 128, W, dtype=torch.float16)
+        cache.k_pages[0].normal_(generator=gen)
+        cache.v_pages[0].normal_(generator=gen)
+        cache.seq_lens.fill_(W)
+        cache._host_len_bound = W
+        tq = f16(B, heads, 128)
+        lab.bandwidth(K, "tower gqa decode", timed(lambda: cache.attend(0, tq)), B * W * kv * 512.0 + 4.0 * tq.numel())
+        tqp, tk, tv = f16(S, heads, 128), f16(S, kv, 128), f16(S, kv, 128)
+        lab.tensor(K, "tower prefill attention", timed(lambda: ops.scaled_dot_product_attention(tqp, tk, tv, True)),
+                   4.0 * heads * 128 * (S * (S + 1) / 2))
+        gu = f16(S, 2 * ff)
+        lab.bandwidth(K, "tower silu_mul (prefill)", timed(lambda: ops.silu_mul_rows(gu, ff)), S * ff * 6.0)
+        gd = f16(B, 2 * ff)
+        lab.bandwidth(K, "tower silu_mul (decode)", timed(lambda: ops.silu_mul_rows(gd, ff)), B * ff * 6.0)
+        del cache, tqp, tk, tv, gu
+        torch.cuda.empty_cache()
+        results[size] = res
+    err = ops.last_error()
+    if err:
+        raise SystemExit(f"device error word {err:#x}")
+    first = next(iter(results.values()))["decode"]["rigozen"]
+    print(json.dumps({
+        "metric": "rigozen_decode_tokens_per_s", "value": first["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+        "warmup": lab.warmup, "ms_per_step": first["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "rigozen", "sizes": list(results), "layers": n_layers, "batch": B, "kv_len": L, "prefill_len": S,
+                   "l2": "steps read more than L2; single kernels after an L2 flush", "peaks": f"of {lab.kind}"},
+        "results": rounded(results), "gpu_launches": launches, "clocks": lab.sampler.summary(),
+    }), flush=True)
+
+
+def rigozen_kernels(lab, model, z, B, S):
+    """The kernels of one model alone, at decode (B rows) and prefill (S rows) sizes."""
+    import torch
+
+    from axono_b200 import ops
+    from axono_b200.models.layers import Rows
+    from axono_b200.serving import ModelRunner
+
+    K, dev, timed, W, width, ff = {}, lab.dev, lab.timed, z["window"], z["width"], z["ff"]
+    bf = lambda *sh: torch.randn(sh, generator=lab.gen, device=dev).to(torch.bfloat16)  # noqa: E731
+    ints = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)  # noqa: E731
+    _, delta, norm2, mlp = model.layers[0]
+    latent, attn = model.layers[2][1], model.layers[3][1]
+    n = max(S, W) + 64
+    runner = ModelRunner(model, B * n, max_seqs=B, max_seq_len=n, shuffle_pages=1)
+    for pool in runner.pages:
+        pool.normal_(generator=lab.gen)
+    for s in [runner.open() for _ in range(B)]:
+        runner.arena.reserve(s, n)
+    runner.arena.sync()
+    state, ring = runner.states[0]
+    state.normal_(generator=lab.gen)
+    pl, pa = runner.pages[latent.cache_layer], runner.pages[attn.cache_layer]
+    pa[..., attn.key_scale:].view(torch.float32).fill_(1.0)
+
+    # decode
+    rows = Rows(ints(list(range(B))), ints([W] * B), runner.block_table, W + 1, B, singles=B)
+    x, y, w = torch.randn((B, width), generator=lab.gen, device=dev), bf(B, width), bf(width)
+    proj, out = bf(B, delta.w_in.shape[0]), bf(B, delta.heads * delta.vdim)
+    lab.bandwidth(K, "decode delta_step", timed(lambda: ops.delta_step(delta, proj, rows, B, state, ring, out)),
+                  8.0 * B * delta.heads * delta.dim * delta.vdim + 2.0 * (proj.numel() + out.numel()), "tower gqa decode")
+    ql = bf(B, latent.heads, latent.kv_rank)
+    lab.bandwidth(K, "decode latent_attend", timed(lambda: ops.latent_attend(ql, None, 0, 0, 0.05, pl, rows, B, W, latent.sink)),
+                  B * W * latent.kv_rank * 2.0 + 4.0 * ql.numel(), "nuderax latent_attend (decode)")
+    pq = bf(B, attn.w_in.shape[0])
+    nq, nk = attn.heads * attn.dim, attn.kv_heads * attn.dim
+    prep = lambda p, r: ops.shared_kv_prepare(p[:, :nq], attn.q_norm, p[:, nq:nq + nk], attn.k_norm, pa, r, attn.heads,  # noqa: E731
+                                              attn.kv_heads, attn.dim, attn.key_scale, 1e-5)
+    lab.bandwidth(K, "decode shared_kv_prepare", timed(lambda: prep(pq, rows)), B * (4.0 * nq + 4.0 * nk), "nuderax norm + rotate + append (decode)")
+    qa = prep(pq, rows)
+    lab.bandwidth(K, "decode shared_kv attend", timed(lambda: ops.latent_attend(qa, None, attn.dim, 0, 0.05, pa, rows, B, W, None, attn.kv_heads,
+                                                                                attn.key_scale)),
+                  B * W * attn.row_elems * 2.0 + 4.0 * qa.numel(), "tower gqa decode")
+    lab.bandwidth(K, "decode residual_post_norm", timed(lambda: ops.residual_post_norm(x, y, w, 1e-5, 1.0)), B * width * 12.0,
+                  "nuderax residual + norm (decode)")
+    gd = bf(B, 2 * ff)
+    lab.bandwidth(K, "decode silu_mul", timed(lambda: ops.silu_mul_rows(gd, ff)), B * ff * 6.0, "tower silu_mul (decode)")
+
+    # prefill: one prompt
+    back = torch.arange(S, dtype=torch.int32, device=dev)
+    prows = Rows(torch.zeros(S, dtype=torch.int32, device=dev), back, runner.block_table, S, 0, [(0, 0, S, 0)], 0, back, [(0, 0, S, 0)],
+                 ints([[0, 0, S, 0]]))
+    x, y = torch.randn((S, width), generator=lab.gen, device=dev), bf(S, width)
+    lab.bandwidth(K, "prefill residual_post_norm", timed(lambda: ops.residual_post_norm(x, y, w, 1e-5, 1.0)), S * width * 12.0,
+                  "nuderax residual + norm (prefill)")
+    del x, y
+    gd = bf(S, 2 * ff)
+    lab.bandwidth(K, "prefill silu_mul", timed(lambda: ops.silu_mul_rows(gd, ff)), S * ff * 6.0, "tower silu_mul (prefill)")
+    del gd
+    proj = bf(S, delta.w_in.shape[0])
+    vv, channels = delta.heads * delta.vdim, delta.conv.shape[1]
+    lab.bandwidth(K, "prefill delta, all", timed(lambda: delta.recur(proj, prows, state, ring)), S * 2.0 * (proj.shape[1] + vv))
+    for name, (fn, nbytes) in delta_parts(ops, delta, proj, prows, state, ring).items():
+        lab.bandwidth(K, f"prefill {name}", timed(fn), nbytes, "nuderax norm + rotate + append (prefill)")
+    del proj
+    pq = bf(S, attn.w_in.shape[0])
+    lab.bandwidth(K, "prefill shared_kv_prepare", timed(lambda: prep(pq, prows)), S * (4.0 * nq + 4.0 * nk), "nuderax norm + rotate + append (prefill)")
+    lab.bandwidth(K, "prefill shared_kv_gather", timed(lambda: ops.shared_kv_gather(pa, runner.block_table[0], 0, S, attn.kv_heads, attn.dim,
+                                                                                    attn.key_scale)), S * nk * 6.0)
+    pairs = sum(min(t + 1, W) for t in range(S))
+    q, k, v = bf(S, nq), bf(S, nk), bf(S, nk)
+    lab.tensor(K, "prefill attention (shared kv)", timed(lambda: ops.latent_prefill(q, 0, k, v, None, attn.heads, 128, 0, 128, 0.05, W, None,
+                                                                                    attn.kv_heads)), pairs * 512.0 * attn.heads, "tower prefill attention")
+    H = latent.heads
+    q, k, v = bf(S, H * 128), bf(S, H * 128), bf(S, H * 128)
+    lab.tensor(K, "prefill attention (latent)", timed(lambda: ops.latent_prefill(q, 0, k, v, None, H, 128, 0, 128, 0.05, W, latent.sink)),
+               pairs * 512.0 * H, "nuderax prefill attention")
+    runner.arena.close()
+    return K
+
+
+def delta_parts(ops, delta, proj, rows, state, ring):
+    """The launches of GatedDelta.recur for one prompt: name -> (call, bytes)."""
+    import torch
+
+    n, vv, qk2 = proj.shape[0], delta.heads * delta.vdim, 2 * delta.kv_heads * delta.dim
+    out = torch.empty((n, vv), dtype=proj.dtype, device=proj.device)
+    qk, v, log_g, beta = ops.delta_prepare(delta, proj, rows, 0, state, ring)
+    return {
+        "delta_prepare": (lambda: ops.delta_prepare(delta, proj, rows, 0, state, ring), n * (2.0 * (qk2 + vv) + 4.0 * qk2 + 2.0 * vv)),
+        "delta_scan": (lambda: ops.delta_scan(delta, rows.portion_table, 0, qk, v, log_g, beta, state, out), n * (4.0 * qk2 + 4.0 * vv)),
+        "delta_finish": (lambda: ops.delta_finish(delta, proj, rows, 0, state, ring, out, out), n * vv * 6.0),
+    }
 
 
 def main():
@@ -1577,12 +1868,12 @@ def main():
     ap.add_argument("--steps", type=int, default=200)
     ap.add_argument("--warmup", type=int, default=10)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "reference-cuda"])
-    ap.add_argument("--workload", default="c3_ragged", choices=sorted(WORKLOADS) + ["c2_block", "c5_tower", "prefill", "ops", "nuderax"])
+    ap.add_argument("--workload", default="c3_ragged", choices=sorted(WORKLOADS) + ["c2_block", "c5_tower", "prefill", "ops", "nuderax", "rigozen"])
     ap.add_argument("--prefill-len", type=int, default=8192)
-    ap.add_argument("--lm-sizes", default="", help="nuderax: comma-separated sizes out of " + ", ".join(LM_SIZES) + " (default 2k,4k)")
-    ap.add_argument("--lm-batch", type=int, default=32, help="nuderax: sequences that decode together")
-    ap.add_argument("--lm-len", type=int, default=16384, help="nuderax: context length of decoding")
-    ap.add_argument("--lm-layers", type=int, default=4, help="nuderax: layers (even ones with direct, odd ones with low-rank queries)")
+    ap.add_argument("--lm-sizes", default="", help="nuderax, rigozen: comma-separated sizes out of " + ", ".join(LM_SIZES) + " (default 2k,4k)")
+    ap.add_argument("--lm-batch", type=int, default=32, help="nuderax, rigozen: sequences that decode together")
+    ap.add_argument("--lm-len", type=int, default=16384, help="nuderax, rigozen: context length of decoding")
+    ap.add_argument("--lm-layers", type=int, default=4, help="nuderax, rigozen: layers (nuderax: even ones with direct, odd ones with low-rank queries)")
     ap.add_argument("--ops-once", action="store_true",
                     help="ops: launch every operator once inside the profiler range and exit (for ncu)")
     ap.add_argument("--runtime", default="native", choices=["native", "torch"],
@@ -1615,12 +1906,15 @@ def main():
         if rank0:
             run_reference_cuda(args)
     elif args.impl == "reference":
-        if args.workload in ("c2_block", "c5_tower", "prefill", "ops", "nuderax"):
+        if args.workload in ("c2_block", "c5_tower", "prefill", "ops", "nuderax", "rigozen"):
             args.workload = "c2_b8_l8k" if args.workload == "c2_block" else "c3_ragged"
         run_reference_arm(args)
     elif args.workload == "nuderax":
         if rank0:
             run_lm(args)
+    elif args.workload == "rigozen":
+        if rank0:
+            run_rigozen(args)
     elif args.workload == "prefill":
         if rank0:
             run_prefill(args)

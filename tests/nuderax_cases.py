@@ -1,8 +1,6 @@
-"""Configurations of the Nuderax tests and the comparison of logits.  Sizes differ from layer to layer and
+"""Configurations of the Nuderax tests.  Sizes differ from layer to layer and
 are awkward on purpose in `odd`; `fast` has the sizes the tensor-core kernels take, and `tiles` some that end
 inside their tiles."""
-import numpy as np
-
 
 def _mixer(low_rank_q, heads, dim, rot_dim, rot_dims, vdim, kv_rank, scale, base, q_rank=None, kv_from=None):
     m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=scale, rot=dict(base=base, dims=rot_dims))
@@ -49,12 +47,3 @@ def fast():
         (_mixer(True, 32, 64, 64, 64, 64, 256, 0.08, 40000.0, q_rank=192), moe),
         (_mixer(False, 20, 128, 64, 64, 128, 512, 0.07, 10000.0, kv_from=0), moe),
     ])
-
-
-def position_errors(got, want):
-    """Per position: rms of the difference (means taken off) over the rms of the wanted logits."""
-    got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
-    d = got - want
-    d -= d.mean(-1, keepdims=True)
-    w = want - want.mean(-1, keepdims=True)
-    return np.sqrt((d * d).mean(-1)) / np.sqrt((w * w).mean())

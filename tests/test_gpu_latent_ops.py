@@ -6,6 +6,7 @@ import pytest
 import torch
 
 import plain_nuderax as plain
+from lm_helpers import Pages, close, rnd
 
 pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16]
@@ -13,17 +14,6 @@ DTYPES = [torch.float32, torch.bfloat16]
 
 def tol(dtype):
     return 3e-6 if dtype == torch.float32 else 1.2e-2
-
-
-def rnd(shape, dtype, seed, scale=1.0):
-    g = torch.Generator().manual_seed(seed)
-    return (scale * torch.randn(shape, generator=g)).to(dtype)
-
-
-def close(got, want, t):
-    got, want = got.double().cpu(), want.double().cpu()
-    err = (got - want).abs().max().item() / max(1e-30, want.abs().max().item())
-    assert err <= t, f"{err:.3e}"
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -65,31 +55,6 @@ def test_embed_layer_norm_and_bad_id(dtype):
     assert ops.last_error() == 0
     ops.embed_layer_norm(torch.tensor([50], device="cuda"), table.cuda(), w.cuda(), 1e-5)
     assert ops.last_error() & 8
-
-
-class Pages:
-    """A paged latent cache with shuffled pages, filled from contiguous rows."""
-
-    def __init__(self, lens, row_elems, dtype, page_tokens=64, seed=0, fill=1e4):
-        blocks = max(-(-n // page_tokens) for n in lens) + 1
-        self.table = torch.full((len(lens), blocks), -1, dtype=torch.int32)
-        perm = torch.randperm(len(lens) * blocks, generator=torch.Generator().manual_seed(seed)).to(torch.int32)
-        for s, n in enumerate(lens):
-            used = -(-n // page_tokens)
-            self.table[s, :used] = perm[s * blocks:s * blocks + used]
-        # what no sequence owns, and what lies behind a sequence's end, is large: reading it would show
-        self.pool = torch.full((len(lens) * blocks, page_tokens, row_elems), fill).to(dtype)
-        self.page_tokens = page_tokens
-
-    def put(self, s, rows):
-        for t in range(rows.shape[0]):
-            self.pool[int(self.table[s, t // self.page_tokens]), t % self.page_tokens] = rows[t]
-
-    def rows(self, seq, pos, max_len, segments=()):
-        from axono_b200.models.layers import Rows
-
-        return Rows(torch.tensor(seq, dtype=torch.int32).cuda(), torch.tensor(pos, dtype=torch.int32).cuda(), self.table.cuda(),
-                    max_len, len(seq), list(segments))
 
 
 @pytest.mark.parametrize("dtype", DTYPES)

@@ -9,6 +9,7 @@ import torch
 
 import nuderax_cases as cases
 import plain_nuderax as plain
+from lm_helpers import SCHEDULES, feed, position_errors, runner_of
 
 pytestmark = pytest.mark.gpu
 
@@ -33,33 +34,12 @@ def built():
     return get
 
 
-def runner_of(cfg, w, dtype, max_tokens, **kw):
-    from axono_b200 import models
-    from axono_b200.serving import ModelRunner
-
-    return ModelRunner(models.create(cfg, w, dtype), max_tokens, **kw)
-
-
-def feed(runner, seq, tokens, portions):
-    """All logits of `tokens` brought in portions of the given sizes (the last size repeats)."""
-    out, at, sizes = [], 0, list(portions)
-    while at < len(tokens):
-        n = min(sizes.pop(0) if len(sizes) > 1 else sizes[0], len(tokens) - at)
-        out.append(runner.step([(seq, tokens[at:at + n], list(range(n)))]).cpu().numpy())
-        at += n
-    assert runner.error_word() == 0
-    return np.concatenate(out)
-
-
 def check(got, ref, dtype):
-    err = cases.position_errors(got, ref)
+    err = position_errors(got, ref)
     if dtype == torch.float32:
         assert err.max() <= F32_TOL, f"worst {err.max():.2e} at {int(err.argmax())}"
     else:
         assert np.quantile(err, 0.8) <= 0.04 and err.max() <= 1.0, f"{np.quantile(err, 0.8):.3f} {err.max():.3f}"
-
-
-SCHEDULES = {"whole": [10000], "tokens": [1], "twos": [2], "mixed": [5, 2, 64, 1, 63, 3, 17, 65, 2, 1], "prompt_then_tokens": [120, 1]}
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
