@@ -115,6 +115,9 @@ SIGNATURES = {
     "axb200_delta_step": (_i, [_vp, _i64, _vp, _vp, _i] + [_vp] * 6 + [_vp] + [_i] * 6 + [_f, _i, _vp]),
     "axb200_delta_prepare": (_i, [_vp, _i64, _vp, _vp, _vp, _i, _i] + [_vp] * 6 + [_vp] * 4 + [_i] * 6 + [_f, _i, _vp]),
     "axb200_delta_scan": (_i, [_vp, _i, _i] + [_vp] * 6 + [_i] * 6 + [_vp]),
+    "axb200_delta_chunks_supported": (_i, [_i] * 3),
+    "axb200_delta_chunks_workspace_bytes": (_sz, [_i64] + [_i] * 5),
+    "axb200_delta_chunks": (_i, [_vp, _i64, _vp, _vp, _vp, _i, _i] + [_vp] * 6 + [_i, _i, _vp] + [_i] * 7 + [_vp, _sz, _vp]),
     "axb200_delta_finish": (_i, [_vp, _i64, _vp, _vp, _vp, _i, _i] + [_vp] * 6 + [_vp] * 2 + [_i] * 6 + [_f, _i, _vp]),
     "axb200_moe_route": (_i, [_vp] * 6 + [_i64, _i, _i, _i, _i, _f, _vp]),
     "axb200_moe_tile_rows": (_i, [_i64, _i, _i, _i, _i]),

@@ -27,7 +27,7 @@ LIB_DIR = os.path.join(PKG, "lib")
 OBJ_DIR = os.path.join(LIB_DIR, "obj")
 LIB = os.path.join(LIB_DIR, "libaxono_b200.so")
 SERVING_LIB = os.path.join(LIB_DIR, "libaxono_b200_lm.so")
-SERVING_SOURCES = ("core.cu", "delta.cu", "fused.cu", "kv_arena.cu", "latent_attn.cu", "latent_prefill.cu", "latent_umma.cu",
+SERVING_SOURCES = ("core.cu", "delta.cu", "delta_chunk.cu", "fused.cu", "kv_arena.cu", "latent_attn.cu", "latent_prefill.cu", "latent_umma.cu",
                    "linear_lt.cpp", "moe.cu", "moe_umma.cu", "residual_norm.cu", "shared_kv.cu")
 
 NVCC_FLAGS = [

@@ -175,6 +175,8 @@ class GatedDelta:
         self.conv = torch.cat([conv_q, conv_k, conv_v]).float().t().contiguous()
         self.a_log, self.dt_bias = a_log.float().contiguous(), dt_bias.float().contiguous()
         self.norm, self.wo = norm, wo
+        # from how many rows on a portion goes through the tensor-core form
+        self.chunk_from = 24 if ops.delta_chunks_supported(dim, vdim, wo.dtype) else 1 << 62
 
     def state_shapes(self, dtype):
         """What one sequence keeps: (shape, dtype) of the matrices and of the convolution's last inputs."""
@@ -190,8 +192,13 @@ class GatedDelta:
         if m:
             ops.delta_step(self, proj, rows, m, state, ring, out)
         if m < n:
-            qk, v, log_g, beta = ops.delta_prepare(self, proj, rows, m, state, ring)
-            ops.delta_scan(self, rows.portion_table, m, qk, v, log_g, beta, state, out[m:])
+            short = sum(p[2] < self.chunk_from for p in rows.portions)  # portions come by length
+            c = rows.portions[short][1] if short < len(rows.portions) else n
+            if short:
+                qk, v, log_g, beta = ops.delta_prepare(self, proj[:c], rows, m, state, ring)
+                ops.delta_scan(self, rows.portion_table[:short], m, qk, v, log_g, beta, state, out[m:c])
+            if c < n:
+                ops.delta_chunks(self, proj, rows, rows.portion_table[short:], rows.portions[-1][2], c, state, ring, out[c:])
             ops.delta_finish(self, proj, rows, m, state, ring, out[m:], out[m:])
         return out
 

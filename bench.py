@@ -1854,10 +1854,8 @@ def delta_parts(ops, delta, proj, rows, state, ring):
 
     n, vv, qk2 = proj.shape[0], delta.heads * delta.vdim, 2 * delta.kv_heads * delta.dim
     out = torch.empty((n, vv), dtype=proj.dtype, device=proj.device)
-    qk, v, log_g, beta = ops.delta_prepare(delta, proj, rows, 0, state, ring)
     return {
-        "delta_prepare": (lambda: ops.delta_prepare(delta, proj, rows, 0, state, ring), n * (2.0 * (qk2 + vv) + 4.0 * qk2 + 2.0 * vv)),
-        "delta_scan": (lambda: ops.delta_scan(delta, rows.portion_table, 0, qk, v, log_g, beta, state, out), n * (4.0 * qk2 + 4.0 * vv)),
+        "delta_chunks": (lambda: ops.delta_chunks(delta, proj, rows, rows.portion_table, n, 0, state, ring, out), n * 2.0 * (qk2 + 2 * vv)),
         "delta_finish": (lambda: ops.delta_finish(delta, proj, rows, 0, state, ring, out, out), n * vv * 6.0),
     }
 

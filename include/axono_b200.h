@@ -573,7 +573,9 @@ int axb200_shared_kv_gather(const void *pages, const int32_t *block_row, void *k
  *     beta (rows - first, heads) fp32;
  *   delta_scan: the recurrence over portions (count x {sequence, first row, rows, start position}, int32), token by
  *     token: out (rows - first, heads * vdim);
- *   delta_finish: norm and gate of that output, and the ring's new entries. */
+ *   delta_finish: norm and gate of that output, and the ring's new entries.
+ *   delta_chunks: delta_prepare and delta_scan in one call for portions of prompts, 64 tokens at a time on tensor cores
+ *     (BFLOAT16; sizes by delta_chunks_supported); `longest` bounds the portions' rows. */
 int axb200_delta_step(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos, int rows,
                       const float *conv, const float *a_log, const float *dt_bias, const void *norm, void *ring,
                       float *state, void *out, int heads, int kv_heads, int dim, int vdim, int taps, int max_seqs,
@@ -586,6 +588,13 @@ int axb200_delta_prepare(const void *proj, int64_t ld, const int32_t *row_seq, c
 int axb200_delta_scan(const int32_t *portions, int count, int first, const float *qk, const void *v, const float *log_g,
                       const float *beta, float *state, void *out, int heads, int kv_heads, int dim, int vdim,
                       int max_seqs, int dtype, void *stream);
+int axb200_delta_chunks_supported(int dim, int vdim, int dtype);
+size_t axb200_delta_chunks_workspace_bytes(int64_t rows, int count, int heads, int kv_heads, int dim, int vdim);
+int axb200_delta_chunks(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos,
+                        const int32_t *row_back, int first, int rows, const float *conv, const float *a_log,
+                        const float *dt_bias, void *ring, float *state, const int32_t *portions, int count, int longest,
+                        void *out, int heads, int kv_heads, int dim, int vdim, int taps, int max_seqs, int dtype,
+                        void *workspace, size_t workspace_bytes, void *stream);
 int axb200_delta_finish(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos,
                         const int32_t *row_back, int first, int rows, const float *conv, const float *a_log,
                         const float *dt_bias, const void *norm, void *ring, float *state, const void *o, void *out,

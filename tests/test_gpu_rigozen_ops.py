@@ -231,7 +231,12 @@ class Mixer:
 
     def weights(self):
         return SimpleNamespace(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, eps=self.eps, conv=self.conv.cuda(),
-                               a_log=self.a_log.cuda(), dt_bias=self.dt_bias.cuda(), norm=self.norm.cuda())
+                               a_log=self.a_log.cuda(), dt_bias=self.dt_bias.cuda(), norm=self.norm.cuda(), chunk_from=self.chunk_from())
+
+    def chunk_from(self):
+        from axono_b200 import ops
+
+        return 24 if ops.delta_chunks_supported(self.dim, self.vdim, self.dtype) else 1 << 62
 
     def inputs(self, n, seed):
         return rnd((n, self.cols + -self.cols % 8), self.dtype, seed)
