@@ -5,16 +5,19 @@
 //     o_t = e^{G_t} S^T q_t + sum_{s <= t} P_ts u_s,                P_ts = e^{G_t - G_s} (q_t . k_s),
 //     S'  = e^{G_64} S + sum_s e^{G_64 - G_s} k_s u_s^T.
 // delta_chunk_prepare does what needs no state, all chunks at once: convolutions and silu, the products of queries and
-// keys, T = (I + A)^-1 diag(beta) by blocked forward substitution in fp32, P, and the scale vectors.  delta_chunk_scan
-// walks a sequence's chunks: a warp owns 16 value columns of a head's state and is independent of all others.
+// keys, T = (I + A)^-1 diag(beta) by blocked forward substitution, P, and the scale vectors.  delta_chunk_scan walks a
+// sequence's chunks: a warp owns 8 value columns of a head's state and is independent of all others.
 //
 // Precision.  The outputs of the short convolutions are bf16, so they are exact tensor-core operands: unit norms and
 // decays stay outside the products, as fp32 factors of rows.  Everything else that enters a product - state, X, U, T, P -
 // is split into two bf16 parts and multiplied part by part (high.high + low.high + high.low), accumulated in fp32.
 //
-// The transposed products chain in registers: S^T (values x keys) is the accumulator of the update and operand A of the
-// next chunk's products, X^T and U^T likewise, so the recurrence touches no shared memory.  Keys, T and P are operand B
-// and come as ready-made, swizzled tiles by bulk copies, two or three chunks ahead.
+// The products chain in registers: S (keys x 8 values) is the accumulator of the update and, transposed in the register
+// file (movmatrix), operand B of the next chunk's products; X and U likewise.  So the recurrence touches no shared memory.
+// Keys, queries, T and P are operand A and come as ready-made, swizzled tiles by bulk copies, some chunks ahead.
+// The walk is bound by the length of this chain, not by the tensor cores of a whole SM: the chain of 64 tokens is 250
+// warp-wide products of 16 x 8 x 16 at about ten cycles each.  Products of tcgen05 size would need 64 or more columns and
+// four round trips through tensor and shared memory per chunk, which together take longer.
 #include <math.h>
 
 #include <mutex>
@@ -25,14 +28,20 @@ namespace axb {
 namespace {
 
 constexpr int kC = 64;                    // tokens of a chunk
-constexpr int kSquare = kC * kC * 2;      // bytes of one bf16 part of T or P
+constexpr int kSquare = 10 * 512;         // bytes of one bf16 part of T or P: its ten lower 16 x 16 blocks
 constexpr int kVec = 4 * kSquare;         // where the scale vectors start in a head's tiles: ek, eq, eu [64], total
 constexpr int kHeadTiles = kVec + 1024;   // T high, T low, P high, P low, vectors
-constexpr int kValueTile = kC * 16 * 2;   // [64 tokens][16 value columns]
+constexpr int kValueTile = kC * 8 * 2;    // [64 tokens][8 value columns]
+constexpr int kPrepHeads = 4;             // heads whose gates a block holds at a time
 constexpr float kUnitEps = 1e-6f;
 
 // Byte offset of 16-byte piece `piece` of row `row` in a tile of rows of `pieces` pieces, swizzled for ldmatrix.
 __device__ __forceinline__ uint32_t tile_at(int row, int piece, int pieces) { return (uint32_t)((row * pieces + (piece ^ (row & 7))) << 4); }
+
+// Byte offset of 16-byte piece `piece` (0, 1) of row `row` of block (m, k), k <= m, in one part of T or P.
+__device__ __forceinline__ uint32_t block_at(int m, int k, int row, int piece) {
+  return (uint32_t)((m * (m + 1) / 2 + k) * 512 + row * 32 + ((piece ^ ((row >> 2) & 1)) << 4));
+}
 
 __device__ __forceinline__ float bf_lo(uint32_t v) { return __uint_as_float(v << 16); }
 __device__ __forceinline__ float bf_hi(uint32_t v) { return __uint_as_float(v & 0xffff0000u); }
@@ -47,13 +56,22 @@ __device__ __forceinline__ void split(float a, float b, uint32_t &high, uint32_t
 __device__ __forceinline__ int first_chunk(const int4 &portion, int i, int first) { return (portion.y - first) / kC + i; }
 
 // ---- chunks by themselves ----------------------------------------------------------------------------
-constexpr int kPrepThreads = 256, kLd = kC + 4;  // fp32 matrices in shared memory have rows of kLd
+constexpr int kPrepThreads = 256, kLd = kC + 8;  // fp32 matrices in shared memory have rows of kLd
 
-// Convolution and silu of four channels from c on over tokens t0 .. t0 + count - 1 of a chunk; put(t, values).
-template <typename Put>
-__device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, int64_t row0, int valid, int c, int t0, int count, Put put) {
+// silu of what a convolution puts out (an activation that is rounded to bf16)
+__device__ __forceinline__ float fast_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
+// Convolution and silu of four channels from c on over kCount tokens from t0 on of a chunk; put(t, values).
+template <int kCount, typename Put>
+__device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, int64_t row0, int valid, int c, int t0, Put put) {
   const int channels = p.channels();
   if (p.taps <= 4) {
+    uint2 raw[kCount];  // all on their way at once
+#pragma unroll
+    for (int i = 0; i < kCount; ++i) {
+      raw[i] = make_uint2(0, 0);
+      if (t0 + i < valid) raw[i] = *reinterpret_cast<const uint2 *>(p.proj + (row0 + t0 + i) * p.ld + c);
+    }
     float w[4][4], past[3][4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -67,24 +85,23 @@ __device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, i
       for (int e = 0; e < 4; ++e) past[j][e] = 0.f;
       if (j + 1 < p.taps && t0 < valid) earlier_input<4>(p, row0 + t0, j + 1, c, past[j]);
     }
-#pragma unroll 4
-    for (int t = t0; t < t0 + count; ++t) {
-      float now[4] = {}, y[4] = {};
-      if (t < valid) {
-        load_vec<4>(p.proj + (row0 + t) * p.ld + c, now);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          y[e] = silu(fmaf(past[2][e], w[3][e], fmaf(past[1][e], w[2][e], fmaf(past[0][e], w[1][e], now[e] * w[0][e]))));
-          past[2][e] = past[1][e];
-          past[1][e] = past[0][e];
-          past[0][e] = now[e];
-        }
+    for (int i = 0; i < kCount; ++i) {
+      const float now[4] = {bf_lo(raw[i].x), bf_hi(raw[i].x), bf_lo(raw[i].y), bf_hi(raw[i].y)};
+      float y[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        y[e] = fmaf(past[2][e], w[3][e], fmaf(past[1][e], w[2][e], fmaf(past[0][e], w[1][e], now[e] * w[0][e])));
+        y[e] = t0 + i < valid ? fast_silu(y[e]) : 0.f;
+        past[2][e] = past[1][e];
+        past[1][e] = past[0][e];
+        past[0][e] = now[e];
       }
-      put(t, y);
+      put(t0 + i, y);
     }
     return;
   }
-  for (int t = t0; t < t0 + count; ++t) {
+  for (int t = t0; t < t0 + kCount; ++t) {
     float y[4] = {};
     if (t < valid) {
       for (int j = 0; j < p.taps; ++j) {
@@ -95,34 +112,40 @@ __device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, i
         for (int e = 0; e < 4; ++e) y[e] = fmaf(in[e], w[e], y[e]);
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) y[e] = silu(y[e]);
+      for (int e = 0; e < 4; ++e) y[e] = fast_silu(y[e]);
     }
     put(t, y);
   }
 }
 
-// out[i0 .. i0 + rows)[j0 .. j0 + 4 per thread) = sign * a (rows x inner) . b (inner x cols), matrices of stride kLd; four
-// neighbouring outputs per thread.
-__device__ __forceinline__ void square_product(float *out, const float *a, const float *b, int rows, int inner, int cols, float sign,
-                                               int tid, int threads) {
-  const int quads = cols / 4;
-  for (int i = tid; i < rows * quads; i += threads) {
-    const int r = i / quads, c = i % quads * 4;
-    float acc[4] = {};
-    for (int k = 0; k < inner; ++k) {
-      const float x = a[r * kLd + k];
-      const float4 y = *reinterpret_cast<const float4 *>(b + k * kLd + c);
-      acc[0] = fmaf(x, y.x, acc[0]), acc[1] = fmaf(x, y.y, acc[1]), acc[2] = fmaf(x, y.z, acc[2]), acc[3] = fmaf(x, y.w, acc[3]);
+// One warp: out (16 x 8) = sign * a (16 x 16 n) . b (16 n x 8), fp32 matrices of stride kLd in shared memory, in bf16
+// parts on the tensor core.
+__device__ __forceinline__ void small_product(float *out, const float *a, const float *b, int n, float sign, int lane) {
+  const int g = lane >> 2, q = (lane & 3) * 2;
+  float acc[4] = {};
+  for (int k = 0; k < n; ++k, a += 16, b += 16 * kLd) {
+    uint32_t ah[4], al[4], bh[2], bl[2];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 v = *reinterpret_cast<const float2 *>(a + (g + (i & 1) * 8) * kLd + q + (i >> 1) * 8);
+      split(v.x, v.y, ah[i], al[i]);
     }
-    *reinterpret_cast<float4 *>(out + r * kLd + c) = make_float4(sign * acc[0], sign * acc[1], sign * acc[2], sign * acc[3]);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) split(b[(q + i * 8) * kLd + g], b[(q + i * 8 + 1) * kLd + g], bh[i], bl[i]);
+    mma_16816_bf16(acc, ah, bh[0], bh[1]);
+    mma_16816_bf16(acc, al, bh[0], bh[1]);
+    mma_16816_bf16(acc, ah, bl[0], bl[1]);
   }
+  *reinterpret_cast<float2 *>(out + g * kLd + q) = make_float2(sign * acc[0], sign * acc[1]);
+  *reinterpret_cast<float2 *>(out + (g + 8) * kLd + q) = make_float2(sign * acc[2], sign * acc[3]);
 }
 
 template <int kDK>
 struct PrepSmem {
   static constexpr int kTile = kC * kDK * 2, kMatrix = kC * kLd * 4;
   static constexpr int kOffKK = 2 * kTile, kOffQK = kOffKK + kMatrix, kOffA = kOffQK + kMatrix, kOffT = kOffA + kMatrix;
-  static constexpr int kOffVec = kOffT + kMatrix, kBytes = kOffVec + 5 * kC * 4;
+  static constexpr int kOffVec = kOffT + kMatrix;
+  static constexpr int kBytes = kOffVec + 4 * kC * 4 + 2 * kPrepHeads * kC * 4;
 };
 
 // Block z < kv_heads: one chunk of one query / key head, and T, P and the vectors of its group of value heads; the others:
@@ -149,16 +172,14 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
 
   if ((int)blockIdx.z >= p.kv_heads) {
     // a quad of channels, a run of 8 tokens at a time
-    const int h = blockIdx.z - p.kv_heads, blocks = (p.vdim + 15) / 16, quads = blocks * 4;
+    const int h = blockIdx.z - p.kv_heads, blocks = p.vdim / 8, quads = blocks * 2;
     uint8_t *dst = values + (chunk * p.heads + h) * (size_t)blocks * kValueTile;
     for (int i = tid; i < quads * (kC / 8); i += kPrepThreads) {
-      const int quad = i % quads, c = quad * 4;
-      auto put = [&](int t, const float (&y)[4]) {
-        *reinterpret_cast<uint2 *>(dst + (c >> 4) * kValueTile + t * 32 + (c & 15) * 2) =
+      const int c = i % quads * 4;
+      conv_walk<8>(p, row0, valid, qk_channels + h * p.vdim + c, i / quads * 8, [&](int t, const float (&y)[4]) {
+        *reinterpret_cast<uint2 *>(dst + (c >> 3) * kValueTile + t * 16 + (c & 7) * 2) =
             make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
-      };
-      // past the last column the tile is zero
-      conv_walk(p, row0, c < p.vdim ? valid : 0, c < p.vdim ? qk_channels + h * p.vdim + c : 0, i / quads * 8, 8, put);
+      });
     }
     return;
   }
@@ -167,9 +188,36 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
   uint8_t *ck = smem, *cq = smem + S::kTile;
   float *kk = reinterpret_cast<float *>(smem + S::kOffKK), *qk = reinterpret_cast<float *>(smem + S::kOffQK);
   float *am = reinterpret_cast<float *>(smem + S::kOffA), *tm = reinterpret_cast<float *>(smem + S::kOffT);
-  float *inv_k = reinterpret_cast<float *>(smem + S::kOffVec), *inv_q = inv_k + kC, *gsum = inv_q + kC, *beta = gsum + kC;
+  float *inv_k = reinterpret_cast<float *>(smem + S::kOffVec), *inv_q = inv_k + kC, *gates = inv_q + 3 * kC;
   constexpr int kPieces = kDK / 8;
 
+  // decays, summed up (in the log2 domain), and steps of up to kPrepHeads heads: a warp per head, two tokens per lane
+  auto gates_of = [&](int g0) {
+    for (int g = g0 + warp; g < min(g0 + kPrepHeads, group); g += kPrepThreads / 32) {
+      const int h = hk * group + g;
+      float lg[2], b[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = 2 * lane + i;
+        lg[i] = b[i] = 0.f;
+        if (t < valid) {
+          const __nv_bfloat16 *x = p.proj + (row0 + t) * p.ld;
+          lg[i] = log_decay(ldf(x + p.a_at() + h), p.a_log[h], p.dt_bias[h]) * 1.4426950408889634f;
+          b[i] = sigmoid(ldf(x + p.b_at() + h));
+        }
+      }
+      float sum = lg[0] + lg[1];
+#pragma unroll
+      for (int d = 1; d < 32; d <<= 1) {
+        const float o = __shfl_up_sync(0xffffffffu, sum, d);
+        if (lane >= d) sum += o;
+      }
+      float *dst = gates + (g - g0) * 2 * kC;
+      *reinterpret_cast<float2 *>(dst + 2 * lane) = make_float2(sum - lg[1], sum);
+      *reinterpret_cast<float2 *>(dst + kC + 2 * lane) = make_float2(b[0], b[1]);
+    }
+  };
+  gates_of(0);
   // convolutions: even warps the keys, odd warps the queries, 16 tokens each; a warp holds a whole row
   {
     const bool is_q = warp & 1;
@@ -177,15 +225,14 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
     uint8_t *tile = is_q ? cq : ck;
     float *inv = is_q ? inv_q : inv_k;
     const float gain = is_q ? 1.0f / sqrtf((float)p.dim) : 1.f;
-    auto put = [&](int t, const float (&y)[4]) {
+    const bool real = c < p.dim;
+    conv_walk<16>(p, row0, real ? valid : 0, real ? (is_q ? hk : p.kv_heads + hk) * p.dim + c : 0, t0, [&](int t, const float (&y)[4]) {
       const uint2 packed = make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
       const float a = bf_lo(packed.x), b = bf_hi(packed.x), d = bf_lo(packed.y), e = bf_hi(packed.y);
       const float sq = warp_sum(a * a + b * b + d * d + e * e);  // of the rounded row: its unit vector is exact
       if (c < kDK) *reinterpret_cast<uint2 *>(tile + tile_at(t, c >> 3, kPieces) + (c & 4) * 2) = packed;
       if (lane == 0) inv[t] = gain / sqrtf(sq + kUnitEps);
-    };
-    const bool real = c < p.dim;
-    conv_walk(p, row0, real ? valid : 0, real ? (is_q ? hk : p.kv_heads + hk) * p.dim + c : 0, t0, 16, put);
+    });
   }
   __syncthreads();
   {
@@ -223,99 +270,72 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
     const int h = hk * group + g;
     uint8_t *dst = heads + (chunk * p.heads + h) * (size_t)kHeadTiles;
     __syncthreads();  // the products (first head); the last head's T has been stored
-    if (warp == 0) {
-      float lg[2], b[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {  // token 2 * lane + i
-        const int t = 2 * lane + i;
-        lg[i] = b[i] = 0.f;
-        if (t < valid) {
-          const __nv_bfloat16 *x = p.proj + (row0 + t) * p.ld;
-          lg[i] = log_decay(ldf(x + p.a_at() + h), p.a_log[h], p.dt_bias[h]);
-          b[i] = sigmoid(ldf(x + p.b_at() + h));
-        }
-      }
-      float sum = lg[0] + lg[1];
-#pragma unroll
-      for (int d = 1; d < 32; d <<= 1) {
-        const float o = __shfl_up_sync(0xffffffffu, sum, d);
-        if (lane >= d) sum += o;
-      }
-      gsum[2 * lane] = sum - lg[1];
-      gsum[2 * lane + 1] = sum;
-      beta[2 * lane] = b[0];
-      beta[2 * lane + 1] = b[1];
-      const float last = __shfl_sync(0xffffffffu, sum, 31);
+    if (g > 0 && g % kPrepHeads == 0) {
+      gates_of(g);
+      __syncthreads();
+    }
+    const float *gsum = gates + g % kPrepHeads * 2 * kC, *beta = gsum + kC;
+    if (tid < kC) {
       float *vec = reinterpret_cast<float *>(dst + kVec);
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = 2 * lane + i;
-        const float gt = i ? sum : sum - lg[1];
-        vec[t] = expf(gt) * inv_k[t];
-        vec[kC + t] = expf(gt) * inv_q[t];
-        vec[2 * kC + t] = expf(last - gt) * inv_k[t];
-      }
-      if (lane == 0) vec[3 * kC] = expf(last);
+      const float last = gsum[kC - 1], e = fast_exp2(gsum[tid]);
+      vec[tid] = e * inv_k[tid];
+      vec[kC + tid] = e * inv_q[tid];
+      vec[2 * kC + tid] = fast_exp2(last - gsum[tid]) * inv_k[tid];
+      if (tid == 0) vec[3 * kC] = fast_exp2(last);
     }
-    __syncthreads();
-    // A in shared memory, P straight to its tiles; a thread takes two neighbouring columns
-    for (int i = tid; i < kC * kC / 2; i += kPrepThreads) {
-      const int t = i / (kC / 2), s = i % (kC / 2) * 2;
-      float a[2] = {}, pr[2] = {};
-#pragma unroll
-      for (int e = 0; e < 2; ++e)
-        if (s + e <= t) {
-          const float f = expf(gsum[t] - gsum[s + e]) * inv_k[s + e];
-          pr[e] = f * inv_q[t] * qk[t * kLd + s + e];
-          if (s + e < t) a[e] = beta[t] * f * inv_k[t] * kk[t * kLd + s + e];
-        }
-      *reinterpret_cast<float2 *>(am + t * kLd + s) = make_float2(a[0], a[1]);
+    // the lower blocks of A in shared memory, of P straight to their place; a thread takes two neighbouring columns
+    for (int i = tid; i < 10 * 128; i += kPrepThreads) {
+      const int blk = i >> 7, m = blk < 1 ? 0 : blk < 3 ? 1 : blk < 6 ? 2 : 3, k = blk - m * (m + 1) / 2;
+      const int r = (i >> 3) & 15, c = (i & 7) * 2, t = m * 16 + r, s = k * 16 + c;
+      const float2 x = *reinterpret_cast<const float2 *>(kk + t * kLd + s), y = *reinterpret_cast<const float2 *>(qk + t * kLd + s);
+      const float2 gs = *reinterpret_cast<const float2 *>(gsum + s), ik = *reinterpret_cast<const float2 *>(inv_k + s);
+      const float gt = gsum[t], f0 = s <= t ? fast_exp2(gt - gs.x) * ik.x : 0.f, f1 = s < t ? fast_exp2(gt - gs.y) * ik.y : 0.f;
+      const float at = beta[t] * inv_k[t], pt = inv_q[t];
+      *reinterpret_cast<float2 *>(am + t * kLd + s) = make_float2(at * f0 * x.x, at * f1 * x.y);  // the diagonal is not read
       uint32_t high, low;
-      split(pr[0], pr[1], high, low);
-      const uint32_t at = tile_at(t, s >> 3, 8) + (s & 7) * 2;
-      *reinterpret_cast<uint32_t *>(dst + 2 * kSquare + at) = high;
-      *reinterpret_cast<uint32_t *>(dst + 3 * kSquare + at) = low;
+      split(pt * f0 * y.x, pt * f1 * y.y, high, low);
+      const uint32_t off = block_at(m, k, r, c >> 3) + (c & 7) * 2;
+      *reinterpret_cast<uint32_t *>(dst + 2 * kSquare + off) = high;
+      *reinterpret_cast<uint32_t *>(dst + 3 * kSquare + off) = low;
     }
     __syncthreads();
-    // (I + A)^-1: the four diagonal blocks of 16, a thread per column; then pairs of blocks
+    // (I + A)^-1: the four diagonal blocks of 16, a thread per column
     if (tid < kC) {
       const int b0 = tid & ~15, j = tid & 15;
       float x[16];
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
-        float acc = 0.f;
+        float acc[2] = {};
 #pragma unroll
-        for (int m = 0; m < i; ++m) acc = fmaf(am[(b0 + i) * kLd + b0 + m], x[m], acc);
-        x[i] = i == j ? 1.f : i < j ? 0.f : -acc;
+        for (int m = 0; m < i; ++m) acc[m & 1] = fmaf(am[(b0 + i) * kLd + b0 + m], x[m], acc[m & 1]);
+        x[i] = i == j ? 1.f : i < j ? 0.f : -(acc[0] + acc[1]);
         tm[(b0 + i) * kLd + b0 + j] = x[i];
       }
     }
     __syncthreads();
-    // lower left blocks: -T_low . (A . T_up); the inner product uses the (still unused) upper right of T
+    // then the lower left blocks, -T_low . (A . T_up), of 16 and of 32; the inner products lie in the unused upper right
     {
-      const int half = tid >> 7, o = half * 32;
-      square_product(tm + o * kLd + o + 16, am + (o + 16) * kLd + o, tm + o * kLd + o, 16, 16, 16, 1.f, tid & 127, 128);
+      const int o = warp & 2 ? 32 : 0, c = (warp & 1) * 8;
+      float *scratch = tm + o * kLd + o + 16 + c;
+      if (warp < 4) small_product(scratch, am + (o + 16) * kLd + o, tm + o * kLd + o + c, 1, 1.f, lane);
       __syncthreads();
-      square_product(tm + (o + 16) * kLd + o, tm + (o + 16) * kLd + o + 16, tm + o * kLd + o + 16, 16, 16, 16, -1.f, tid & 127, 128);
+      if (warp < 4) small_product(tm + (o + 16) * kLd + o + c, tm + (o + 16) * kLd + o + 16, scratch, 1, -1.f, lane);
       __syncthreads();
-      if ((tid & 127) < 64) {  // clear the scratch: level two reads whole blocks
-        const int r = (tid & 63) / 4, c = tid % 4 * 4;
-        *reinterpret_cast<float4 *>(tm + (o + r) * kLd + o + 16 + c) = make_float4(0.f, 0.f, 0.f, 0.f);
-      }
+      const int m = warp >> 2, n = (warp & 3) * 8, k0 = n >> 4;  // blocks of T_up above its diagonal are zero, and not read
+      small_product(tm + m * 16 * kLd + 32 + n, am + (32 + m * 16) * kLd + k0 * 16, tm + k0 * 16 * kLd + n, 2 - k0, 1.f, lane);
       __syncthreads();
-      square_product(tm + 32, am + 32 * kLd, tm, 32, 32, 32, 1.f, tid, kPrepThreads);
-      __syncthreads();
-      square_product(tm + 32 * kLd, tm + 32 * kLd + 32, tm + 32, 32, 32, 32, -1.f, tid, kPrepThreads);
+      small_product(tm + (32 + m * 16) * kLd + n, tm + (32 + m * 16) * kLd + 32, tm + 32 + n, m + 1, -1.f, lane);
       __syncthreads();
     }
-    for (int i = tid; i < kC * kC / 2; i += kPrepThreads) {
-      const int t = i / (kC / 2), s = i % (kC / 2) * 2;
-      const float a = s <= t ? tm[t * kLd + s] * beta[s] : 0.f, b = s + 1 <= t ? tm[t * kLd + s + 1] * beta[s + 1] : 0.f;
+    for (int i = tid; i < 10 * 128; i += kPrepThreads) {
+      const int blk = i >> 7, m = blk < 1 ? 0 : blk < 3 ? 1 : blk < 6 ? 2 : 3, k = blk - m * (m + 1) / 2;
+      const int r = (i >> 3) & 15, c = (i & 7) * 2, s = k * 16 + c;
+      const float2 v = *reinterpret_cast<const float2 *>(tm + (m * 16 + r) * kLd + s), b = *reinterpret_cast<const float2 *>(beta + s);
       uint32_t high, low;
-      split(a, b, high, low);
-      const uint32_t at = tile_at(t, s >> 3, 8) + (s & 7) * 2;
-      *reinterpret_cast<uint32_t *>(dst + at) = high;
-      *reinterpret_cast<uint32_t *>(dst + kSquare + at) = low;
+      split(v.x * b.x, v.y * b.y, high, low);
+      const uint32_t off = block_at(m, k, r, c >> 3) + (c & 7) * 2;
+      *reinterpret_cast<uint32_t *>(dst + off) = high;
+      *reinterpret_cast<uint32_t *>(dst + kSquare + off) = low;
     }
   }
 }
@@ -325,8 +345,8 @@ template <int kDK, int kWarps>
 struct ScanSmem {
   static constexpr int kTile = kC * kDK * 2;
   static constexpr int kOffHead = 2 * kTile, kOffValues = kOffHead + kHeadTiles, kStage = kOffValues + kWarps * kValueTile;
-  static constexpr int kStages = 3 * kStage + kWarps * kValueTile + 256 <= 227 * 1024 ? 3 : 2;
-  static constexpr int kOffOut = kStages * kStage, kOffBar = kOffOut + kWarps * kValueTile, kBytes = kOffBar + 256;
+  static constexpr int kStages = 4 * kStage + 256 <= 227 * 1024 ? 4 : 3;
+  static constexpr int kOffBar = kStages * kStage, kBytes = kOffBar + 256;
 };
 
 __device__ __forceinline__ void bulk_load(void *dst, const void *src, uint32_t bytes, uint64_t *bar) {
@@ -335,37 +355,42 @@ __device__ __forceinline__ void bulk_load(void *dst, const void *src, uint32_t b
                : "memory");
 }
 
-__device__ __forceinline__ void stmatrix_x4_trans(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
-  asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(r0), "r"(r1), "r"(r2), "r"(r3)
-               : "memory");
+// An 8 x 8 matrix of 16-bit elements, a row's pairs in four lanes, transposed.
+__device__ __forceinline__ uint32_t transposed(uint32_t v) {
+  uint32_t r;
+  asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+  return r;
 }
 
-// Operand A (16 x 16) in two parts from two neighbouring accumulator tiles.
-__device__ __forceinline__ void split_operand(const float (&c0)[4], const float (&c1)[4], uint32_t (&high)[4], uint32_t (&low)[4]) {
-  split(c0[0], c0[1], high[0], low[0]);
-  split(c0[2], c0[3], high[1], low[1]);
-  split(c1[0], c1[1], high[2], low[2]);
-  split(c1[2], c1[3], high[3], low[3]);
+// Operand B (16 x 8) in two parts from an accumulator tile (16 x 8).
+__device__ __forceinline__ void split_operand(const float (&c)[4], uint32_t (&high)[2], uint32_t (&low)[2]) {
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    uint32_t h, l;
+    split(c[2 * i], c[2 * i + 1], h, l);
+    high[i] = transposed(h);
+    low[i] = transposed(l);
+  }
 }
 
-// acc (16 x 64) += x (16 x 64, in two parts) . m^T for a lower triangular m (64 x 64) in two parts.
-__device__ __forceinline__ void triangular_product(float (&acc)[8][4], const uint32_t (&high)[4][4], const uint32_t (&low)[4][4],
-                                                   uint32_t m_high, uint32_t m_low, int lane) {
+// acc (64 x 8) += m (lower triangular, 64 x 64, in two parts) . x (64 x 8, in two parts)
+__device__ __forceinline__ void triangular_product(float (&acc)[4][4], uint32_t m_high, uint32_t m_low, const uint32_t (&high)[4][2],
+                                                   const uint32_t (&low)[4][2], int lane) {
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
+    uint32_t a[4][4], b[4][4];
 #pragma unroll
-    for (int j = 2 * k; j < 8; j += 2) {
-      const uint32_t at = tile_at(8 * (j + (lane >> 4)) + (lane & 7), 2 * k + ((lane >> 3) & 1), 8);
-      uint32_t b[4], c[4];
-      ldmatrix_x4(b[0], b[1], b[2], b[3], m_high + at);
-      ldmatrix_x4(c[0], c[1], c[2], c[3], m_low + at);
-      mma_16816_bf16(acc[j], high[k], b[0], b[1]);
-      mma_16816_bf16(acc[j + 1], high[k], b[2], b[3]);
-      mma_16816_bf16(acc[j], low[k], b[0], b[1]);
-      mma_16816_bf16(acc[j + 1], low[k], b[2], b[3]);
-      mma_16816_bf16(acc[j], high[k], c[0], c[1]);
-      mma_16816_bf16(acc[j + 1], high[k], c[2], c[3]);
+    for (int m = k; m < 4; ++m) {
+      const uint32_t at = block_at(m, k, lane & 15, lane >> 4);
+      ldmatrix_x4(a[m][0], a[m][1], a[m][2], a[m][3], m_high + at);
+      ldmatrix_x4(b[m][0], b[m][1], b[m][2], b[m][3], m_low + at);
     }
+#pragma unroll
+    for (int m = k; m < 4; ++m) mma_16816_bf16(acc[m], a[m], high[k][0], high[k][1]);
+#pragma unroll
+    for (int m = k; m < 4; ++m) mma_16816_bf16(acc[m], a[m], low[k][0], low[k][1]);
+#pragma unroll
+    for (int m = k; m < 4; ++m) mma_16816_bf16(acc[m], b[m], high[k][0], high[k][1]);
   }
 }
 
@@ -382,12 +407,12 @@ struct ScanParams {
 template <int kDK, int kWarps>
 __global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(const ScanParams p) {
   using L = ScanSmem<kDK, kWarps>;
-  constexpr int kPieces = kDK / 8, kKeyTiles = kDK / 8;  // 8-wide tiles of S^T
+  constexpr int kPieces = kDK / 8, kKeyTiles = kDK / 16;  // 16-high tiles of S
   extern __shared__ __align__(128) uint8_t smem[];
   uint64_t *full = reinterpret_cast<uint64_t *>(smem + L::kOffBar), *empty = full + L::kStages;
   volatile int *abort_flag = reinterpret_cast<volatile int *>(empty + L::kStages);
   const int warp = __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0), lane = threadIdx.x & 31;
-  const int h = blockIdx.y, hk = h / (p.heads / p.kv_heads), blocks = (p.vdim + 15) / 16, block0 = blockIdx.z * kWarps;
+  const int h = blockIdx.y, hk = h / (p.heads / p.kv_heads), blocks = p.vdim / 8, block0 = blockIdx.z * kWarps;
   const int warps = min(kWarps, blocks - block0);  // with columns of their own
   if (threadIdx.x == 0) {
     for (int i = 0; i < L::kStages; ++i) {
@@ -434,125 +459,113 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(
   }
   if (warp >= warps) return;
 
-  // S^T: tile j holds keys 8j .. 8j + 7; rows lane / 4 and + 8 are value columns, (lane % 4) * 2 and + 1 the keys
-  const int v0 = (block0 + warp) * 16, va = v0 + (lane >> 2), vb = va + 8, kc = (lane & 3) * 2;
+  // S: tile j holds keys 16j .. 16j + 15 (rows lane / 4 and + 8), 8 value columns ((lane % 4) * 2 and + 1)
+  const int g = lane >> 2, v0 = (block0 + warp) * 8 + (lane & 3) * 2;
   float *state = p.state + ((size_t)portion.x * p.heads + h) * p.dim * p.vdim;
   float st[kKeyTiles][4];
 #pragma unroll
   for (int j = 0; j < kKeyTiles; ++j)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int k = 8 * j + kc + (e & 1), v = e < 2 ? va : vb;
-      st[j][e] = portion.w > 0 && k < p.dim && v < p.vdim ? state[(size_t)k * p.vdim + v] : 0.f;
+    for (int i = 0; i < 2; ++i) {
+      const int k = 16 * j + g + 8 * i;
+      float2 v = make_float2(0.f, 0.f);
+      if (portion.w > 0 && k < p.dim) v = *reinterpret_cast<const float2 *>(state + (size_t)k * p.vdim + v0);
+      st[j][2 * i] = v.x, st[j][2 * i + 1] = v.y;
     }
-  uint8_t *staged = smem + L::kOffOut + warp * kValueTile;
 
   for (int n = 0; n < chunks; ++n) {
     const int s = n % L::kStages;
     if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[s], (n / L::kStages) & 1, abort_flag, p.wait_ns))) return;
     const uint32_t base = smem_u32(smem + s * L::kStage), ck = base, cq = base + L::kTile, tiles = base + L::kOffHead;
     const float *vec = reinterpret_cast<const float *>(smem + s * L::kStage + L::kOffHead + kVec);
+    const uint8_t *value = smem + s * L::kStage + L::kOffValues + warp * kValueTile + (lane & 3) * 4;
 
-    // S^T k and S^T q of all tokens
-    float x[8][4] = {}, o[8][4] = {};
+    // k S and q S of all tokens
+    float x[4][4] = {}, o[4][4] = {};
 #pragma unroll
-    for (int k = 0; k < kDK / 16; ++k) {
-      uint32_t high[4], low[4];
-      split_operand(st[2 * k], st[2 * k + 1], high, low);
+    for (int k = 0; k < kKeyTiles; ++k) {
+      uint32_t high[2], low[2], a[4][4], b[4][4];
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        float(&acc)[8][4] = half ? o : x;
-        const uint32_t tile = half ? cq : ck;
-        uint32_t b[4][4];
+      for (int m = 0; m < 4; ++m) {
+        const uint32_t at = tile_at(16 * m + (lane & 15), 2 * k + (lane >> 4), kPieces);
+        ldmatrix_x4(a[m][0], a[m][1], a[m][2], a[m][3], ck + at);
+        ldmatrix_x4(b[m][0], b[m][1], b[m][2], b[m][3], cq + at);
+      }
+      split_operand(st[k], high, low);
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          ldmatrix_x4(b[j][0], b[j][1], b[j][2], b[j][3],
-                      tile + tile_at(8 * (2 * j + (lane >> 4)) + (lane & 7), 2 * k + ((lane >> 3) & 1), kPieces));
+      for (int m = 0; m < 4; ++m) {
+        mma_16816_bf16(x[m], a[m], high[0], high[1]);
+        mma_16816_bf16(o[m], b[m], high[0], high[1]);
+      }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) mma_16816_bf16(acc[j], high, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) mma_16816_bf16(acc[j], low, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
+      for (int m = 0; m < 4; ++m) {
+        mma_16816_bf16(x[m], a[m], low[0], low[1]);
+        mma_16816_bf16(o[m], b[m], low[0], low[1]);
       }
     }
-    // X^T = v^T - e^G S^T k
+    // X = v - e^G k S
+    uint32_t high[4][2], low[4][2];
 #pragma unroll
-    for (int j = 0; j < 8; j += 2) {
-      uint32_t v[4];
-      ldmatrix_x4_trans(v[0], v[1], v[2], v[3], base + L::kOffValues + warp * kValueTile + (8 * (j + (lane >> 4)) + (lane & 7)) * 32 +
-                                                    ((lane >> 3) & 1) * 16);
+    for (int m = 0; m < 4; ++m) {
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
-        const float2 e = *reinterpret_cast<const float2 *>(vec + 8 * (j + i) + kc);
-        x[j + i][0] = fmaf(-e.x, x[j + i][0], bf_lo(v[2 * i]));
-        x[j + i][1] = fmaf(-e.y, x[j + i][1], bf_hi(v[2 * i]));
-        x[j + i][2] = fmaf(-e.x, x[j + i][2], bf_lo(v[2 * i + 1]));
-        x[j + i][3] = fmaf(-e.y, x[j + i][3], bf_hi(v[2 * i + 1]));
+        const int t = 16 * m + g + 8 * i;
+        const uint32_t v = *reinterpret_cast<const uint32_t *>(value + t * 16);
+        const float e = vec[t];
+        x[m][2 * i] = fmaf(-e, x[m][2 * i], bf_lo(v));
+        x[m][2 * i + 1] = fmaf(-e, x[m][2 * i + 1], bf_hi(v));
       }
+      split_operand(x[m], high[m], low[m]);
     }
-    uint32_t high[4][4], low[4][4];
-#pragma unroll
-    for (int k = 0; k < 4; ++k) split_operand(x[2 * k], x[2 * k + 1], high[k], low[k]);
-    float u[8][4] = {};
-    triangular_product(u, high, low, tiles, tiles + kSquare, lane);
-    // S'^T = e^G_64 S^T + (e^{G_64 - G} u)^T k
+    float u[4][4] = {};
+    triangular_product(u, tiles, tiles + kSquare, high, low, lane);
+    // S' = e^G_64 S + k^T (e^{G_64 - G} u)
     const float total = vec[3 * kC];
 #pragma unroll
     for (int j = 0; j < kKeyTiles; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) st[j][e] *= total;
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      float w[2][4];
+    for (int m = 0; m < 4; ++m) {
+      const float e0 = vec[2 * kC + 16 * m + g], e1 = vec[2 * kC + 16 * m + g + 8];
+      const float w[4] = {e0 * u[m][0], e0 * u[m][1], e1 * u[m][2], e1 * u[m][3]};
+      uint32_t wh[2], wl[2], a[kKeyTiles][4];
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const float2 e = *reinterpret_cast<const float2 *>(vec + 2 * kC + 8 * (2 * k + i) + kc);
-        w[i][0] = e.x * u[2 * k + i][0], w[i][1] = e.y * u[2 * k + i][1];
-        w[i][2] = e.x * u[2 * k + i][2], w[i][3] = e.y * u[2 * k + i][3];
-      }
-      split_operand(w[0], w[1], high[k], low[k]);
+      for (int j = 0; j < kKeyTiles; ++j)
+        ldmatrix_x4_trans(a[j][0], a[j][1], a[j][2], a[j][3],
+                          ck + tile_at(16 * m + ((lane >> 4) & 1) * 8 + (lane & 7), 2 * j + ((lane >> 3) & 1), kPieces));
+      split_operand(w, wh, wl);
 #pragma unroll
-      for (int j = 0; j < kKeyTiles; j += 2) {
-        uint32_t b[4];
-        ldmatrix_x4_trans(b[0], b[1], b[2], b[3], ck + tile_at(16 * k + 8 * ((lane >> 3) & 1) + (lane & 7), j + (lane >> 4), kPieces));
-        mma_16816_bf16(st[j], high[k], b[0], b[1]);
-        mma_16816_bf16(st[j + 1], high[k], b[2], b[3]);
-        mma_16816_bf16(st[j], low[k], b[0], b[1]);
-        mma_16816_bf16(st[j + 1], low[k], b[2], b[3]);
-      }
+      for (int j = 0; j < kKeyTiles; ++j) mma_16816_bf16(st[j], a[j], wh[0], wh[1]);
+#pragma unroll
+      for (int j = 0; j < kKeyTiles; ++j) mma_16816_bf16(st[j], a[j], wl[0], wl[1]);
     }
-    // o^T = e^G S^T q + u^T P^T
+    // o = e^G q S + P u
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const float2 e = *reinterpret_cast<const float2 *>(vec + kC + 8 * j + kc);
-      o[j][0] *= e.x, o[j][1] *= e.y, o[j][2] *= e.x, o[j][3] *= e.y;
+    for (int m = 0; m < 4; ++m) {
+      const float e0 = vec[kC + 16 * m + g], e1 = vec[kC + 16 * m + g + 8];
+      o[m][0] *= e0, o[m][1] *= e0, o[m][2] *= e1, o[m][3] *= e1;
+      split_operand(u[m], high[m], low[m]);
     }
-#pragma unroll
-    for (int k = 0; k < 4; ++k) split_operand(u[2 * k], u[2 * k + 1], high[k], low[k]);
-    triangular_product(o, high, low, tiles + 2 * kSquare, tiles + 3 * kSquare, lane);
+    triangular_product(o, tiles + 2 * kSquare, tiles + 3 * kSquare, high, low, lane);
     __syncwarp();
     if (lane == 0) mbar_arrive(&empty[s]);
-    // through shared memory into rows of 16 columns
+    const int valid = portion.z - n * kC;
+    __nv_bfloat16 *dst = p.out + ((int64_t)(portion.y - p.first + n * kC) * p.heads + h) * p.vdim + v0;
 #pragma unroll
-    for (int j = 0; j < 8; j += 2)
-      stmatrix_x4_trans(smem_u32(staged) + (8 * (j + (lane >> 4)) + (lane & 7)) * 32 + ((lane >> 3) & 1) * 16, pack_bf16x2(o[j][0], o[j][1]),
-                        pack_bf16x2(o[j][2], o[j][3]), pack_bf16x2(o[j + 1][0], o[j + 1][1]), pack_bf16x2(o[j + 1][2], o[j + 1][3]));
-    __syncwarp();
-    const int valid = min(kC, portion.z - n * kC);
+    for (int m = 0; m < 4; ++m)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int t = (i * 32 + lane) >> 1, c = v0 + (lane & 1) * 8;
-      if (t < valid && c < p.vdim)
-        *reinterpret_cast<uint4 *>(p.out + ((int64_t)(portion.y - p.first + n * kC + t) * p.heads + h) * p.vdim + c) =
-            *reinterpret_cast<const uint4 *>(staged + t * 32 + (lane & 1) * 16);
-    }
-    __syncwarp();
+      for (int i = 0; i < 2; ++i) {
+        const int t = 16 * m + g + 8 * i;
+        if (t < valid) *reinterpret_cast<uint32_t *>(dst + (int64_t)t * p.heads * p.vdim) = pack_bf16x2(o[m][2 * i], o[m][2 * i + 1]);
+      }
   }
 #pragma unroll
   for (int j = 0; j < kKeyTiles; ++j)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int k = 8 * j + kc + (e & 1), v = e < 2 ? va : vb;
-      if (k < p.dim && v < p.vdim) state[(size_t)k * p.vdim + v] = st[j][e];
+    for (int i = 0; i < 2; ++i) {
+      const int k = 16 * j + g + 8 * i;
+      if (k < p.dim) *reinterpret_cast<float2 *>(state + (size_t)k * p.vdim + v0) = make_float2(st[j][2 * i], st[j][2 * i + 1]);
     }
 }
 
@@ -575,7 +588,7 @@ template <int kDK, int kWarps>
 int run_scan(const ScanParams &p, int count, cudaStream_t st) {
   using L = ScanSmem<kDK, kWarps>;
   if (int rc = opt_in<delta_chunk_scan_kernel<kDK, kWarps>>(L::kBytes)) return rc;
-  const int blocks = (p.vdim + 15) / 16;
+  const int blocks = p.vdim / 8;
   return launch_dependent(delta_chunk_scan_kernel<kDK, kWarps>, dim3(count, p.heads, (blocks + kWarps - 1) / kWarps),
                           dim3((kWarps + 1) * 32), (size_t)L::kBytes, st, p);
 }
@@ -593,10 +606,11 @@ int run(const DeltaParams<__nv_bfloat16> &d, const ScanParams &s, int count, int
   int dev = 0, sms = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess)
     return AXB200_DEVICE_ERROR;
-  const int64_t warps = (int64_t)count * d.heads * ((d.vdim + 15) / 16);
+  const int64_t warps = (int64_t)count * d.heads * (d.vdim / 8);
   if (warps <= sms) return run_scan<kDK, 1>(s, count, st);
   if (warps <= 2 * sms) return run_scan<kDK, 2>(s, count, st);
-  return run_scan<kDK, 4>(s, count, st);
+  if (warps <= 4 * sms) return run_scan<kDK, 4>(s, count, st);
+  return run_scan<kDK, 8>(s, count, st);
 }
 
 int padded_dim(int dim) { return dim <= 64 ? 64 : 128; }
@@ -615,7 +629,7 @@ size_t axb200_delta_chunks_workspace_bytes(int64_t rows, int count, int heads, i
   if (rows <= 0 || count <= 0) return 0;
   return (size_t)axb::chunk_slots(rows, count) *
          ((size_t)kv_heads * 2 * axb::kC * axb::padded_dim(dim) * 2 +
-          (size_t)heads * (axb::kHeadTiles + (size_t)((vdim + 15) / 16) * axb::kValueTile));
+          (size_t)heads * (axb::kHeadTiles + (size_t)(vdim / 8) * axb::kValueTile));
 }
 
 int axb200_delta_chunks(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos, const int32_t *row_back,
