@@ -3,7 +3,9 @@
 // with q, k and v behind a short causal convolution over time and silu, q and k unit vectors (q also over sqrt(dim)), one
 // decay g and one step beta per head; o is normed over vdim, weighted and gated.
 //
-//   delta_step_kernel     decoded tokens: convolution, norms, recurrence, norm and gate of one token in one launch
+//   delta_step_bulk_kernel  decoded tokens: convolution, norms, recurrence, norm and gate of one token in one launch, the
+//                         state through shared memory by bulk copies; delta_step_kernel: the same through registers, for
+//                         states that are too large or oddly sized
 //   delta_prepare_kernel  portions: convolution, silu and unit norms of every row, decays and steps
 //   delta_scan_kernel     portions, token by token with S in registers
 //   delta_finish_kernel   portions: norm and gate of the outputs; the ring of inputs for the next step's convolution
@@ -31,7 +33,7 @@ __device__ __forceinline__ bool bad_seq(int seq, int max_seqs, bool report) {
 constexpr int kStepThreads = 256, kStepWarps = kStepThreads / 32;
 
 template <typename T, int kVec, int kRowsPerWarp>
-__global__ void __launch_bounds__(kStepThreads, kVec == 4 && kRowsPerWarp == 16 ? 2 : 1)
+__global__ void __launch_bounds__(kStepThreads)
 delta_step_kernel(const DeltaParams<T> p, T *out) {
   extern __shared__ float sm[];
   __shared__ float scratch[32], part[2][kStepWarps][32 * kVec];
@@ -145,6 +147,143 @@ delta_step_kernel(const DeltaParams<T> p, T *out) {
   const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)p.vdim + p.eps);  // also: o is complete
   for (int i = threadIdx.x; i < p.vdim; i += kStepThreads)
     stf(out + (r * p.heads + h) * p.vdim + i, o[i] * inv * ldf(p.norm + i) * silu(ldf(x + p.gate_at() + h * p.vdim + i)));
+}
+
+// The same with the state in shared memory: one bulk copy fetches it while the inputs are prepared, one bulk copy puts it
+// back, and with no registers tied up several CTAs per SM keep enough bytes on their way.  dim and vdim are multiples of 4.
+template <typename T>
+__global__ void __launch_bounds__(kStepThreads, 3) delta_step_bulk_kernel(const DeltaParams<T> p, T *out, unsigned long long wait_ns) {
+  extern __shared__ __align__(128) float sm[];
+  __shared__ float scratch[3][kStepWarps];
+  __shared__ alignas(8) uint64_t bar;
+  __shared__ int abort_flag;
+  float *s = sm, *q = s + p.dim * p.vdim, *k = q + p.dim, *v = k + p.dim, *o = v + p.vdim, *part = o + p.vdim;
+  const int64_t r = blockIdx.x;
+  const int h = blockIdx.y, group = p.heads / p.kv_heads, hk = h / group, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    mbar_init(&bar, 1);
+    abort_flag = 0;
+    mbar_fence_init();
+  }
+  __syncthreads();
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const int seq = p.row_seq[r], pos = p.row_pos[r];
+  if (bad_seq(seq, p.max_seqs, threadIdx.x == 0)) return;
+  const bool fresh = pos == 0;
+  float *state = p.state + ((size_t)seq * p.heads + h) * p.dim * p.vdim;
+  const uint32_t bytes = (uint32_t)(p.dim * p.vdim) * 4;
+  if (threadIdx.x == 0 && !fresh) {
+    mbar_arrive_expect_tx(&bar, bytes);
+    bulk_load(s, state, bytes, &bar);
+  }
+  if (fresh)
+    for (int i = threadIdx.x * 4; i < p.dim * p.vdim; i += kStepThreads * 4) *reinterpret_cast<float4 *>(s + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+
+  const int channels = p.channels(), slot = pos % p.taps;
+  const T *x = p.proj + r * p.ld;
+  T *ring = p.ring + (size_t)seq * p.taps * channels;
+  const bool owns_qk = h % group == 0;
+  const float a_in = ldf(x + p.a_at() + h), b_in = ldf(x + p.b_at() + h), a_log = p.a_log[h], dt_bias = p.dt_bias[h];
+  // two neighbouring channels per thread; query and key elements stay with the threads whose sums they enter
+  float sq[3] = {};  // q.q, k.k, k.q come out of one reduction each, k.q after the exchange
+  for (int i = threadIdx.x * 2; i < 2 * p.dim + p.vdim; i += kStepThreads * 2) {
+    const int c = i < p.dim ? hk * p.dim + i : i < 2 * p.dim ? (p.kv_heads + hk) * p.dim + i - p.dim
+                                                             : 2 * p.kv_heads * p.dim + h * p.vdim + i - 2 * p.dim;
+    float acc[2], in[2], w[2];
+    load_vec<2>(x + c, in);
+    load_vec<2>(p.conv + (size_t)(p.taps - 1) * channels + c, w);
+    acc[0] = in[0] * w[0], acc[1] = in[1] * w[1];
+    for (int j = 1; j < p.taps && j <= pos; ++j) {
+      float old[2];
+      load_vec<2>(ring + (size_t)((pos - j) % p.taps) * channels + c, old);
+      load_vec<2>(p.conv + (size_t)(p.taps - 1 - j) * channels + c, w);
+      acc[0] = fmaf(old[0], w[0], acc[0]), acc[1] = fmaf(old[1], w[1], acc[1]);
+    }
+    if (owns_qk || i >= 2 * p.dim) store_vec<2>(ring + (size_t)slot * channels + c, in);
+    acc[0] = silu(acc[0]), acc[1] = silu(acc[1]);
+    *reinterpret_cast<float2 *>(q + i) = make_float2(acc[0], acc[1]);
+    const float both = fmaf(acc[0], acc[0], acc[1] * acc[1]);
+    if (i < p.dim)
+      sq[0] += both;
+    else if (i < 2 * p.dim)
+      sq[1] += both;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < p.dim; i += kStepThreads) sq[2] = fmaf(q[i], k[i], sq[2]);
+#pragma unroll
+  for (int i = 0; i < 3; ++i) {
+    sq[i] = warp_sum(sq[i]);
+    if (lane == 0) scratch[i][warp] = sq[i];
+  }
+  const float g = expf(log_decay(a_in, a_log, dt_bias)), beta = sigmoid(b_in);
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < 3; ++i) {
+    sq[i] = 0.f;
+#pragma unroll
+    for (int w = 0; w < kStepWarps; ++w) sq[i] += scratch[i][w];
+  }
+  const float inv_q = 1.0f / (sqrtf(sq[0] + kUnitEps) * sqrtf((float)p.dim)), inv_k = 1.0f / sqrtf(sq[1] + kUnitEps);
+  const float kq = sq[2] * inv_q * inv_k;
+  if (!fresh && !mbar_wait_bounded(&bar, 0, &abort_flag, wait_ns)) {  // no copy may still be on its way when the CTA leaves
+    const unsigned long long t0 = global_timer_ns();
+    while (!mbar_try_wait(&bar, 0) && global_timer_ns() - t0 < 100000000ull) {
+    }
+    return;
+  }
+
+  // g S^T k and g S^T q: a warp's rows, a lane's four columns
+  const int rows = (p.dim + kStepWarps - 1) / kStepWarps, row0 = warp * rows, row1 = min(row0 + rows, p.dim);
+  for (int col = lane * 4; col < p.vdim; col += 128) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+#pragma unroll 8
+    for (int i = row0; i < row1; ++i) {
+      const float4 e = *reinterpret_cast<const float4 *>(s + i * p.vdim + col);
+      const float ki = k[i], qi = q[i];
+      a.x = fmaf(e.x, ki, a.x), a.y = fmaf(e.y, ki, a.y), a.z = fmaf(e.z, ki, a.z), a.w = fmaf(e.w, ki, a.w);
+      b.x = fmaf(e.x, qi, b.x), b.y = fmaf(e.y, qi, b.y), b.z = fmaf(e.z, qi, b.z), b.w = fmaf(e.w, qi, b.w);
+    }
+    *reinterpret_cast<float4 *>(part + warp * 2 * p.vdim + col) = a;
+    *reinterpret_cast<float4 *>(part + (warp * 2 + 1) * p.vdim + col) = b;
+  }
+  __syncthreads();
+  float oo = 0.f;
+  for (int c = threadIdx.x; c < p.vdim; c += kStepThreads) {
+    float a = 0.f, b = 0.f;
+#pragma unroll
+    for (int w = 0; w < kStepWarps; ++w) {
+      a += part[w * 2 * p.vdim + c];
+      b += part[(w * 2 + 1) * p.vdim + c];
+    }
+    const float u = beta * (v[c] - g * inv_k * a), y = fmaf(kq, u, g * inv_q * b);
+    v[c] = u * inv_k;  // what the rows of S are updated with, times k
+    o[c] = y;
+    oo = fmaf(y, y, oo);
+  }
+  oo = warp_sum(oo);
+  if (lane == 0) scratch[0][warp] = oo;
+  __syncthreads();
+  for (int col = lane * 4; col < p.vdim; col += 128) {
+    const float4 u = *reinterpret_cast<const float4 *>(v + col);
+#pragma unroll 8
+    for (int i = row0; i < row1; ++i) {
+      float4 e = *reinterpret_cast<const float4 *>(s + i * p.vdim + col);
+      const float ki = k[i];
+      e.x = fmaf(ki, u.x, g * e.x), e.y = fmaf(ki, u.y, g * e.y), e.z = fmaf(ki, u.z, g * e.z), e.w = fmaf(ki, u.w, g * e.w);
+      *reinterpret_cast<float4 *>(s + i * p.vdim + col) = e;
+    }
+  }
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  __syncthreads();
+  if (threadIdx.x == 0) bulk_store(state, s, bytes);
+  oo = 0.f;
+#pragma unroll
+  for (int w = 0; w < kStepWarps; ++w) oo += scratch[0][w];
+  const float inv = 1.0f / sqrtf(oo / (float)p.vdim + p.eps);
+  for (int i = threadIdx.x; i < p.vdim; i += kStepThreads)
+    stf(out + (r * p.heads + h) * p.vdim + i, o[i] * inv * ldf(p.norm + i) * silu(ldf(x + p.gate_at() + h * p.vdim + i)));
+  if (threadIdx.x == 0) bulk_store_wait();
 }
 
 // ---- portions: convolution, unit norms, decays ----------------------------------------------------------
@@ -301,8 +440,66 @@ delta_scan_kernel(const DeltaParams<T> p, const int4 *portions, int first, const
 }
 
 // ---- portions: norm and gate; the ring ----------------------------------------------------------------
-// A warp per (row, head).  o (rows - first, heads, vdim) may be the output itself.
+// o (rows - first, heads, vdim) may be the output itself.
 constexpr int kFinishWarps = 8;
+
+// The last `taps` rows of a portion are what the next step's convolution may look back at: filed by the threads of a CTA.
+template <typename T, int kVec>
+__device__ __forceinline__ void file_inputs(const DeltaParams<T> &p, int64_t r) {
+  const bool last = r + p.taps >= p.rows || p.row_back[r + p.taps] < p.taps;
+  const int seq = p.row_seq[r];
+  if (!last || bad_seq(seq, p.max_seqs, false)) return;
+  const int channels = p.channels();
+  T *slot = p.ring + ((size_t)seq * p.taps + p.row_pos[r] % p.taps) * channels;
+  for (int c = threadIdx.x * kVec; c < channels; c += blockDim.x * kVec) {
+    float in[kVec];
+    load_vec<kVec>(p.proj + r * p.ld + c, in);
+    store_vec<kVec>(slot + c, in);
+  }
+}
+
+// Heads of 8 * kLanes elements: kLanes lanes per head, eight elements each, four heads of a lane on their way at a time.
+template <typename T, int kLanes>
+__global__ void __launch_bounds__(kFinishWarps * 32)
+delta_finish_lanes_kernel(const DeltaParams<T> p, int first, const T *o, T *out) {
+  constexpr int kVdim = 8 * kLanes, kAtOnce = kFinishWarps * 32 / kLanes, kDeep = 4;
+  const int at = threadIdx.x % kLanes * 8;
+  const int64_t r = first + (int64_t)blockIdx.x;
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const T *gates = p.proj + r * p.ld + p.gate_at();
+  const size_t base = (size_t)(r - first) * p.heads * kVdim;
+  float w[8];
+  load_vec<8>(p.norm + at, w);
+  for (int h0 = threadIdx.x / kLanes; h0 - threadIdx.x / kLanes < p.heads; h0 += kAtOnce * kDeep) {
+    float y[kDeep][8], gate[kDeep][8];
+#pragma unroll
+    for (int d = 0; d < kDeep; ++d)
+      if (h0 + d * kAtOnce < p.heads) {
+        load_vec<8>(o + base + (size_t)(h0 + d * kAtOnce) * kVdim + at, y[d]);
+        load_vec<8>(gates + (size_t)(h0 + d * kAtOnce) * kVdim + at, gate[d]);
+      }
+#pragma unroll
+    for (int d = 0; d < kDeep; ++d) {
+      if (h0 - threadIdx.x / kLanes + d * kAtOnce >= p.heads) break;  // the same for the whole CTA
+      const bool mine = h0 + d * kAtOnce < p.heads;
+      float sq = 0.f;
+      if (mine)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sq = fmaf(y[d][e], y[d][e], sq);
+#pragma unroll
+      for (int off = kLanes / 2; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
+      const float inv = 1.0f / sqrtf(sq / (float)kVdim + p.eps);
+      if (!mine) continue;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[d][e] = y[d][e] * inv * w[e] * __fdividef(gate[d][e], 1.0f + __expf(-gate[d][e]));
+      store_vec<8>(out + base + (size_t)(h0 + d * kAtOnce) * kVdim + at, y[d]);
+    }
+  }
+  file_inputs<T, 8>(p, r);
+}
+
+// Any size: a warp per head.
 
 template <typename T, int kVec>
 __global__ void __launch_bounds__(kFinishWarps * 32)
@@ -330,17 +527,7 @@ delta_finish_kernel(const DeltaParams<T> p, int first, const T *o, T *out) {
       store_vec<kVec>(out + ((r - first) * p.heads + h) * p.vdim + i, y);
     }
   }
-  // the last `taps` rows of a portion are what the next step's convolution may look back at
-  const bool last = r + p.taps >= p.rows || p.row_back[r + p.taps] < p.taps;
-  const int seq = p.row_seq[r];
-  if (!last || bad_seq(seq, p.max_seqs, false)) return;
-  const int channels = p.channels();
-  T *slot = p.ring + ((size_t)seq * p.taps + p.row_pos[r] % p.taps) * channels;
-  for (int c = threadIdx.x * kVec; c < channels; c += kFinishWarps * 32 * kVec) {
-    float in[kVec];
-    load_vec<kVec>(x + c, in);
-    store_vec<kVec>(slot + c, in);
-  }
+  file_inputs<T, kVec>(p, r);
 }
 
 bool al16(const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
@@ -360,6 +547,13 @@ int step(const DeltaParams<T> &p, void *out, cudaStream_t st) {
     return launch_dependent(kernel, dim3(p.rows, p.heads), dim3(kStepThreads), smem, st, p, static_cast<T *>(out));
   };
   const bool vec = quads(p);
+  const size_t bulk = ((size_t)p.dim * p.vdim + 2 * p.dim + (2 + 2 * kStepWarps) * p.vdim) * sizeof(float);
+  if (vec && bulk <= 220 * 1024) {
+    auto *kernel = delta_step_bulk_kernel<T>;
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bulk) != cudaSuccess)
+      return (int)AXB200_DEVICE_ERROR;
+    return launch_dependent(kernel, dim3(p.rows, p.heads), dim3(kStepThreads), bulk, st, p, static_cast<T *>(out), wait_limit_ns());
+  }
   if (p.dim <= 8 * 4) return vec ? go(delta_step_kernel<T, 4, 4>) : go(delta_step_kernel<T, 1, 4>);
   if (p.dim <= 8 * 8) return vec ? go(delta_step_kernel<T, 4, 8>) : go(delta_step_kernel<T, 1, 8>);
   if (p.dim <= 8 * 16) return vec ? go(delta_step_kernel<T, 4, 16>) : go(delta_step_kernel<T, 1, 16>);
@@ -397,6 +591,15 @@ int scan(const DeltaParams<T> &p, const int32_t *portions, int count, int first,
 template <typename T>
 int finish(const DeltaParams<T> &p, int first, const void *o, void *out, cudaStream_t st) {
   const bool vec = quads(p) && al16(o) && al16(out);
+  auto lanes = [&](auto *kernel) {
+    return launch_dependent(kernel, dim3(p.rows - first), dim3(kFinishWarps * 32), 0, st, p, first, static_cast<const T *>(o),
+                            static_cast<T *>(out));
+  };
+  if (vec && p.ld % 8 == 0 && p.gate_at() % 8 == 0 && sizeof(T) == 2) {
+    if (p.vdim == 64) return lanes(delta_finish_lanes_kernel<T, 8>);
+    if (p.vdim == 128) return lanes(delta_finish_lanes_kernel<T, 16>);
+    if (p.vdim == 256) return lanes(delta_finish_lanes_kernel<T, 32>);
+  }
   auto *kernel = vec ? delta_finish_kernel<T, 4> : delta_finish_kernel<T, 1>;
   return launch_dependent(kernel, dim3(p.rows - first), dim3(kFinishWarps * 32), 0, st, p, first, static_cast<const T *>(o),
                           static_cast<T *>(out));

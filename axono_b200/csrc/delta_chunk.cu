@@ -349,12 +349,6 @@ struct ScanSmem {
   static constexpr int kOffBar = kStages * kStage, kBytes = kOffBar + 256;
 };
 
-__device__ __forceinline__ void bulk_load(void *dst, const void *src, uint32_t bytes, uint64_t *bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
-               "l"(__cvta_generic_to_global(src)), "r"(bytes), "r"(smem_u32(bar))
-               : "memory");
-}
-
 // An 8 x 8 matrix of 16-bit elements, a row's pairs in four lanes, transposed.
 __device__ __forceinline__ uint32_t transposed(uint32_t v) {
   uint32_t r;

@@ -44,6 +44,7 @@ struct UmmaAttend {
   int pairs, singles;            // per tile
   int pair_slots, single_slots;  // in the rings
   int chunks;                    // per row: ceil(elements / 64)
+  int ahead;                     // the rings hold two tiles: a tile's scores are computed before the sum of the one before
   float *part_o;                 // (2 * CTAs, N, kv_rank)
   float2 *part_ml;               // (2 * CTAs, N): reference (log2 domain), sum
 };
@@ -281,53 +282,58 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
     const uint64_t dv = smem_desc(smem_u32(smem), kChunk, 1024);       // a pair as latent elements x keys
     const uint64_t dq = smem_desc(smem_u32(smem + S::off_q(u)), 16, 1024), dp = smem_desc(smem_u32(smem + S::off_p(u)), 16, 1024);
     RingPos rp, rs, pv;  // pairs and singles of the scores, pairs of the sum
-    int tile = 0, seg = 0;
-    bool ok = true;
-    for (int r = r_first, g = lo; g < hi && ok; ++r) {
-      if (start[r + 1] <= g) continue;
-      const int g_end = min(hi, start[r + 1]);
-      ok = mbar_wait_warp(bar_q, seg & 1, abort_flag, p.wait_ns);  // this item's queries are in place
-      ++seg;
-      for (const int g_first = g; g < g_end && ok; ++g, ++tile) {
-        const uint32_t ts = tmem + (tile & 1) * kN;
-        bool first = true;
-        auto score_chunk = [&](int offset, int c) {
-          const uint64_t a = da + (uint64_t)(offset >> 4), b = dq + (uint64_t)(c * (S::kQBox >> 4));
-#pragma unroll
-          for (int ks = 0; ks < 4; ++ks) umma_f16_lead(ts, a + ks * 2, b + ks * 2, idesc_s, !first || ks > 0, lead);
-          first = false;
-        };
-        for (int i = 0; i < u.singles && ok; ++i, rs.next(u.single_slots)) {
-          const int s = rs.slot;
-          ok = mbar_wait_warp(&full_s[s], rs.parity, abort_flag, p.wait_ns);
-          if (!ok) break;
-          tc_fence_after();
-          score_chunk(off_single + s * kChunk, 2 * u.pairs + i);
-          umma_commit_lead(&empty_s[s], lead);
-        }
-        for (int i = 0; i < u.pairs && ok; ++i, rp.next(u.pair_slots)) {
-          const int s = rp.slot;
-          ok = mbar_wait_warp(&full_p[s], rp.parity, abort_flag, p.wait_ns);
-          if (!ok) break;
-          tc_fence_after();
-          for (int c = 0; c < 2 && 2 * i + c < u.chunks; ++c) score_chunk(s * 2 * kChunk + c * kChunk, 2 * i + c);
-        }
-        if (!ok) break;
-        umma_commit_lead(&bar_s[tile & 1], lead);
-        ok = mbar_wait_warp(bar_p, tile & 1, abort_flag, p.wait_ns);
-        if (!ok) break;
-        tc_fence_after();
-        for (int i = 0; i < u.pairs; ++i, pv.next(u.pair_slots)) {
-          const int s = pv.slot;
-          const uint64_t a = dv + (uint64_t)(s * (2 * kChunk >> 4));
-#pragma unroll
-          for (int ks = 0; ks < kKeys / 16; ++ks)  // 16 keys: 2 KB of the chunk, 32 bytes of P
-            umma_f16_lead(tmem_o + i * kN, a + (uint64_t)(ks * (2048 >> 4)),
-                          dp + (uint64_t)(((ks >> 2) * (kN * 128) + (ks & 3) * 32) >> 4), idesc_o, g > g_first || ks > 0, lead);
-          umma_commit_lead(&empty_p[s], lead);
-        }
-        if (g + 1 == g_end) umma_commit_lead(bar_o, lead);
+    int r_s = r_first, g_s = lo, tile_s = 0, seg = 0;
+    auto scores = [&]() -> bool {  // of tile g_s
+      while (start[r_s + 1] <= g_s) ++r_s;
+      if (g_s == lo || g_s == start[r_s]) {  // a new item: its queries are in place
+        if (!mbar_wait_warp(bar_q, seg & 1, abort_flag, p.wait_ns)) return false;
+        ++seg;
       }
+      const uint32_t ts = tmem + (tile_s & 1) * kN;
+      bool first = true;
+      auto score_chunk = [&](int offset, int c) {
+        const uint64_t a = da + (uint64_t)(offset >> 4), b = dq + (uint64_t)(c * (S::kQBox >> 4));
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) umma_f16_lead(ts, a + ks * 2, b + ks * 2, idesc_s, !first || ks > 0, lead);
+        first = false;
+      };
+      for (int i = 0; i < u.singles; ++i, rs.next(u.single_slots)) {
+        const int s = rs.slot;
+        if (!mbar_wait_warp(&full_s[s], rs.parity, abort_flag, p.wait_ns)) return false;
+        tc_fence_after();
+        score_chunk(off_single + s * kChunk, 2 * u.pairs + i);
+        umma_commit_lead(&empty_s[s], lead);
+      }
+      for (int i = 0; i < u.pairs; ++i, rp.next(u.pair_slots)) {
+        const int s = rp.slot;
+        if (!mbar_wait_warp(&full_p[s], rp.parity, abort_flag, p.wait_ns)) return false;
+        tc_fence_after();
+        for (int c = 0; c < 2 && 2 * i + c < u.chunks; ++c) score_chunk(s * 2 * kChunk + c * kChunk, 2 * i + c);
+      }
+      umma_commit_lead(&bar_s[tile_s & 1], lead);
+      ++g_s;
+      ++tile_s;
+      return true;
+    };
+    bool ok = scores();
+    for (int r = r_first, g = lo, tile = 0; g < hi && ok; ++g, ++tile) {
+      while (start[r + 1] <= g) ++r;
+      if (u.ahead && g_s < hi) ok = scores();
+      ok = ok && mbar_wait_warp(bar_p, tile & 1, abort_flag, p.wait_ns);
+      if (!ok) break;
+      tc_fence_after();
+      const bool fresh = g == lo || g == start[r];
+      for (int i = 0; i < u.pairs; ++i, pv.next(u.pair_slots)) {
+        const int s = pv.slot;
+        const uint64_t a = dv + (uint64_t)(s * (2 * kChunk >> 4));
+#pragma unroll
+        for (int ks = 0; ks < kKeys / 16; ++ks)  // 16 keys: 2 KB of the chunk, 32 bytes of P
+          umma_f16_lead(tmem_o + i * kN, a + (uint64_t)(ks * (2048 >> 4)),
+                        dp + (uint64_t)(((ks >> 2) * (kN * 128) + (ks & 3) * 32) >> 4), idesc_o, !fresh || ks > 0, lead);
+        umma_commit_lead(&empty_p[s], lead);
+      }
+      umma_commit_lead(bar_o, lead);
+      if (!u.ahead && g_s < hi) ok = scores();
     }
   } else {
     // ================= softmax warps: thread = key of the tile =================
@@ -368,8 +374,13 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         const int t0 = key0 + (g - start[r]) * kKeys, valid = min(kKeys, keys - t0);
         const bool seen = tid < valid && (g > start[r] || tid >= hidden);
         const float factor = p.key_scale < 0 ? scale_log2 : seen ? scale_log2 * key_factor(p, r, t0 + tid) : 0.f;
-        ok = mbar_wait_warp(&bar_s[tile & 1], (tile >> 1) & 1, abort_flag, p.wait_ns);
+        ok = mbar_wait_warp(&bar_s[tile & 1], (tile >> 1) & 1, abort_flag, p.wait_ns) && ok;
         tc_fence_after();
+        // the last tile's sum has to be done before O^T is rescaled and before its weights are overwritten
+        auto wait_sum = [&] {
+          if (tile > 0) ok = mbar_wait_warp(bar_o, (tile - 1) & 1, abort_flag, p.wait_ns) && ok;
+          tc_fence_after();
+        };
         float s[kN], rf[kN];
         load_refs<kN>(ref, rf);
         if (ok) {
@@ -411,7 +422,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
           if (g > g_first) {
 #pragma unroll
             for (int h = 0; h < kN; ++h) l[h] *= corr_s[h];
-            // bar_s of this tile was committed after the last tile's sum: O^T may be rescaled
+            wait_sum();
             for (int i = 0; i < u.pairs; ++i) {
               float o[kN];
               tmem_ld_heads<kN>(tmem_o + i * kN + lane_base, o);
@@ -427,10 +438,13 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         const int chunk = (tid >> 3) & 7;
 #pragma unroll
         for (int h = 0; h < kN; ++h) {
-          const float w = fast_exp2(s[h] - rf[h]);
-          l[h] += w;
-          *reinterpret_cast<__nv_bfloat16 *>(pk + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16_rn(w);
+          s[h] = fast_exp2(s[h] - rf[h]);
+          l[h] += s[h];
         }
+        wait_sum();
+#pragma unroll
+        for (int h = 0; h < kN; ++h)
+          *reinterpret_cast<__nv_bfloat16 *>(pk + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16_rn(s[h]);
         if (valid < kKeys) {
           // the sequence's last tile: what stands in the rows past its end is not its own, and weight 0 is not
           // enough against a NaN: clear them where the sum will read them
@@ -456,7 +470,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       // ---- the item, or this range's part of it ----
       const float sum = reduce_heads<kN>(l, lane, [](float a, float b) { return a + b; });
       if (kN == 32 || (lane & 1) == 0) red[warp][lane * kN / 32] = sum;
-      ok = mbar_wait_warp(bar_o, (seg - 1) & 1, abort_flag, p.wait_ns);
+      ok = mbar_wait_warp(bar_o, (tile - 1) & 1, abort_flag, p.wait_ns) && ok;
       tc_fence_after();
       if (any_of_softmax(!ok)) {  // also: red is complete
         ok = false;
@@ -583,6 +597,7 @@ bool layout(UmmaAttend &u) {
     ++u.single_slots;
     if (Smem<kN>::bytes(u, kMaxRows) > kSmemLimit) --u.single_slots;
   }
+  u.ahead = u.pair_slots >= 2 * u.pairs && u.single_slots >= 2 * u.singles;
   return true;
 }
 
