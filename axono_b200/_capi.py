@@ -103,13 +103,13 @@ SIGNATURES = {
                               [_i, _i, _i64] + [_i] * 5 + [_vp]),
     "axb200_latent_attend_workspace_bytes": (_sz, [_i, _i, _i, _i, _i64, _i]),
     # q_lat, q, q_ld, dim | out, pages, block_table, row_seq, row_pos, sink | rows, heads, kv_heads, kv_rank, rot_dim,
-    # row_elems, key_scale, window | scale | page_tokens, max_blocks, num_pages, max_seqs | max_len, dtype, workspace
-    "axb200_latent_attend": (_i, [_vp, _vp, _i64, _i] + [_vp] * 6 + [_i] * 8 + [_f] + [_i] * 4 + [_i64, _i, _vp, _sz, _vp]),
+    # key_scale, window | scale | page_tokens, max_blocks, num_pages, max_seqs | max_len, dtype, workspace
+    "axb200_latent_attend": (_i, [_vp, _vp, _i64, _i] + [_vp] * 6 + [_i] * 7 + [_f] + [_i] * 4 + [_i64, _i, _vp, _sz, _vp]),
     "axb200_latent_gather": (_i, [_vp, _vp, _vp, _i64, _i64, _i, _i, _i, _i, _i, _vp]),
     "axb200_latent_prefill_supported": (_i, [_i] * 5),
     "axb200_latent_prefill": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _i, _i64] + [_i] * 6 + [_f, _i, _vp]),
-    "axb200_shared_kv_prepare": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _f] + [_vp] * 4 + [_i64] + [_i] * 10 + [_vp]),
-    "axb200_shared_kv_gather": (_i, [_vp] * 4 + [_i64] * 2 + [_i] * 8 + [_vp]),
+    "axb200_shared_kv_prepare": (_i, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _f] + [_vp] * 4 + [_i64] + [_i] * 8 + [_vp]),
+    "axb200_shared_kv_gather": (_i, [_vp] * 4 + [_i64] * 2 + [_i] * 6 + [_vp]),
     # proj, ld, row_seq, row_pos[, row_back, first], rows, conv, a_log, dt_bias, norm, ring, state | operands | heads,
     # kv_heads, dim, vdim, taps, max_seqs, eps, dtype, stream
     "axb200_delta_step": (_i, [_vp, _i64, _vp, _vp, _i] + [_vp] * 6 + [_vp] + [_i] * 6 + [_f, _i, _vp]),

@@ -458,45 +458,50 @@ __device__ __forceinline__ void file_inputs(const DeltaParams<T> &p, int64_t r) 
   }
 }
 
-// Heads of 8 * kLanes elements: kLanes lanes per head, eight elements each, four heads of a lane on their way at a time.
+// Heads of 8 * kLanes elements: kLanes lanes per head, eight elements each, kDeep heads of a lane on their way at a time.
 template <typename T, int kLanes>
-__global__ void __launch_bounds__(kFinishWarps * 32)
+__global__ void __launch_bounds__(kFinishWarps * 32, 4)
 delta_finish_lanes_kernel(const DeltaParams<T> p, int first, const T *o, T *out) {
   constexpr int kVdim = 8 * kLanes, kAtOnce = kFinishWarps * 32 / kLanes, kDeep = 4;
   const int at = threadIdx.x % kLanes * 8;
-  const int64_t r = first + (int64_t)blockIdx.x;
+  const int64_t items = (int64_t)(p.rows - first) * p.heads, i0 = (int64_t)blockIdx.x * kAtOnce * kDeep;
   grid_dependency_wait();
   grid_dependency_launch();
-  const T *gates = p.proj + r * p.ld + p.gate_at();
-  const size_t base = (size_t)(r - first) * p.heads * kVdim;
-  float w[8];
-  load_vec<8>(p.norm + at, w);
-  for (int h0 = threadIdx.x / kLanes; h0 - threadIdx.x / kLanes < p.heads; h0 += kAtOnce * kDeep) {
-    float y[kDeep][8], gate[kDeep][8];
+  uint4 y[kDeep], gate[kDeep];
 #pragma unroll
-    for (int d = 0; d < kDeep; ++d)
-      if (h0 + d * kAtOnce < p.heads) {
-        load_vec<8>(o + base + (size_t)(h0 + d * kAtOnce) * kVdim + at, y[d]);
-        load_vec<8>(gates + (size_t)(h0 + d * kAtOnce) * kVdim + at, gate[d]);
-      }
-#pragma unroll
-    for (int d = 0; d < kDeep; ++d) {
-      if (h0 - threadIdx.x / kLanes + d * kAtOnce >= p.heads) break;  // the same for the whole CTA
-      const bool mine = h0 + d * kAtOnce < p.heads;
-      float sq = 0.f;
-      if (mine)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) sq = fmaf(y[d][e], y[d][e], sq);
-#pragma unroll
-      for (int off = kLanes / 2; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
-      const float inv = 1.0f / sqrtf(sq / (float)kVdim + p.eps);
-      if (!mine) continue;
-#pragma unroll
-      for (int e = 0; e < 8; ++e) y[d][e] = y[d][e] * inv * w[e] * __fdividef(gate[d][e], 1.0f + __expf(-gate[d][e]));
-      store_vec<8>(out + base + (size_t)(h0 + d * kAtOnce) * kVdim + at, y[d]);
+  for (int d = 0; d < kDeep; ++d) {
+    const int64_t i = i0 + d * kAtOnce + threadIdx.x / kLanes;
+    y[d] = gate[d] = make_uint4(0, 0, 0, 0);
+    if (i < items) {
+      const int64_t r = i / p.heads;
+      y[d] = *reinterpret_cast<const uint4 *>(o + i * kVdim + at);
+      gate[d] = *reinterpret_cast<const uint4 *>(p.proj + (first + r) * p.ld + p.gate_at() + (i - r * p.heads) * kVdim + at);
     }
   }
-  file_inputs<T, 8>(p, r);
+  float w[8];
+  load_vec<8>(p.norm + at, w);
+#pragma unroll
+  for (int d = 0; d < kDeep; ++d) {
+    const int64_t i = i0 + d * kAtOnce + threadIdx.x / kLanes;
+    const T *ye = reinterpret_cast<const T *>(&y[d]), *ge = reinterpret_cast<const T *>(&gate[d]);
+    float v[8], sq = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      v[e] = ldf(ye + e);
+      sq = fmaf(v[e], v[e], sq);
+    }
+#pragma unroll
+    for (int off = kLanes / 2; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
+    const float inv = 1.0f / sqrtf(sq / (float)kVdim + p.eps);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float z = ldf(ge + e);
+      v[e] = v[e] * inv * w[e] * __fdividef(z, 1.0f + __expf(-z));
+    }
+    if (i < items) store_vec<8>(out + i * kVdim + at, v);
+  }
+  // the rows whose first head is among this CTA's
+  for (int64_t r = (i0 + p.heads - 1) / p.heads; r * p.heads < i0 + kAtOnce * kDeep && first + r < p.rows; ++r) file_inputs<T, 8>(p, first + r);
 }
 
 // Any size: a warp per head.
@@ -592,13 +597,16 @@ template <typename T>
 int finish(const DeltaParams<T> &p, int first, const void *o, void *out, cudaStream_t st) {
   const bool vec = quads(p) && al16(o) && al16(out);
   auto lanes = [&](auto *kernel) {
-    return launch_dependent(kernel, dim3(p.rows - first), dim3(kFinishWarps * 32), 0, st, p, first, static_cast<const T *>(o),
+    const int64_t per = kFinishWarps * 32 / (p.vdim / 8) * 4, items = (int64_t)(p.rows - first) * p.heads;
+    return launch_dependent(kernel, dim3((unsigned)((items + per - 1) / per)), dim3(kFinishWarps * 32), 0, st, p, first, static_cast<const T *>(o),
                             static_cast<T *>(out));
   };
-  if (vec && p.ld % 8 == 0 && p.gate_at() % 8 == 0 && sizeof(T) == 2) {
-    if (p.vdim == 64) return lanes(delta_finish_lanes_kernel<T, 8>);
-    if (p.vdim == 128) return lanes(delta_finish_lanes_kernel<T, 16>);
-    if (p.vdim == 256) return lanes(delta_finish_lanes_kernel<T, 32>);
+  if constexpr (sizeof(T) == 2) {
+    if (vec && p.ld % 8 == 0 && p.channels() % 8 == 0) {
+      if (p.vdim == 64) return lanes(delta_finish_lanes_kernel<T, 8>);
+      if (p.vdim == 128) return lanes(delta_finish_lanes_kernel<T, 16>);
+      if (p.vdim == 256) return lanes(delta_finish_lanes_kernel<T, 32>);
+    }
   }
   auto *kernel = vec ? delta_finish_kernel<T, 4> : delta_finish_kernel<T, 1>;
   return launch_dependent(kernel, dim3(p.rows - first), dim3(kFinishWarps * 32), 0, st, p, first, static_cast<const T *>(o),

@@ -143,8 +143,8 @@ __device__ __forceinline__ void small_product(float *out, const float *a, const 
 template <int kDK>
 struct PrepSmem {
   static constexpr int kTile = kC * kDK * 2, kMatrix = kC * kLd * 4;
-  static constexpr int kOffKK = 2 * kTile, kOffQK = kOffKK + kMatrix, kOffA = kOffQK + kMatrix, kOffT = kOffA + kMatrix;
-  static constexpr int kOffVec = kOffT + kMatrix;
+  static constexpr int kOffKK = 2 * kTile, kOffQK = kOffKK + kMatrix, kOffA = kOffQK + kMatrix;  // A: one per half
+  static constexpr int kOffVec = kOffA + 2 * kMatrix;
   static constexpr int kBytes = kOffVec + 4 * kC * 4 + 2 * kPrepHeads * kC * 4;
 };
 
@@ -187,7 +187,6 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
   const int hk = blockIdx.z, group = p.heads / p.kv_heads;
   uint8_t *ck = smem, *cq = smem + S::kTile;
   float *kk = reinterpret_cast<float *>(smem + S::kOffKK), *qk = reinterpret_cast<float *>(smem + S::kOffQK);
-  float *am = reinterpret_cast<float *>(smem + S::kOffA), *tm = reinterpret_cast<float *>(smem + S::kOffT);
   float *inv_k = reinterpret_cast<float *>(smem + S::kOffVec), *inv_q = inv_k + kC, *gates = inv_q + 3 * kC;
   constexpr int kPieces = kDK / 8;
 
@@ -226,13 +225,25 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
     float *inv = is_q ? inv_q : inv_k;
     const float gain = is_q ? 1.0f / sqrtf((float)p.dim) : 1.f;
     const bool real = c < p.dim;
+    float sq[16];  // of the rounded rows: their unit vectors are exact
     conv_walk<16>(p, row0, real ? valid : 0, real ? (is_q ? hk : p.kv_heads + hk) * p.dim + c : 0, t0, [&](int t, const float (&y)[4]) {
       const uint2 packed = make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
       const float a = bf_lo(packed.x), b = bf_hi(packed.x), d = bf_lo(packed.y), e = bf_hi(packed.y);
-      const float sq = warp_sum(a * a + b * b + d * d + e * e);  // of the rounded row: its unit vector is exact
+      sq[t & 15] = a * a + b * b + d * d + e * e;
       if (c < kDK) *reinterpret_cast<uint2 *>(tile + tile_at(t, c >> 3, kPieces) + (c & 4) * 2) = packed;
-      if (lane == 0) inv[t] = gain / sqrtf(sq + kUnitEps);
     });
+    // all sixteen sums over the warp by halving exchanges: lanes 2 i and 2 i + 1 end with row i's
+#pragma unroll
+    for (int n = 8, off = 16; n > 0; n >>= 1, off >>= 1) {
+      const bool upper = lane & off;
+#pragma unroll
+      for (int i = 0; i < n; ++i) {
+        const float send = upper ? sq[i] : sq[i + n], keep = upper ? sq[i + n] : sq[i];
+        sq[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+      }
+    }
+    sq[0] += __shfl_xor_sync(0xffffffffu, sq[0], 1);
+    if ((lane & 1) == 0) inv[t0 + (lane >> 1)] = gain / sqrtf(sq[0] + kUnitEps);
   }
   __syncthreads();
   {
@@ -266,27 +277,35 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
     }
   }
 
-  for (int g = 0; g < group; ++g) {
-    const int h = hk * group + g;
-    uint8_t *dst = heads + (chunk * p.heads + h) * (size_t)kHeadTiles;
-    __syncthreads();  // the products (first head); the last head's T has been stored
-    if (g > 0 && g % kPrepHeads == 0) {
-      gates_of(g);
+  // T and P: each half of the block (four warps) takes every second head
+  __syncthreads();
+  const int half = warp >> 2, ht = tid & 127, hw = warp & 3;
+  auto half_sync = [&] { named_bar_sync(1 + half, 128); };
+  float *am = reinterpret_cast<float *>(smem + S::kOffA) + half * kC * kLd;  // A, and in its place (I + A)^-1
+  for (int g0 = 0; g0 < group; g0 += 2) {
+    const int g = g0 + half, h = hk * group + g;
+    if (g0 > 0 && g0 % kPrepHeads == 0) {
+      __syncthreads();
+      gates_of(g0);
       __syncthreads();
     }
+    if (g >= group) continue;  // the other half has the last head
+    uint8_t *dst = heads + (chunk * p.heads + h) * (size_t)kHeadTiles;
     const float *gsum = gates + g % kPrepHeads * 2 * kC, *beta = gsum + kC;
-    if (tid < kC) {
+    if (ht < kC) {
       float *vec = reinterpret_cast<float *>(dst + kVec);
-      const float last = gsum[kC - 1], e = fast_exp2(gsum[tid]);
-      vec[tid] = e * inv_k[tid];
-      vec[kC + tid] = e * inv_q[tid];
-      vec[2 * kC + tid] = fast_exp2(last - gsum[tid]) * inv_k[tid];
-      if (tid == 0) vec[3 * kC] = fast_exp2(last);
+      const float last = gsum[kC - 1], e = fast_exp2(gsum[ht]);
+      vec[ht] = e * inv_k[ht];
+      vec[kC + ht] = e * inv_q[ht];
+      vec[2 * kC + ht] = fast_exp2(last - gsum[ht]) * inv_k[ht];
+      if (ht == 0) vec[3 * kC] = fast_exp2(last);
     }
+    half_sync();  // the last head's T has been stored
     // the lower blocks of A in shared memory, of P straight to their place; a thread takes two neighbouring columns
-    for (int i = tid; i < 10 * 128; i += kPrepThreads) {
-      const int blk = i >> 7, m = blk < 1 ? 0 : blk < 3 ? 1 : blk < 6 ? 2 : 3, k = blk - m * (m + 1) / 2;
-      const int r = (i >> 3) & 15, c = (i & 7) * 2, t = m * 16 + r, s = k * 16 + c;
+#pragma unroll
+    for (int blk = 0; blk < 10; ++blk) {
+      const int m = blk < 1 ? 0 : blk < 3 ? 1 : blk < 6 ? 2 : 3, k = blk - m * (m + 1) / 2;
+      const int r = ht >> 3, c = (ht & 7) * 2, t = m * 16 + r, s = k * 16 + c;
       const float2 x = *reinterpret_cast<const float2 *>(kk + t * kLd + s), y = *reinterpret_cast<const float2 *>(qk + t * kLd + s);
       const float2 gs = *reinterpret_cast<const float2 *>(gsum + s), ik = *reinterpret_cast<const float2 *>(inv_k + s);
       const float gt = gsum[t], f0 = s <= t ? fast_exp2(gt - gs.x) * ik.x : 0.f, f1 = s < t ? fast_exp2(gt - gs.y) * ik.y : 0.f;
@@ -298,39 +317,47 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
       *reinterpret_cast<uint32_t *>(dst + 2 * kSquare + off) = high;
       *reinterpret_cast<uint32_t *>(dst + 3 * kSquare + off) = low;
     }
-    __syncthreads();
-    // (I + A)^-1: the four diagonal blocks of 16, a thread per column
-    if (tid < kC) {
-      const int b0 = tid & ~15, j = tid & 15;
-      float x[16];
+    half_sync();
+    // the four diagonal blocks of 16 by forward substitution, a thread per column
+    float inv[16];
+    const int b0 = ht & 48, bj = ht & 15;
+    if (ht < kC) {
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         float acc[2] = {};
 #pragma unroll
-        for (int m = 0; m < i; ++m) acc[m & 1] = fmaf(am[(b0 + i) * kLd + b0 + m], x[m], acc[m & 1]);
-        x[i] = i == j ? 1.f : i < j ? 0.f : -(acc[0] + acc[1]);
-        tm[(b0 + i) * kLd + b0 + j] = x[i];
+        for (int m = 0; m < i; ++m) acc[m & 1] = fmaf(am[(b0 + i) * kLd + b0 + m], inv[m], acc[m & 1]);
+        inv[i] = i == bj ? 1.f : i < bj ? 0.f : -(acc[0] + acc[1]);
       }
     }
-    __syncthreads();
+    half_sync();
+    if (ht < kC) {
+#pragma unroll
+      for (int i = 0; i < 16; ++i) am[(b0 + i) * kLd + b0 + bj] = inv[i];
+    }
+    half_sync();
     // then the lower left blocks, -T_low . (A . T_up), of 16 and of 32; the inner products lie in the unused upper right
     {
-      const int o = warp & 2 ? 32 : 0, c = (warp & 1) * 8;
-      float *scratch = tm + o * kLd + o + 16 + c;
-      if (warp < 4) small_product(scratch, am + (o + 16) * kLd + o, tm + o * kLd + o + c, 1, 1.f, lane);
-      __syncthreads();
-      if (warp < 4) small_product(tm + (o + 16) * kLd + o + c, tm + (o + 16) * kLd + o + 16, scratch, 1, -1.f, lane);
-      __syncthreads();
-      const int m = warp >> 2, n = (warp & 3) * 8, k0 = n >> 4;  // blocks of T_up above its diagonal are zero, and not read
-      small_product(tm + m * 16 * kLd + 32 + n, am + (32 + m * 16) * kLd + k0 * 16, tm + k0 * 16 * kLd + n, 2 - k0, 1.f, lane);
-      __syncthreads();
-      small_product(tm + (32 + m * 16) * kLd + n, tm + (32 + m * 16) * kLd + 32, tm + 32 + n, m + 1, -1.f, lane);
-      __syncthreads();
+      const int o = hw & 2 ? 32 : 0, c = (hw & 1) * 8;
+      float *scratch = am + o * kLd + o + 16 + c;
+      small_product(scratch, am + (o + 16) * kLd + o, am + o * kLd + o + c, 1, 1.f, lane);
+      half_sync();
+      small_product(am + (o + 16) * kLd + o + c, am + (o + 16) * kLd + o + 16, scratch, 1, -1.f, lane);
+      half_sync();
+      const int n = hw * 8, k0 = n >> 4;  // blocks of T_up above its diagonal are zero, and not read
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
+        small_product(am + m * 16 * kLd + 32 + n, am + (32 + m * 16) * kLd + k0 * 16, am + k0 * 16 * kLd + n, 2 - k0, 1.f, lane);
+      half_sync();
+#pragma unroll
+      for (int m = 0; m < 2; ++m) small_product(am + (32 + m * 16) * kLd + n, am + (32 + m * 16) * kLd + 32, am + 32 + n, m + 1, -1.f, lane);
+      half_sync();
     }
-    for (int i = tid; i < 10 * 128; i += kPrepThreads) {
-      const int blk = i >> 7, m = blk < 1 ? 0 : blk < 3 ? 1 : blk < 6 ? 2 : 3, k = blk - m * (m + 1) / 2;
-      const int r = (i >> 3) & 15, c = (i & 7) * 2, s = k * 16 + c;
-      const float2 v = *reinterpret_cast<const float2 *>(tm + (m * 16 + r) * kLd + s), b = *reinterpret_cast<const float2 *>(beta + s);
+#pragma unroll
+    for (int blk = 0; blk < 10; ++blk) {
+      const int m = blk < 1 ? 0 : blk < 3 ? 1 : blk < 6 ? 2 : 3, k = blk - m * (m + 1) / 2;
+      const int r = ht >> 3, c = (ht & 7) * 2, s = k * 16 + c;
+      const float2 v = *reinterpret_cast<const float2 *>(am + (m * 16 + r) * kLd + s), b = *reinterpret_cast<const float2 *>(beta + s);
       uint32_t high, low;
       split(v.x * b.x, v.y * b.y, high, low);
       const uint32_t off = block_at(m, k, r, c >> 3) + (c & 7) * 2;

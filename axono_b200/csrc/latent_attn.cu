@@ -12,7 +12,7 @@
 // mixtures of both.  A per-head sink may join the denominator.
 //
 // The same kernels attend plain cached keys that are also the values: kv_heads parts per row, each read by its group of
-// query heads, and a factor per row that turns its keys - not its values - into normed ones (shared_kv.cu).
+// query heads, and a factor per row, behind the rows of its page, that turns its keys - not its values - into normed ones (shared_kv.cu).
 #include <math.h>
 
 #include "latent_attn.cuh"
@@ -290,9 +290,9 @@ __global__ void __launch_bounds__(kGenThreads) latent_attend_generic_kernel(cons
         atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
         page = 0;
       }
-      const T *row = pages + ((size_t)page * p.page_tokens + t % p.page_tokens) * p.row_elems;
-      key[threadIdx.x] = row + part;
-      factor[threadIdx.x] = p.key_scale >= 0 ? p.scale * *reinterpret_cast<const float *>(row + p.key_scale) : p.scale;
+      const T *base = pages + (size_t)page * p.page_elems;
+      key[threadIdx.x] = base + (size_t)(t % p.page_tokens) * p.row_elems + part;
+      factor[threadIdx.x] = p.key_scale ? p.scale * page_factors(base, p)[t % p.page_tokens] : p.scale;
     }
     __syncthreads();
     for (int j = warp; j < n; j += kGenThreads / 32) {
@@ -390,20 +390,12 @@ size_t axb200_latent_attend_workspace_bytes(int rows, int heads, int kv_rank, in
 
 int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim, void *out, const void *pages,
                          const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, const float *sink,
-                         int rows, int heads, int kv_heads, int kv_rank, int rot_dim, int row_elems, int key_scale, int window,
+                         int rows, int heads, int kv_heads, int kv_rank, int rot_dim, int key_scale, int window,
                          float scale, int page_tokens, int max_blocks, int num_pages, int max_seqs, int64_t max_len, int dtype,
                          void *workspace, size_t workspace_bytes, void *stream) {
   if (dtype != AXB200_FLOAT32 && dtype != AXB200_BFLOAT16) return AXB200_UNSUPPORTED_TYPE;
   if (!q_lat || (!q && rot_dim > 0) || !out || !pages || !block_table || !row_seq || !row_pos) return AXB200_INVALID_PTR;
-  if (kv_heads <= 0 || heads % kv_heads != 0 || (kv_heads > 1 && rot_dim > 0) || window < 0 ||
-      row_elems < kv_heads * kv_rank + rot_dim)
-    return AXB200_INVALID_ARGUMENT;
-  // the factor is an aligned float inside the row, behind its parts
-  if (key_scale >= 0) {
-    const int es = (int)axb::dtype_size(dtype), per = 4 / es;
-    if (key_scale < kv_heads * kv_rank + rot_dim || key_scale + per > row_elems || key_scale % per || row_elems % per)
-      return AXB200_INVALID_ARGUMENT;
-  }
+  if (kv_heads <= 0 || heads % kv_heads != 0 || (kv_heads > 1 && rot_dim > 0) || window < 0) return AXB200_INVALID_ARGUMENT;
   if (rows < 0 || heads <= 0 || heads > 65535 || kv_rank <= 0 || rot_dim < 0 || dim < 0 || page_tokens <= 0 || max_blocks <= 0 ||
       num_pages <= 0 || max_seqs <= 0 || max_len <= 0 || max_len > 0x7fffffff - 4096)
     return AXB200_INVALID_ARGUMENT;
@@ -412,8 +404,9 @@ int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   axb::AttendParams p{};
   p.kv_heads = kv_heads;
-  p.row_elems = row_elems;
-  p.key_scale = key_scale < 0 ? -1 : key_scale;
+  p.row_elems = kv_heads * kv_rank + rot_dim;
+  p.page_elems = page_tokens * p.row_elems + (key_scale ? page_tokens * (4 / (int)axb::dtype_size(dtype)) : 0);
+  p.key_scale = key_scale;
   p.window = window;
   p.sink = sink;
   p.q_lat = q_lat;

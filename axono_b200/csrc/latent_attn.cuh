@@ -17,8 +17,9 @@ struct AttendParams {
   float scale;
   unsigned long long wait_ns;
   int kv_heads;       // a cached row holds kv_heads parts of kv_rank elements, each for heads / kv_heads query heads
-  int row_elems;      // elements from one cached row to the next
-  int key_scale;      // element of the row at which the fp32 factor of its keys stands, or -1: none
+  int row_elems;      // elements from one cached row of a page to the next
+  int page_elems;     // elements from one page to the next
+  int key_scale;      // whether a page ends, behind its rows, with an fp32 factor of the keys of each row
   int window;         // keys a row sees, itself included; 0: all
   const float *sink;  // (heads): logit that takes part in the softmax's denominator only, or null
 };
@@ -34,6 +35,12 @@ __device__ __forceinline__ int visible_keys(const AttendParams &p, int r) {
 // The first key row r sees.
 __device__ __forceinline__ int first_key(const AttendParams &p, int r) {
   return p.window > 0 ? max(0, p.row_pos[r] + 1 - p.window) : 0;
+}
+
+// The factors of a page's rows (see shared_kv.cu).
+template <typename T>
+__device__ __forceinline__ const float *page_factors(const T *page, const AttendParams &p) {
+  return reinterpret_cast<const float *>(page + (size_t)p.page_tokens * p.row_elems);
 }
 
 // tcgen05 form for bf16 (latent_umma.cu)

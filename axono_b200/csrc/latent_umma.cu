@@ -87,8 +87,7 @@ __device__ __forceinline__ void scan_tiles(const AttendParams &p, int *start) {
 __device__ __forceinline__ float key_factor(const AttendParams &p, int r, int t) {
   const int page = p.block_table[(size_t)p.row_seq[r] * p.max_blocks + t / p.page_tokens];
   if (page < 0 || page >= p.num_pages) return 0.f;
-  const __nv_bfloat16 *row = static_cast<const __nv_bfloat16 *>(p.pages) + ((size_t)page * p.page_tokens + t % p.page_tokens) * p.row_elems;
-  return *reinterpret_cast<const float *>(row + p.key_scale);
+  return page_factors(static_cast<const __nv_bfloat16 *>(p.pages) + (size_t)page * p.page_elems, p)[t % p.page_tokens];
 }
 
 // What un-normalised results with sum l at reference ref (log2 domain) are multiplied by when a sink joins the sum.
@@ -109,7 +108,7 @@ __device__ __forceinline__ bool any_of_softmax(bool mine) {
 }
 
 // Reduces v[h], h < kN, over the 32 lanes by halving exchanges; a lane ends with the result of head
-// lane * kN / 32 (kN == 16: two lanes per head).
+// lane * kN / 32 (below 32 heads several lanes have the same one).
 template <int kN, typename Op>
 __device__ __forceinline__ float reduce_heads(float (&v)[kN], int lane, Op op) {
   int n = kN;
@@ -133,9 +132,31 @@ __device__ __forceinline__ float reduce_heads(float (&v)[kN], int lane, Op op) {
 
 template <int kN>
 __device__ __forceinline__ void tmem_ld_heads(uint32_t taddr, float (&v)[kN]) {
+  if constexpr (kN == 4) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x4.b32 {%0,%1,%2,%3}, [%4];" : "=f"(v[0]), "=f"(v[1]), "=f"(v[2]), "=f"(v[3]) : "r"(taddr));
+  } else if constexpr (kN == 8) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
+                 : "=f"(v[0]), "=f"(v[1]), "=f"(v[2]), "=f"(v[3]), "=f"(v[4]), "=f"(v[5]), "=f"(v[6]), "=f"(v[7])
+                 : "r"(taddr));
+  } else {
 #pragma unroll
-  for (int c = 0; c < kN; c += 16) tmem_ld16_async(taddr + c, reinterpret_cast<uint32_t(&)[16]>(v[c]));
+    for (int c = 0; c < kN; c += 16) tmem_ld16_async(taddr + c, reinterpret_cast<uint32_t(&)[16]>(v[c]));
+  }
   tmem_wait_ld();
+}
+
+template <int kN>
+__device__ __forceinline__ void tmem_st_heads(uint32_t taddr, float (&v)[kN]) {
+  if constexpr (kN == 4) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x4.b32 [%0], {%1,%2,%3,%4};" ::"r"(taddr), "f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]) : "memory");
+  } else if constexpr (kN == 8) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"r"(taddr), "f"(v[0]), "f"(v[1]), "f"(v[2]),
+                 "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7])
+                 : "memory");
+  } else {
+#pragma unroll
+    for (int c = 0; c < kN; c += 16) tmem_st16(taddr + c, reinterpret_cast<uint32_t(&)[16]>(v[c]));
+  }
 }
 
 // The heads' references out of shared memory; before an item's first tile they may be anything.
@@ -162,7 +183,9 @@ struct Smem {
   __host__ __device__ static int bytes(const UmmaAttend &u, int rows) { return off_start(u) + (rows + 1) * 4; }
 };
 
-template <int kN>
+// kN: heads of a tile, the products' N side; kH <= kN: how many of them a part can have (the softmax skips the rest, whose
+// columns hold nothing that is read).
+template <int kN, int kH>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_constant__ UmmaAttend u) {
   using S = Smem<kN>;
@@ -232,7 +255,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
           const int t0 = key0 + (g - start[r]) * kKeys;
           // two halves of 64 keys, each within one page; a half past the end is not loaded
           const int halves = keys - t0 > 64 ? 2 : 1;
-          int at[2];
+          int at[2], page_at[2];
 #pragma unroll
           for (int i = 0; i < 2; ++i) {
             const int t = t0 + 64 * (i < halves ? i : 0);
@@ -241,10 +264,11 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
               atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
               page = 0;
             }
-            at[i] = page * p.page_tokens + t % p.page_tokens;
+            at[i] = t % p.page_tokens;
+            page_at[i] = page;
           }
           auto load_chunk = [&](uint8_t *dst, uint64_t *bar, int c) {
-            for (int i = 0; i < halves; ++i) tma_load_3d(dst + i * (kChunk / 2), &tmPages, bar, c * 64, part, at[i]);
+            for (int i = 0; i < halves; ++i) tma_load_4d(dst + i * (kChunk / 2), &tmPages, bar, c * 64, part, at[i], page_at[i]);
           };
           for (int i = 0; i < u.singles && ok; ++i, ++ns, rs.next(u.single_slots)) {
             const int s = rs.slot;
@@ -361,19 +385,27 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_q);
     };
+    // the factor of this thread's key in tile g (of row r or a later one), fetched a tile ahead
+    auto factor_of = [&](int r, int g) {
+      while (start[r + 1] <= g) ++r;
+      const int t = first_tile_key(p, r) + (g - start[r]) * kKeys + tid;
+      return t < visible_keys(p, r) ? key_factor(p, r, t) : 0.f;
+    };
+    float next_factor = p.key_scale ? factor_of(r_first, lo) : 1.f;
     for (int r = r_first, g = lo; g < hi && ok; ++r) {
       if (start[r + 1] <= g) continue;
       const int k_first = g - start[r], g_end = min(hi, start[r + 1]), keys = visible_keys(p, r);
       const int key0 = first_tile_key(p, r), hidden = first_key(p, r) - key0;  // keys of the first tile before the window
       if (seg == 0) put_queries(r);
       ++seg;
-      float l[kN];
+      float l[kH];
 #pragma unroll
-      for (int h = 0; h < kN; ++h) l[h] = 0.f;
+      for (int h = 0; h < kH; ++h) l[h] = 0.f;
       for (const int g_first = g; g < g_end; ++g, ++tile, np += u.pairs) {
-        const int t0 = key0 + (g - start[r]) * kKeys, valid = min(kKeys, keys - t0);
+        const int valid = min(kKeys, keys - key0 - (g - start[r]) * kKeys);
         const bool seen = tid < valid && (g > start[r] || tid >= hidden);
-        const float factor = p.key_scale < 0 ? scale_log2 : seen ? scale_log2 * key_factor(p, r, t0 + tid) : 0.f;
+        const float factor = scale_log2 * next_factor;
+        if (p.key_scale && g + 1 < hi) next_factor = factor_of(r, g + 1);
         ok = mbar_wait_warp(&bar_s[tile & 1], (tile >> 1) & 1, abort_flag, p.wait_ns) && ok;
         tc_fence_after();
         // the last tile's sum has to be done before O^T is rescaled and before its weights are overwritten
@@ -381,17 +413,17 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
           if (tile > 0) ok = mbar_wait_warp(bar_o, (tile - 1) & 1, abort_flag, p.wait_ns) && ok;
           tc_fence_after();
         };
-        float s[kN], rf[kN];
-        load_refs<kN>(ref, rf);
+        float s[kH], rf[kH];
+        load_refs<kH>(ref, rf);
         if (ok) {
-          tmem_ld_heads<kN>(tmem + (tile & 1) * kN + lane_base, s);
+          tmem_ld_heads<kH>(tmem + (tile & 1) * kN + lane_base, s);
         } else {
 #pragma unroll
-          for (int h = 0; h < kN; ++h) s[h] = 0.f;
+          for (int h = 0; h < kH; ++h) s[h] = 0.f;
         }
         float most = -INFINITY;  // how far a score exceeds its head's reference
 #pragma unroll
-        for (int h = 0; h < kN; ++h) {
+        for (int h = 0; h < kH; ++h) {
           s[h] = seen ? s[h] * factor : -INFINITY;
           most = fmaxf(most, s[h] - rf[h]);
         }
@@ -403,13 +435,13 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
             break;
           }
           // the references move: the maximum over the tile, head by head
-          float t[kN];
+          float t[kH];
 #pragma unroll
-          for (int h = 0; h < kN; ++h) t[h] = s[h];
-          const float best = reduce_heads<kN>(t, lane, [](float a, float b) { return fmaxf(a, b); });
-          if (kN == 32 || (lane & 1) == 0) red[warp][lane * kN / 32] = best;
+          for (int h = 0; h < kH; ++h) t[h] = s[h];
+          const float best = reduce_heads<kH>(t, lane, [](float a, float b) { return fmaxf(a, b); });
+          if (lane % (32 / kH) == 0) red[warp][lane * kH / 32] = best;
           named_bar_sync(1, kSoftmax);
-          if (tid < kN) {
+          if (tid < kH) {
             float m = fmaxf(fmaxf(red[0][tid], red[1][tid]), fmaxf(red[2][tid], red[3][tid]));
             const float old = g == g_first ? -INFINITY : ref[tid];
             m = fmaxf(m, old);
@@ -418,18 +450,17 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
             ref[tid] = m;
           }
           named_bar_sync(1, kSoftmax);
-          load_refs<kN>(ref, rf);
+          load_refs<kH>(ref, rf);
           if (g > g_first) {
 #pragma unroll
-            for (int h = 0; h < kN; ++h) l[h] *= corr_s[h];
+            for (int h = 0; h < kH; ++h) l[h] *= corr_s[h];
             wait_sum();
             for (int i = 0; i < u.pairs; ++i) {
-              float o[kN];
-              tmem_ld_heads<kN>(tmem_o + i * kN + lane_base, o);
+              float o[kH];
+              tmem_ld_heads<kH>(tmem_o + i * kN + lane_base, o);
 #pragma unroll
-              for (int h = 0; h < kN; ++h) o[h] *= corr_s[h];
-#pragma unroll
-              for (int c = 0; c < kN; c += 16) tmem_st16(tmem_o + i * kN + lane_base + c, reinterpret_cast<uint32_t(&)[16]>(o[c]));
+              for (int h = 0; h < kH; ++h) o[h] *= corr_s[h];
+              tmem_st_heads<kH>(tmem_o + i * kN + lane_base, o);
             }
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
           }
@@ -437,13 +468,13 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         uint8_t *pk = ps + (tid >> 6) * (kN * 128) + (tid & 7) * 2;
         const int chunk = (tid >> 3) & 7;
 #pragma unroll
-        for (int h = 0; h < kN; ++h) {
+        for (int h = 0; h < kH; ++h) {
           s[h] = fast_exp2(s[h] - rf[h]);
           l[h] += s[h];
         }
         wait_sum();
 #pragma unroll
-        for (int h = 0; h < kN; ++h)
+        for (int h = 0; h < kH; ++h)
           *reinterpret_cast<__nv_bfloat16 *>(pk + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16_rn(s[h]);
         if (valid < kKeys) {
           // the sequence's last tile: what stands in the rows past its end is not its own, and weight 0 is not
@@ -468,8 +499,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         put_queries(r_next);
       }
       // ---- the item, or this range's part of it ----
-      const float sum = reduce_heads<kN>(l, lane, [](float a, float b) { return a + b; });
-      if (kN == 32 || (lane & 1) == 0) red[warp][lane * kN / 32] = sum;
+      const float sum = reduce_heads<kH>(l, lane, [](float a, float b) { return a + b; });
+      if (lane % (32 / kH) == 0) red[warp][lane * kH / 32] = sum;
       ok = mbar_wait_warp(bar_o, (tile - 1) & 1, abort_flag, p.wait_ns) && ok;
       tc_fence_after();
       if (any_of_softmax(!ok)) {  // also: red is complete
@@ -478,14 +509,14 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       }
       const bool whole = k_first == 0 && g_end == start[r + 1];
       const int slot = (int)blockIdx.x * 2 + (k_first == 0 ? 1 : 0);
-      if (!whole && tid < kN) u.part_ml[slot * kN + tid] = make_float2(ref[tid], red[0][tid] + red[1][tid] + red[2][tid] + red[3][tid]);
+      if (!whole && tid < kH) u.part_ml[slot * kN + tid] = make_float2(ref[tid], red[0][tid] + red[1][tid] + red[2][tid] + red[3][tid]);
       for (int i = 0; i < u.pairs; ++i) {
-        float o[kN];
-        tmem_ld_heads<kN>(tmem_o + i * kN + lane_base, o);
+        float o[kH];
+        tmem_ld_heads<kH>(tmem_o + i * kN + lane_base, o);
         const int e = i * 128 + tid;
         if (e >= p.kv_rank) continue;
 #pragma unroll
-        for (int h = 0; h < kN; ++h) {
+        for (int h = 0; h < kH; ++h) {
           if (whole) {
             if (h0 + h < h_end) {
               const float lt = red[0][h] + red[1][h] + red[2][h] + red[3][h];
@@ -601,9 +632,9 @@ bool layout(UmmaAttend &u) {
   return true;
 }
 
-template <int kN>
+template <int kN, int kH>
 int run(const AttendParams &p, void *workspace, cudaStream_t st) {
-  auto *kernel = latent_umma_kernel<kN>;
+  auto *kernel = latent_umma_kernel<kN, kH>;
   static std::mutex mu;
   static bool opted[64] = {false};
   int dev = 0;
@@ -616,12 +647,14 @@ int run(const AttendParams &p, void *workspace, cudaStream_t st) {
       opted[dev] = true;
     }
   }
-  // a part's elements, the parts of a row, the rows: a box ends with its part and is zero-filled beyond
+  // a part's elements, the parts of a row, the rows of a page, the pages: a box ends with its part, zero-filled beyond
   CUtensorMap map;
-  const cuuint64_t dims[3] = {(cuuint64_t)(p.kv_rank + p.rot_dim), (cuuint64_t)p.kv_heads, (cuuint64_t)p.num_pages * p.page_tokens};
-  const cuuint64_t strides[2] = {(cuuint64_t)(p.kv_heads > 1 ? p.kv_rank : p.row_elems) * 2, (cuuint64_t)p.row_elems * 2};
-  const cuuint32_t box[3] = {64, 1, 64}, es[3] = {1, 1, 1};
-  if (tensor_map_encoder()(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void *>(p.pages), dims, strides, box, es,
+  const cuuint64_t dims[4] = {(cuuint64_t)(p.kv_rank + p.rot_dim), (cuuint64_t)p.kv_heads, (cuuint64_t)p.page_tokens,
+                              (cuuint64_t)p.num_pages};
+  const cuuint64_t strides[3] = {(cuuint64_t)(p.kv_heads > 1 ? p.kv_rank : p.row_elems) * 2, (cuuint64_t)p.row_elems * 2,
+                                 (cuuint64_t)p.page_elems * 2};
+  const cuuint32_t box[4] = {64, 1, 64, 1}, es[4] = {1, 1, 1, 1};
+  if (tensor_map_encoder()(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void *>(p.pages), dims, strides, box, es,
                            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
     return AXB200_INTERNAL_ERROR;
@@ -666,14 +699,16 @@ bool latent_umma_supported(const AttendParams &p) {
   const int n = heads_per_tile(p.heads / p.kv_heads), sms = sm_count();
   UmmaAttend u{};
   u.a = p;
-  return p.kv_rank % 8 == 0 && p.rot_dim % 8 == 0 && p.row_elems % 8 == 0 && (p.rot_dim == 0 || (p.dim % 8 == 0 && p.q_ld % 8 == 0)) &&
+  return p.kv_rank % 8 == 0 && p.rot_dim % 8 == 0 && p.row_elems % 8 == 0 && p.page_elems % 8 == 0 && (p.rot_dim == 0 || (p.dim % 8 == 0 && p.q_ld % 8 == 0)) &&
          (bits & 15u) == 0 && p.page_tokens % 64 == 0 && p.kv_heads * ((p.heads / p.kv_heads + n - 1) / n) <= kMaxCtas && sms > 0 && sms <= kMaxCtas && tensor_map_encoder() &&
-         (int64_t)p.num_pages * p.page_tokens < 0x7fffffff && (p.max_len / kKeys + 1) * (int64_t)kMaxRows < 0x7fffffff &&
+         (p.max_len / kKeys + 1) * (int64_t)kMaxRows < 0x7fffffff &&
          (n == 16 ? layout<16>(u) : layout<32>(u));
 }
 
 int latent_umma(const AttendParams &p, void *workspace, cudaStream_t st) {
-  return heads_per_tile(p.heads / p.kv_heads) == 16 ? run<16>(p, workspace, st) : run<32>(p, workspace, st);
+  const int part_heads = p.heads / p.kv_heads;
+  if (heads_per_tile(part_heads) == 32) return run<32, 32>(p, workspace, st);
+  return part_heads <= 4 ? run<16, 4>(p, workspace, st) : part_heads <= 8 ? run<16, 8>(p, workspace, st) : run<16, 16>(p, workspace, st);
 }
 
 }  // namespace axb

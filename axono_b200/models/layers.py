@@ -139,7 +139,7 @@ class SharedKVAttention:
         self.window, self.cache_layer = window, cache_layer
         self.w_in = _padded_rows(torch.cat([wq, wk]))
         self.q_norm, self.k_norm, self.wo = q_norm, k_norm, wo
-        self.row_elems, self.key_scale = ops.shared_kv_row(kv_heads, dim, wo.dtype)
+        self.row_elems = ops.shared_kv_row(kv_heads, dim, wo.dtype)
         self.expandable = ops.latent_prefill_supported(heads, dim, 0, dim, wo.dtype) and scale > 0
 
     def takes_segment(self, n: int) -> bool:
@@ -149,17 +149,16 @@ class SharedKVAttention:
         pages, nq, nk = cache.pages[self.cache_layer], self.heads * self.dim, self.kv_heads * self.dim
         proj = ops.linear(h, self.w_in)
         q = ops.shared_kv_prepare(proj[:, :nq], self.q_norm, proj[:, nq:nq + nk], self.k_norm, pages, rows, self.heads,
-                                  self.kv_heads, self.dim, self.key_scale, self.eps)
+                                  self.kv_heads, self.dim, self.eps)
         return ops.linear(_by_form(self, q, rows, pages), self.wo)
 
     def _latent_form(self, q, rows, pages, m):
         return ops.latent_attend(q[:m], None, self.dim, 0, self.scale, pages, rows, m, self.window, None, self.kv_heads,
-                                 self.key_scale).view(m, -1)
+                                 True).view(m, -1)
 
     def _expanded_form(self, q, rows, pages, seq, start):
         first = _first_key(start, self.window)
-        k, v = ops.shared_kv_gather(pages, rows.block_table[seq], first, start + q.shape[0] - first, self.kv_heads, self.dim,
-                                    self.key_scale)
+        k, v = ops.shared_kv_gather(pages, rows.block_table[seq], first, start + q.shape[0] - first, self.kv_heads, self.dim)
         return ops.latent_prefill(q.view(q.shape[0], -1), start - first, k, v, None, self.heads, self.dim, 0, self.dim, self.scale,
                                   self.window, None, self.kv_heads)
 

@@ -683,14 +683,15 @@ def latent_prepare(rows, inv_freq, rot_dim, q=None, heads=0, dim=0, dq=None, dq_
     return cq
 
 
-def latent_attend(q_lat, q, dim, rot_dim, scale, pages, rows, n, window=0, sink=None, kv_heads=1, key_scale=-1):
+def latent_attend(q_lat, q, dim, rot_dim, scale, pages, rows, n, window=0, sink=None, kv_heads=1, key_scale=False):
     """Latent attention of the first n rows: q_lat (n, heads, kv_rank), the rotated query parts inside q (strided
     rows of heads x (dim + rot_dim); None without them) -> (n, heads, kv_rank).  window: keys a row sees (0: all); sink
-    (heads) fp32: logit in the denominator; kv_heads parts per cached row; key_scale: where its scores' factor stands."""
+    (heads) fp32: logit in the denominator; kv_heads parts per cached row; key_scale: pages end with a factor per row (`shared_kv_prepare`)."""
     op = "latent_attend"
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != q_lat.shape[1]):
         _capi.check(4, op)
-    if not q_lat.is_contiguous() or q_lat.dtype != pages.dtype:
+    elems = kv_heads * q_lat.shape[2] + rot_dim + (4 // pages.element_size() if key_scale else 0)
+    if not q_lat.is_contiguous() or q_lat.dtype != pages.dtype or pages.shape[2] != elems:
         _capi.check(4, op)
     dt = _lm_dt(q_lat, op)
     heads, rank = q_lat.shape[1], q_lat.shape[2]
@@ -700,7 +701,7 @@ def latent_attend(q_lat, q, dim, rot_dim, scale, pages, rows, n, window=0, sink=
     _call(lib.axb200_latent_attend(
         q_lat.data_ptr(), _ptr(q), q.stride(0) if q is not None else 0, dim, out.data_ptr(), pages.data_ptr(),
         rows.block_table.data_ptr(), rows.seq.data_ptr(), rows.pos.data_ptr(), _ptr(sink), n, heads, kv_heads, rank, rot_dim,
-        pages.shape[2], int(key_scale), int(window), float(scale), pages.shape[1], rows.block_table.shape[1], pages.shape[0],
+        int(key_scale), int(window), float(scale), pages.shape[1], rows.block_table.shape[1], pages.shape[0],
         rows.block_table.shape[0], int(rows.max_len), dt, ws.data_ptr(), ws.numel(), _stream(q_lat)), op)
     return out
 
@@ -739,38 +740,41 @@ def latent_prefill(q, start, k, v, rot, heads, dim, rot_dim, vdim, scale, window
 
 
 def shared_kv_row(kv_heads, dim, dtype):
-    """(elements of a cached row of raw keys, element at which its factor stands)."""
-    per = 16 // torch.empty((), dtype=dtype).element_size()
-    at = -(-kv_heads * dim // per) * per
-    return at + per, at
+    """Elements a token takes in the cache of raw keys: the row itself and its share of the page's factors."""
+    return kv_heads * dim + 4 // torch.empty((), dtype=dtype).element_size()
 
 
-def shared_kv_prepare(q, q_weight, k, k_weight, pages, rows, heads, kv_heads, dim, key_scale, eps):
+def shared_kv_factors(pages):
+    """The factors (num_pages, page_tokens) at the end of each page."""
+    per = 4 // pages.element_size()
+    return pages.view(pages.shape[0], -1)[:, pages.shape[1] * (pages.shape[2] - per):].view(torch.float32)
+
+
+def shared_kv_prepare(q, q_weight, k, k_weight, pages, rows, heads, kv_heads, dim, eps):
     """Norms q (rows, heads * dim) over the whole row with both weights folded in -> (rows, heads, dim), and appends the
     raw k (rows, kv_heads * dim) with its factor; both may be column slices of a wider matrix."""
     op = "shared_kv_prepare"
     dt = _lm_dt(q, op)
     n = q.shape[0]
     if k.dtype != q.dtype or k.shape[0] != n or q.stride(1) != 1 or k.stride(1) != 1 or q.shape[1] != heads * dim or \
-            k.shape[1] != kv_heads * dim or pages.dtype != q.dtype or q_weight.dtype != q.dtype or k_weight.dtype != q.dtype:
+            k.shape[1] != kv_heads * dim or pages.dtype != q.dtype or pages.shape[2] != shared_kv_row(kv_heads, dim, q.dtype) or q_weight.dtype != q.dtype or k_weight.dtype != q.dtype:
         _capi.check(4, op)
     out = torch.empty((n, heads, dim), dtype=q.dtype, device=q.device)
     _call(_capi.lib().axb200_shared_kv_prepare(
         q.data_ptr(), q.stride(0), q_weight.data_ptr(), out.data_ptr(), k.data_ptr(), k.stride(0), k_weight.data_ptr(), float(eps),
         pages.data_ptr(), rows.block_table.data_ptr(), rows.seq.data_ptr(), rows.pos.data_ptr(), n, heads, kv_heads, dim,
-        pages.shape[2], key_scale, pages.shape[1], rows.block_table.shape[1], pages.shape[0], rows.block_table.shape[0], dt,
-        _stream(q)), op)
+        pages.shape[1], rows.block_table.shape[1], pages.shape[0], rows.block_table.shape[0], dt, _stream(q)), op)
     return out
 
 
-def shared_kv_gather(pages, block_row, first, n, kv_heads, dim, key_scale):
+def shared_kv_gather(pages, block_row, first, n, kv_heads, dim):
     """Cached rows first .. first + n - 1 of a sequence -> normed keys (without their weight), values; (n, kv_heads * dim)."""
     op = "shared_kv_gather"
     keys = torch.empty((n, kv_heads * dim), dtype=pages.dtype, device=pages.device)
     values = torch.empty_like(keys)
     _call(_capi.lib().axb200_shared_kv_gather(
-        pages.data_ptr(), block_row.data_ptr(), keys.data_ptr(), values.data_ptr(), int(first), n, kv_heads, dim, pages.shape[2],
-        key_scale, pages.shape[1], block_row.numel(), pages.shape[0], _lm_dt(pages, op), _stream(pages)), op)
+        pages.data_ptr(), block_row.data_ptr(), keys.data_ptr(), values.data_ptr(), int(first), n, kv_heads, dim,
+        pages.shape[1], block_row.numel(), pages.shape[0], _lm_dt(pages, op), _stream(pages)), op)
     return keys, values
 
 

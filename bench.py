@@ -1790,7 +1790,7 @@ def rigozen_kernels(lab, model, z, B, S):
     state, ring = runner.states[0]
     state.normal_(generator=lab.gen)
     pl, pa = runner.pages[latent.cache_layer], runner.pages[attn.cache_layer]
-    pa[..., attn.key_scale:].view(torch.float32).fill_(1.0)
+    ops.shared_kv_factors(pa).fill_(1.0)
 
     # decode
     rows = Rows(ints(list(range(B))), ints([W] * B), runner.block_table, W + 1, B, singles=B)
@@ -1804,11 +1804,11 @@ def rigozen_kernels(lab, model, z, B, S):
     pq = bf(B, attn.w_in.shape[0])
     nq, nk = attn.heads * attn.dim, attn.kv_heads * attn.dim
     prep = lambda p, r: ops.shared_kv_prepare(p[:, :nq], attn.q_norm, p[:, nq:nq + nk], attn.k_norm, pa, r, attn.heads,  # noqa: E731
-                                              attn.kv_heads, attn.dim, attn.key_scale, 1e-5)
+                                              attn.kv_heads, attn.dim, 1e-5)
     lab.bandwidth(K, "decode shared_kv_prepare", timed(lambda: prep(pq, rows)), B * (4.0 * nq + 4.0 * nk), "nuderax norm + rotate + append (decode)")
     qa = prep(pq, rows)
     lab.bandwidth(K, "decode shared_kv attend", timed(lambda: ops.latent_attend(qa, None, attn.dim, 0, 0.05, pa, rows, B, W, None, attn.kv_heads,
-                                                                                attn.key_scale)),
+                                                                                True)),
                   B * W * attn.row_elems * 2.0 + 4.0 * qa.numel(), "tower gqa decode")
     lab.bandwidth(K, "decode residual_post_norm", timed(lambda: ops.residual_post_norm(x, y, w, 1e-5, 1.0)), B * width * 12.0,
                   "nuderax residual + norm (decode)")
@@ -1834,8 +1834,8 @@ def rigozen_kernels(lab, model, z, B, S):
     del proj
     pq = bf(S, attn.w_in.shape[0])
     lab.bandwidth(K, "prefill shared_kv_prepare", timed(lambda: prep(pq, prows)), S * (4.0 * nq + 4.0 * nk), "nuderax norm + rotate + append (prefill)")
-    lab.bandwidth(K, "prefill shared_kv_gather", timed(lambda: ops.shared_kv_gather(pa, runner.block_table[0], 0, S, attn.kv_heads, attn.dim,
-                                                                                    attn.key_scale)), S * nk * 6.0)
+    lab.bandwidth(K, "prefill shared_kv_gather", timed(lambda: ops.shared_kv_gather(pa, runner.block_table[0], 0, S, attn.kv_heads, attn.dim)),
+                  S * nk * 6.0)
     pairs = sum(min(t + 1, W) for t in range(S))
     q, k, v = bf(S, nq), bf(S, nk), bf(S, nk)
     lab.tensor(K, "prefill attention (shared kv)", timed(lambda: ops.latent_prefill(q, 0, k, v, None, attn.heads, 128, 0, 128, 0.05, W, None,

@@ -511,8 +511,8 @@ int axb200_residual_post_norm(float *x, const void *y, const void *w, float offs
  *     q_rot . rot_j) * scale) c_j, with q_lat (rows, heads, kv_rank) = q . W_uk and q_rot read from q.
  *     max_len bounds row_pos + 1 and sizes the grid.  window > 0: only the keys j > row_pos[r] - window take part.
  *     sink (heads) or NULL: exp(sink_h) joins the denominator.  kv_heads > 1 (then rot_dim = 0): the row holds kv_heads
- *     parts of kv_rank elements, query head h reads part h / (heads / kv_heads).  key_scale >= 0: the row's element at
- *     which an fp32 factor of its scores stands (key_scale < 0: none).  workspace_bytes takes the heads per part.
+ *     parts of kv_rank elements, query head h reads part h / (heads / kv_heads).  key_scale != 0: a page ends, behind
+ *     its rows, with page_tokens fp32 factors of its rows' scores.  workspace_bytes takes the heads per part.
  *   latent_gather: rows first .. first + n - 1 of one sequence's pages, contiguous.
  *   latent_prefill: the expanded form for n rows of ONE sequence at positions start .. start + n - 1: q (n, q_ld)
  *     rotated, k (skv, heads * dim) and v (skv, heads * vdim) expanded from the latents of positions 0 .. skv - 1
@@ -529,8 +529,8 @@ int axb200_latent_prepare(void *q, int64_t q_ld, int heads, int dim, const void 
 size_t axb200_latent_attend_workspace_bytes(int rows, int heads, int kv_rank, int rot_dim, int64_t max_len, int dtype);
 int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim, void *out, const void *pages,
                          const int32_t *block_table, const int32_t *row_seq, const int32_t *row_pos, const float *sink,
-                         int rows, int heads, int kv_heads, int kv_rank, int rot_dim, int row_elems, int key_scale,
-                         int window, float scale, int page_tokens, int max_blocks, int num_pages, int max_seqs,
+                         int rows, int heads, int kv_heads, int kv_rank, int rot_dim, int key_scale, int window,
+                         float scale, int page_tokens, int max_blocks, int num_pages, int max_seqs,
                          int64_t max_len, int dtype, void *workspace, size_t workspace_bytes, void *stream);
 int axb200_latent_gather(const void *pages, const int32_t *block_row, void *out, int64_t first, int64_t n, int row_elems,
                          int page_tokens, int max_blocks, int num_pages, int dtype, void *stream);
@@ -540,21 +540,21 @@ int axb200_latent_prefill(const void *q, int64_t q_ld, const void *k, const void
                           int rot_dim, int vdim, int window, float scale, int dtype, void *stream);
 
 /* ---- grouped attention whose values are the raw keys ------------------------------------------------------
- * The cache row is [kv_heads parts of dim raw key elements | ... | fp32 factor at element key_scale], the factor
- * 1 / rms of all raw elements of the row: factor * part * k_w is the normed key, the part itself the value.
+ * A page holds page_tokens rows of kv_heads parts of dim raw key elements and, behind them, page_tokens fp32 factors,
+ * 1 / rms of all raw elements of a row: factor * part * k_w is the normed key, the part itself the value.
  *   shared_kv_prepare: per row q_out (rows, heads * dim) = rms_norm(q) * q_w * (k_w of the head's part), the norm over
  *     all heads at once, and the append of the raw keys and their factor.  latent_attend with kv_rank = dim, kv_heads
- *     and key_scale then is the attention.
+ *     and key_scale set then is the attention.
  *   shared_kv_gather: rows first .. first + n - 1 of one sequence as keys (part * factor) and values (part), both (n,
  *     kv_heads * dim), for latent_prefill. */
 int axb200_shared_kv_prepare(const void *q, int64_t q_ld, const void *q_w, void *q_out, const void *k, int64_t k_ld,
                              const void *k_w, float eps, void *pages, const int32_t *block_table,
                              const int32_t *row_seq, const int32_t *row_pos, int64_t rows, int heads, int kv_heads,
-                             int dim, int row_elems, int key_scale, int page_tokens, int max_blocks, int num_pages,
-                             int max_seqs, int dtype, void *stream);
+                             int dim, int page_tokens, int max_blocks, int num_pages, int max_seqs, int dtype,
+                             void *stream);
 int axb200_shared_kv_gather(const void *pages, const int32_t *block_row, void *keys, void *values, int64_t first,
-                            int64_t n, int kv_heads, int dim, int row_elems, int key_scale, int page_tokens,
-                            int max_blocks, int num_pages, int dtype, void *stream);
+                            int64_t n, int kv_heads, int dim, int page_tokens, int max_blocks, int num_pages, int dtype,
+                            void *stream);
 
 /* ---- gated delta rule -------------------------------------------------------------------------------------
  * A recurrent mixer.  proj (rows, ld) holds per row [q | k | v | gate | a | b]: kv_heads * dim twice, heads * vdim

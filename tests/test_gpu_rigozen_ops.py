@@ -122,14 +122,11 @@ def test_window_edge_of_one_key(heads, rank, dtype):
     assert ops.last_error() == 0
 
 
-class SharedPages(Pages):
-    """Cached rows as shared_kv_prepare leaves them."""
+def shared_pages(lens, kv_heads, dim, dtype, seed=0):
+    """Pages for rows and factors as shared_kv_prepare leaves them."""
+    from axono_b200 import ops
 
-    def __init__(self, lens, kv_heads, dim, dtype, seed=0):
-        from axono_b200 import ops
-
-        row, self.at = ops.shared_kv_row(kv_heads, dim, dtype)
-        super().__init__(lens, row, dtype, seed=seed)
+    return Pages(lens, ops.shared_kv_row(kv_heads, dim, dtype), dtype, seed=seed)
 
 
 SHARED_SIZES = [(6, 3, 20), (6, 1, 48), (12, 2, 40), (32, 4, 128), (8, 8, 64), (40, 1, 128), (4, 2, 9), (64, 2, 256)]
@@ -146,16 +143,16 @@ def test_shared_kv_prepare_attend_gather(heads, kv_heads, dim, dtype):
     proj = rnd((n, nq + nk + (-(nq + nk)) % 8), dtype, 1)
     proj[:, nq:nq + nk] *= torch.linspace(0.1, 6, n).to(dtype)[:, None]  # the norm's factor differs from row to row
     qw, kw = rnd((nq,), dtype, 2) + 1, rnd((nk,), dtype, 3) + 1
-    pages = SharedPages([n], kv_heads, dim, dtype, seed=dim)
+    pages = shared_pages([n], kv_heads, dim, dtype, seed=dim)
     pool, rows, wd = pages.pool.cuda(), pages.rows([0] * n, list(range(n)), n), proj.cuda()
-    q = ops.shared_kv_prepare(wd[:, :nq], qw.cuda(), wd[:, nq:nq + nk], kw.cuda(), pool, rows, heads, kv_heads, dim, pages.at, eps)
+    q = ops.shared_kv_prepare(wd[:, :nq], qw.cuda(), wd[:, nq:nq + nk], kw.cuda(), pool, rows, heads, kv_heads, dim, eps)
     assert ops.last_error() == 0
     raw = proj[:, nq:nq + nk].double()
     group = heads // kv_heads
     fold = kw.double().view(kv_heads, 1, dim).expand(-1, group, -1).reshape(-1)
     want_q = plain.rms(proj[:, :nq].double(), eps) * qw.double() * fold
     close(q.view(n, -1), want_q, tol(dtype))
-    keys, values = ops.shared_kv_gather(pool, rows.block_table[0], 70, 200, kv_heads, dim, pages.at)
+    keys, values = ops.shared_kv_gather(pool, rows.block_table[0], 70, 200, kv_heads, dim)
     assert torch.equal(values.cpu(), proj[70:270, nq:nq + nk])
     close(keys, plain.rms(raw, eps)[70:270], tol(dtype))
     k = plain.rms(raw, eps).view(n, kv_heads, dim).transpose(0, 1).repeat_interleave(group, 0)
@@ -163,7 +160,7 @@ def test_shared_kv_prepare_attend_gather(heads, kv_heads, dim, dtype):
     qd = q.cpu().double()
     picks = [0, 1, 63, 64, 65, 127, 128, 191, 256, 299]
     for window in (1, 64, 65, 130, 0):
-        got = ops.latent_attend(q, None, dim, 0, scale, pool, rows, n, window, None, kv_heads, pages.at).cpu()
+        got = ops.latent_attend(q, None, dim, 0, scale, pool, rows, n, window, None, kv_heads, True).cpu()
         assert ops.last_error() == 0
         for i in picks:
             close(got[i], plain_rows(qd[i], k, v, i, scale, window, None), 4e-6 if dtype == torch.float32 else 1.5e-2)
@@ -172,10 +169,10 @@ def test_shared_kv_prepare_attend_gather(heads, kv_heads, dim, dtype):
 def test_shared_kv_append_without_room_is_reported():
     from axono_b200 import ops
 
-    pages = SharedPages([64], 1, 8, torch.float32)
+    pages = shared_pages([64], 1, 8, torch.float32)
     pool, one = pages.pool.cuda(), torch.ones(1, 8, device="cuda")
     for pos, word in ((64, 2), (64 * pages.table.shape[1], 4)):
-        ops.shared_kv_prepare(one, one[0], one, one[0], pool, pages.rows([0], [pos], 256), 1, 1, 8, pages.at, 1e-5)
+        ops.shared_kv_prepare(one, one[0], one, one[0], pool, pages.rows([0], [pos], 256), 1, 1, 8, 1e-5)
         assert ops.last_error() == word
     assert torch.equal(pool.cpu(), pages.pool)
 
