@@ -45,6 +45,7 @@ struct UmmaAttend {
   int pair_slots, single_slots;  // in the rings
   int chunks;                    // per row: ceil(elements / 64)
   int ahead;                     // the rings hold two tiles: a tile's scores are computed before the sum of the one before
+  int p_slots;                   // buffers of P: two where there is room ahead
   float *part_o;                 // (2 * CTAs, N, kv_rank)
   float2 *part_ml;               // (2 * CTAs, N): reference (log2 domain), sum
 };
@@ -176,7 +177,7 @@ struct Smem {
   // after the rings: Q (chunks boxes), P, reference and reduction scratch, barriers, row starts
   __host__ __device__ static int off_q(const UmmaAttend &u) { return u.pair_slots * 2 * kChunk + u.single_slots * kChunk; }
   __host__ __device__ static int off_p(const UmmaAttend &u) { return off_q(u) + u.chunks * kQBox; }
-  __host__ __device__ static int off_ref(const UmmaAttend &u) { return off_p(u) + kP; }
+  __host__ __device__ static int off_ref(const UmmaAttend &u) { return off_p(u) + u.p_slots * kP; }
   __host__ __device__ static int off_red(const UmmaAttend &u) { return off_ref(u) + 2 * kN * 4; }
   __host__ __device__ static int off_bar(const UmmaAttend &u) { return off_red(u) + 4 * kN * 4; }
   __host__ __device__ static int off_start(const UmmaAttend &u) { return off_bar(u) + 512; }
@@ -193,9 +194,9 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
   const AttendParams &p = u.a;
   uint64_t *full_p = reinterpret_cast<uint64_t *>(smem + S::off_bar(u)), *empty_p = full_p + kMaxSlots;
   uint64_t *full_s = empty_p + kMaxSlots, *empty_s = full_s + kMaxSlots;
-  uint64_t *bar_s = empty_s + kMaxSlots, *bar_p = bar_s + 2, *bar_q = bar_p + 1, *bar_o = bar_q + 1;
-  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(bar_o + 1);
-  volatile int *abort_flag = reinterpret_cast<volatile int *>(bar_o + 2);
+  uint64_t *bar_s = empty_s + kMaxSlots, *bar_o = bar_s + 2, *bar_p = bar_o + 2, *bar_q = bar_p + 1;
+  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(bar_q + 1);
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(bar_q + 2);
   int *start = reinterpret_cast<int *>(smem + S::off_start(u));
   if ((smem_u32(smem) & 1023u) != 0) {
     if (threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_WAIT_TIMEOUT);
@@ -203,10 +204,9 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
   }
   const int warp = uniform_warp(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 4 * kMaxSlots + 2; ++i) mbar_init(&full_p[i], 1);  // rings and bar_s
+    for (int i = 0; i < 4 * kMaxSlots + 4; ++i) mbar_init(&full_p[i], 1);  // rings, bar_s and bar_o
     mbar_init(bar_p, 4);
     mbar_init(bar_q, 4);
-    mbar_init(bar_o, 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -347,16 +347,17 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       if (!ok) break;
       tc_fence_after();
       const bool fresh = g == lo || g == start[r];
+      const uint64_t dpt = dp + (uint64_t)((u.p_slots == 2 ? tile & 1 : 0) * (S::kP >> 4));
       for (int i = 0; i < u.pairs; ++i, pv.next(u.pair_slots)) {
         const int s = pv.slot;
         const uint64_t a = dv + (uint64_t)(s * (2 * kChunk >> 4));
 #pragma unroll
         for (int ks = 0; ks < kKeys / 16; ++ks)  // 16 keys: 2 KB of the chunk, 32 bytes of P
           umma_f16_lead(tmem_o + i * kN, a + (uint64_t)(ks * (2048 >> 4)),
-                        dp + (uint64_t)(((ks >> 2) * (kN * 128) + (ks & 3) * 32) >> 4), idesc_o, !fresh || ks > 0, lead);
+                        dpt + (uint64_t)(((ks >> 2) * (kN * 128) + (ks & 3) * 32) >> 4), idesc_o, !fresh || ks > 0, lead);
         umma_commit_lead(&empty_p[s], lead);
       }
-      umma_commit_lead(bar_o, lead);
+      umma_commit_lead(&bar_o[tile & 1], lead);
       if (!u.ahead && g_s < hi) ok = scores();
     }
   } else {
@@ -408,9 +409,10 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         if (p.key_scale && g + 1 < hi) next_factor = factor_of(r, g + 1);
         ok = mbar_wait_warp(&bar_s[tile & 1], (tile >> 1) & 1, abort_flag, p.wait_ns) && ok;
         tc_fence_after();
-        // the last tile's sum has to be done before O^T is rescaled and before its weights are overwritten
-        auto wait_sum = [&] {
-          if (tile > 0) ok = mbar_wait_warp(bar_o, (tile - 1) & 1, abort_flag, p.wait_ns) && ok;
+        // the last tile's sum has to be done before O^T is rescaled, that of `p_slots` tiles back before its weights are
+        // overwritten
+        auto wait_sum = [&](int back) {
+          if (tile >= back) ok = mbar_wait_warp(&bar_o[(tile - back) & 1], ((tile - back) >> 1) & 1, abort_flag, p.wait_ns) && ok;
           tc_fence_after();
         };
         float s[kH], rf[kH];
@@ -454,7 +456,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
           if (g > g_first) {
 #pragma unroll
             for (int h = 0; h < kH; ++h) l[h] *= corr_s[h];
-            wait_sum();
+            wait_sum(1);
             for (int i = 0; i < u.pairs; ++i) {
               float o[kH];
               tmem_ld_heads<kH>(tmem_o + i * kN + lane_base, o);
@@ -465,14 +467,14 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
           }
         }
-        uint8_t *pk = ps + (tid >> 6) * (kN * 128) + (tid & 7) * 2;
+        uint8_t *pk = ps + (u.p_slots == 2 ? tile & 1 : 0) * S::kP + (tid >> 6) * (kN * 128) + (tid & 7) * 2;
         const int chunk = (tid >> 3) & 7;
 #pragma unroll
         for (int h = 0; h < kH; ++h) {
           s[h] = fast_exp2(s[h] - rf[h]);
           l[h] += s[h];
         }
-        wait_sum();
+        wait_sum(u.p_slots);
 #pragma unroll
         for (int h = 0; h < kH; ++h)
           *reinterpret_cast<__nv_bfloat16 *>(pk + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16_rn(s[h]);
@@ -501,7 +503,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       // ---- the item, or this range's part of it ----
       const float sum = reduce_heads<kH>(l, lane, [](float a, float b) { return a + b; });
       if (lane % (32 / kH) == 0) red[warp][lane * kH / 32] = sum;
-      ok = mbar_wait_warp(bar_o, (tile - 1) & 1, abort_flag, p.wait_ns) && ok;
+      ok = mbar_wait_warp(&bar_o[(tile - 1) & 1], ((tile - 1) >> 1) & 1, abort_flag, p.wait_ns) && ok;
       tc_fence_after();
       if (any_of_softmax(!ok)) {  // also: red is complete
         ok = false;
@@ -616,6 +618,7 @@ bool layout(UmmaAttend &u) {
   // every pair of a tile has to be in place before the first is freed; what is left is read-ahead
   u.single_slots = u.singles;
   u.pair_slots = u.pairs;
+  u.p_slots = 1;
   if (Smem<kN>::bytes(u, kMaxRows) > kSmemLimit) return false;
   while (u.pair_slots < kMaxSlots) {
     ++u.pair_slots;
@@ -629,6 +632,12 @@ bool layout(UmmaAttend &u) {
     if (Smem<kN>::bytes(u, kMaxRows) > kSmemLimit) --u.single_slots;
   }
   u.ahead = u.pair_slots >= 2 * u.pairs && u.single_slots >= 2 * u.singles;
+  if (u.ahead) {
+    UmmaAttend two = u;
+    two.p_slots = 2;
+    while (Smem<kN>::bytes(two, kMaxRows) > kSmemLimit && two.pair_slots > 2 * u.pairs) --two.pair_slots;
+    if (Smem<kN>::bytes(two, kMaxRows) <= kSmemLimit) u = two;
+  }
   return true;
 }
 
