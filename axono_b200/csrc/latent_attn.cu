@@ -11,8 +11,8 @@
 // 0 .. row_pos[r], or the last `window` of them, so one launch serves decode batches, portions of prompts and
 // mixtures of both.  A per-head sink may join the denominator.
 //
-// The same kernels attend plain cached keys that are also the values: kv_heads parts per row, each read by its group of
-// query heads, and a factor per row, behind the rows of its page, that turns its keys - not its values - into normed ones (shared_kv.cu).
+// The same kernels attend plain cached keys that are also the values: kv_heads rows per token, each read by its group of
+// query heads, and a factor per token, behind the rows of its page, that turns its keys - not its values - into normed ones (shared_kv.cu).
 #include <math.h>
 
 #include "latent_attn.cuh"
@@ -269,7 +269,7 @@ __global__ void __launch_bounds__(kGenThreads) latent_attend_generic_kernel(cons
   const int part_elems = p.kv_rank + p.rot_dim;
   float *q = sm, *acc = sm + part_elems;
   const int r = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int part = h / (p.heads / p.kv_heads) * p.kv_rank;
+  const size_t part = (size_t)(h / (p.heads / p.kv_heads)) * p.page_tokens;
   grid_dependency_wait();
   grid_dependency_launch();
   const T *ql = static_cast<const T *>(p.q_lat) + ((size_t)r * p.heads + h) * p.kv_rank;
@@ -291,7 +291,7 @@ __global__ void __launch_bounds__(kGenThreads) latent_attend_generic_kernel(cons
         page = 0;
       }
       const T *base = pages + (size_t)page * p.page_elems;
-      key[threadIdx.x] = base + (size_t)(t % p.page_tokens) * p.row_elems + part;
+      key[threadIdx.x] = base + (part + t % p.page_tokens) * p.row_elems;
       factor[threadIdx.x] = p.key_scale ? p.scale * page_factors(base, p)[t % p.page_tokens] : p.scale;
     }
     __syncthreads();
@@ -404,8 +404,8 @@ int axb200_latent_attend(const void *q_lat, const void *q, int64_t q_ld, int dim
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   axb::AttendParams p{};
   p.kv_heads = kv_heads;
-  p.row_elems = kv_heads * kv_rank + rot_dim;
-  p.page_elems = page_tokens * p.row_elems + (key_scale ? page_tokens * (4 / (int)axb::dtype_size(dtype)) : 0);
+  p.row_elems = kv_rank + rot_dim;
+  p.page_elems = page_tokens * kv_heads * p.row_elems + (key_scale ? page_tokens * (4 / (int)axb::dtype_size(dtype)) : 0);
   p.key_scale = key_scale;
   p.window = window;
   p.sink = sink;

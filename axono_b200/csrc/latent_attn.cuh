@@ -16,8 +16,8 @@ struct AttendParams {
   int rows, heads, dim, kv_rank, rot_dim, page_tokens, max_blocks, num_pages, max_seqs, max_len;
   float scale;
   unsigned long long wait_ns;
-  int kv_heads;       // a cached row holds kv_heads parts of kv_rank elements, each for heads / kv_heads query heads
-  int row_elems;      // elements from one cached row of a page to the next
+  int kv_heads;       // a token caches kv_heads rows, each for heads / kv_heads query heads; in a page head by head
+  int row_elems;      // of one such row: kv_rank + rot_dim
   int page_elems;     // elements from one page to the next
   int key_scale;      // whether a page ends, behind its rows, with an fp32 factor of the keys of each row
   int window;         // keys a row sees, itself included; 0: all
@@ -40,7 +40,7 @@ __device__ __forceinline__ int first_key(const AttendParams &p, int r) {
 // The factors of a page's rows (see shared_kv.cu).
 template <typename T>
 __device__ __forceinline__ const float *page_factors(const T *page, const AttendParams &p) {
-  return reinterpret_cast<const float *>(page + (size_t)p.page_tokens * p.row_elems);
+  return reinterpret_cast<const float *>(page + (size_t)p.kv_heads * p.page_tokens * p.row_elems);
 }
 
 // tcgen05 form for bf16 (latent_umma.cu)

@@ -84,13 +84,6 @@ __device__ __forceinline__ void scan_tiles(const AttendParams &p, int *start) {
   }
 }
 
-// The factor of key t's row of row r's sequence (the loader reports a bad page).
-__device__ __forceinline__ float key_factor(const AttendParams &p, int r, int t) {
-  const int page = p.block_table[(size_t)p.row_seq[r] * p.max_blocks + t / p.page_tokens];
-  if (page < 0 || page >= p.num_pages) return 0.f;
-  return page_factors(static_cast<const __nv_bfloat16 *>(p.pages) + (size_t)page * p.page_elems, p)[t % p.page_tokens];
-}
-
 // What un-normalised results with sum l at reference ref (log2 domain) are multiplied by when a sink joins the sum.
 __device__ __forceinline__ float inverse_with_sink(float ref, float l, float sink) {
   const float s = sink * kLog2e, top = fmaxf(ref, s), w = fast_exp2(ref - top);
@@ -174,10 +167,12 @@ template <int kN>
 struct Smem {
   static constexpr int kP = kN * kKeys * 2;
   static constexpr int kQBox = kN * 128;
-  // after the rings: Q (chunks boxes), P, reference and reduction scratch, barriers, row starts
+  // after the rings: Q (chunks boxes), P, the keys' factors (for each pair slot, filled with a tile's first pair),
+  // reference and reduction scratch, barriers, row starts
   __host__ __device__ static int off_q(const UmmaAttend &u) { return u.pair_slots * 2 * kChunk + u.single_slots * kChunk; }
   __host__ __device__ static int off_p(const UmmaAttend &u) { return off_q(u) + u.chunks * kQBox; }
-  __host__ __device__ static int off_ref(const UmmaAttend &u) { return off_p(u) + u.p_slots * kP; }
+  __host__ __device__ static int off_factor(const UmmaAttend &u) { return off_p(u) + u.p_slots * kP; }
+  __host__ __device__ static int off_ref(const UmmaAttend &u) { return off_factor(u) + (u.a.key_scale ? u.pair_slots * kKeys * 4 : 0); }
   __host__ __device__ static int off_red(const UmmaAttend &u) { return off_ref(u) + 2 * kN * 4; }
   __host__ __device__ static int off_bar(const UmmaAttend &u) { return off_red(u) + 4 * kN * 4; }
   __host__ __device__ static int off_start(const UmmaAttend &u) { return off_bar(u) + 512; }
@@ -281,7 +276,13 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
             const int s = rp.slot, n = min(2, u.chunks - 2 * i);
             if (np >= u.pair_slots) ok = mbar_wait_bounded(&empty_p[s], rp.parity ^ 1, abort_flag, p.wait_ns);
             if (!ok) break;
-            mbar_arrive_expect_tx(&full_p[s], n * halves * (kChunk / 2));
+            const bool factors = p.key_scale && i == 0;
+            mbar_arrive_expect_tx(&full_p[s], n * halves * (kChunk / 2) + (factors ? halves * 256 : 0));
+            if (factors)
+              for (int k = 0; k < halves; ++k)
+                bulk_load(smem + S::off_factor(u) + s * kKeys * 4 + k * 256,
+                          page_factors(static_cast<const __nv_bfloat16 *>(p.pages) + (size_t)page_at[k] * p.page_elems, p) + at[k], 256,
+                          &full_p[s]);
             for (int c = 0; c < n; ++c) load_chunk(smem + s * 2 * kChunk + c * kChunk, &full_p[s], 2 * i + c);
           }
         }
@@ -386,13 +387,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_q);
     };
-    // the factor of this thread's key in tile g (of row r or a later one), fetched a tile ahead
-    auto factor_of = [&](int r, int g) {
-      while (start[r + 1] <= g) ++r;
-      const int t = first_tile_key(p, r) + (g - start[r]) * kKeys + tid;
-      return t < visible_keys(p, r) ? key_factor(p, r, t) : 0.f;
-    };
-    float next_factor = p.key_scale ? factor_of(r_first, lo) : 1.f;
+    const float *factors = reinterpret_cast<const float *>(smem + S::off_factor(u));
+    RingPos fp;  // of a tile's first pair
     for (int r = r_first, g = lo; g < hi && ok; ++r) {
       if (start[r + 1] <= g) continue;
       const int k_first = g - start[r], g_end = min(hi, start[r + 1]), keys = visible_keys(p, r);
@@ -405,10 +401,14 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       for (const int g_first = g; g < g_end; ++g, ++tile, np += u.pairs) {
         const int valid = min(kKeys, keys - key0 - (g - start[r]) * kKeys);
         const bool seen = tid < valid && (g > start[r] || tid >= hidden);
-        const float factor = scale_log2 * next_factor;
-        if (p.key_scale && g + 1 < hi) next_factor = factor_of(r, g + 1);
+        float factor = scale_log2;
         ok = mbar_wait_warp(&bar_s[tile & 1], (tile >> 1) & 1, abort_flag, p.wait_ns) && ok;
         tc_fence_after();
+        if (p.key_scale) {
+          ok = mbar_wait_warp(&full_p[fp.slot], fp.parity, abort_flag, p.wait_ns) && ok;
+          factor *= factors[fp.slot * kKeys + tid];
+          for (int i = 0; i < u.pairs; ++i) fp.next(u.pair_slots);
+        }
         // the last tile's sum has to be done before O^T is rescaled, that of `p_slots` tiles back before its weights are
         // overwritten
         auto wait_sum = [&](int back) {
@@ -656,11 +656,11 @@ int run(const AttendParams &p, void *workspace, cudaStream_t st) {
       opted[dev] = true;
     }
   }
-  // a part's elements, the parts of a row, the rows of a page, the pages: a box ends with its part, zero-filled beyond
+  // a row's elements, the heads and the tokens of a page, the pages: a box ends with its row, zero-filled beyond
   CUtensorMap map;
-  const cuuint64_t dims[4] = {(cuuint64_t)(p.kv_rank + p.rot_dim), (cuuint64_t)p.kv_heads, (cuuint64_t)p.page_tokens,
+  const cuuint64_t dims[4] = {(cuuint64_t)p.row_elems, (cuuint64_t)p.kv_heads, (cuuint64_t)p.page_tokens,
                               (cuuint64_t)p.num_pages};
-  const cuuint64_t strides[3] = {(cuuint64_t)(p.kv_heads > 1 ? p.kv_rank : p.row_elems) * 2, (cuuint64_t)p.row_elems * 2,
+  const cuuint64_t strides[3] = {(cuuint64_t)p.page_tokens * p.row_elems * 2, (cuuint64_t)p.row_elems * 2,
                                  (cuuint64_t)p.page_elems * 2};
   const cuuint32_t box[4] = {64, 1, 64, 1}, es[4] = {1, 1, 1, 1};
   if (tensor_map_encoder()(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void *>(p.pages), dims, strides, box, es,

@@ -1,6 +1,6 @@
-// Grouped attention whose values are the keys as projected: the cache holds one row of kv_heads parts of dim raw key
-// elements per token, and a page ends, behind its rows, with one fp32 factor per row.  The factor, 1 / rms of the whole
-// raw row, makes the parts the normed keys.  The key norm's weight is folded into
+// Grouped attention whose values are the keys as projected: the cache holds kv_heads rows of dim raw key elements per
+// token, head by head within a page, and a page ends with one fp32 factor per token.  The factor, 1 / rms of all the
+// token's elements, makes the rows the normed keys.  The key norm's weight is folded into
 // the queries, so a score is factor_j * (q' . k_j) and a value is k_j itself: one read of the row serves both, where a
 // cache of keys and values would take two.  The attention over these rows is latent_attn.cu / latent_umma.cu; for long
 // portions of prompts the rows are gathered into normed keys and raw values for the kernel of latent_prefill.cu.
@@ -25,7 +25,7 @@ struct SharedKvParams {
   const T *k;    // (rows, k_ld): kv_heads * dim
   int64_t k_ld;
   const T *k_w;  // (kv_heads * dim)
-  T *pages;      // per page: (page_tokens, kv_heads * dim) and page_tokens fp32 factors
+  T *pages;      // per page: (kv_heads, page_tokens, dim) and page_tokens fp32 factors
   const int32_t *block_table, *row_seq, *row_pos;
   int heads, kv_heads, dim, max_blocks, page_tokens, num_pages, max_seqs;
   float eps;
@@ -71,10 +71,10 @@ __global__ void __launch_bounds__(kThreads) shared_kv_prepare_kernel(const Share
     if (threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
     return;
   }
-  T *base = p.pages + page * page_elems<T>(p.page_tokens, nk), *dst = base + (size_t)(pos % p.page_tokens) * nk;
+  T *base = p.pages + page * page_elems<T>(p.page_tokens, nk);
   for (int i = threadIdx.x * kVec; i < nk; i += kThreads * kVec) {
     load_vec<kVec>(k + i, v);
-    store_vec<kVec>(dst + i, v);
+    store_vec<kVec>(base + ((size_t)(i / p.dim) * p.page_tokens + pos % p.page_tokens) * p.dim + i % p.dim, v);
   }
   if (threadIdx.x == 0) reinterpret_cast<float *>(base + (size_t)p.page_tokens * nk)[pos % p.page_tokens] = inv_k;
 }
@@ -82,7 +82,7 @@ __global__ void __launch_bounds__(kThreads) shared_kv_prepare_kernel(const Share
 // Cached rows first .. first + n - 1 of one sequence as normed keys and raw values, both (n, elems); a warp per row.
 template <typename T, int kVec>
 __global__ void __launch_bounds__(kThreads)
-shared_kv_gather_kernel(const T *pages, const int32_t *table, T *keys, T *values, int first, int n, int elems, int page_tokens, int max_blocks, int num_pages) {
+shared_kv_gather_kernel(const T *pages, const int32_t *table, T *keys, T *values, int first, int n, int elems, int dim, int page_tokens, int max_blocks, int num_pages) {
   grid_dependency_wait();
   grid_dependency_launch();
   const int lane = threadIdx.x & 31;
@@ -92,11 +92,11 @@ shared_kv_gather_kernel(const T *pages, const int32_t *table, T *keys, T *values
       if (lane == 0) atomicOr(&g_error_word, AXB200_ERR_BAD_PAGE);
       continue;
     }
-    const T *base = pages + page * page_elems<T>(page_tokens, elems), *src = base + (size_t)(t % page_tokens) * elems;
+    const T *base = pages + page * page_elems<T>(page_tokens, elems);
     const float inv = reinterpret_cast<const float *>(base + (size_t)page_tokens * elems)[t % page_tokens];
     for (int i = lane * kVec; i < elems; i += 32 * kVec) {
       float v[kVec];
-      load_vec<kVec>(src + i, v);
+      load_vec<kVec>(base + ((size_t)(i / dim) * page_tokens + t % page_tokens) * dim + i % dim, v);
       store_vec<kVec>(values + (size_t)r * elems + i, v);
 #pragma unroll
       for (int e = 0; e < kVec; ++e) v[e] *= inv;
@@ -153,12 +153,12 @@ int axb200_shared_kv_gather(const void *pages, const int32_t *block_row, void *k
   auto go = [&](auto tag) {
     using T = decltype(tag);
     const int elems = kv_heads * dim;
-    const bool vec = elems % 8 == 0 && page_tokens % 8 == 0 && axb::al16(pages) && axb::al16(keys) && axb::al16(values);
+    const bool vec = dim % 8 == 0 && page_tokens % 8 == 0 && axb::al16(pages) && axb::al16(keys) && axb::al16(values);
     auto *kernel = vec ? axb::shared_kv_gather_kernel<T, 8> : axb::shared_kv_gather_kernel<T, 1>;
     const int64_t want = (n + axb::kThreads / 32 - 1) / (axb::kThreads / 32);
     return axb::launch_dependent(kernel, dim3((unsigned)(want < 148 * 8 ? want : 148 * 8)), dim3(axb::kThreads), 0,
                                  static_cast<cudaStream_t>(stream), static_cast<const T *>(pages), block_row,
-                                 static_cast<T *>(keys), static_cast<T *>(values), (int)first, (int)n, elems,
+                                 static_cast<T *>(keys), static_cast<T *>(values), (int)first, (int)n, elems, dim,
                                  page_tokens, max_blocks, num_pages);
   };
   return dtype == AXB200_FLOAT32 ? go(float{}) : go(__nv_bfloat16{});

@@ -686,7 +686,8 @@ def latent_prepare(rows, inv_freq, rot_dim, q=None, heads=0, dim=0, dq=None, dq_
 def latent_attend(q_lat, q, dim, rot_dim, scale, pages, rows, n, window=0, sink=None, kv_heads=1, key_scale=False):
     """Latent attention of the first n rows: q_lat (n, heads, kv_rank), the rotated query parts inside q (strided
     rows of heads x (dim + rot_dim); None without them) -> (n, heads, kv_rank).  window: keys a row sees (0: all); sink
-    (heads) fp32: logit in the denominator; kv_heads parts per cached row; key_scale: pages end with a factor per row (`shared_kv_prepare`)."""
+    (heads) fp32: logit in the denominator; kv_heads rows per
+    cached token; key_scale: pages end with a factor per token (`shared_kv_prepare`)."""
     op = "latent_attend"
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != q_lat.shape[1]):
         _capi.check(4, op)
@@ -740,7 +741,7 @@ def latent_prefill(q, start, k, v, rot, heads, dim, rot_dim, vdim, scale, window
 
 
 def shared_kv_row(kv_heads, dim, dtype):
-    """Elements a token takes in the cache of raw keys: the row itself and its share of the page's factors."""
+    """Elements a token takes in the cache of raw keys: its rows and its share of the page's factors."""
     return kv_heads * dim + 4 // torch.empty((), dtype=dtype).element_size()
 
 

@@ -510,9 +510,9 @@ int axb200_residual_post_norm(float *x, const void *y, const void *w, float offs
  *   latent_attend: out (rows, heads, kv_rank) = sum over j <= row_pos[r] of softmax((q_lat . c_j +
  *     q_rot . rot_j) * scale) c_j, with q_lat (rows, heads, kv_rank) = q . W_uk and q_rot read from q.
  *     max_len bounds row_pos + 1 and sizes the grid.  window > 0: only the keys j > row_pos[r] - window take part.
- *     sink (heads) or NULL: exp(sink_h) joins the denominator.  kv_heads > 1 (then rot_dim = 0): the row holds kv_heads
- *     parts of kv_rank elements, query head h reads part h / (heads / kv_heads).  key_scale != 0: a page ends, behind
- *     its rows, with page_tokens fp32 factors of its rows' scores.  workspace_bytes takes the heads per part.
+ *     sink (heads) or NULL: exp(sink_h) joins the denominator.  kv_heads > 1 (then rot_dim = 0): a page is (kv_heads,
+ *     page_tokens, kv_rank), query head h reads the rows of head h / (heads / kv_heads).  key_scale != 0: a page ends, behind
+ *     its rows, with page_tokens fp32 factors of its tokens' scores.  workspace_bytes takes the heads per part.
  *   latent_gather: rows first .. first + n - 1 of one sequence's pages, contiguous.
  *   latent_prefill: the expanded form for n rows of ONE sequence at positions start .. start + n - 1: q (n, q_ld)
  *     rotated, k (skv, heads * dim) and v (skv, heads * vdim) expanded from the latents of positions 0 .. skv - 1
@@ -540,12 +540,12 @@ int axb200_latent_prefill(const void *q, int64_t q_ld, const void *k, const void
                           int rot_dim, int vdim, int window, float scale, int dtype, void *stream);
 
 /* ---- grouped attention whose values are the raw keys ------------------------------------------------------
- * A page holds page_tokens rows of kv_heads parts of dim raw key elements and, behind them, page_tokens fp32 factors,
- * 1 / rms of all raw elements of a row: factor * part * k_w is the normed key, the part itself the value.
- *   shared_kv_prepare: per row q_out (rows, heads * dim) = rms_norm(q) * q_w * (k_w of the head's part), the norm over
+ * A page holds (kv_heads, page_tokens, dim) raw key elements and, behind them, page_tokens fp32 factors, 1 / rms of all
+ * raw elements of a token: factor * row * k_w is the normed key, the row itself the value.
+ *   shared_kv_prepare: per row q_out (rows, heads * dim) = rms_norm(q) * q_w * (k_w of the head's row), the norm over
  *     all heads at once, and the append of the raw keys and their factor.  latent_attend with kv_rank = dim, kv_heads
  *     and key_scale set then is the attention.
- *   shared_kv_gather: rows first .. first + n - 1 of one sequence as keys (part * factor) and values (part), both (n,
+ *   shared_kv_gather: rows first .. first + n - 1 of one sequence as keys (row * factor) and values (row), both (n,
  *     kv_heads * dim), for latent_prefill. */
 int axb200_shared_kv_prepare(const void *q, int64_t q_ld, const void *q_w, void *q_out, const void *k, int64_t k_ld,
                              const void *k_w, float eps, void *pages, const int32_t *block_table,
