@@ -152,12 +152,16 @@ __device__ __forceinline__ bool mbar_wait_bounded(uint64_t *bar, uint32_t parity
                                                   volatile int *abort_flag,
                                                   unsigned long long limit_ns = kWaitNanos) {
   if (mbar_try_wait(bar, parity)) return true;
-  const unsigned long long t0 = global_timer_ns();
+  unsigned long long t0 = 0;  // taken after the first spins: short waits do not pay for reading the timer
   for (uint32_t spin = 1;; ++spin) {
     if (mbar_try_wait(bar, parity)) return true;
     if ((spin & 255u) == 0u) {
       if (*abort_flag) return false;
-      if (global_timer_ns() - t0 > limit_ns) break;
+      const unsigned long long now = global_timer_ns();
+      if (t0 == 0)
+        t0 = now;
+      else if (now - t0 > limit_ns)
+        break;
     }
   }
   *abort_flag = 1;

@@ -19,7 +19,8 @@
 // graph stays balanced as the cache grows.  An item that lies in one range is finished there; otherwise every range
 // leaves an un-normalised record, and the merge kernel adds them up.
 //
-// Warps 0-3: softmax, queries into shared memory, results; warp 4: MMAs; one lane of warp 5: TMA.  The staged chunks
+// Warps 0-3: softmax, queries into shared memory, results; warps 4 and 6: the products of the scores and of the sum (one
+// warp's issue of small products, not the tensor core, would set the pace of both); one lane of warp 5: TMA.  The staged chunks
 // (128 keys x 64 elements) lie in rings: pairs of chunks that hold latent elements, freed when their part of the sum
 // is done, and single chunks with the rest of the row (the rotated part), freed after the scores.  Every wait is
 // bounded.
@@ -33,7 +34,7 @@ namespace axb {
 namespace {
 
 constexpr int kKeys = 128, kChunk = kKeys * 128;  // bytes of a chunk
-constexpr int kThreads = 192, kMmaWarp = 4, kLoadWarp = 5, kSoftmax = 128;
+constexpr int kThreads = 224, kMmaWarp = 4, kLoadWarp = 5, kSumWarp = 6, kSoftmax = 128;
 constexpr int kMaxRows = 1024, kMinTiles = 2, kMaxCtas = 256, kMaxSlots = 8;
 constexpr float kLog2e = 1.4426950408889634f, kLazy = 8.0f;
 
@@ -44,8 +45,7 @@ struct UmmaAttend {
   int pairs, singles;            // per tile
   int pair_slots, single_slots;  // in the rings
   int chunks;                    // per row: ceil(elements / 64)
-  int ahead;                     // the rings hold two tiles: a tile's scores are computed before the sum of the one before
-  int p_slots;                   // buffers of P: two where there is room ahead
+  int p_slots;                   // buffers of P: two where the rings hold two tiles, so that scores run ahead of sums
   float *part_o;                 // (2 * CTAs, N, kv_rank)
   float2 *part_ml;               // (2 * CTAs, N): reference (log2 domain), sum
 };
@@ -163,6 +163,10 @@ __device__ __forceinline__ void load_refs(const float *ref, float (&v)[kN]) {
   }
 }
 
+// fp32 accumulators, bf16 operands, M = 128, N = kN
+template <int kN>
+constexpr uint32_t kIdesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(kN >> 3) << 17) | ((128u >> 4) << 24);
+
 template <int kN>
 struct Smem {
   static constexpr int kP = kN * kKeys * 2;
@@ -189,7 +193,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
   const AttendParams &p = u.a;
   uint64_t *full_p = reinterpret_cast<uint64_t *>(smem + S::off_bar(u)), *empty_p = full_p + kMaxSlots;
   uint64_t *full_s = empty_p + kMaxSlots, *empty_s = full_s + kMaxSlots;
-  uint64_t *bar_s = empty_s + kMaxSlots, *bar_o = bar_s + 2, *bar_p = bar_o + 2, *bar_q = bar_p + 1;
+  uint64_t *bar_s = empty_s + kMaxSlots, *bar_o = bar_s + 2, *bar_p = bar_o + 2, *bar_q = bar_p + 2;
   uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(bar_q + 1);
   volatile int *abort_flag = reinterpret_cast<volatile int *>(bar_q + 2);
   int *start = reinterpret_cast<int *>(smem + S::off_start(u));
@@ -200,7 +204,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
   const int warp = uniform_warp(), lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     for (int i = 0; i < 4 * kMaxSlots + 4; ++i) mbar_init(&full_p[i], 1);  // rings, bar_s and bar_o
-    mbar_init(bar_p, 4);
+    mbar_init(&bar_p[0], 4);
+    mbar_init(&bar_p[1], 4);
     mbar_init(bar_q, 4);
     *abort_flag = 0;
     mbar_fence_init();
@@ -299,53 +304,56 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
       }
     }
   } else if (warp == kMmaWarp) {
-    // ================= MMA (the warp walks, one lane issues) =================
+    // ================= products of the scores (the warp walks, one lane issues) =================
     const uint32_t lead = lane == 0;
-    constexpr uint32_t kBf16 = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(kN >> 3) << 17) | ((128u >> 4) << 24);
-    constexpr uint32_t idesc_s = kBf16, idesc_o = kBf16 | (1u << 15);  // A K-major; A MN-major
-    const uint64_t da = smem_desc(smem_u32(smem), 16, 1024);           // a chunk as [keys][elements]
-    const uint64_t dv = smem_desc(smem_u32(smem), kChunk, 1024);       // a pair as latent elements x keys
-    const uint64_t dq = smem_desc(smem_u32(smem + S::off_q(u)), 16, 1024), dp = smem_desc(smem_u32(smem + S::off_p(u)), 16, 1024);
-    RingPos rp, rs, pv;  // pairs and singles of the scores, pairs of the sum
-    int r_s = r_first, g_s = lo, tile_s = 0, seg = 0;
-    auto scores = [&]() -> bool {  // of tile g_s
-      while (start[r_s + 1] <= g_s) ++r_s;
-      if (g_s == lo || g_s == start[r_s]) {  // a new item: its queries are in place
-        if (!mbar_wait_warp(bar_q, seg & 1, abort_flag, p.wait_ns)) return false;
+    constexpr uint32_t idesc = kIdesc<kN>;                                // A K-major
+    const uint64_t da = smem_desc(smem_u32(smem), 16, 1024);             // a chunk as [keys][elements]
+    const uint64_t dq = smem_desc(smem_u32(smem + S::off_q(u)), 16, 1024);
+    RingPos rp, rs;
+    bool ok = true;
+    for (int r = r_first, g = lo, tile = 0, seg = 0; g < hi && ok; ++g, ++tile) {
+      while (start[r + 1] <= g) ++r;
+      if (g == lo || g == start[r]) {  // a new item: its queries are in place
+        ok = mbar_wait_warp(bar_q, seg & 1, abort_flag, p.wait_ns);
         ++seg;
       }
-      const uint32_t ts = tmem + (tile_s & 1) * kN;
+      // the scores two tiles back have been read
+      if (tile >= 2) ok = ok && mbar_wait_warp(&bar_p[tile & 1], ((tile - 2) >> 1) & 1, abort_flag, p.wait_ns);
+      const uint32_t ts = tmem + (tile & 1) * kN;
       bool first = true;
       auto score_chunk = [&](int offset, int c) {
         const uint64_t a = da + (uint64_t)(offset >> 4), b = dq + (uint64_t)(c * (S::kQBox >> 4));
 #pragma unroll
-        for (int ks = 0; ks < 4; ++ks) umma_f16_lead(ts, a + ks * 2, b + ks * 2, idesc_s, !first || ks > 0, lead);
+        for (int ks = 0; ks < 4; ++ks) umma_f16_lead(ts, a + ks * 2, b + ks * 2, idesc, !first || ks > 0, lead);
         first = false;
       };
-      for (int i = 0; i < u.singles; ++i, rs.next(u.single_slots)) {
+      for (int i = 0; i < u.singles && ok; ++i, rs.next(u.single_slots)) {
         const int s = rs.slot;
-        if (!mbar_wait_warp(&full_s[s], rs.parity, abort_flag, p.wait_ns)) return false;
+        ok = mbar_wait_warp(&full_s[s], rs.parity, abort_flag, p.wait_ns);
+        if (!ok) break;
         tc_fence_after();
         score_chunk(off_single + s * kChunk, 2 * u.pairs + i);
         umma_commit_lead(&empty_s[s], lead);
       }
-      for (int i = 0; i < u.pairs; ++i, rp.next(u.pair_slots)) {
+      for (int i = 0; i < u.pairs && ok; ++i, rp.next(u.pair_slots)) {
         const int s = rp.slot;
-        if (!mbar_wait_warp(&full_p[s], rp.parity, abort_flag, p.wait_ns)) return false;
+        ok = mbar_wait_warp(&full_p[s], rp.parity, abort_flag, p.wait_ns);
+        if (!ok) break;
         tc_fence_after();
         for (int c = 0; c < 2 && 2 * i + c < u.chunks; ++c) score_chunk(s * 2 * kChunk + c * kChunk, 2 * i + c);
       }
-      umma_commit_lead(&bar_s[tile_s & 1], lead);
-      ++g_s;
-      ++tile_s;
-      return true;
-    };
-    bool ok = scores();
-    for (int r = r_first, g = lo, tile = 0; g < hi && ok; ++g, ++tile) {
+      if (ok) umma_commit_lead(&bar_s[tile & 1], lead);
+    }
+  } else if (warp == kSumWarp) {
+    // ================= products of the sum =================
+    const uint32_t lead = lane == 0;
+    constexpr uint32_t idesc = kIdesc<kN> | (1u << 15);             // A MN-major
+    const uint64_t dv = smem_desc(smem_u32(smem), kChunk, 1024);    // a pair as latent elements x keys
+    const uint64_t dp = smem_desc(smem_u32(smem + S::off_p(u)), 16, 1024);
+    RingPos pv;
+    for (int r = r_first, g = lo, tile = 0; g < hi; ++g, ++tile) {
       while (start[r + 1] <= g) ++r;
-      if (u.ahead && g_s < hi) ok = scores();
-      ok = ok && mbar_wait_warp(bar_p, tile & 1, abort_flag, p.wait_ns);
-      if (!ok) break;
+      if (!mbar_wait_warp(&bar_p[tile & 1], (tile >> 1) & 1, abort_flag, p.wait_ns)) break;
       tc_fence_after();
       const bool fresh = g == lo || g == start[r];
       const uint64_t dpt = dp + (uint64_t)((u.p_slots == 2 ? tile & 1 : 0) * (S::kP >> 4));
@@ -355,11 +363,10 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
 #pragma unroll
         for (int ks = 0; ks < kKeys / 16; ++ks)  // 16 keys: 2 KB of the chunk, 32 bytes of P
           umma_f16_lead(tmem_o + i * kN, a + (uint64_t)(ks * (2048 >> 4)),
-                        dpt + (uint64_t)(((ks >> 2) * (kN * 128) + (ks & 3) * 32) >> 4), idesc_o, !fresh || ks > 0, lead);
+                        dpt + (uint64_t)(((ks >> 2) * (kN * 128) + (ks & 3) * 32) >> 4), idesc, !fresh || ks > 0, lead);
         umma_commit_lead(&empty_p[s], lead);
       }
       umma_commit_lead(&bar_o[tile & 1], lead);
-      if (!u.ahead && g_s < hi) ok = scores();
     }
   } else {
     // ================= softmax warps: thread = key of the tile =================
@@ -490,7 +497,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap tmPages, const __grid_con
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
         tc_fence_before();
         __syncwarp();
-        if (lane == 0) mbar_arrive(bar_p);
+        if (lane == 0) mbar_arrive(&bar_p[tile & 1]);
       }
       if (!ok) break;
       // The scores of the item's last tile are done (bar_s), so its queries may be replaced: the next item's first
@@ -631,8 +638,7 @@ bool layout(UmmaAttend &u) {
     ++u.single_slots;
     if (Smem<kN>::bytes(u, kMaxRows) > kSmemLimit) --u.single_slots;
   }
-  u.ahead = u.pair_slots >= 2 * u.pairs && u.single_slots >= 2 * u.singles;
-  if (u.ahead) {
+  if (u.pair_slots >= 2 * u.pairs && u.single_slots >= 2 * u.singles) {
     UmmaAttend two = u;
     two.p_slots = 2;
     while (Smem<kN>::bytes(two, kMaxRows) > kSmemLimit && two.pair_slots > 2 * u.pairs) --two.pair_slots;
