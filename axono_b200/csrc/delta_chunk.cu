@@ -15,9 +15,10 @@
 // The products chain in registers: S (keys x 8 values) is the accumulator of the update and, transposed in the register
 // file (movmatrix), operand B of the next chunk's products; X and U likewise.  So the recurrence touches no shared memory.
 // Keys, queries, T and P are operand A and come as ready-made, swizzled tiles by bulk copies, some chunks ahead.
-// The walk is bound by the length of this chain, not by the tensor cores of a whole SM: the chain of 64 tokens is 250
-// warp-wide products of 16 x 8 x 16 at about ten cycles each.  Products of tcgen05 size would need 64 or more columns and
-// four round trips through tensor and shared memory per chunk, which together take longer.
+// The walk is bound by the length of this chain, not by the tensor cores of a whole SM: 64 tokens take 250 warp-wide
+// products of 16 x 8 x 16 at about ten cycles each, of which the 94 of the read-out (q S + P U) move to a second warp that
+// gets S and U through shared memory.  Products of tcgen05 size would need 64 or more columns and four round trips
+// through tensor and shared memory per chunk, which together take longer.
 #include <math.h>
 
 #include <mutex>
@@ -370,10 +371,14 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
 // ---- the walk over a sequence's chunks ------------------------------------------------------------------
 template <int kDK, int kWarps>
 struct ScanSmem {
+  static constexpr bool kSplit = kWarps <= 4;  // a second warp per 8 columns for the read-out
   static constexpr int kTile = kC * kDK * 2;
   static constexpr int kOffHead = 2 * kTile, kOffValues = kOffHead + kHeadTiles, kStage = kOffValues + kWarps * kValueTile;
-  static constexpr int kStages = 4 * kStage + 256 <= 227 * 1024 ? 4 : 3;
-  static constexpr int kOffBar = kStages * kStage, kBytes = kOffBar + 256;
+  static constexpr int kState = kDK / 16 * 512, kHandOver = kSplit ? kState + 4 * 512 : 0;  // S as operands B, U as accumulators
+  static constexpr int kRest = kWarps * kHandOver + 512;
+  static constexpr int kStages = 4 * kStage + kRest <= 227 * 1024 ? 4 : 3;
+  static constexpr int kOffHand = kStages * kStage, kOffBar = kOffHand + kWarps * kHandOver, kBytes = kOffBar + 512;
+  static constexpr int kThreads = ((kSplit ? 2 : 1) * kWarps + 1) * 32;
 };
 
 // An 8 x 8 matrix of 16-bit elements, a row's pairs in four lanes, transposed.
@@ -425,21 +430,62 @@ struct ScanParams {
   unsigned long long wait_ns;
 };
 
+// One chunk's o = e^G q S + P u of 8 columns; S comes as operands B tile by tile (state(k, high, low)), u when it is ready.
+template <int kDK, typename State, typename Update>
+__device__ __forceinline__ void read_out(const ScanParams &p, uint32_t cq, uint32_t tiles, const float *vec, int lane, int valid,
+                                         __nv_bfloat16 *dst, State state, Update update) {
+  constexpr int kPieces = kDK / 8;
+  const int g = lane >> 2;
+  float o[4][4] = {};
+#pragma unroll
+  for (int k = 0; k < kDK / 16; ++k) {
+    uint32_t high[2], low[2], b[4][4];
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+      ldmatrix_x4(b[m][0], b[m][1], b[m][2], b[m][3], cq + tile_at(16 * m + (lane & 15), 2 * k + (lane >> 4), kPieces));
+    state(k, high, low);
+#pragma unroll
+    for (int m = 0; m < 4; ++m) mma_16816_bf16(o[m], b[m], high[0], high[1]);
+#pragma unroll
+    for (int m = 0; m < 4; ++m) mma_16816_bf16(o[m], b[m], low[0], low[1]);
+  }
+  float u[4][4];
+  update(u);
+  uint32_t high[4][2], low[4][2];
+#pragma unroll
+  for (int m = 0; m < 4; ++m) {
+    const float e0 = vec[kC + 16 * m + g], e1 = vec[kC + 16 * m + g + 8];
+    o[m][0] *= e0, o[m][1] *= e0, o[m][2] *= e1, o[m][3] *= e1;
+    split_operand(u[m], high[m], low[m]);
+  }
+  triangular_product(o, tiles + 2 * kSquare, tiles + 3 * kSquare, high, low, lane);
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = 16 * m + g + 8 * i;
+      if (t < valid) *reinterpret_cast<uint32_t *>(dst + (int64_t)t * p.heads * p.vdim) = pack_bf16x2(o[m][2 * i], o[m][2 * i + 1]);
+    }
+}
+
 template <int kDK, int kWarps>
-__global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(const ScanParams p) {
+__global__ void __launch_bounds__(ScanSmem<kDK, kWarps>::kThreads, 1) delta_chunk_scan_kernel(const ScanParams p) {
   using L = ScanSmem<kDK, kWarps>;
   constexpr int kPieces = kDK / 8, kKeyTiles = kDK / 16;  // 16-high tiles of S
+  constexpr int kProducer = (L::kSplit ? 2 : 1) * kWarps;
   extern __shared__ __align__(128) uint8_t smem[];
   uint64_t *full = reinterpret_cast<uint64_t *>(smem + L::kOffBar), *empty = full + L::kStages;
-  volatile int *abort_flag = reinterpret_cast<volatile int *>(empty + L::kStages);
+  uint64_t *s_full = empty + L::kStages, *s_empty = s_full + kWarps, *u_full = s_empty + kWarps, *u_empty = u_full + kWarps;
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(u_empty + kWarps);
   const int warp = __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0), lane = threadIdx.x & 31;
   const int h = blockIdx.y, hk = h / (p.heads / p.kv_heads), blocks = p.vdim / 8, block0 = blockIdx.z * kWarps;
   const int warps = min(kWarps, blocks - block0);  // with columns of their own
   if (threadIdx.x == 0) {
     for (int i = 0; i < L::kStages; ++i) {
       mbar_init(&full[i], 1);
-      mbar_init(&empty[i], warps);
+      mbar_init(&empty[i], (L::kSplit ? 2 : 1) * warps);
     }
+    for (int i = 0; i < 4 * kWarps; ++i) mbar_init(&s_full[i], 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -454,7 +500,7 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(
   const int chunks = (portion.z + kC - 1) / kC;
   const size_t chunk0 = first_chunk(portion, blockIdx.x, p.first);
 
-  if (warp == kWarps) {
+  if (warp == kProducer) {
     if (lane == 0) {
       bool ok = true;
       int n = 0;
@@ -478,10 +524,49 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(
     }
     return;
   }
-  if (warp >= warps) return;
+  const int w = warp % kWarps;
+  if (w >= warps) return;
+  auto wait = [&](uint64_t *bar, int phase) { return __all_sync(0xffffffffu, mbar_wait_bounded(bar, phase & 1, abort_flag, p.wait_ns)); };
+  auto release = [&](uint64_t *bar) {
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar);
+  };
+  const int g = lane >> 2, v0 = (block0 + w) * 8 + (lane & 3) * 2;
+  auto rows_of = [&](int n) { return p.out + ((int64_t)(portion.y - p.first + n * kC) * p.heads + h) * p.vdim + v0; };
+  uint4 *hand_s = reinterpret_cast<uint4 *>(smem + L::kOffHand + w * L::kHandOver) + lane;
+  float4 *hand_u = reinterpret_cast<float4 *>(smem + L::kOffHand + w * L::kHandOver + L::kState) + lane;
 
-  // S: tile j holds keys 16j .. 16j + 15 (rows lane / 4 and + 8), 8 value columns ((lane % 4) * 2 and + 1)
-  const int g = lane >> 2, v0 = (block0 + warp) * 8 + (lane & 3) * 2;
+  if (L::kSplit && warp >= kWarps) {
+    // ---- the read-out ----
+    for (int n = 0; n < chunks; ++n) {
+      const int s = n % L::kStages;
+      if (!wait(&full[s], n / L::kStages) || !wait(&s_full[w], n)) return;
+      const uint32_t base = smem_u32(smem + s * L::kStage);
+      bool ok = true;
+      read_out<kDK>(
+          p, base + L::kTile, base + L::kOffHead, reinterpret_cast<const float *>(smem + s * L::kStage + L::kOffHead + kVec), lane,
+          portion.z - n * kC, rows_of(n),
+          [&](int k, uint32_t(&high)[2], uint32_t(&low)[2]) {
+            const uint4 v = hand_s[k * 32];
+            high[0] = v.x, high[1] = v.y, low[0] = v.z, low[1] = v.w;
+          },
+          [&](float(&u)[4][4]) {
+            release(&s_empty[w]);
+            ok = wait(&u_full[w], n);
+#pragma unroll
+            for (int m = 0; m < 4; ++m) {
+              const float4 v = hand_u[m * 32];
+              u[m][0] = v.x, u[m][1] = v.y, u[m][2] = v.z, u[m][3] = v.w;
+            }
+            release(&u_empty[w]);
+          });
+      if (!ok) return;
+      release(&empty[s]);
+    }
+    return;
+  }
+
+  // ---- the chain.  S: tile j holds keys 16j .. 16j + 15 (rows lane / 4 and + 8), 8 value columns ((lane % 4) * 2 and + 1) ----
   float *state = p.state + ((size_t)portion.x * p.heads + h) * p.dim * p.vdim;
   float st[kKeyTiles][4];
 #pragma unroll
@@ -496,33 +581,32 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(
 
   for (int n = 0; n < chunks; ++n) {
     const int s = n % L::kStages;
-    if (!__all_sync(0xffffffffu, mbar_wait_bounded(&full[s], (n / L::kStages) & 1, abort_flag, p.wait_ns))) return;
-    const uint32_t base = smem_u32(smem + s * L::kStage), ck = base, cq = base + L::kTile, tiles = base + L::kOffHead;
+    uint32_t sh[kKeyTiles][2], sl[kKeyTiles][2];
+#pragma unroll
+    for (int k = 0; k < kKeyTiles; ++k) split_operand(st[k], sh[k], sl[k]);
+    if (L::kSplit) {
+      if (n > 0 && !wait(&s_empty[w], n - 1)) return;
+#pragma unroll
+      for (int k = 0; k < kKeyTiles; ++k) hand_s[k * 32] = make_uint4(sh[k][0], sh[k][1], sl[k][0], sl[k][1]);
+      release(&s_full[w]);
+    }
+    if (!wait(&full[s], n / L::kStages)) return;
+    const uint32_t base = smem_u32(smem + s * L::kStage), ck = base, tiles = base + L::kOffHead;
     const float *vec = reinterpret_cast<const float *>(smem + s * L::kStage + L::kOffHead + kVec);
-    const uint8_t *value = smem + s * L::kStage + L::kOffValues + warp * kValueTile + (lane & 3) * 4;
+    const uint8_t *value = smem + s * L::kStage + L::kOffValues + w * kValueTile + (lane & 3) * 4;
 
-    // k S and q S of all tokens
-    float x[4][4] = {}, o[4][4] = {};
+    // k S of all tokens
+    float x[4][4] = {};
 #pragma unroll
     for (int k = 0; k < kKeyTiles; ++k) {
-      uint32_t high[2], low[2], a[4][4], b[4][4];
+      uint32_t a[4][4];
 #pragma unroll
-      for (int m = 0; m < 4; ++m) {
-        const uint32_t at = tile_at(16 * m + (lane & 15), 2 * k + (lane >> 4), kPieces);
-        ldmatrix_x4(a[m][0], a[m][1], a[m][2], a[m][3], ck + at);
-        ldmatrix_x4(b[m][0], b[m][1], b[m][2], b[m][3], cq + at);
-      }
-      split_operand(st[k], high, low);
+      for (int m = 0; m < 4; ++m)
+        ldmatrix_x4(a[m][0], a[m][1], a[m][2], a[m][3], ck + tile_at(16 * m + (lane & 15), 2 * k + (lane >> 4), kPieces));
 #pragma unroll
-      for (int m = 0; m < 4; ++m) {
-        mma_16816_bf16(x[m], a[m], high[0], high[1]);
-        mma_16816_bf16(o[m], b[m], high[0], high[1]);
-      }
+      for (int m = 0; m < 4; ++m) mma_16816_bf16(x[m], a[m], sh[k][0], sh[k][1]);
 #pragma unroll
-      for (int m = 0; m < 4; ++m) {
-        mma_16816_bf16(x[m], a[m], low[0], low[1]);
-        mma_16816_bf16(o[m], b[m], low[0], low[1]);
-      }
+      for (int m = 0; m < 4; ++m) mma_16816_bf16(x[m], a[m], sl[k][0], sl[k][1]);
     }
     // X = v - e^G k S
     uint32_t high[4][2], low[4][2];
@@ -540,6 +624,12 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(
     }
     float u[4][4] = {};
     triangular_product(u, tiles, tiles + kSquare, high, low, lane);
+    if (L::kSplit) {
+      if (n > 0 && !wait(&u_empty[w], n - 1)) return;
+#pragma unroll
+      for (int m = 0; m < 4; ++m) hand_u[m * 32] = make_float4(u[m][0], u[m][1], u[m][2], u[m][3]);
+      release(&u_full[w]);
+    }
     // S' = e^G_64 S + k^T (e^{G_64 - G} u)
     const float total = vec[3 * kC];
 #pragma unroll
@@ -549,37 +639,31 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 1) delta_chunk_scan_kernel(
 #pragma unroll
     for (int m = 0; m < 4; ++m) {
       const float e0 = vec[2 * kC + 16 * m + g], e1 = vec[2 * kC + 16 * m + g + 8];
-      const float w[4] = {e0 * u[m][0], e0 * u[m][1], e1 * u[m][2], e1 * u[m][3]};
+      const float wu[4] = {e0 * u[m][0], e0 * u[m][1], e1 * u[m][2], e1 * u[m][3]};
       uint32_t wh[2], wl[2], a[kKeyTiles][4];
 #pragma unroll
       for (int j = 0; j < kKeyTiles; ++j)
         ldmatrix_x4_trans(a[j][0], a[j][1], a[j][2], a[j][3],
                           ck + tile_at(16 * m + ((lane >> 4) & 1) * 8 + (lane & 7), 2 * j + ((lane >> 3) & 1), kPieces));
-      split_operand(w, wh, wl);
+      split_operand(wu, wh, wl);
 #pragma unroll
       for (int j = 0; j < kKeyTiles; ++j) mma_16816_bf16(st[j], a[j], wh[0], wh[1]);
 #pragma unroll
       for (int j = 0; j < kKeyTiles; ++j) mma_16816_bf16(st[j], a[j], wl[0], wl[1]);
     }
-    // o = e^G q S + P u
+    if (!L::kSplit)
+      read_out<kDK>(
+          p, base + L::kTile, tiles, vec, lane, portion.z - n * kC, rows_of(n),
+          [&](int k, uint32_t(&high)[2], uint32_t(&low)[2]) {
+            high[0] = sh[k][0], high[1] = sh[k][1], low[0] = sl[k][0], low[1] = sl[k][1];
+          },
+          [&](float(&out)[4][4]) {
 #pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      const float e0 = vec[kC + 16 * m + g], e1 = vec[kC + 16 * m + g + 8];
-      o[m][0] *= e0, o[m][1] *= e0, o[m][2] *= e1, o[m][3] *= e1;
-      split_operand(u[m], high[m], low[m]);
-    }
-    triangular_product(o, tiles + 2 * kSquare, tiles + 3 * kSquare, high, low, lane);
-    __syncwarp();
-    if (lane == 0) mbar_arrive(&empty[s]);
-    const int valid = portion.z - n * kC;
-    __nv_bfloat16 *dst = p.out + ((int64_t)(portion.y - p.first + n * kC) * p.heads + h) * p.vdim + v0;
+            for (int m = 0; m < 4; ++m)
 #pragma unroll
-    for (int m = 0; m < 4; ++m)
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = 16 * m + g + 8 * i;
-        if (t < valid) *reinterpret_cast<uint32_t *>(dst + (int64_t)t * p.heads * p.vdim) = pack_bf16x2(o[m][2 * i], o[m][2 * i + 1]);
-      }
+              for (int e = 0; e < 4; ++e) out[m][e] = u[m][e];
+          });
+    release(&empty[s]);
   }
 #pragma unroll
   for (int j = 0; j < kKeyTiles; ++j)
@@ -611,7 +695,7 @@ int run_scan(const ScanParams &p, int count, cudaStream_t st) {
   if (int rc = opt_in<delta_chunk_scan_kernel<kDK, kWarps>>(L::kBytes)) return rc;
   const int blocks = p.vdim / 8;
   return launch_dependent(delta_chunk_scan_kernel<kDK, kWarps>, dim3(count, p.heads, (blocks + kWarps - 1) / kWarps),
-                          dim3((kWarps + 1) * 32), (size_t)L::kBytes, st, p);
+                          dim3(L::kThreads), (size_t)L::kBytes, st, p);
 }
 
 template <int kDK>
