@@ -1,5 +1,8 @@
 """What the tests of the language models share: random tensors, a paged cache filled by hand, comparisons, and feeding a
-runner in portions."""
+runner in portions, and writing model folders."""
+import json
+import struct
+
 import numpy as np
 import torch
 
@@ -68,3 +71,15 @@ def position_errors(got, want):
     d -= d.mean(-1, keepdims=True)
     w = want - want.mean(-1, keepdims=True)
     return np.sqrt((d * d).mean(-1)) / np.sqrt((w * w).mean())
+
+
+def write_safetensors(path, tensors, extra_header=None):
+    names = {torch.bfloat16: "BF16", torch.float32: "F32", torch.int32: "I32"}
+    header, data = dict(extra_header or {}), b""
+    for k, t in tensors.items():
+        raw = t.contiguous().view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        header[k] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [len(data), len(data) + len(raw)]}
+        data += raw
+    head = json.dumps(header).encode()
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(head)) + head + data)

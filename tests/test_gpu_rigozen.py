@@ -1,14 +1,20 @@
 """The Rigozen model on the GPU against the plain CPU evaluation (tests/plain_rigozen.py): whole prompts, token by token,
 portions, batches, pages and slots used again, and generation through the scheduler."""
+import json
+import os
+import subprocess
+import sys
+
 import numpy as np
 import pytest
 import torch
 
 import plain_rigozen as plain
 import rigozen_cases as cases
-from lm_helpers import SCHEDULES, feed, position_errors, runner_of
+from lm_helpers import SCHEDULES, feed, position_errors, runner_of, write_safetensors
 
 pytestmark = pytest.mark.gpu
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 F32_TOL = 3e-5
 DTYPES = [torch.float32, torch.bfloat16]
@@ -193,3 +199,30 @@ def test_long_decoding_by_graph(built, dtype):
         # a tie within rounding may go either way: the decoded token must be (nearly) the largest logit
         gap = max(float(logits[i].max() - logits[i, t]) for i, t in enumerate(out)) / float(logits.std())
         assert gap <= (2e-4 if dtype == torch.float32 else 0.3), gap
+
+
+def test_command_lines_on_a_model_folder(built, tmp_path):
+    """A folder with config.json and model.safetensors through the generation command line and the trace runner."""
+    cfg, w, tokens, ref = built("odd", 150)
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    write_safetensors(str(tmp_path / "model.safetensors"), w)
+    wd = {k: v.double() for k, v in w.items()}
+    prompts = [tokens[:6], tokens[40:61]]
+    cmd = [sys.executable, "-m", "axono_b200.generate", "--model", str(tmp_path), "--dtype", "float32", "--max-new", "8"]
+    for p in prompts:
+        cmd += ["--tokens", ",".join(map(str, p))]
+    out = subprocess.run(cmd, capture_output=True, text=True, timeout=600, cwd=ROOT)
+    assert out.returncode == 0, out.stderr
+    assert [[int(t) for t in line.split()] for line in out.stdout.splitlines()] == [plain.greedy(cfg, wd, p, 8) for p in prompts]
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": tokens[:31], "want": [0, 30]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": tokens[31:33], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "a", "tokens": tokens[33:80], "want": [46]}, {"id": "b", "tokens": tokens[:1], "want": [0]}], "end": ["a", "b"]},
+             {"step": 3, "entries": [{"id": "a", "tokens": tokens[:2], "want": [1]}], "end": ["a"]}]
+    out = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", str(tmp_path), "--dtype", "float32", "--out", str(tmp_path),
+                          "--max-tokens", "160"], input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600)
+    assert out.returncode == 0, out.stderr
+    assert [line for line in out.stdout.splitlines() if line.startswith("done")] == [f"done {i}" for i in range(4)]
+    for step, places in ((0, [0, 30]), (2, [79, 0]), (3, [1])):
+        got = np.fromfile(tmp_path / f"{step}.f32", dtype="<f4").reshape(len(places), cfg["vocab"])
+        check(got, ref[places], torch.float32)
+    assert not (tmp_path / "1.f32").exists()

@@ -294,7 +294,8 @@ def run_delta(mixer, w, projs, steps, state, ring):
 
 
 DELTA_SIZES = [(6, 2, 20, 12, 3), (3, 3, 33, 7, 1), (4, 1, 72, 136, 4), (2, 2, 136, 40, 5), (8, 4, 128, 128, 4), (6, 2, 64, 96, 2),
-               (4, 4, 32, 64, 4), (2, 1, 256, 256, 3), (3, 1, 16, 300, 7)]
+               (4, 4, 32, 64, 4), (2, 1, 256, 256, 3), (3, 1, 16, 300, 7), (4, 2, 32, 64, 6), (9, 1, 64, 16, 4), (10, 2, 100, 8, 5),
+               (64, 16, 32, 128, 4)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)

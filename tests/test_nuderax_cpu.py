@@ -1,7 +1,6 @@
 """What of the language models needs no GPU: configuration, weights, the arena of rows, the scheduler, the command
 lines, and the plain evaluation against itself."""
 import copy
-import json
 import os
 import struct
 import subprocess
@@ -12,20 +11,9 @@ import torch
 
 import nuderax_cases as cases
 import plain_nuderax as plain
+from lm_helpers import write_safetensors
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-
-
-def write_safetensors(path, tensors, extra_header=None):
-    names = {torch.bfloat16: "BF16", torch.float32: "F32", torch.int32: "I32"}
-    header, data = dict(extra_header or {}), b""
-    for k, t in tensors.items():
-        raw = t.contiguous().view(torch.uint8).numpy().tobytes() if t.numel() else b""
-        header[k] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [len(data), len(data) + len(raw)]}
-        data += raw
-    head = json.dumps(header).encode()
-    with open(path, "wb") as f:
-        f.write(struct.pack("<Q", len(head)) + head + data)
 
 
 def test_safetensors_reader(tmp_path):
