@@ -117,7 +117,7 @@ SIGNATURES = {
     "axb200_delta_scan": (_i, [_vp, _i, _i] + [_vp] * 6 + [_i] * 6 + [_vp]),
     "axb200_delta_chunks_supported": (_i, [_i] * 3),
     "axb200_delta_chunks_workspace_bytes": (_sz, [_i64] + [_i] * 5),
-    "axb200_delta_chunks": (_i, [_vp, _i64, _vp, _vp, _vp, _i, _i] + [_vp] * 6 + [_i, _i, _vp] + [_i] * 7 + [_vp, _sz, _vp]),
+    "axb200_delta_chunks": (_i, [_vp, _i64, _i, _i] + [_vp] * 6 + [_i, _i, _vp] + [_i] * 7 + [_vp, _sz, _vp]),
     "axb200_delta_finish": (_i, [_vp, _i64, _vp, _vp, _vp, _i, _i] + [_vp] * 6 + [_vp] * 2 + [_i] * 6 + [_f, _i, _vp]),
     "axb200_moe_route": (_i, [_vp] * 6 + [_i64, _i, _i, _i, _i, _f, _vp]),
     "axb200_moe_tile_rows": (_i, [_i64, _i, _i, _i, _i]),
@@ -146,12 +146,12 @@ def library_path() -> str:
     return _path or _build.LIB
 
 
-def use_serving_library() -> str:
-    """For processes that serve a model: builds what they need if it is missing or stale (the full library when
+def use_serving_library(architecture: str, kernel_sources) -> str:
+    """For processes that serve one design: builds what they need if it is missing or stale (the full library when
     that is up to date) and makes it the one `lib()` loads.  Without effect once a library is loaded."""
     global _path
     if _lib is None:
-        _path = _build.build_serving()
+        _path = _build.build_serving(architecture, kernel_sources)
     return library_path()
 
 
@@ -166,7 +166,7 @@ def lib() -> C.CDLL:
                 "axono_b200 has no fallback path.")
         handle = C.CDLL(path)
         for name, (res, args) in SIGNATURES.items():
-            if path == _build.SERVING_LIB and not hasattr(handle, name):
+            if path != _build.LIB and not hasattr(handle, name):
                 continue  # the subset library has no such operator
             fn = getattr(handle, name)
             fn.restype = res

@@ -1,13 +1,13 @@
 """Builds the C-ABI library (axono_b200/lib/libaxono_b200.so) for sm_100a with nvcc, and the native
 Python module `libaxono` (host runtime + operator adapters + pybind11 binding) that links against it.
 
-    python -m axono_b200.build [--force] [--verbose] [--serving]
+    python -m axono_b200.build [--force] [--verbose] [--serving DESIGN]
 
 nvcc cross-compiles without a GPU; the library is kept in-tree so it travels with the
 source checkout.  Sources compile to objects side by side and only where a source or header is newer.
 
-`build_serving()` links the subset of the same objects that the language-model serving path calls into
-libaxono_b200_lm.so: a fresh checkout that only serves a model compiles that much and no more.
+`build_serving()` links the subset of the same objects that serving a language model calls into a library of its own
+(libaxono_b200_lm_<design>.so): a fresh checkout that only serves a model compiles that much and no more.
 """
 from __future__ import annotations
 
@@ -26,9 +26,9 @@ CSRC = os.path.join(PKG, "csrc")
 LIB_DIR = os.path.join(PKG, "lib")
 OBJ_DIR = os.path.join(LIB_DIR, "obj")
 LIB = os.path.join(LIB_DIR, "libaxono_b200.so")
-SERVING_LIB = os.path.join(LIB_DIR, "libaxono_b200_lm.so")
-SERVING_SOURCES = ("core.cu", "delta.cu", "delta_chunk.cu", "fused.cu", "kv_arena.cu", "latent_attn.cu", "latent_prefill.cu", "latent_umma.cu",
-                   "linear_lt.cpp", "moe.cu", "moe_umma.cu", "residual_norm.cu", "shared_kv.cu")
+# what serving any language model takes; a model class names the rest as `kernel_sources`
+SERVING_SOURCES = ("core.cu", "fused.cu", "kv_arena.cu", "latent_attn.cu", "latent_prefill.cu", "latent_umma.cu", "linear_lt.cpp",
+                   "residual_norm.cu")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -41,8 +41,8 @@ def sources():
     return sorted(glob.glob(os.path.join(CSRC, "*.cu")) + glob.glob(os.path.join(CSRC, "*.cpp")))
 
 
-def serving_sources():
-    return [os.path.join(CSRC, name) for name in SERVING_SOURCES]
+def serving_lib(architecture: str) -> str:
+    return os.path.join(LIB_DIR, f"libaxono_b200_lm_{architecture.lower()}.so")
 
 
 def _headers():
@@ -95,11 +95,12 @@ def build(force: bool = False, verbose: bool = False) -> str:
     return _link(LIB, sources(), force, verbose)
 
 
-def build_serving(force: bool = False, verbose: bool = False) -> str:
-    """The library a serving process loads: the full one when it is there and up to date, else the subset."""
+def build_serving(architecture: str, kernel_sources=(), force: bool = False, verbose: bool = False) -> str:
+    """The library a process that serves one design loads: the full one when it is there and up to date, else the subset."""
     if not force and not _newer(sources() + _headers(), LIB):
         return LIB
-    return _link(SERVING_LIB, serving_sources(), force, verbose)
+    srcs = [os.path.join(CSRC, name) for name in (*SERVING_SOURCES, *kernel_sources)]
+    return _link(serving_lib(architecture), srcs, force, verbose)
 
 
 HOST = os.path.join(CSRC, "host")
@@ -137,7 +138,10 @@ def build_native(force: bool = False) -> str:
 
 if __name__ == "__main__":
     if "--serving" in sys.argv:
-        print(build_serving(force="--force" in sys.argv, verbose="--verbose" in sys.argv))
+        from axono_b200.models import model_class
+
+        design = sys.argv[sys.argv.index("--serving") + 1]
+        print(build_serving(design, model_class(design).kernel_sources, "--force" in sys.argv, "--verbose" in sys.argv))
         sys.exit(0)
     print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv))
     print(build_native(force="--force" in sys.argv))

@@ -464,25 +464,29 @@ __global__ void __launch_bounds__(kFinishWarps * 32, 4)
 delta_finish_lanes_kernel(const DeltaParams<T> p, int first, const T *o, T *out) {
   constexpr int kVdim = 8 * kLanes, kAtOnce = kFinishWarps * 32 / kLanes, kDeep = 4;
   const int at = threadIdx.x % kLanes * 8;
-  const int64_t items = (int64_t)(p.rows - first) * p.heads, i0 = (int64_t)blockIdx.x * kAtOnce * kDeep;
+  const uint32_t items = (uint32_t)(p.rows - first) * p.heads, i0 = blockIdx.x * (kAtOnce * kDeep);
   grid_dependency_wait();
   grid_dependency_launch();
   uint4 y[kDeep], gate[kDeep];
 #pragma unroll
   for (int d = 0; d < kDeep; ++d) {
-    const int64_t i = i0 + d * kAtOnce + threadIdx.x / kLanes;
+    const uint32_t i = i0 + d * kAtOnce + threadIdx.x / kLanes;
     y[d] = gate[d] = make_uint4(0, 0, 0, 0);
     if (i < items) {
-      const int64_t r = i / p.heads;
-      y[d] = *reinterpret_cast<const uint4 *>(o + i * kVdim + at);
-      gate[d] = *reinterpret_cast<const uint4 *>(p.proj + (first + r) * p.ld + p.gate_at() + (i - r * p.heads) * kVdim + at);
+      const uint32_t r = i / (uint32_t)p.heads;
+      y[d] = *reinterpret_cast<const uint4 *>(o + (size_t)i * kVdim + at);
+      gate[d] = *reinterpret_cast<const uint4 *>(p.proj + (int64_t)(first + r) * p.ld + p.gate_at() + (size_t)(i - r * p.heads) * kVdim + at);
     }
   }
+  // the rows whose first head is among this CTA's: which of them the next step may look back at
+  const int r0 = first + (int)((i0 + p.heads - 1) / p.heads), r1 = min(p.rows, first + (int)((i0 + kAtOnce * kDeep + p.heads - 1) / p.heads));
+  const int mine = r0 + (int)threadIdx.x;
+  const bool files = __syncthreads_or(mine < r1 && (mine + p.taps >= p.rows || p.row_back[mine + p.taps] < p.taps));
   float w[8];
   load_vec<8>(p.norm + at, w);
 #pragma unroll
   for (int d = 0; d < kDeep; ++d) {
-    const int64_t i = i0 + d * kAtOnce + threadIdx.x / kLanes;
+    const uint32_t i = i0 + d * kAtOnce + threadIdx.x / kLanes;
     const T *ye = reinterpret_cast<const T *>(&y[d]), *ge = reinterpret_cast<const T *>(&gate[d]);
     float v[8], sq = 0.f;
 #pragma unroll
@@ -498,10 +502,10 @@ delta_finish_lanes_kernel(const DeltaParams<T> p, int first, const T *o, T *out)
       const float z = ldf(ge + e);
       v[e] = v[e] * inv * w[e] * __fdividef(z, 1.0f + __expf(-z));
     }
-    if (i < items) store_vec<8>(out + i * kVdim + at, v);
+    if (i < items) store_vec<8>(out + (size_t)i * kVdim + at, v);
   }
-  // the rows whose first head is among this CTA's
-  for (int64_t r = (i0 + p.heads - 1) / p.heads; r * p.heads < i0 + kAtOnce * kDeep && first + r < p.rows; ++r) file_inputs<T, 8>(p, first + r);
+  if (files)
+    for (int r = r0; r < r1; ++r) file_inputs<T, 8>(p, r);
 }
 
 // Any size: a warp per head.
@@ -602,7 +606,7 @@ int finish(const DeltaParams<T> &p, int first, const void *o, void *out, cudaStr
                             static_cast<T *>(out));
   };
   if constexpr (sizeof(T) == 2) {
-    if (vec && p.ld % 8 == 0 && p.channels() % 8 == 0) {
+    if (vec && p.ld % 8 == 0 && p.channels() % 8 == 0 && (int64_t)(p.rows - first) * p.heads < 0x7fff0000) {
       if (p.vdim == 64) return lanes(delta_finish_lanes_kernel<T, 8>);
       if (p.vdim == 128) return lanes(delta_finish_lanes_kernel<T, 16>);
       if (p.vdim == 256) return lanes(delta_finish_lanes_kernel<T, 32>);

@@ -4,9 +4,9 @@
 //     X_t = v_t - e^{G_t} S^T k_t,      (I + A) U = diag(beta) X,   A_ts = beta_t e^{G_t - G_s} (k_t . k_s), s < t,
 //     o_t = e^{G_t} S^T q_t + sum_{s <= t} P_ts u_s,                P_ts = e^{G_t - G_s} (q_t . k_s),
 //     S'  = e^{G_64} S + sum_s e^{G_64 - G_s} k_s u_s^T.
-// delta_chunk_prepare does what needs no state, all chunks at once: convolutions and silu, the products of queries and
-// keys, T = (I + A)^-1 diag(beta) by blocked forward substitution, P, and the scale vectors.  delta_chunk_scan walks a
-// sequence's chunks: a warp owns 8 value columns of a head's state and is independent of all others.
+// Two kernels do what needs no state, all chunks at once: delta_chunk_conv the convolutions and silu, into tiles;
+// delta_chunk_prepare the products of queries and keys, T = (I + A)^-1 diag(beta) by blocked forward substitution, P, and
+// the scale vectors.  delta_chunk_scan walks a sequence's chunks: a warp owns 8 value columns of a head's state and is independent of all others.
 //
 // Precision.  The outputs of the short convolutions are bf16, so they are exact tensor-core operands: unit norms and
 // decays stay outside the products, as fp32 factors of rows.  Everything else that enters a product - state, X, U, T, P -
@@ -44,6 +44,13 @@ __device__ __forceinline__ uint32_t block_at(int m, int k, int row, int piece) {
   return (uint32_t)((m * (m + 1) / 2 + k) * 512 + row * 32 + ((piece ^ ((row >> 2) & 1)) << 4));
 }
 
+// A chunk of one query / key head: the tiles of k and q as the convolutions put them out, and 1 / norm of their rows (of q
+// also / sqrt(dim)).
+template <int kDK>
+struct KeyTiles {
+  static constexpr int kTile = kC * kDK * 2, kOffInv = 2 * kTile, kBytes = kOffInv + 2 * kC * 4;
+};
+
 __device__ __forceinline__ float bf_lo(uint32_t v) { return __uint_as_float(v << 16); }
 __device__ __forceinline__ float bf_hi(uint32_t v) { return __uint_as_float(v & 0xffff0000u); }
 
@@ -62,16 +69,29 @@ constexpr int kPrepThreads = 256, kLd = kC + 8;  // fp32 matrices in shared memo
 // silu of what a convolution puts out (an activation that is rounded to bf16)
 __device__ __forceinline__ float fast_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 
-// Convolution and silu of four channels from c on over kCount tokens from t0 on of a chunk; put(t, values).
+// The inputs of four channels at token t of a portion: a row of this step, the ring, or zero before the sequence's start.
+__device__ __forceinline__ void portion_input(const DeltaParams<__nv_bfloat16> &p, const int4 &portion, int t, int c, float (&v)[4]) {
+  if (t >= 0) {
+    load_vec<4>(p.proj + (int64_t)(portion.y + t) * p.ld + c, v);
+  } else if (portion.w + t >= 0) {
+    load_vec<4>(p.ring + ((size_t)portion.x * p.taps + (portion.w + t) % p.taps) * p.channels() + c, v);
+  } else {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = 0.f;
+  }
+}
+
+// Convolution and silu of four channels from c on over kCount tokens from t0 on of a portion, of which `valid` are real;
+// put(i, values).
 template <int kCount, typename Put>
-__device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, int64_t row0, int valid, int c, int t0, Put put) {
+__device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, const int4 &portion, int t0, int valid, int c, Put put) {
   const int channels = p.channels();
   if (p.taps <= 4) {
     uint2 raw[kCount];  // all on their way at once
 #pragma unroll
     for (int i = 0; i < kCount; ++i) {
       raw[i] = make_uint2(0, 0);
-      if (t0 + i < valid) raw[i] = *reinterpret_cast<const uint2 *>(p.proj + (row0 + t0 + i) * p.ld + c);
+      if (i < valid) raw[i] = *reinterpret_cast<const uint2 *>(p.proj + (int64_t)(portion.y + t0 + i) * p.ld + c);
     }
     float w[4][4], past[3][4];
 #pragma unroll
@@ -84,7 +104,7 @@ __device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, i
     for (int j = 0; j < 3; ++j) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) past[j][e] = 0.f;
-      if (j + 1 < p.taps && t0 < valid) earlier_input<4>(p, row0 + t0, j + 1, c, past[j]);
+      if (j + 1 < p.taps && valid > 0) portion_input(p, portion, t0 - j - 1, c, past[j]);
     }
 #pragma unroll
     for (int i = 0; i < kCount; ++i) {
@@ -93,21 +113,22 @@ __device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, i
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         y[e] = fmaf(past[2][e], w[3][e], fmaf(past[1][e], w[2][e], fmaf(past[0][e], w[1][e], now[e] * w[0][e])));
-        y[e] = t0 + i < valid ? fast_silu(y[e]) : 0.f;
+        y[e] = i < valid ? fast_silu(y[e]) : 0.f;
         past[2][e] = past[1][e];
         past[1][e] = past[0][e];
         past[0][e] = now[e];
       }
-      put(t0 + i, y);
+      put(i, y);
     }
     return;
   }
-  for (int t = t0; t < t0 + kCount; ++t) {
+#pragma unroll
+  for (int i = 0; i < kCount; ++i) {
     float y[4] = {};
-    if (t < valid) {
+    if (i < valid) {
       for (int j = 0; j < p.taps; ++j) {
         float in[4], w[4];
-        earlier_input<4>(p, row0 + t, j, c, in);
+        portion_input(p, portion, t0 + i - j, c, in);
         load_vec<4>(p.conv + (size_t)(p.taps - 1 - j) * channels + c, w);
 #pragma unroll
         for (int e = 0; e < 4; ++e) y[e] = fmaf(in[e], w[e], y[e]);
@@ -115,8 +136,62 @@ __device__ __forceinline__ void conv_walk(const DeltaParams<__nv_bfloat16> &p, i
 #pragma unroll
       for (int e = 0; e < 4; ++e) y[e] = fast_silu(y[e]);
     }
-    put(t, y);
+    put(i, y);
   }
+}
+
+// A warp takes 16 tokens of a query or key head (all its channels: the unit norm stays inside the warp) or of 128 value
+// channels; the four warps of a block the four runs of a chunk.
+template <int kDK>
+__global__ void __launch_bounds__(128)
+delta_chunk_conv_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *portions, int first, uint8_t *keys, uint8_t *values) {
+  using K = KeyTiles<kDK>;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.z;
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const int4 portion = portions[blockIdx.y];
+  const int c_first = blockIdx.x * kC;
+  if (c_first >= portion.z) return;
+  if (portion.x < 0 || portion.x >= p.max_seqs) {
+    if (threadIdx.x == 0) atomicOr(&g_error_word, AXB200_ERR_CAPACITY);
+    return;
+  }
+  const size_t chunk = first_chunk(portion, blockIdx.y, first) + blockIdx.x;
+  const int run = warp * 16, t0 = c_first + run, valid = portion.z - t0;
+  if (unit >= 2 * p.kv_heads) {
+    const int c = (unit - 2 * p.kv_heads) * 128 + lane * 4;
+    if (c >= p.heads * p.vdim) return;
+    uint8_t *dst = values + (chunk * (p.heads * p.vdim / 8) + c / 8) * (size_t)kValueTile + (c & 7) * 2;
+    conv_walk<16>(p, portion, t0, valid, 2 * p.kv_heads * p.dim + c, [&](int i, const float (&y)[4]) {
+      *reinterpret_cast<uint2 *>(dst + (run + i) * 16) = make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
+    });
+    return;
+  }
+  const bool is_k = unit >= p.kv_heads;
+  const int hk = is_k ? unit - p.kv_heads : unit, c = lane * 4;
+  uint8_t *tiles = keys + (chunk * p.kv_heads + hk) * (size_t)K::kBytes, *tile = tiles + (is_k ? 0 : K::kTile);
+  const bool real = c < p.dim;
+  float sq[16];  // of the rounded rows: their unit vectors are exact
+  conv_walk<16>(p, portion, t0, real ? valid : 0, real ? unit * p.dim + c : 0, [&](int i, const float (&y)[4]) {
+    const uint2 packed = make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
+    const float a = bf_lo(packed.x), b = bf_hi(packed.x), d = bf_lo(packed.y), e = bf_hi(packed.y);
+    sq[i] = a * a + b * b + d * d + e * e;
+    if (c < kDK) *reinterpret_cast<uint2 *>(tile + tile_at(run + i, c >> 3, kDK / 8) + (c & 4) * 2) = packed;
+  });
+  // all sixteen sums over the warp by halving exchanges: lanes 2 i and 2 i + 1 end with row i's
+#pragma unroll
+  for (int n = 8, off = 16; n > 0; n >>= 1, off >>= 1) {
+    const bool upper = lane & off;
+#pragma unroll
+    for (int i = 0; i < n; ++i) {
+      const float send = upper ? sq[i] : sq[i + n], keep = upper ? sq[i + n] : sq[i];
+      sq[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+    }
+  }
+  sq[0] += __shfl_xor_sync(0xffffffffu, sq[0], 1);
+  const float gain = is_k ? 1.f : 1.0f / sqrtf((float)p.dim);
+  if ((lane & 1) == 0)
+    reinterpret_cast<float *>(tiles + K::kOffInv)[(is_k ? 0 : kC) + run + (lane >> 1)] = gain / sqrtf(sq[0] + kUnitEps);
 }
 
 // One warp: out (16 x 8) = sign * a (16 x 16 n) . b (16 n x 8), fp32 matrices of stride kLd in shared memory, in bf16
@@ -143,52 +218,44 @@ __device__ __forceinline__ void small_product(float *out, const float *a, const 
 
 template <int kDK>
 struct PrepSmem {
-  static constexpr int kTile = kC * kDK * 2, kMatrix = kC * kLd * 4;
-  static constexpr int kOffKK = 2 * kTile, kOffQK = kOffKK + kMatrix, kOffA = kOffQK + kMatrix;  // A: one per half
-  static constexpr int kOffVec = kOffA + 2 * kMatrix;
-  static constexpr int kBytes = kOffVec + 4 * kC * 4 + 2 * kPrepHeads * kC * 4;
+  static constexpr int kMatrix = kC * kLd * 4;
+  static constexpr int kOffKK = KeyTiles<kDK>::kBytes, kOffQK = kOffKK + kMatrix, kOffA = kOffQK + kMatrix;  // A: one per half
+  static constexpr int kOffGates = kOffA + 2 * kMatrix, kOffBar = kOffGates + 2 * kPrepHeads * kC * 4, kBytes = kOffBar + 16;
 };
 
-// Block z < kv_heads: one chunk of one query / key head, and T, P and the vectors of its group of value heads; the others:
-// the values of one head.
+// One chunk of one query / key head: T, P and the vectors of its group of value heads.
 template <int kDK>
 __global__ void __launch_bounds__(kPrepThreads, 2)
-delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *portions, int first, uint8_t *keys, uint8_t *heads,
-                           uint8_t *values) {
+delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *portions, int first, const uint8_t *keys, uint8_t *heads,
+                           unsigned long long wait_ns) {
   using S = PrepSmem<kDK>;
+  using K = KeyTiles<kDK>;
   extern __shared__ __align__(128) uint8_t smem[];
+  uint64_t *bar = reinterpret_cast<uint64_t *>(smem + S::kOffBar);
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(bar + 1);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (tid == 0) {
+    mbar_init(bar, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  __syncthreads();
   grid_dependency_wait();
   grid_dependency_launch();
   const int4 portion = portions[blockIdx.y];
   const int t_first = blockIdx.x * kC, valid = min(kC, portion.z - t_first);
-  if (valid <= 0) return;
-  if (portion.x < 0 || portion.x >= p.max_seqs) {
-    if (tid == 0) atomicOr(&g_error_word, AXB200_ERR_CAPACITY);
-    return;
-  }
+  if (valid <= 0 || portion.x < 0 || portion.x >= p.max_seqs) return;
   const int64_t row0 = portion.y + t_first;
   const size_t chunk = first_chunk(portion, blockIdx.y, first) + blockIdx.x;
-  const int qk_channels = 2 * p.kv_heads * p.dim;
-
-  if ((int)blockIdx.z >= p.kv_heads) {
-    // a quad of channels, a run of 8 tokens at a time
-    const int h = blockIdx.z - p.kv_heads, blocks = p.vdim / 8, quads = blocks * 2;
-    uint8_t *dst = values + (chunk * p.heads + h) * (size_t)blocks * kValueTile;
-    for (int i = tid; i < quads * (kC / 8); i += kPrepThreads) {
-      const int c = i % quads * 4;
-      conv_walk<8>(p, row0, valid, qk_channels + h * p.vdim + c, i / quads * 8, [&](int t, const float (&y)[4]) {
-        *reinterpret_cast<uint2 *>(dst + (c >> 3) * kValueTile + t * 16 + (c & 7) * 2) =
-            make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
-      });
-    }
-    return;
-  }
-
   const int hk = blockIdx.z, group = p.heads / p.kv_heads;
-  uint8_t *ck = smem, *cq = smem + S::kTile;
+  if (tid == 0) {
+    mbar_arrive_expect_tx(bar, K::kBytes);
+    bulk_load(smem, keys + (chunk * p.kv_heads + hk) * K::kBytes, K::kBytes, bar);
+  }
+  const uint8_t *ck = smem, *cq = smem + K::kTile;
   float *kk = reinterpret_cast<float *>(smem + S::kOffKK), *qk = reinterpret_cast<float *>(smem + S::kOffQK);
-  float *inv_k = reinterpret_cast<float *>(smem + S::kOffVec), *inv_q = inv_k + kC, *gates = inv_q + 3 * kC;
+  const float *inv_k = reinterpret_cast<const float *>(smem + K::kOffInv), *inv_q = inv_k + kC;
+  float *gates = reinterpret_cast<float *>(smem + S::kOffGates);
   constexpr int kPieces = kDK / 8;
 
   // decays, summed up (in the log2 domain), and steps of up to kPrepHeads heads: a warp per head, two tokens per lane
@@ -218,39 +285,11 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
     }
   };
   gates_of(0);
-  // convolutions: even warps the keys, odd warps the queries, 16 tokens each; a warp holds a whole row
-  {
-    const bool is_q = warp & 1;
-    const int c = lane * 4, t0 = (warp >> 1) * 16;
-    uint8_t *tile = is_q ? cq : ck;
-    float *inv = is_q ? inv_q : inv_k;
-    const float gain = is_q ? 1.0f / sqrtf((float)p.dim) : 1.f;
-    const bool real = c < p.dim;
-    float sq[16];  // of the rounded rows: their unit vectors are exact
-    conv_walk<16>(p, row0, real ? valid : 0, real ? (is_q ? hk : p.kv_heads + hk) * p.dim + c : 0, t0, [&](int t, const float (&y)[4]) {
-      const uint2 packed = make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
-      const float a = bf_lo(packed.x), b = bf_hi(packed.x), d = bf_lo(packed.y), e = bf_hi(packed.y);
-      sq[t & 15] = a * a + b * b + d * d + e * e;
-      if (c < kDK) *reinterpret_cast<uint2 *>(tile + tile_at(t, c >> 3, kPieces) + (c & 4) * 2) = packed;
-    });
-    // all sixteen sums over the warp by halving exchanges: lanes 2 i and 2 i + 1 end with row i's
-#pragma unroll
-    for (int n = 8, off = 16; n > 0; n >>= 1, off >>= 1) {
-      const bool upper = lane & off;
-#pragma unroll
-      for (int i = 0; i < n; ++i) {
-        const float send = upper ? sq[i] : sq[i + n], keep = upper ? sq[i + n] : sq[i];
-        sq[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
-      }
+  if (!mbar_wait_bounded(bar, 0, abort_flag, wait_ns)) {  // no copy may still be on its way when the CTA leaves
+    const unsigned long long t0 = global_timer_ns();
+    while (!mbar_try_wait(bar, 0) && global_timer_ns() - t0 < 100000000ull) {
     }
-    sq[0] += __shfl_xor_sync(0xffffffffu, sq[0], 1);
-    if ((lane & 1) == 0) inv[t0 + (lane >> 1)] = gain / sqrtf(sq[0] + kUnitEps);
-  }
-  __syncthreads();
-  {
-    uint8_t *dst = keys + (chunk * p.kv_heads + hk) * (size_t)(2 * S::kTile);
-    for (int i = tid * 16; i < 2 * S::kTile; i += kPrepThreads * 16)
-      *reinterpret_cast<uint4 *>(dst + i) = *reinterpret_cast<const uint4 *>(smem + i);
+    return;
   }
   // K.K^T (even warps) and Q.K^T (odd warps), 16 rows each
   {
@@ -372,7 +411,7 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
 template <int kDK, int kWarps>
 struct ScanSmem {
   static constexpr bool kSplit = kWarps <= 4;  // a second warp per 8 columns for the read-out
-  static constexpr int kTile = kC * kDK * 2;
+  static constexpr int kTile = KeyTiles<kDK>::kTile;
   static constexpr int kOffHead = 2 * kTile, kOffValues = kOffHead + kHeadTiles, kStage = kOffValues + kWarps * kValueTile;
   static constexpr int kState = kDK / 16 * 512, kHandOver = kSplit ? kState + 4 * 512 : 0;  // S as operands B, U as accumulators
   static constexpr int kRest = kWarps * kHandOver + 512;
@@ -511,7 +550,7 @@ __global__ void __launch_bounds__(ScanSmem<kDK, kWarps>::kThreads, 1) delta_chun
         const size_t chunk = chunk0 + n;
         uint8_t *dst = smem + s * L::kStage;
         mbar_arrive_expect_tx(&full[s], 2 * L::kTile + kHeadTiles + warps * kValueTile);
-        bulk_load(dst, p.keys + (chunk * p.kv_heads + hk) * (2 * L::kTile), 2 * L::kTile, &full[s]);
+        bulk_load(dst, p.keys + (chunk * p.kv_heads + hk) * KeyTiles<kDK>::kBytes, 2 * L::kTile, &full[s]);
         bulk_load(dst + L::kOffHead, p.heads_tiles + (chunk * p.heads + h) * kHeadTiles, kHeadTiles, &full[s]);
         bulk_load(dst + L::kOffValues, p.values + ((chunk * p.heads + h) * blocks + block0) * kValueTile, warps * kValueTile, &full[s]);
       }
@@ -703,9 +742,12 @@ int run(const DeltaParams<__nv_bfloat16> &d, const ScanParams &s, int count, int
         cudaStream_t st) {
   using P = PrepSmem<kDK>;
   if (int rc = opt_in<delta_chunk_prepare_kernel<kDK>>(P::kBytes)) return rc;
-  const dim3 grid((longest + kC - 1) / kC, count, d.kv_heads + d.heads);
-  if (int rc = launch_dependent(delta_chunk_prepare_kernel<kDK>, grid, dim3(kPrepThreads), (size_t)P::kBytes, st, d, s.portions, s.first, keys,
-                                heads, values))
+  const int chunks = (longest + kC - 1) / kC;
+  if (int rc = launch_dependent(delta_chunk_conv_kernel<kDK>, dim3(chunks, count, 2 * d.kv_heads + (d.heads * d.vdim + 127) / 128), dim3(128),
+                                0, st, d, s.portions, s.first, keys, values))
+    return rc;
+  if (int rc = launch_dependent(delta_chunk_prepare_kernel<kDK>, dim3(chunks, count, d.kv_heads), dim3(kPrepThreads), (size_t)P::kBytes, st, d,
+                                s.portions, s.first, keys, heads, s.wait_ns))
     return rc;
   // as few warps in a CTA as give every SM at most one
   int dev = 0, sms = 0;
@@ -719,6 +761,7 @@ int run(const DeltaParams<__nv_bfloat16> &d, const ScanParams &s, int count, int
 }
 
 int padded_dim(int dim) { return dim <= 64 ? 64 : 128; }
+size_t key_bytes(int dim) { return padded_dim(dim) == 64 ? KeyTiles<64>::kBytes : KeyTiles<128>::kBytes; }
 int64_t chunk_slots(int64_t rows, int count) { return rows / kC + count; }
 
 }  // namespace
@@ -733,19 +776,18 @@ int axb200_delta_chunks_supported(int dim, int vdim, int dtype) {
 size_t axb200_delta_chunks_workspace_bytes(int64_t rows, int count, int heads, int kv_heads, int dim, int vdim) {
   if (rows <= 0 || count <= 0) return 0;
   return (size_t)axb::chunk_slots(rows, count) *
-         ((size_t)kv_heads * 2 * axb::kC * axb::padded_dim(dim) * 2 +
+         ((size_t)kv_heads * axb::key_bytes(dim) +
           (size_t)heads * (axb::kHeadTiles + (size_t)(vdim / 8) * axb::kValueTile));
 }
 
-int axb200_delta_chunks(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos, const int32_t *row_back,
-                        int first, int rows, const float *conv, const float *a_log, const float *dt_bias, void *ring, float *state,
-                        const int32_t *portions, int count, int longest, void *out, int heads, int kv_heads, int dim, int vdim,
+int axb200_delta_chunks(const void *proj, int64_t ld, int first, int rows, const float *conv, const float *a_log,
+                        const float *dt_bias, const void *ring, float *state, const int32_t *portions, int count, int longest, void *out, int heads, int kv_heads, int dim, int vdim,
                         int taps, int max_seqs, int dtype, void *workspace, size_t workspace_bytes, void *stream) {
   if (!axb200_delta_chunks_supported(dim, vdim, dtype)) return AXB200_UNSUPPORTED_TYPE;
-  if (!proj || !row_seq || !row_pos || !row_back || !conv || !a_log || !dt_bias || !ring || !state || !portions || !out || !workspace)
+  if (!proj || !conv || !a_log || !dt_bias || !ring || !state || !portions || !out || !workspace)
     return AXB200_INVALID_PTR;
   if (first < 0 || first > rows || count < 0 || count > 65535 || longest < 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 ||
-      heads + kv_heads > 65535 || taps <= 0 || max_seqs <= 0)
+      heads > 65535 || 2 * (int64_t)kv_heads + ((int64_t)heads * vdim + 127) / 128 > 65535 || taps <= 0 || max_seqs <= 0)
     return AXB200_INVALID_ARGUMENT;
   if (ld < (int64_t)2 * kv_heads * dim + (int64_t)heads * (2 * vdim + 2)) return AXB200_SHAPE_MISMATCH;
   if (ld % 4 || !axb::al16(proj) || !axb::al16(conv) || !axb::al16(ring) || !axb::al16(portions) || !axb::al16(out) ||
@@ -753,12 +795,12 @@ int axb200_delta_chunks(const void *proj, int64_t ld, const int32_t *row_seq, co
     return AXB200_UNSUPPORTED_TYPE;
   if (count == 0 || first == rows) return AXB200_OK;
   if (workspace_bytes < axb200_delta_chunks_workspace_bytes(rows - first, count, heads, kv_heads, dim, vdim)) return AXB200_OUT_OF_MEMORY;
-  const axb::DeltaParams<__nv_bfloat16> d{static_cast<const __nv_bfloat16 *>(proj), ld, row_seq, row_pos, row_back, rows, conv, a_log,
-                                          dt_bias, nullptr, static_cast<__nv_bfloat16 *>(ring), state, heads, kv_heads, dim, vdim, taps,
+  const axb::DeltaParams<__nv_bfloat16> d{static_cast<const __nv_bfloat16 *>(proj), ld, nullptr, nullptr, nullptr, rows, conv, a_log,
+                                          dt_bias, nullptr, static_cast<__nv_bfloat16 *>(const_cast<void *>(ring)), state, heads, kv_heads, dim, vdim, taps,
                                           max_seqs, 0.f};
   const size_t slots = (size_t)axb::chunk_slots(rows - first, count);
   uint8_t *keys = static_cast<uint8_t *>(workspace);
-  uint8_t *tiles = keys + slots * kv_heads * 2 * axb::kC * axb::padded_dim(dim) * 2;
+  uint8_t *tiles = keys + slots * kv_heads * axb::key_bytes(dim);
   uint8_t *values = tiles + slots * heads * axb::kHeadTiles;
   const axb::ScanParams s{reinterpret_cast<const int4 *>(portions), first, keys, tiles, values, state, static_cast<__nv_bfloat16 *>(out),
                           heads, kv_heads, dim, vdim, max_seqs, axb::wait_limit_ns()};

@@ -33,10 +33,10 @@ def main(argv=None) -> int:
 
     import torch  # first: the library then shares PyTorch's cuBLASLt
 
-    from . import _capi, models
+    from . import models
     from .serving import ModelRunner, generate
 
-    _capi.use_serving_library()
+    models.use_library_for(args.model)
     torch.cuda.set_device(0)
     model = models.load(args.model, getattr(torch, args.dtype))
     longest = max(len(p) for p in prompts) + args.max_new

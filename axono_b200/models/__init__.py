@@ -6,7 +6,8 @@
 
 A registered class takes (config, weights, dtype, device) and offers what `axono_b200.serving` drives:
 `cache_rows` (elements one token caches in each cache layer), `state_shapes` (what one sequence keeps in each state
-layer, as (shape, dtype) pairs), `vocab`, `takes_segment(n)` and `forward(tokens, rows, cache, want)`.
+layer, as (shape, dtype) pairs), `vocab`, `takes_segment(n)` and `forward(tokens, rows, cache, want)`; `kernel_sources` names the CUDA sources it needs
+beyond those that every model does.
 `TextTower`, the decode step of the reference's own model, is listed by name for `config_of`; it makes its
 random weights itself and is stepped directly (axono_b200.decode, axono_b200.native_tower).
 """
@@ -45,6 +46,15 @@ def config_of(config: dict):
 
         return TextTowerConfig(**{k: tuple(v) if isinstance(v, list) else v for k, v in config.items() if k != "architecture"})
     return model_class(config.get("architecture")).config_class.parse(config)
+
+
+def use_library_for(folder: str) -> None:
+    """Makes the library that the folder's design needs the one this process loads (see axono_b200.build)."""
+    from .. import _capi
+
+    with open(os.path.join(folder, "config.json")) as f:
+        architecture = json.load(f).get("architecture")
+    _capi.use_serving_library(architecture, model_class(architecture).kernel_sources)
 
 
 def create(config: dict, weights, dtype, device="cuda"):

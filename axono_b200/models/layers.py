@@ -197,7 +197,7 @@ class GatedDelta:
                 qk, v, log_g, beta = ops.delta_prepare(self, proj[:c], rows, m, state, ring)
                 ops.delta_scan(self, rows.portion_table[:short], m, qk, v, log_g, beta, state, out[m:c])
             if c < n:
-                ops.delta_chunks(self, proj, rows, rows.portion_table[short:], rows.portions[-1][2], c, state, ring, out[c:])
+                ops.delta_chunks(self, proj, rows.portion_table[short:], rows.portions[-1][2], c, state, ring, out[c:])
             ops.delta_finish(self, proj, rows, m, state, ring, out[m:], out[m:])
         return out
 

@@ -133,6 +133,7 @@ def tensor_shapes(cfg: NuderaxConfig):
 @register("Nuderax")
 class Nuderax:
     config_class = NuderaxConfig
+    kernel_sources = ("moe.cu", "moe_umma.cu")
     state_shapes = ()  # no recurrent layers
 
     def __init__(self, cfg: NuderaxConfig, weights, dtype=torch.bfloat16, device="cuda"):

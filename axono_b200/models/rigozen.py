@@ -159,6 +159,7 @@ def tensor_shapes(cfg: RigozenConfig):
 @register("Rigozen")
 class Rigozen:
     config_class = RigozenConfig
+    kernel_sources = ("delta.cu", "delta_chunk.cu", "shared_kv.cu")
 
     def __init__(self, cfg: RigozenConfig, weights, dtype=torch.bfloat16, device="cuda"):
         self.cfg, self.dtype, self.device, self.vocab = cfg, dtype, torch.device(device), cfg.vocab

@@ -824,7 +824,7 @@ def delta_chunks_supported(dim, vdim, dtype) -> bool:
     return bool(_capi.lib().axb200_delta_chunks_supported(dim, vdim, _LM_DTYPES[dtype]))
 
 
-def delta_chunks(m, proj, rows, portions, longest, first, state, ring, out):
+def delta_chunks(m, proj, portions, longest, first, state, ring, out):
     """`delta_prepare` and `delta_scan` of the portions (int32 (count, 4), rows first..) in chunks of 64 tokens, bf16."""
     op = "delta_chunks"
     (conv, a_log, dt_bias, _, ring_ptr, state_ptr), sizes = _delta_args(m, proj, state, ring)
@@ -834,9 +834,8 @@ def delta_chunks(m, proj, rows, portions, longest, first, state, ring, out):
     ws = torch.empty(lib.axb200_delta_chunks_workspace_bytes(n, portions.shape[0], m.heads, m.kv_heads, m.dim, m.vdim),
                      dtype=torch.uint8, device=proj.device)
     _call(lib.axb200_delta_chunks(
-        proj.data_ptr(), proj.stride(0), rows.seq.data_ptr(), rows.pos.data_ptr(), rows.back.data_ptr(), first, proj.shape[0], conv,
-        a_log, dt_bias, ring_ptr, state_ptr, portions.data_ptr(), portions.shape[0], int(longest), out.data_ptr(), *sizes[:-1],
-        _lm_dt(proj, op), ws.data_ptr(), ws.numel(), _stream(proj)), op)
+        proj.data_ptr(), proj.stride(0), first, proj.shape[0], conv, a_log, dt_bias, ring_ptr, state_ptr, portions.data_ptr(),
+        portions.shape[0], int(longest), out.data_ptr(), *sizes[:-1], _lm_dt(proj, op), ws.data_ptr(), ws.numel(), _stream(proj)), op)
 
 
 def delta_finish(m, proj, rows, first, state, ring, o, out):

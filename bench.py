@@ -1855,7 +1855,7 @@ def delta_parts(ops, delta, proj, rows, state, ring):
     n, vv, qk2 = proj.shape[0], delta.heads * delta.vdim, 2 * delta.kv_heads * delta.dim
     out = torch.empty((n, vv), dtype=proj.dtype, device=proj.device)
     return {
-        "delta_chunks": (lambda: ops.delta_chunks(delta, proj, rows, rows.portion_table, n, 0, state, ring, out), n * 2.0 * (qk2 + 2 * vv)),
+        "delta_chunks": (lambda: ops.delta_chunks(delta, proj, rows.portion_table, n, 0, state, ring, out), n * 2.0 * (qk2 + 2 * vv)),
         "delta_finish": (lambda: ops.delta_finish(delta, proj, rows, 0, state, ring, out, out), n * vv * 6.0),
     }
 

@@ -590,10 +590,9 @@ int axb200_delta_scan(const int32_t *portions, int count, int first, const float
                       int max_seqs, int dtype, void *stream);
 int axb200_delta_chunks_supported(int dim, int vdim, int dtype);
 size_t axb200_delta_chunks_workspace_bytes(int64_t rows, int count, int heads, int kv_heads, int dim, int vdim);
-int axb200_delta_chunks(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos,
-                        const int32_t *row_back, int first, int rows, const float *conv, const float *a_log,
-                        const float *dt_bias, void *ring, float *state, const int32_t *portions, int count, int longest,
-                        void *out, int heads, int kv_heads, int dim, int vdim, int taps, int max_seqs, int dtype,
+int axb200_delta_chunks(const void *proj, int64_t ld, int first, int rows, const float *conv, const float *a_log,
+                        const float *dt_bias, const void *ring, float *state, const int32_t *portions, int count,
+                        int longest, void *out, int heads, int kv_heads, int dim, int vdim, int taps, int max_seqs, int dtype,
                         void *workspace, size_t workspace_bytes, void *stream);
 int axb200_delta_finish(const void *proj, int64_t ld, const int32_t *row_seq, const int32_t *row_pos,
                         const int32_t *row_back, int first, int rows, const float *conv, const float *a_log,

@@ -74,6 +74,17 @@ def test_arena_with_state_and_without_rows():
     a.close()
 
 
+def test_a_design_names_the_sources_it_needs():
+    import os
+
+    from axono_b200 import build, models
+
+    for design in models.architectures():
+        for name in (*build.SERVING_SOURCES, *models.model_class(design).kernel_sources):
+            assert os.path.exists(os.path.join(build.CSRC, name)), name
+        assert design.lower() in build.serving_lib(design)
+
+
 # ---- the plain evaluation itself ---------------------------------------------------------------------------
 def test_plain_windows_end_exactly():
     """With window n a row's output depends on the key n - 1 before it and not on the one before that."""
