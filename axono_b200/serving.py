@@ -12,6 +12,7 @@ import collections
 from dataclasses import dataclass, field
 from typing import List, Optional, Sequence
 
+import numpy as np
 import torch
 
 from . import ops
@@ -74,33 +75,33 @@ class ModelRunner:
         self.arena.sync()
         # single tokens first, then portions by length: those that attend through the cache, then the long ones
         order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]))
-        ids, seqs, pos, back, first, segments, portions, latent, max_len = [], [], [], [], {}, [], [], 0, 1
+        total, wanted = sum(len(e[1]) for e in entries), sum(len(e[2]) for e in entries)
+        # two copies for the step's integers: token ids and wanted rows; sequences, positions, rows before, portions
+        wide, ints = np.empty(total + wanted, np.int64), np.empty((3, total), np.int32)
+        first, segments, portions, latent, max_len, at = {}, [], [], 0, 1, 0
         for i in order:
             seq, tokens, _ = entries[i]
             start, n = self.lengths[seq], len(tokens)
-            first[i] = len(ids)
+            first[i] = at
             if n > 1:
-                portions.append((seq, len(ids), n, start))
+                portions.append((seq, at, n, start))
             if self.model.takes_segment(n):
-                segments.append((seq, len(ids), n, start))
+                segments.append((seq, at, n, start))
             elif segments:
                 raise RuntimeError("a model that takes a portion as a segment must take every longer one")
             else:
                 latent += n
                 max_len = max(max_len, start + n)
-            ids.extend(tokens)
-            seqs.extend([seq] * n)
-            pos.extend(range(start, start + n))
-            back.extend(range(n))
-        want = [first[i] + w for i, (_, _, places) in enumerate(entries) for w in places]
-        dev = self.model.device
-        # two copies for the step's integers: token ids and wanted rows; portions, sequences, positions, rows before
-        wide = torch.tensor(ids + want, dtype=torch.int64).to(dev)
-        n, at = len(ids), 4 * len(portions)
-        ints = torch.tensor([v for p in portions for v in p] + seqs + pos + back, dtype=torch.int32).to(dev)
-        rows = Rows(ints[at:at + n], ints[at + n:at + 2 * n], self.block_table, max_len, latent, segments, n - sum(p[2] for p in portions),
-                    ints[at + 2 * n:], portions, ints[:at].view(-1, 4))
-        logits = self.model.forward(wide[:n], rows, self.cache, wide[n:], trace=trace)
+            wide[at:at + n] = tokens
+            ints[0, at:at + n], ints[1, at:at + n], ints[2, at:at + n] = seq, np.arange(start, start + n), np.arange(n)
+            at += n
+        wide[total:] = [first[i] + w for i, (_, _, places) in enumerate(entries) for w in places]
+        dev, k = self.model.device, 4 * len(portions)
+        packed = torch.from_numpy(np.concatenate([np.array(portions, np.int32).reshape(-1), ints.reshape(-1)])).to(dev)
+        ids, (seqs, pos, back) = torch.from_numpy(wide).to(dev), packed[k:].view(3, total)
+        rows = Rows(seqs, pos, self.block_table, max_len, latent, segments, total - sum(p[2] for p in portions), back, portions,
+                    packed[:k].view(-1, 4))
+        logits = self.model.forward(ids[:total], rows, self.cache, ids[total:], trace=trace)
         for seq, tokens, _ in entries:
             self.lengths[seq] += len(tokens)
         return logits
