@@ -6,13 +6,14 @@
 //     S'  = e^{G_64} S + sum_s e^{G_64 - G_s} k_s u_s^T.
 // Two kernels do what needs no state, all chunks at once: delta_chunk_conv the convolutions and silu, into tiles;
 // delta_chunk_prepare the products of queries and keys, T = (I + A)^-1 diag(beta) by blocked forward substitution, P, and
-// the scale vectors.  delta_chunk_scan walks a sequence's chunks: a warp owns 8 value columns of a head's state and is independent of all others.
+// the scale vectors.  delta_chunk_scan walks a sequence's chunks: a warp owns 8 or 16 value columns of a head's state and
+// is independent of all others.
 //
 // Precision.  The outputs of the short convolutions are bf16, so they are exact tensor-core operands: unit norms and
 // decays stay outside the products, as fp32 factors of rows.  Everything else that enters a product - state, X, U, T, P -
 // is split into two bf16 parts and multiplied part by part (high.high + low.high + high.low), accumulated in fp32.
 //
-// The products chain in registers: S (keys x 8 values) is the accumulator of the update and, transposed in the register
+// The products chain in registers: S (keys x values) is the accumulator of the update and, transposed in the register
 // file (movmatrix), operand B of the next chunk's products; X and U likewise.  So the recurrence touches no shared memory.
 // Keys, queries, T and P are operand A and come as ready-made, swizzled tiles by bulk copies, some chunks ahead.
 // The walk is bound by the length of this chain, not by the tensor cores of a whole SM: 64 tokens take 250 warp-wide
@@ -408,16 +409,17 @@ delta_chunk_prepare_kernel(const DeltaParams<__nv_bfloat16> p, const int4 *porti
 }
 
 // ---- the walk over a sequence's chunks ------------------------------------------------------------------
-template <int kDK, int kWarps>
+// kWarps pairs of warps (the chain and the read-out) per CTA, kN tiles of 8 value columns each.  One tile makes the shorter
+// chain; two read the operands from shared memory once for both, whose bandwidth is the limit when an SM has many pairs.
+template <int kDK, int kWarps, int kN>
 struct ScanSmem {
-  static constexpr bool kSplit = kWarps <= 4;  // a second warp per 8 columns for the read-out
-  static constexpr int kTile = KeyTiles<kDK>::kTile;
-  static constexpr int kOffHead = 2 * kTile, kOffValues = kOffHead + kHeadTiles, kStage = kOffValues + kWarps * kValueTile;
-  static constexpr int kState = kDK / 16 * 512, kHandOver = kSplit ? kState + 4 * 512 : 0;  // S as operands B, U as accumulators
-  static constexpr int kRest = kWarps * kHandOver + 512;
-  static constexpr int kStages = 4 * kStage + kRest <= 227 * 1024 ? 4 : 3;
+  static constexpr int kTile = KeyTiles<kDK>::kTile, kTiles = kWarps * kN;
+  static constexpr int kOffHead = 2 * kTile, kOffValues = kOffHead + kHeadTiles, kStage = kOffValues + kTiles * kValueTile;
+  static constexpr int kState = kDK / 16 * kN * 512, kHandOver = kState + 4 * kN * 512;  // S as operands B, U as accumulators
+  static constexpr int kRest = kWarps * kHandOver + 512, kRoom = 227 * 1024 - kRest;
+  static constexpr int kStages = kRoom >= 4 * kStage ? 4 : kRoom >= 3 * kStage ? 3 : 2;
   static constexpr int kOffHand = kStages * kStage, kOffBar = kOffHand + kWarps * kHandOver, kBytes = kOffBar + 512;
-  static constexpr int kThreads = ((kSplit ? 2 : 1) * kWarps + 1) * 32;
+  static constexpr int kThreads = (2 * kWarps + 1) * 32;
 };
 
 // An 8 x 8 matrix of 16-bit elements, a row's pairs in four lanes, transposed.
@@ -438,9 +440,10 @@ __device__ __forceinline__ void split_operand(const float (&c)[4], uint32_t (&hi
   }
 }
 
-// acc (64 x 8) += m (lower triangular, 64 x 64, in two parts) . x (64 x 8, in two parts)
-__device__ __forceinline__ void triangular_product(float (&acc)[4][4], uint32_t m_high, uint32_t m_low, const uint32_t (&high)[4][2],
-                                                   const uint32_t (&low)[4][2], int lane) {
+// acc (64 x 8 kN) += m (lower triangular, 64 x 64, in two parts) . x (64 x 8 kN, in two parts)
+template <int kN>
+__device__ __forceinline__ void triangular_product(float (&acc)[kN][4][4], uint32_t m_high, uint32_t m_low, const uint32_t (&high)[kN][4][2],
+                                                   const uint32_t (&low)[kN][4][2], int lane) {
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     uint32_t a[4][4], b[4][4];
@@ -451,12 +454,36 @@ __device__ __forceinline__ void triangular_product(float (&acc)[4][4], uint32_t 
       ldmatrix_x4(b[m][0], b[m][1], b[m][2], b[m][3], m_low + at);
     }
 #pragma unroll
-    for (int m = k; m < 4; ++m) mma_16816_bf16(acc[m], a[m], high[k][0], high[k][1]);
+    for (int c = 0; c < kN; ++c)
 #pragma unroll
-    for (int m = k; m < 4; ++m) mma_16816_bf16(acc[m], a[m], low[k][0], low[k][1]);
+      for (int m = k; m < 4; ++m) mma_16816_bf16(acc[c][m], a[m], high[c][k][0], high[c][k][1]);
 #pragma unroll
-    for (int m = k; m < 4; ++m) mma_16816_bf16(acc[m], b[m], high[k][0], high[k][1]);
+    for (int c = 0; c < kN; ++c)
+#pragma unroll
+      for (int m = k; m < 4; ++m) mma_16816_bf16(acc[c][m], a[m], low[c][k][0], low[c][k][1]);
+#pragma unroll
+    for (int c = 0; c < kN; ++c)
+#pragma unroll
+      for (int m = k; m < 4; ++m) mma_16816_bf16(acc[c][m], b[m], high[c][k][0], high[c][k][1]);
   }
+}
+
+// acc (64 x 8 kN) += rows of a tile . s, for one slice of 16 keys, s in two parts
+template <int kN>
+__device__ __forceinline__ void slice_product(float (&acc)[kN][4][4], uint32_t tile, int k, int pieces, const uint32_t (&high)[kN][2],
+                                              const uint32_t (&low)[kN][2], int lane) {
+  uint32_t a[4][4];
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+    ldmatrix_x4(a[m][0], a[m][1], a[m][2], a[m][3], tile + tile_at(16 * m + (lane & 15), 2 * k + (lane >> 4), pieces));
+#pragma unroll
+  for (int c = 0; c < kN; ++c)
+#pragma unroll
+    for (int m = 0; m < 4; ++m) mma_16816_bf16(acc[c][m], a[m], high[c][0], high[c][1]);
+#pragma unroll
+  for (int c = 0; c < kN; ++c)
+#pragma unroll
+    for (int m = 0; m < 4; ++m) mma_16816_bf16(acc[c][m], a[m], low[c][0], low[c][1]);
 }
 
 struct ScanParams {
@@ -469,60 +496,21 @@ struct ScanParams {
   unsigned long long wait_ns;
 };
 
-// One chunk's o = e^G q S + P u of 8 columns; S comes as operands B tile by tile (state(k, high, low)), u when it is ready.
-template <int kDK, typename State, typename Update>
-__device__ __forceinline__ void read_out(const ScanParams &p, uint32_t cq, uint32_t tiles, const float *vec, int lane, int valid,
-                                         __nv_bfloat16 *dst, State state, Update update) {
-  constexpr int kPieces = kDK / 8;
-  const int g = lane >> 2;
-  float o[4][4] = {};
-#pragma unroll
-  for (int k = 0; k < kDK / 16; ++k) {
-    uint32_t high[2], low[2], b[4][4];
-#pragma unroll
-    for (int m = 0; m < 4; ++m)
-      ldmatrix_x4(b[m][0], b[m][1], b[m][2], b[m][3], cq + tile_at(16 * m + (lane & 15), 2 * k + (lane >> 4), kPieces));
-    state(k, high, low);
-#pragma unroll
-    for (int m = 0; m < 4; ++m) mma_16816_bf16(o[m], b[m], high[0], high[1]);
-#pragma unroll
-    for (int m = 0; m < 4; ++m) mma_16816_bf16(o[m], b[m], low[0], low[1]);
-  }
-  float u[4][4];
-  update(u);
-  uint32_t high[4][2], low[4][2];
-#pragma unroll
-  for (int m = 0; m < 4; ++m) {
-    const float e0 = vec[kC + 16 * m + g], e1 = vec[kC + 16 * m + g + 8];
-    o[m][0] *= e0, o[m][1] *= e0, o[m][2] *= e1, o[m][3] *= e1;
-    split_operand(u[m], high[m], low[m]);
-  }
-  triangular_product(o, tiles + 2 * kSquare, tiles + 3 * kSquare, high, low, lane);
-#pragma unroll
-  for (int m = 0; m < 4; ++m)
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int t = 16 * m + g + 8 * i;
-      if (t < valid) *reinterpret_cast<uint32_t *>(dst + (int64_t)t * p.heads * p.vdim) = pack_bf16x2(o[m][2 * i], o[m][2 * i + 1]);
-    }
-}
-
-template <int kDK, int kWarps>
-__global__ void __launch_bounds__(ScanSmem<kDK, kWarps>::kThreads, 1) delta_chunk_scan_kernel(const ScanParams p) {
-  using L = ScanSmem<kDK, kWarps>;
+template <int kDK, int kWarps, int kN>
+__global__ void __launch_bounds__(ScanSmem<kDK, kWarps, kN>::kThreads, 1) delta_chunk_scan_kernel(const ScanParams p) {
+  using L = ScanSmem<kDK, kWarps, kN>;
   constexpr int kPieces = kDK / 8, kKeyTiles = kDK / 16;  // 16-high tiles of S
-  constexpr int kProducer = (L::kSplit ? 2 : 1) * kWarps;
   extern __shared__ __align__(128) uint8_t smem[];
   uint64_t *full = reinterpret_cast<uint64_t *>(smem + L::kOffBar), *empty = full + L::kStages;
   uint64_t *s_full = empty + L::kStages, *s_empty = s_full + kWarps, *u_full = s_empty + kWarps, *u_empty = u_full + kWarps;
   volatile int *abort_flag = reinterpret_cast<volatile int *>(u_empty + kWarps);
   const int warp = __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0), lane = threadIdx.x & 31;
-  const int h = blockIdx.y, hk = h / (p.heads / p.kv_heads), blocks = p.vdim / 8, block0 = blockIdx.z * kWarps;
-  const int warps = min(kWarps, blocks - block0);  // with columns of their own
+  const int h = blockIdx.y, hk = h / (p.heads / p.kv_heads), blocks = p.vdim / 8, block0 = blockIdx.z * L::kTiles;
+  const int tiles_here = min(L::kTiles, blocks - block0), warps = (tiles_here + kN - 1) / kN;  // with columns of their own
   if (threadIdx.x == 0) {
     for (int i = 0; i < L::kStages; ++i) {
       mbar_init(&full[i], 1);
-      mbar_init(&empty[i], (L::kSplit ? 2 : 1) * warps);
+      mbar_init(&empty[i], 2 * warps);
     }
     for (int i = 0; i < 4 * kWarps; ++i) mbar_init(&s_full[i], 1);
     *abort_flag = 0;
@@ -539,7 +527,8 @@ __global__ void __launch_bounds__(ScanSmem<kDK, kWarps>::kThreads, 1) delta_chun
   const int chunks = (portion.z + kC - 1) / kC;
   const size_t chunk0 = first_chunk(portion, blockIdx.x, p.first);
 
-  if (warp == kProducer) {
+  if (warp == 2 * kWarps) {
+    // ---- bulk copies ----
     if (lane == 0) {
       bool ok = true;
       int n = 0;
@@ -549,10 +538,10 @@ __global__ void __launch_bounds__(ScanSmem<kDK, kWarps>::kThreads, 1) delta_chun
         if (!ok) break;
         const size_t chunk = chunk0 + n;
         uint8_t *dst = smem + s * L::kStage;
-        mbar_arrive_expect_tx(&full[s], 2 * L::kTile + kHeadTiles + warps * kValueTile);
+        mbar_arrive_expect_tx(&full[s], 2 * L::kTile + kHeadTiles + tiles_here * kValueTile);
         bulk_load(dst, p.keys + (chunk * p.kv_heads + hk) * KeyTiles<kDK>::kBytes, 2 * L::kTile, &full[s]);
         bulk_load(dst + L::kOffHead, p.heads_tiles + (chunk * p.heads + h) * kHeadTiles, kHeadTiles, &full[s]);
-        bulk_load(dst + L::kOffValues, p.values + ((chunk * p.heads + h) * blocks + block0) * kValueTile, warps * kValueTile, &full[s]);
+        bulk_load(dst + L::kOffValues, p.values + ((chunk * p.heads + h) * blocks + block0) * kValueTile, tiles_here * kValueTile, &full[s]);
       }
       if (*abort_flag) {  // no copy may still be on its way when the CTA leaves
         const unsigned long long t0 = global_timer_ns();
@@ -570,147 +559,169 @@ __global__ void __launch_bounds__(ScanSmem<kDK, kWarps>::kThreads, 1) delta_chun
     __syncwarp();
     if (lane == 0) mbar_arrive(bar);
   };
-  const int g = lane >> 2, v0 = (block0 + w) * 8 + (lane & 3) * 2;
-  auto rows_of = [&](int n) { return p.out + ((int64_t)(portion.y - p.first + n * kC) * p.heads + h) * p.vdim + v0; };
+  // an accumulator tile's rows are lane / 4 and + 8, its columns (lane % 4) * 2 and + 1
+  const int g = lane >> 2, v0 = (block0 + w * kN) * 8 + (lane & 3) * 2;
+  auto mine = [&](int c) { return v0 + 8 * c < p.vdim; };  // a last tile of a pair may not exist: its columns are never stored
   uint4 *hand_s = reinterpret_cast<uint4 *>(smem + L::kOffHand + w * L::kHandOver) + lane;
   float4 *hand_u = reinterpret_cast<float4 *>(smem + L::kOffHand + w * L::kHandOver + L::kState) + lane;
 
-  if (L::kSplit && warp >= kWarps) {
-    // ---- the read-out ----
+  if (warp >= kWarps) {
+    // ---- the read-out: o = e^G q S + P u ----
     for (int n = 0; n < chunks; ++n) {
       const int s = n % L::kStages;
       if (!wait(&full[s], n / L::kStages) || !wait(&s_full[w], n)) return;
-      const uint32_t base = smem_u32(smem + s * L::kStage);
-      bool ok = true;
-      read_out<kDK>(
-          p, base + L::kTile, base + L::kOffHead, reinterpret_cast<const float *>(smem + s * L::kStage + L::kOffHead + kVec), lane,
-          portion.z - n * kC, rows_of(n),
-          [&](int k, uint32_t(&high)[2], uint32_t(&low)[2]) {
-            const uint4 v = hand_s[k * 32];
-            high[0] = v.x, high[1] = v.y, low[0] = v.z, low[1] = v.w;
-          },
-          [&](float(&u)[4][4]) {
-            release(&s_empty[w]);
-            ok = wait(&u_full[w], n);
+      const uint32_t cq = smem_u32(smem + s * L::kStage + L::kTile), tiles = smem_u32(smem + s * L::kStage + L::kOffHead);
+      const float *vec = reinterpret_cast<const float *>(smem + s * L::kStage + L::kOffHead + kVec);
+      float o[kN][4][4] = {};
 #pragma unroll
-            for (int m = 0; m < 4; ++m) {
-              const float4 v = hand_u[m * 32];
-              u[m][0] = v.x, u[m][1] = v.y, u[m][2] = v.z, u[m][3] = v.w;
-            }
-            release(&u_empty[w]);
-          });
-      if (!ok) return;
+      for (int k = 0; k < kKeyTiles; ++k) {
+        uint32_t sh[kN][2], sl[kN][2];
+#pragma unroll
+        for (int c = 0; c < kN; ++c) {
+          const uint4 v = hand_s[(k * kN + c) * 32];
+          sh[c][0] = v.x, sh[c][1] = v.y, sl[c][0] = v.z, sl[c][1] = v.w;
+        }
+        slice_product<kN>(o, cq, k, kPieces, sh, sl, lane);
+      }
+      release(&s_empty[w]);
+      if (!wait(&u_full[w], n)) return;
+      uint32_t high[kN][4][2], low[kN][4][2];
+#pragma unroll
+      for (int m = 0; m < 4; ++m) {
+        const float e0 = vec[kC + 16 * m + g], e1 = vec[kC + 16 * m + g + 8];
+#pragma unroll
+        for (int c = 0; c < kN; ++c) {
+          o[c][m][0] *= e0, o[c][m][1] *= e0, o[c][m][2] *= e1, o[c][m][3] *= e1;
+          const float4 v = hand_u[(m * kN + c) * 32];
+          const float u[4] = {v.x, v.y, v.z, v.w};
+          split_operand(u, high[c][m], low[c][m]);
+        }
+      }
+      release(&u_empty[w]);
+      triangular_product<kN>(o, tiles + 2 * kSquare, tiles + 3 * kSquare, high, low, lane);
       release(&empty[s]);
+      const int valid = portion.z - n * kC;
+      __nv_bfloat16 *dst = p.out + ((int64_t)(portion.y - p.first + n * kC) * p.heads + h) * p.vdim + v0;
+#pragma unroll
+      for (int c = 0; c < kN; ++c)
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const int t = 16 * m + g + 8 * i;
+            if (t < valid && mine(c))
+              *reinterpret_cast<uint32_t *>(dst + (int64_t)t * p.heads * p.vdim + 8 * c) = pack_bf16x2(o[c][m][2 * i], o[c][m][2 * i + 1]);
+          }
     }
     return;
   }
 
-  // ---- the chain.  S: tile j holds keys 16j .. 16j + 15 (rows lane / 4 and + 8), 8 value columns ((lane % 4) * 2 and + 1) ----
+  // ---- the chain ----
   float *state = p.state + ((size_t)portion.x * p.heads + h) * p.dim * p.vdim;
-  float st[kKeyTiles][4];
+  float st[kN][kKeyTiles][4];  // S: tile j holds keys 16j .. 16j + 15
 #pragma unroll
-  for (int j = 0; j < kKeyTiles; ++j)
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int k = 16 * j + g + 8 * i;
-      float2 v = make_float2(0.f, 0.f);
-      if (portion.w > 0 && k < p.dim) v = *reinterpret_cast<const float2 *>(state + (size_t)k * p.vdim + v0);
-      st[j][2 * i] = v.x, st[j][2 * i + 1] = v.y;
-    }
-
-  for (int n = 0; n < chunks; ++n) {
-    const int s = n % L::kStages;
-    uint32_t sh[kKeyTiles][2], sl[kKeyTiles][2];
-#pragma unroll
-    for (int k = 0; k < kKeyTiles; ++k) split_operand(st[k], sh[k], sl[k]);
-    if (L::kSplit) {
-      if (n > 0 && !wait(&s_empty[w], n - 1)) return;
-#pragma unroll
-      for (int k = 0; k < kKeyTiles; ++k) hand_s[k * 32] = make_uint4(sh[k][0], sh[k][1], sl[k][0], sl[k][1]);
-      release(&s_full[w]);
-    }
-    if (!wait(&full[s], n / L::kStages)) return;
-    const uint32_t base = smem_u32(smem + s * L::kStage), ck = base, tiles = base + L::kOffHead;
-    const float *vec = reinterpret_cast<const float *>(smem + s * L::kStage + L::kOffHead + kVec);
-    const uint8_t *value = smem + s * L::kStage + L::kOffValues + w * kValueTile + (lane & 3) * 4;
-
-    // k S of all tokens
-    float x[4][4] = {};
-#pragma unroll
-    for (int k = 0; k < kKeyTiles; ++k) {
-      uint32_t a[4][4];
-#pragma unroll
-      for (int m = 0; m < 4; ++m)
-        ldmatrix_x4(a[m][0], a[m][1], a[m][2], a[m][3], ck + tile_at(16 * m + (lane & 15), 2 * k + (lane >> 4), kPieces));
-#pragma unroll
-      for (int m = 0; m < 4; ++m) mma_16816_bf16(x[m], a[m], sh[k][0], sh[k][1]);
-#pragma unroll
-      for (int m = 0; m < 4; ++m) mma_16816_bf16(x[m], a[m], sl[k][0], sl[k][1]);
-    }
-    // X = v - e^G k S
-    uint32_t high[4][2], low[4][2];
-#pragma unroll
-    for (int m = 0; m < 4; ++m) {
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = 16 * m + g + 8 * i;
-        const uint32_t v = *reinterpret_cast<const uint32_t *>(value + t * 16);
-        const float e = vec[t];
-        x[m][2 * i] = fmaf(-e, x[m][2 * i], bf_lo(v));
-        x[m][2 * i + 1] = fmaf(-e, x[m][2 * i + 1], bf_hi(v));
-      }
-      split_operand(x[m], high[m], low[m]);
-    }
-    float u[4][4] = {};
-    triangular_product(u, tiles, tiles + kSquare, high, low, lane);
-    if (L::kSplit) {
-      if (n > 0 && !wait(&u_empty[w], n - 1)) return;
-#pragma unroll
-      for (int m = 0; m < 4; ++m) hand_u[m * 32] = make_float4(u[m][0], u[m][1], u[m][2], u[m][3]);
-      release(&u_full[w]);
-    }
-    // S' = e^G_64 S + k^T (e^{G_64 - G} u)
-    const float total = vec[3 * kC];
+  for (int c = 0; c < kN; ++c)
 #pragma unroll
     for (int j = 0; j < kKeyTiles; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) st[j][e] *= total;
+      for (int i = 0; i < 2; ++i) {
+        const int k = 16 * j + g + 8 * i;
+        float2 v = make_float2(0.f, 0.f);
+        if (portion.w > 0 && k < p.dim && mine(c)) v = *reinterpret_cast<const float2 *>(state + (size_t)k * p.vdim + v0 + 8 * c);
+        st[c][j][2 * i] = v.x, st[c][j][2 * i + 1] = v.y;
+      }
+
+  for (int n = 0; n < chunks; ++n) {
+    const int s = n % L::kStages;
+    if (n > 0 && !wait(&s_empty[w], n - 1)) return;
+    if (!wait(&full[s], n / L::kStages)) return;
+    const uint32_t base = smem_u32(smem + s * L::kStage), ck = base, tiles = base + L::kOffHead;
+    const float *vec = reinterpret_cast<const float *>(smem + s * L::kStage + L::kOffHead + kVec);
+    const uint8_t *value = smem + s * L::kStage + L::kOffValues + w * kN * kValueTile + (lane & 3) * 4;
+
+    // k S of all tokens; S is handed over on the way
+    float x[kN][4][4] = {};
+#pragma unroll
+    for (int k = 0; k < kKeyTiles; ++k) {
+      uint32_t sh[kN][2], sl[kN][2];
+#pragma unroll
+      for (int c = 0; c < kN; ++c) {
+        split_operand(st[c][k], sh[c], sl[c]);
+        hand_s[(k * kN + c) * 32] = make_uint4(sh[c][0], sh[c][1], sl[c][0], sl[c][1]);
+      }
+      slice_product<kN>(x, ck, k, kPieces, sh, sl, lane);
+    }
+    release(&s_full[w]);
+    // X = v - e^G k S
+    uint32_t high[kN][4][2], low[kN][4][2];
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+      for (int c = 0; c < kN; ++c) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int t = 16 * m + g + 8 * i;
+          const uint32_t v = *reinterpret_cast<const uint32_t *>(value + c * kValueTile + t * 16);
+          const float e = vec[t];
+          x[c][m][2 * i] = fmaf(-e, x[c][m][2 * i], bf_lo(v));
+          x[c][m][2 * i + 1] = fmaf(-e, x[c][m][2 * i + 1], bf_hi(v));
+        }
+        split_operand(x[c][m], high[c][m], low[c][m]);
+      }
+    float u[kN][4][4] = {};
+    triangular_product<kN>(u, tiles, tiles + kSquare, high, low, lane);
+    if (n > 0 && !wait(&u_empty[w], n - 1)) return;
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+      for (int c = 0; c < kN; ++c) hand_u[(m * kN + c) * 32] = make_float4(u[c][m][0], u[c][m][1], u[c][m][2], u[c][m][3]);
+    release(&u_full[w]);
+    // S' = e^G_64 S + k^T (e^{G_64 - G} u)
+    const float total = vec[3 * kC];
+#pragma unroll
+    for (int c = 0; c < kN; ++c)
+#pragma unroll
+      for (int j = 0; j < kKeyTiles; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) st[c][j][e] *= total;
 #pragma unroll
     for (int m = 0; m < 4; ++m) {
       const float e0 = vec[2 * kC + 16 * m + g], e1 = vec[2 * kC + 16 * m + g + 8];
-      const float wu[4] = {e0 * u[m][0], e0 * u[m][1], e1 * u[m][2], e1 * u[m][3]};
-      uint32_t wh[2], wl[2], a[kKeyTiles][4];
+      uint32_t wh[kN][2], wl[kN][2];
 #pragma unroll
-      for (int j = 0; j < kKeyTiles; ++j)
-        ldmatrix_x4_trans(a[j][0], a[j][1], a[j][2], a[j][3],
-                          ck + tile_at(16 * m + ((lane >> 4) & 1) * 8 + (lane & 7), 2 * j + ((lane >> 3) & 1), kPieces));
-      split_operand(wu, wh, wl);
+      for (int c = 0; c < kN; ++c) {
+        const float wu[4] = {e0 * u[c][m][0], e0 * u[c][m][1], e1 * u[c][m][2], e1 * u[c][m][3]};
+        split_operand(wu, wh[c], wl[c]);
+      }
 #pragma unroll
-      for (int j = 0; j < kKeyTiles; ++j) mma_16816_bf16(st[j], a[j], wh[0], wh[1]);
+      for (int j0 = 0; j0 < kKeyTiles; j0 += 4) {
+        uint32_t a[4][4];
 #pragma unroll
-      for (int j = 0; j < kKeyTiles; ++j) mma_16816_bf16(st[j], a[j], wl[0], wl[1]);
+        for (int j = 0; j < 4; ++j)
+          ldmatrix_x4_trans(a[j][0], a[j][1], a[j][2], a[j][3],
+                            ck + tile_at(16 * m + ((lane >> 4) & 1) * 8 + (lane & 7), 2 * (j0 + j) + ((lane >> 3) & 1), kPieces));
+#pragma unroll
+        for (int c = 0; c < kN; ++c)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) mma_16816_bf16(st[c][j0 + j], a[j], wh[c][0], wh[c][1]);
+#pragma unroll
+        for (int c = 0; c < kN; ++c)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) mma_16816_bf16(st[c][j0 + j], a[j], wl[c][0], wl[c][1]);
+      }
     }
-    if (!L::kSplit)
-      read_out<kDK>(
-          p, base + L::kTile, tiles, vec, lane, portion.z - n * kC, rows_of(n),
-          [&](int k, uint32_t(&high)[2], uint32_t(&low)[2]) {
-            high[0] = sh[k][0], high[1] = sh[k][1], low[0] = sl[k][0], low[1] = sl[k][1];
-          },
-          [&](float(&out)[4][4]) {
-#pragma unroll
-            for (int m = 0; m < 4; ++m)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) out[m][e] = u[m][e];
-          });
     release(&empty[s]);
   }
 #pragma unroll
-  for (int j = 0; j < kKeyTiles; ++j)
+  for (int c = 0; c < kN; ++c)
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int k = 16 * j + g + 8 * i;
-      if (k < p.dim) *reinterpret_cast<float2 *>(state + (size_t)k * p.vdim + v0) = make_float2(st[j][2 * i], st[j][2 * i + 1]);
-    }
+    for (int j = 0; j < kKeyTiles; ++j)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int k = 16 * j + g + 8 * i;
+        if (k < p.dim && mine(c))
+          *reinterpret_cast<float2 *>(state + (size_t)k * p.vdim + v0 + 8 * c) = make_float2(st[c][j][2 * i], st[c][j][2 * i + 1]);
+      }
 }
 
 bool al16(const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
@@ -728,12 +739,11 @@ int opt_in(int bytes) {
   return AXB200_OK;
 }
 
-template <int kDK, int kWarps>
+template <int kDK, int kWarps, int kN>
 int run_scan(const ScanParams &p, int count, cudaStream_t st) {
-  using L = ScanSmem<kDK, kWarps>;
-  if (int rc = opt_in<delta_chunk_scan_kernel<kDK, kWarps>>(L::kBytes)) return rc;
-  const int blocks = p.vdim / 8;
-  return launch_dependent(delta_chunk_scan_kernel<kDK, kWarps>, dim3(count, p.heads, (blocks + kWarps - 1) / kWarps),
+  using L = ScanSmem<kDK, kWarps, kN>;
+  if (int rc = opt_in<delta_chunk_scan_kernel<kDK, kWarps, kN>>(L::kBytes)) return rc;
+  return launch_dependent(delta_chunk_scan_kernel<kDK, kWarps, kN>, dim3(count, p.heads, (p.vdim / 8 + L::kTiles - 1) / L::kTiles),
                           dim3(L::kThreads), (size_t)L::kBytes, st, p);
 }
 
@@ -749,15 +759,15 @@ int run(const DeltaParams<__nv_bfloat16> &d, const ScanParams &s, int count, int
   if (int rc = launch_dependent(delta_chunk_prepare_kernel<kDK>, dim3(chunks, count, d.kv_heads), dim3(kPrepThreads), (size_t)P::kBytes, st, d,
                                 s.portions, s.first, keys, heads, s.wait_ns))
     return rc;
-  // as few warps in a CTA as give every SM at most one
+  // as few columns in a CTA as give every SM at most one
   int dev = 0, sms = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess)
     return AXB200_DEVICE_ERROR;
-  const int64_t warps = (int64_t)count * d.heads * (d.vdim / 8);
-  if (warps <= sms) return run_scan<kDK, 1>(s, count, st);
-  if (warps <= 2 * sms) return run_scan<kDK, 2>(s, count, st);
-  if (warps <= 4 * sms) return run_scan<kDK, 4>(s, count, st);
-  return run_scan<kDK, 8>(s, count, st);
+  const int64_t tiles = (int64_t)count * d.heads * (d.vdim / 8);
+  if (tiles <= sms) return run_scan<kDK, 1, 1>(s, count, st);
+  if (tiles <= 2 * sms) return run_scan<kDK, 2, 1>(s, count, st);
+  if (tiles <= 4 * sms) return run_scan<kDK, 4, 1>(s, count, st);
+  return run_scan<kDK, 4, 2>(s, count, st);
 }
 
 int padded_dim(int dim) { return dim <= 64 ? 64 : 128; }
