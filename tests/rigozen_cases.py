@@ -58,7 +58,7 @@ def fast():
         0,
         (latent(40, 64, 64, 256, 0.12, 333), 192),
         (delta(6, 2, 64, 96, 2), 256),
-        (attention(6, 1, 48, 0.14, 64), 192),
+        (attention(10, 1, 56, 0.14, 64), 192),
     ])
 
 

@@ -129,7 +129,7 @@ def shared_pages(lens, kv_heads, dim, dtype, seed=0):
     return Pages(lens, ops.shared_kv_row(kv_heads, dim, dtype), dtype, seed=seed)
 
 
-SHARED_SIZES = [(6, 3, 20), (6, 1, 48), (12, 2, 40), (32, 4, 128), (8, 8, 64), (40, 1, 128), (4, 2, 9), (64, 2, 256)]
+SHARED_SIZES = [(6, 3, 20), (10, 1, 48), (12, 2, 40), (32, 4, 128), (8, 8, 64), (40, 1, 128), (4, 2, 9), (64, 2, 256)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -294,7 +294,7 @@ def run_delta(mixer, w, projs, steps, state, ring):
 
 
 DELTA_SIZES = [(6, 2, 20, 12, 3), (3, 3, 33, 7, 1), (4, 1, 72, 136, 4), (2, 2, 136, 40, 5), (8, 4, 128, 128, 4), (6, 2, 64, 96, 2),
-               (4, 4, 32, 64, 4), (2, 1, 256, 256, 3), (3, 1, 16, 300, 7), (4, 2, 32, 64, 6), (9, 1, 64, 16, 4), (10, 2, 100, 8, 5),
+               (5, 5, 32, 56, 4), (2, 1, 256, 256, 3), (3, 1, 16, 300, 7), (4, 2, 32, 64, 6), (9, 1, 64, 16, 4), (10, 2, 100, 8, 5),
                (64, 16, 32, 128, 4)]
 
 
