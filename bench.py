@@ -1373,9 +1373,12 @@ class LmLab:
         self.sampler.pause()
         return e0.elapsed_time(e1) / steps
 
-    def weights(self, shapes, around_zero=("correction", "norm1", "norm2", "final.norm", "A_log", "dt_bias", "sink")):
-        """name -> random tensor; vectors named in around_zero have mean 0, the others 1."""
-        lab, torch = self, self.torch
+    # vectors with mean 0 instead of 1, by the end of their names
+    AROUND_ZERO = {"Nuderax": ("correction",), "Rigozen": ("norm1", "norm2", "final.norm", "A_log", "dt_bias", "sink")}
+
+    def weights(self, cfg, shapes):
+        """name -> random tensor of a configuration's design."""
+        lab, torch, around_zero = self, self.torch, self.AROUND_ZERO[cfg["architecture"]]
 
         class RandomWeights(dict):
             def __missing__(self, name):
@@ -1464,7 +1467,7 @@ def run_lm(args):
         z = LM_SIZES[size]
         cfg = lm_config(size, n_layers)
         shapes = dict(tensor_shapes(models.config_of(cfg)))
-        model = models.create(cfg, lab.weights(shapes), torch.bfloat16)
+        model = models.create(cfg, lab.weights(cfg, shapes), torch.bfloat16)
         res = {"decode": {}, "prefill": {}, "kernels": {}}
 
         # ---- decode: whole steps as graph replays ----
@@ -1678,7 +1681,7 @@ def run_rigozen(args):
         for name, cfg in (("rigozen", rigozen_config(size, n_layers)), ("nuderax", lm_config(size, n_layers))):
             parsed = models.config_of(cfg)
             module = sys.modules[type(parsed).__module__]
-            model = models.create(cfg, lab.weights(dict(module.tensor_shapes(parsed))), torch.bfloat16)
+            model = models.create(cfg, lab.weights(cfg, dict(module.tensor_shapes(parsed))), torch.bfloat16)
             ms, nodes = lab.decode(model, B, L, args.steps)
             launches += nodes * args.steps
             res["decode"][name] = {"ms_per_step": ms, "tokens_per_s": B / ms * 1e3, "launches": nodes}
